@@ -31,6 +31,7 @@ class MemberSpec:
     v_head_dim: int = 0
     keep_first: int = 0
     values_in_keys: bool = False
+    chunk: int = 0  # c > 0 (without a window): a row at p reads the keys of its own chunk, [p // c * c, p]
 
     @property
     def value_dim(self) -> int:
@@ -41,9 +42,9 @@ class MemberSpec:
         return 0 if self.values_in_keys else self.value_dim
 
     @property
-    def lifetime(self) -> tuple[int, int]:
-        """Members whose pages live equally long: without a window every position is kept anyway."""
-        return (self.window, self.keep_first if self.window > 0 else 0)
+    def lifetime(self) -> tuple[int, int, int]:
+        """Members whose pages live equally long: without a window or chunks every position is kept anyway."""
+        return (self.window, self.keep_first if self.window > 0 else 0, self.chunk)
 
 
 @dataclass
@@ -64,17 +65,17 @@ class CacheMember:
 
 
 def derive_groups(members: list[MemberSpec], page_size: int, num_pages: int) -> tuple[list[GroupSpec], list[int]]:
-    """Members with the same lifetime (here: the same window and the same kept first tokens) share a group
+    """Members with the same lifetime (here: the same window, kept first tokens and chunk size) share a group
     (kelpie-models/kelpie_models/sdk/groups.py:268-294). -> (groups, group index per member)."""
-    keys: list[tuple[int, int]] = []
+    keys: list[tuple[int, int, int]] = []
     index: list[int] = []
     for m in members:
         if m.lifetime not in keys:
             keys.append(m.lifetime)
         index.append(keys.index(m.lifetime))
     if not keys:  # a model without any per-token cache still gets one (empty) group
-        keys.append((0, 0))
-    return [GroupSpec(page_size, w, num_pages, keep) for w, keep in keys], index
+        keys.append((0, 0, 0))
+    return [GroupSpec(page_size, w, num_pages, keep, chunk) for w, keep, chunk in keys], index
 
 
 class KVArena:

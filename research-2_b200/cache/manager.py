@@ -40,6 +40,7 @@ class GroupSpec:
     window: int = 0  # 0 = every position is kept; w > 0 = a query at p reads keys (p - w, p]
     num_pages: int = 1  # pages that can be handed out; page id 0 (the null page) is extra
     keep_first: int = 0  # with a window: the request's first keep_first positions stay readable as well
+    chunk: int = 0  # c > 0 (without a window): a query at p reads the keys of its own chunk, [p // c * c, p]
 
 
 def _ptr(a: np.ndarray):
@@ -50,7 +51,7 @@ def _ptr(a: np.ndarray):
 def group_array(groups: list[GroupSpec]):
     arr = (_host.GroupSpecC * len(groups))()
     for i, g in enumerate(groups):
-        arr[i] = _host.GroupSpecC(g.page_size, g.window, g.num_pages, g.keep_first)
+        arr[i] = _host.GroupSpecC(g.page_size, g.window, g.num_pages, g.keep_first, g.chunk)
     return arr
 
 
@@ -94,7 +95,7 @@ class CacheManager:
         return bool(self._lib.r2_cache_can_reserve(self._h, req, n_computed, n_total, spare_pages))
 
     def slide(self, req: int, n_computed: int) -> None:
-        """Window groups give back the pages that the window has passed."""
+        """Window and chunk groups give back the pages that no later row of the request can read."""
         self._check(self._lib.r2_cache_slide(self._h, req, n_computed), f"slide request {req}")
 
     # ---- queries ---------------------------------------------------------------------------

@@ -100,7 +100,8 @@ def _headers(folder: Path) -> list[Path]:
 
 
 def _build_and_load(key: str, sources: list[Path], deps: list[Path], cmd_prefix: list[str], flags: list[str],
-                    link_flags: list[str], compiler: str) -> ctypes.CDLL:
+                    link_flags: list[str], compiler: str, include: list[str] = ()) -> ctypes.CDLL:
+    """`include`: the folder of the headers in `deps`, whose contents (not whose path) decide whether a library is current."""
     with _lock:
         if key in _loaded:
             return _loaded[key]
@@ -109,7 +110,7 @@ def _build_and_load(key: str, sources: list[Path], deps: list[Path], cmd_prefix:
         if not out.is_file():
             _say(f"compiling {key} (first use)")
             tmp = out.with_suffix(f".tmp{os.getpid()}.so")
-            _run(cmd_prefix + flags + ["-shared", "-o", str(tmp)] + [str(s) for s in sources] + link_flags, key)
+            _run(cmd_prefix + flags + list(include) + ["-shared", "-o", str(tmp)] + [str(s) for s in sources] + link_flags, key)
             os.replace(tmp, out)
             for stale in out.parent.glob(f"{key}.*.so"):
                 if stale != out and ".tmp" not in stale.name:
@@ -148,5 +149,4 @@ def kernel_library(source: str, defines: dict[str, int | str] | None = None) -> 
     tag = "_".join(f"{k.lower()}{v}" for k, v in sorted(defines.items()))
     key = f"r2k_{source}" + (f"_{tag}" if tag else "")
     nvcc = find_nvcc()
-    flags = NVCC_ARCH + NVCC_FLAGS + dflags + ["-I", str(folder)]
-    return _build_and_load(key, [path], _headers(folder), [nvcc], flags, [], nvcc)
+    return _build_and_load(key, [path], _headers(folder), [nvcc], NVCC_ARCH + NVCC_FLAGS + dflags, [], nvcc, include=["-I", str(folder)])

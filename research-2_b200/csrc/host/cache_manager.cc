@@ -61,6 +61,7 @@ int32_t CacheManager::close(int32_t req) {
 
 int32_t CacheManager::first_needed_page(int32_t g, int32_t n_computed) const {
   const GroupSpec& spec = groups_[g];
+  if (spec.chunk > 0) return n_computed / spec.chunk * spec.chunk / spec.page_size;
   if (spec.window <= 0) return 0;
   int32_t first_key = std::max(0, n_computed - spec.window + 1);
   return first_key / spec.page_size;
@@ -110,7 +111,7 @@ int32_t CacheManager::reserve(int32_t req, int32_t n_computed, int32_t n_total) 
 int32_t CacheManager::slide(int32_t req, int32_t n_computed) {
   if (!is_open(req)) return CACHE_BAD_REQUEST;
   for (int32_t g = 0; g < n_groups(); ++g) {
-    if (groups_[g].window <= 0) continue;
+    if (!slides(g)) continue;
     int32_t* t = &tables_[g][size_t(req) * widths_[g]];
     int32_t first = std::min(first_needed_page(g, n_computed), widths_[g]);
     for (int32_t i = kept_pages(g); i < first; ++i) {
@@ -127,8 +128,8 @@ int32_t CacheManager::slide(int32_t req, int32_t n_computed) {
 int32_t CacheManager::worst_pages(int32_t g, int32_t n_total, int32_t max_chunk, int32_t grain) const {
   const GroupSpec& spec = groups_[g];
   int32_t all = ceil_div(n_total, spec.page_size);
-  if (spec.window <= 0) return all;
-  // A portion of rows [s, e) needs the keys from s - window + 1 up to e - 1. Portions are
+  if (!slides(g)) return all;
+  // A portion of rows [s, e) needs the keys from s - window + 1 (or from the start of s's chunk) up to e - 1. Portions are
   // either one decoded row at any s, or a piece of a history: it starts on a multiple of
   // `grain` and ends on one unless it reaches the history's end. The most pages over all of them:
   // (kept first pages that lie before the window's first page come on top)
@@ -137,7 +138,7 @@ int32_t CacheManager::worst_pages(int32_t g, int32_t n_total, int32_t max_chunk,
   grain = std::max(1, grain);
   const int32_t kept = kept_pages(g);
   for (int32_t s = 0; s < n_total; ++s) {
-    int32_t first_page = std::max(0, s - spec.window + 1) / spec.page_size;
+    int32_t first_page = first_needed_page(g, s);
     int32_t e = s + 1;  // the single decoded row
     if (s % grain == 0) {
       e = std::min(n_total, s + max_chunk);

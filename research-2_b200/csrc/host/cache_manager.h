@@ -4,7 +4,8 @@
 // It owns indices only; the tensors that the indices point into belong to the model side.
 // A cache group is a set of layers whose pages live and die together: "all" groups keep every
 // position of a request, "window" groups keep the last `window` positions (and, with `keep_first`,
-// the request's first positions) and give the pages between back as soon as the window has passed them. Every group has a pool of its own. Page id 0 of each
+// the request's first positions) and give the pages between back as soon as the window has passed them, "chunk" groups keep the
+// positions of the chunk that the request has reached (chunks are counted from its position 0). Every group has a pool of its own. Page id 0 of each
 // pool is the null page: real memory that is never handed out; holes in a block table point
 // at it. This restates the block pool of the reference's core (kelpie-core/src/kv_pool.zig:
 // 17-25,183-188,254-301; block tables kelpie-core/src/request.zig:78-81,218-278) without its
@@ -23,6 +24,7 @@ struct GroupSpec {
   int32_t window;     // 0: keep every position; w > 0: a query at p reads keys (p - w, p]
   int32_t num_pages;  // pages that can be handed out (the null page is extra)
   int32_t keep_first; // with a window: the request's first keep_first positions stay readable for good
+  int32_t chunk = 0;  // 0: none; c > 0 (without a window): a query at p reads the keys of its own chunk, [p / c * c, p]
 };
 
 // One group's pages. Freed pages are reused in the order in which they were freed.
@@ -66,7 +68,9 @@ class CacheManager {
   // Every page of the request goes back to its pool; the state slot is released.
   int32_t close(int32_t req);
 
-  // First page index that group g's window still needs when the request's next row is at `n_computed`.
+  // Whether group g gives pages back while a request lives.
+  bool slides(int32_t g) const { return groups_[g].window > 0 || groups_[g].chunk > 0; }
+  // First page index that group g's window or chunk still needs when the request's next row is at `n_computed`.
   int32_t first_needed_page(int32_t g, int32_t n_computed) const;
   // Pages at a table's start that hold kept first positions and are never given back while the request lives.
   int32_t kept_pages(int32_t g) const;
@@ -79,7 +83,7 @@ class CacheManager {
   bool can_reserve(int32_t req, int32_t n_computed, int32_t n_total, int32_t spare_tokens) const;
   // All groups or nothing.
   int32_t reserve(int32_t req, int32_t n_computed, int32_t n_total);
-  // Window groups give back the pages that no later row can read.
+  // Window and chunk groups give back the pages that no later row can read.
   int32_t slide(int32_t req, int32_t n_computed);
   // The most pages of group g that a lone request of n_total positions ever holds, when it is
   // fed in portions of at most max_chunk rows that end on multiples of `grain`.

@@ -13,13 +13,14 @@
 extern "C" {
 #endif
 
-#define R2_ABI_VERSION 5
+#define R2_ABI_VERSION 6
 
 typedef struct {
   int32_t page_size;
   int32_t window;
   int32_t num_pages;
   int32_t keep_first; /* with a window: a request's first keep_first positions are kept for good */
+  int32_t chunk;      /* 0: none; c > 0 (without a window): a query at p reads the keys of its own chunk, [p / c * c, p] */
 } R2GroupSpec;
 
 typedef struct {
