@@ -48,6 +48,10 @@ struct DecodeParams {
   // exp(sinks[h]) instead of exp(0) into head h's denominator; `head_gate` (may be null; float [rows, n_heads])
   // multiplies head h's output by the sigmoid of its entry.
   float softcap; const float* sinks; const float* head_gate; int head_gate_stride;
+  // The form X == 2 alone: `chunk` > 0 (without a window) limits a row at position p to its own chunk's keys, [p / chunk * chunk, p];
+  // `dist_bias` (may be null; [n_heads][bias_len]) is added to head h's score of a key n positions back (entry n, the last entry
+  // for every larger n); `out_scale` multiplies the output.
+  int chunk; const float* dist_bias; int bias_len; float out_scale;
   int n_slices;
   float* part_o;   // [rows, n_heads, n_slices, HD]
   float* part_ml;  // [rows, n_heads, n_slices, 2]
@@ -86,9 +90,9 @@ __device__ __forceinline__ uint32_t pack_rest(float lo, float hi, uint32_t packe
 // The end of a row's softmax: with a sink the denominator counts one more key of score 0; with a gate the
 // output is multiplied by the sigmoid of the gate's value.
 __device__ __forceinline__ float finish(float o, float l, float mx, int sink, const bf16* gate, float sink_value = 0.f,
-                                        const float* head_gate = nullptr) {
+                                        const float* head_gate = nullptr, float scale = 1.f) {
   if (sink) l += mx > -INFINITY ? __expf(sink_value - mx) : 1.f;   // (no key seen: o is zero whatever l is)
-  float y = l > 0.f ? o / l : 0.f;
+  float y = l > 0.f ? o * scale / l : 0.f;
   if (gate != nullptr) y *= 1.f / (1.f + __expf(-__bfloat162float(*gate)));
   if (head_gate != nullptr) y *= 1.f / (1.f + __expf(-*head_gate));
   return y;
@@ -106,9 +110,9 @@ bool g_decode_mma = true;              // r2_attention_decode_set_mma (tests com
 // A tile then costs a warp 32 mma and 16 ldmatrix instead of some 500 scalar instructions, which
 // is what bounds this kernel at large batches (at batch 64 it read the cache at 0.57 of the copy
 // bandwidth with the scalar form).
-// X: the form with kept first keys, a sink, a gate and two-term weights; without it those parameters are not
-// read and the plain form compiles to what it was.
-template <int G, bool MMA, bool X>
+// X 1: the form with kept first keys, a sink, a gate and two-term weights; without it those parameters are not
+// read and the plain form compiles to what it was. X 2: chunks, a bias by distance and a factor on the output besides.
+template <int G, bool MMA, int X>
 __global__ void __launch_bounds__(WARPS * 32, (MMA && HD <= 64) ? 5 : 1)  // five CTAs to an SM is what the tiles' shared memory allows
 decode_kernel(const DecodeParams p) {
   pdl_launch_dependents();  // the next kernel may begin its prologue
@@ -129,13 +133,19 @@ decode_kernel(const DecodeParams p) {
   const int pos = p.positions[t];
   const int seq_len = p.seq_lens[e];
   const int last = pos < seq_len - 1 ? pos : seq_len - 1;
-  const int first = p.window > 0 ? (pos - p.window + 1 > 0 ? pos - p.window + 1 : 0) : 0;
+  const int first = (X == 2 && p.chunk > 0) ? pos / p.chunk * p.chunk
+                                            : (p.window > 0 ? (pos - p.window + 1 > 0 ? pos - p.window + 1 : 0) : 0);
   // The keys that the row sees are walked by a running index v: first the kept first keys (those below
   // the window's start), then the window's. Key v of the walk lies at position v, or first + (v - kept).
   const int kept = (X && p.window > 0) ? min(p.keep_first, first) : 0;
   const int n_keys = kept + last - first + 1;
   const int v_of_pos = kept + pos - first;   // where the newest key stands in the walk
   auto key_at = [&](int v) { return (X && v < kept) ? v : first + (v - kept); };
+  // what distance adds to the score of query head h0 + g for key v of the walk
+  auto bias_at = [&](int g, int v) {
+    const int n = pos - key_at(v);
+    return p.dist_bias[size_t(h0 + g) * p.bias_len + (n < p.bias_len ? n : p.bias_len - 1)];
+  };
   // this slice's keys: equal runs of whole 32-key tiles
   const int tiles = (n_keys + 31) / 32;
   const int tiles_per = (tiles + p.n_slices - 1) / p.n_slices;
@@ -296,6 +306,10 @@ decode_kernel(const DecodeParams p) {
             if (seen) sc[nt][c] = soft_cap(sc[nt][c], p.softcap);
             if (seen) sc[nt][2 + c] = soft_cap(sc[nt][2 + c], p.softcap);
           }
+          if (X == 2 && p.dist_bias != nullptr && seen) {
+            if (gq < G) sc[nt][c] += bias_at(gq, v0 + nt * 8 + 2 * tq + c);
+            if (gq + 8 < G) sc[nt][2 + c] += bias_at(gq + 8, v0 + nt * 8 + 2 * tq + c);
+          }
           mx_a = fmaxf(mx_a, sc[nt][c]);
           mx_b = fmaxf(mx_b, sc[nt][2 + c]);
         }
@@ -390,6 +404,7 @@ decode_kernel(const DecodeParams p) {
     for (int g = 0; g < G; ++g) {
       float sv = valid ? s[g] : -INFINITY;
       if (X && p.softcap > 0.f && valid) sv = soft_cap(sv, p.softcap);
+      if (X == 2 && p.dist_bias != nullptr && valid) sv += bias_at(g, v0 + lane);
       float m_new = fmaxf(m[g], warp_max(sv));
       float corr = __expf(m[g] - m_new);
       pr[g] = valid ? __expf(sv - m_new) : 0.f;
@@ -482,7 +497,7 @@ decode_kernel(const DecodeParams p) {
       const bf16* gate = (X && p.gate != nullptr) ? p.gate + size_t(t) * p.gate_row_stride + size_t(h0 + g) * HD + d : nullptr;
       p.out[size_t(t) * p.out_row_stride + size_t(h0 + g) * HD + d] = __float2bfloat16_rn(finish(
           o, lsum, mx, X ? p.sink : 0, gate, (X && p.sinks != nullptr) ? p.sinks[h0 + g] : 0.f,
-          (X && p.head_gate != nullptr) ? p.head_gate + size_t(t) * p.head_gate_stride + h0 + g : nullptr));
+          (X && p.head_gate != nullptr) ? p.head_gate + size_t(t) * p.head_gate_stride + h0 + g : nullptr, X == 2 ? p.out_scale : 1.f));
     } else {
       size_t at = (size_t(t) * p.n_heads + h0 + g) * p.n_slices + slice;
       p.part_o[at * HD + d] = o;
@@ -521,7 +536,7 @@ decode_kernel(const DecodeParams p) {
         const bf16* gate = (X && p.gate != nullptr) ? p.gate + size_t(t) * p.gate_row_stride + size_t(h0 + g) * HD + d : nullptr;
         p.out[size_t(t) * p.out_row_stride + size_t(h0 + g) * HD + d] = __float2bfloat16_rn(finish(
           o, lsum, mx, X ? p.sink : 0, gate, (X && p.sinks != nullptr) ? p.sinks[h0 + g] : 0.f,
-          (X && p.head_gate != nullptr) ? p.head_gate + size_t(t) * p.head_gate_stride + h0 + g : nullptr));
+          (X && p.head_gate != nullptr) ? p.head_gate + size_t(t) * p.head_gate_stride + h0 + g : nullptr, X == 2 ? p.out_scale : 1.f));
       }
     }
   }
@@ -553,7 +568,7 @@ __global__ void merge_kernel(const float* __restrict__ part_o, const float* __re
   }
 }
 
-template <int G, bool MMA, bool X>
+template <int G, bool MMA, int X>
 bool configure_smem() {
   // once per kernel instance and device (function attributes belong to a device's context): room for
   // the tiles beyond the default 48 KB
@@ -570,7 +585,7 @@ bool configure_smem() {
   return true;
 }
 
-template <int G, bool MMA, bool X>
+template <int G, bool MMA, int X>
 int launch_form(const DecodeParams& p, int n_rows, cudaStream_t stream) {
   dim3 grid(p.n_slices, p.n_kv_heads, n_rows);
   if (!configure_smem<G, MMA, X>()) return R2_UNSUPPORTED;
@@ -578,7 +593,7 @@ int launch_form(const DecodeParams& p, int n_rows, cudaStream_t stream) {
   return launch_status();
 }
 
-template <int G, bool X = false>
+template <int G, int X = 0>
 int launch(const DecodeParams& p, int n_rows, cudaStream_t stream) {
   if constexpr (MMA_FITS) {
     if (g_decode_mma) return launch_form<G, true, X>(p, n_rows, stream);
@@ -616,6 +631,7 @@ extern "C" int r2_attention_decode(const void* q, int q_row_stride, void* out, i
   p.scale = scale; p.window = window; p.n_slices = n_slices;
   p.keep_first = 0; p.sink = 0; p.gate = nullptr; p.gate_row_stride = 0; p.split_p = 0;
   p.softcap = 0.f; p.sinks = nullptr; p.head_gate = nullptr; p.head_gate_stride = 0;
+  p.chunk = 0; p.dist_bias = nullptr; p.bias_len = 0; p.out_scale = 1.f;
   p.part_o = scratch;
   p.part_ml = scratch != nullptr ? scratch + (long long)n_rows * n_heads * n_slices * HD : nullptr;
   p.k_new = nullptr; p.v_new = nullptr; p.new_row_stride = 0; p.slot_mapping = nullptr;
@@ -639,12 +655,13 @@ namespace {
 // The plain form for groups of 1, 2, 4 and 8 query heads; the form with extras for every group up to 8.
 template <int G>
 int launch_fused(const DecodeParams& p, int n_rows, cudaStream_t stream) {
+  if (p.chunk > 0 || p.dist_bias != nullptr || p.out_scale != 1.f) return launch<G, 2>(p, n_rows, stream);
   const bool extras = p.keep_first > 0 || p.sink != 0 || p.gate != nullptr || p.split_p != 0 || p.softcap > 0.f ||
                       p.sinks != nullptr || p.head_gate != nullptr;
   if constexpr (G == 1 || G == 2 || G == 4 || G == 8) {
-    if (!extras) return launch<G, false>(p, n_rows, stream);
+    if (!extras) return launch<G, 0>(p, n_rows, stream);
   }
-  return launch<G, true>(p, n_rows, stream);
+  return launch<G, 1>(p, n_rows, stream);
 }
 
 }  // namespace
@@ -655,7 +672,8 @@ int launch_fused(const DecodeParams& p, int n_rows, cudaStream_t stream) {
 // finishes last, so there is neither a separate cache-write kernel nor a merge kernel.
 // `scratch` as for r2_attention_decode; `counters` holds n_rows * n_kv_heads ints that are
 // zero before the call and zero again after it. `keep_first`, `sink`, `gate` and `split_p`: see DecodeParams.
-extern "C" int r2_attention_decode_fused_capped(const void* q, int q_row_stride, void* out, int out_row_stride, void* k_cache,
+// `chunk`, `dist_bias`, `bias_len` and `out_scale` (0, null, 0 and 1: none of them) likewise.
+extern "C" int r2_attention_decode_fused_biased(const void* q, int q_row_stride, void* out, int out_row_stride, void* k_cache,
                                          void* v_cache, long long page_stride, int page_size, int n_pages,
                                          const int32_t* block_tables, int table_width, const int32_t* row_entry,
                                          const int32_t* positions, const int32_t* seq_lens, int n_rows, int n_heads,
@@ -664,9 +682,9 @@ extern "C" int r2_attention_decode_fused_capped(const void* q, int q_row_stride,
                                          float* scratch, long long scratch_floats, int* counters, int n_counters,
                                          int keep_first, int sink, const void* gate, int gate_row_stride, int split_p,
                                          float softcap, const float* sinks, const float* head_gate, int head_gate_stride,
-                                         cudaStream_t stream) {
+                                         int chunk, const float* dist_bias, int bias_len, float out_scale, cudaStream_t stream) {
   if (n_rows <= 0) return R2_OK;
-  if (keep_first < 0) return R2_BAD_SHAPE;
+  if (keep_first < 0 || chunk < 0 || (chunk > 0 && window > 0) || (dist_bias != nullptr && bias_len < 1)) return R2_BAD_SHAPE;
   if (n_heads < 1 || n_kv_heads < 1 || n_heads % n_kv_heads != 0 || page_size < 1 || window < 0 || n_slices < 1) return R2_BAD_SHAPE;
   if (n_slices > 1 && (scratch == nullptr || counters == nullptr || n_counters < n_rows * n_kv_heads ||
                        scratch_floats < r2_attention_decode_scratch_floats(n_rows, n_heads, n_slices))) return R2_BAD_SHAPE;
@@ -684,6 +702,7 @@ extern "C" int r2_attention_decode_fused_capped(const void* q, int q_row_stride,
   p.scale = scale; p.window = window; p.n_slices = n_slices;
   p.keep_first = keep_first; p.sink = (sink || sinks != nullptr) ? 1 : 0; p.gate = (const bf16*)gate; p.gate_row_stride = gate_row_stride; p.split_p = split_p;
   p.softcap = softcap; p.sinks = sinks; p.head_gate = head_gate; p.head_gate_stride = head_gate_stride;
+  p.chunk = chunk; p.dist_bias = dist_bias; p.bias_len = bias_len; p.out_scale = out_scale;
   p.part_o = scratch;
   p.part_ml = scratch != nullptr ? scratch + (long long)n_rows * n_heads * n_slices * HD : nullptr;
   p.k_new = (const bf16*)k_new; p.v_new = (const bf16*)v_new; p.new_row_stride = new_row_stride;
@@ -712,10 +731,10 @@ extern "C" int r2_attention_decode_fused(const void* q, int q_row_stride, void* 
                                          float* scratch, long long scratch_floats, int* counters, int n_counters,
                                          int keep_first, int sink, const void* gate, int gate_row_stride, int split_p,
                                          cudaStream_t stream) {
-  return r2_attention_decode_fused_capped(q, q_row_stride, out, out_row_stride, k_cache, v_cache, page_stride, page_size, n_pages,
+  return r2_attention_decode_fused_biased(q, q_row_stride, out, out_row_stride, k_cache, v_cache, page_stride, page_size, n_pages,
                                           block_tables, table_width, row_entry, positions, seq_lens, n_rows, n_heads, n_kv_heads, scale,
                                           window, n_slices, k_new, v_new, new_row_stride, slot_mapping, scratch, scratch_floats, counters,
-                                          n_counters, keep_first, sink, gate, gate_row_stride, split_p, 0.f, nullptr, nullptr, 0, stream);
+                                          n_counters, keep_first, sink, gate, gate_row_stride, split_p, 0.f, nullptr, nullptr, 0, 0, nullptr, 0, 1.f, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

@@ -63,10 +63,15 @@ struct PrefillParams {
   // exp(sinks[h]) instead of exp(0) into head h's denominator; `head_gate` (may be null; float [rows, n_heads])
   // multiplies head h's output by the sigmoid of its entry.
   float softcap; const float* sinks; const float* head_gate; int head_gate_stride;
+  // The form X alone: `chunk` > 0 (without a window) limits a row at position p to its own chunk's keys, [p / chunk * chunk, p];
+  // `dist_bias` (may be null; [n_heads][bias_len]) is added to head h's score of a key n positions back (entry n, the last entry
+  // for every larger n; the first bias_smem of them lie in shared memory); `out_scale` multiplies the output.
+  int chunk; const float* dist_bias; int bias_len; int bias_smem; float out_scale;
   int box_rows;      // TMA form: key rows per tensor copy (the page size, or 64 for larger pages)
   int* error_flag;   // TMA form: where a bounded wait that ran out is recorded
 };
 
+constexpr int BIAS_SMEM = 2048;               // entries of a distance bias kept in shared memory at most
 bool g_prefill_tma = true;                    // r2_attention_prefill_set_tma
 constexpr int TMA_TILE_BYTES = BN * 128;       // TMA form (head size 64): unpadded 128-byte rows
 using namespace r2ptx;
@@ -75,7 +80,9 @@ using namespace r2ptx;
 // Threads: four warps that compute; the TMA form adds a fifth that only issues the tensor copies
 // (a tile's two or more copies cost the issuing thread several hundred cycles, which would
 // otherwise come out of one computing warp and hold the other three at the next barrier).
-template <bool TMA>
+// X: the form with chunks, a bias by distance and a factor on the output; without it those parameters are not read and the
+// kernel compiles to what it is without them.
+template <bool TMA, bool X>
 __global__ void __launch_bounds__(WARPS * 32 + (TMA ? 32 : 0))
 prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const PrefillParams p) {
   pdl_launch_dependents();  // the next kernel may begin its prologue
@@ -88,6 +95,7 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
   uint8_t* k_s = TMA ? reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem + TILE_BYTES) + 1023) & ~uintptr_t(1023))
                      : smem + TILE_BYTES;
   uint8_t* v_s = k_s + STAGES * KV_TILE;
+  float* bias_s = reinterpret_cast<float*>(v_s + STAGES * KV_TILE);   // form X: [bias_smem], in units of log2 e
   __shared__ int tile_entry, tile_row0;
   __shared__ __align__(8) uint64_t full[STAGES];    // TMA form: a stage's copies have landed
   __shared__ __align__(8) uint64_t empty[STAGES];   // TMA form: the four computing warps are done with a stage
@@ -124,10 +132,13 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
   const int start = seq_len - n_rows;           // position of the entry's first row
   const int rows_here = min(BM, n_rows - r0);
   const int pmin = start + r0, pmax = start + r0 + rows_here - 1;
-  const int lo = p.window > 0 ? max(0, pmin - p.window + 1) : 0;
+  const int lo = (X && p.chunk > 0) ? pmin / p.chunk * p.chunk : (p.window > 0 ? max(0, pmin - p.window + 1) : 0);
   const int keep = p.window > 0 ? p.keep_first : 0;   // keys below it stay visible however far the window has moved
   const int32_t* table = p.block_tables + size_t(e) * p.table_width;
 
+  if (X && p.dist_bias != nullptr) {   // (every role of the CTA waits at a barrier before a score is made)
+    for (int n = tid; n < p.bias_smem; n += blockDim.x) bias_s[n] = p.dist_bias[size_t(h) * p.bias_len + n] * 1.4426950408889634f;
+  }
   // ---- the query tile ----
   for (int id = tid; id < BM * (HD / 8) && tid < WARPS * 32; id += WARPS * 32) {
     int row = id / (HD / 8), c = id % (HD / 8);
@@ -299,7 +310,9 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       }
     }
     // a warp whose 16 rows all lie past the entry's rows, or before every key of this tile, rests
-    const bool warp_active = warp * 16 < rows_here && j0 <= pmin + min(warp * 16 + 15, rows_here - 1);
+    // (and, with chunks, one whose rows all belong to later chunks than the tile's keys)
+    const bool warp_active = warp * 16 < rows_here && j0 <= pmin + min(warp * 16 + 15, rows_here - 1) &&
+                             !(X && p.chunk > 0 && j0 + BN - 1 < (pmin + warp * 16) / p.chunk * p.chunk);
     if (warp_active) {
       const uint32_t kt = smem_u32(k_s) + uint32_t(stage * KV_TILE);
       const uint32_t vt = smem_u32(v_s) + uint32_t(stage * KV_TILE);
@@ -333,11 +346,31 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
           for (int c = 0; c < 4; ++c) s[nt][c] = back * (1.f - __fdividef(2.f, __expf(s[nt][c] * in) + 1.f));
         }
       }
+      if (X) {
+        // the bias by distance; the scores go on in units of log2 e, with the scale inside
+        const bool biased = p.dist_bias != nullptr;
+        const float* far = biased ? p.dist_bias + size_t(h) * p.bias_len : nullptr;
+        auto bias_at = [&](int n) {
+          n = min(max(n, 0), p.bias_len - 1);   // (keys after the row are masked below)
+          return n < p.bias_smem ? bias_s[n] : far[n] * 1.4426950408889634f;
+        };
+#pragma unroll
+        for (int nt = 0; nt < BN / 8; ++nt) {
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const int n = pos_a - (j0 + nt * 8 + 2 * tq + c);
+            s[nt][c] = fmaf(s[nt][c], scale2, biased ? bias_at(n) : 0.f);
+            s[nt][2 + c] = fmaf(s[nt][2 + c], scale2, biased ? bias_at(n + 8) : 0.f);
+          }
+        }
+      }
+      const float units = X ? 1.f : scale2;   // what is left to multiply the scores by
       float mx_a = -INFINITY, mx_b = -INFINITY;
       // every key of this tile is visible to every row of this warp: no mask to evaluate
       const int warp_pmin = pmin + warp * 16, warp_pmax = pmin + min(warp * 16 + 15, rows_here - 1);
       const bool all_visible = j0 + BN - 1 <= warp_pmin && warp * 16 + 15 < rows_here &&
-                               (p.window == 0 || j0 > warp_pmax - p.window || j0 + BN <= keep);
+                               (p.window == 0 || j0 > warp_pmax - p.window || j0 + BN <= keep) &&
+                               !(X && p.chunk > 0 && j0 < warp_pmax / p.chunk * p.chunk);
       // (the scale is positive, so the largest raw score is the largest scaled one; it goes into
       // the exponent's multiply-add)
       if (all_visible) {
@@ -353,7 +386,11 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
         // key k of the tile is seen by a row if lo <= k <= hi (two compares against registers: the same test
         // written with && and || over the position compiles to a chain of branches per element)
         const int hi_a = row_a < rows_here ? pos_a - j0 : -1, hi_b = row_b < rows_here ? pos_b - j0 : -1;
-        const int lo_a = p.window > 0 ? pos_a - p.window + 1 - j0 : 0, lo_b = p.window > 0 ? pos_b - p.window + 1 - j0 : 0;
+        int lo_a = p.window > 0 ? pos_a - p.window + 1 - j0 : 0, lo_b = p.window > 0 ? pos_b - p.window + 1 - j0 : 0;
+        if (X && p.chunk > 0) {
+          lo_a = pos_a / p.chunk * p.chunk - j0;
+          lo_b = pos_b / p.chunk * p.chunk - j0;
+        }
         const int kf = keep - j0;   // keys of the tile below it are kept first keys
 #pragma unroll
         for (int nt = 0; nt < BN / 8; ++nt) {
@@ -373,7 +410,7 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
       mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
       mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
-      const float m_a = fmaxf(m_run[0], mx_a * scale2), m_b = fmaxf(m_run[1], mx_b * scale2);
+      const float m_a = fmaxf(m_run[0], mx_a * units), m_b = fmaxf(m_run[1], mx_b * units);
       // a row that has seen no key yet keeps exp(-inf - -inf) out of the way
       const float base_a = m_a == -INFINITY ? 0.f : m_a, base_b = m_b == -INFINITY ? 0.f : m_b;
       const float corr_a = fast_exp2(m_run[0] - base_a), corr_b = fast_exp2(m_run[1] - base_b);
@@ -382,8 +419,8 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       for (int nt = 0; nt < BN / 8; ++nt) {
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
-          s[nt][c] = fast_exp2(fmaf(s[nt][c], scale2, -base_a));
-          s[nt][2 + c] = fast_exp2(fmaf(s[nt][2 + c], scale2, -base_b));
+          s[nt][c] = fast_exp2(fmaf(s[nt][c], units, -base_a));
+          s[nt][2 + c] = fast_exp2(fmaf(s[nt][2 + c], units, -base_b));
           sum_a += s[nt][c];
           sum_b += s[nt][2 + c];
         }
@@ -442,6 +479,10 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
     l_run[1] += m_run[1] > -INFINITY ? fast_exp2(sv - m_run[1]) : 1.f;
   }
   float inv_a = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, inv_b = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
+  if (X) {
+    inv_a *= p.out_scale;
+    inv_b *= p.out_scale;
+  }
   if (p.head_gate != nullptr) {  // one gate per head
     if (row_a < rows_here) inv_a *= 1.f / (1.f + __expf(-p.head_gate[size_t(t0 + r0 + row_a) * p.head_gate_stride + h]));
     if (row_b < rows_here) inv_b *= 1.f / (1.f + __expf(-p.head_gate[size_t(t0 + r0 + row_b) * p.head_gate_stride + h]));
@@ -476,19 +517,21 @@ extern "C" int r2_attention_prefill_head_dim(void) { return HD; }
 
 namespace {
 
-template <bool TMA>
+template <bool TMA, bool X>
 int launch(const CUtensorMap& mk, const CUtensorMap& mv, const PrefillParams& p, int n_tiles, cudaStream_t stream) {
   const size_t smem = TMA ? size_t(TILE_BYTES) + 1024 + 2 * STAGES * size_t(TMA_TILE_BYTES) : (1 + 2 * STAGES) * size_t(TILE_BYTES);
+  const size_t smem_most = smem + (X ? BIAS_SMEM * sizeof(float) : 0);
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_kernel<TMA>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    cudaError_t e = cudaFuncSetAttribute(prefill_kernel<TMA, X>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_most));
     if (e != cudaSuccess) return int(e);
     // several CTAs per SM hide each other's waits: ask for the shared memory that takes
-    e = cudaFuncSetAttribute(prefill_kernel<TMA>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    e = cudaFuncSetAttribute(prefill_kernel<TMA, X>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     if (e != cudaSuccess) return int(e);
     configured = true;
   }
-  r2_launch(prefill_kernel<TMA>, dim3(dim3(n_tiles, p.n_heads)), dim3(WARPS * 32 + (TMA ? 32 : 0)), size_t(smem), stream, mk, mv, p);
+  const size_t smem_here = smem + (X ? size_t(p.bias_smem) * sizeof(float) : 0);
+  r2_launch(prefill_kernel<TMA, X>, dim3(dim3(n_tiles, p.n_heads)), dim3(WARPS * 32 + (TMA ? 32 : 0)), smem_here, stream, mk, mv, p);
   return launch_status();
 }
 
@@ -498,15 +541,18 @@ int launch(const CUtensorMap& mk, const CUtensorMap& mv, const PrefillParams& p,
 // harmless: the CTAs beyond find no tile). error_flag: a device word in which a bounded wait that
 // ran out is recorded (may be null; the tensor-copy form is then not used). `keep_first`, `sink`, `gate`
 // and `split_p`: see PrefillParams.
-extern "C" int r2_attention_prefill_capped(const void* q, int q_row_stride, void* out, int out_row_stride, const void* k_cache,
+// `chunk`, `dist_bias`, `bias_len` and `out_scale` (0, null, 0 and 1: none of them): see PrefillParams.
+extern "C" int r2_attention_prefill_biased(const void* q, int q_row_stride, void* out, int out_row_stride, const void* k_cache,
                                     const void* v_cache, long long page_stride, int page_size, int n_pages,
                                     const int32_t* block_tables, int table_width, const int32_t* q_start,
                                     const int32_t* seq_lens, int n_entries, int n_tiles, int n_heads, int n_kv_heads,
                                     float scale, int window, int* error_flag, int keep_first, int sink, const void* gate,
                                     int gate_row_stride, int split_p, float softcap, const float* sinks, const float* head_gate,
-                                    int head_gate_stride, cudaStream_t stream) {
+                                    int head_gate_stride, int chunk, const float* dist_bias, int bias_len, float out_scale,
+                                    cudaStream_t stream) {
   if (n_entries <= 0 || n_tiles <= 0) return R2_OK;
-  if (n_heads < 1 || n_kv_heads < 1 || n_heads % n_kv_heads != 0 || page_size < 1 || window < 0 || keep_first < 0) return R2_BAD_SHAPE;
+  if (n_heads < 1 || n_kv_heads < 1 || n_heads % n_kv_heads != 0 || page_size < 1 || window < 0 || keep_first < 0 || chunk < 0) return R2_BAD_SHAPE;
+  if ((chunk > 0 && window > 0) || (dist_bias != nullptr && bias_len < 1)) return R2_BAD_SHAPE;
   if (gate != nullptr && (gate_row_stride % 2 != 0 || (reinterpret_cast<uintptr_t>(gate) & 3))) return R2_BAD_ALIGN;
   if (page_stride % 8 != 0 || q_row_stride % 8 != 0 || out_row_stride % 2 != 0 || (reinterpret_cast<uintptr_t>(k_cache) & 15) ||
       (reinterpret_cast<uintptr_t>(v_cache) & 15) || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(out) & 3)) {
@@ -524,6 +570,9 @@ extern "C" int r2_attention_prefill_capped(const void* q, int q_row_stride, void
   p.scale = scale; p.window = window;
   p.keep_first = keep_first; p.sink = (sink || sinks != nullptr) ? 1 : 0; p.gate = (const bf16*)gate; p.gate_row_stride = gate_row_stride; p.split_p = split_p;
   p.softcap = softcap; p.sinks = sinks; p.head_gate = head_gate; p.head_gate_stride = head_gate_stride;
+  p.chunk = chunk; p.dist_bias = dist_bias; p.bias_len = dist_bias != nullptr ? bias_len : 0; p.out_scale = out_scale;
+  p.bias_smem = p.bias_len < BIAS_SMEM ? p.bias_len : BIAS_SMEM;
+  const bool extra = chunk > 0 || dist_bias != nullptr || out_scale != 1.f;
   p.box_rows = 0;
   p.error_flag = error_flag;
   CUtensorMap mk, mv;
@@ -532,13 +581,26 @@ extern "C" int r2_attention_prefill_capped(const void* q, int q_row_stride, void
     p.box_rows = page_size < 64 ? page_size : 64;
     if (r2::page_map(&mk, k_cache, page_stride, page_size, n_kv_heads, n_pages, p.box_rows, HD) &&
         r2::page_map(&mv, v_cache, page_stride, page_size, n_kv_heads, n_pages, p.box_rows, HD)) {
-      return launch<true>(mk, mv, p, n_tiles, stream);
+      return extra ? launch<true, true>(mk, mv, p, n_tiles, stream) : launch<true, false>(mk, mv, p, n_tiles, stream);
     }
     p.box_rows = 0;
   }
   memset(&mk, 0, sizeof(mk));
   memset(&mv, 0, sizeof(mv));
-  return launch<false>(mk, mv, p, n_tiles, stream);
+  return extra ? launch<false, true>(mk, mv, p, n_tiles, stream) : launch<false, false>(mk, mv, p, n_tiles, stream);
+}
+
+extern "C" int r2_attention_prefill_capped(const void* q, int q_row_stride, void* out, int out_row_stride, const void* k_cache,
+                                    const void* v_cache, long long page_stride, int page_size, int n_pages,
+                                    const int32_t* block_tables, int table_width, const int32_t* q_start,
+                                    const int32_t* seq_lens, int n_entries, int n_tiles, int n_heads, int n_kv_heads,
+                                    float scale, int window, int* error_flag, int keep_first, int sink, const void* gate,
+                                    int gate_row_stride, int split_p, float softcap, const float* sinks, const float* head_gate,
+                                    int head_gate_stride, cudaStream_t stream) {
+  return r2_attention_prefill_biased(q, q_row_stride, out, out_row_stride, k_cache, v_cache, page_stride, page_size, n_pages, block_tables,
+                                     table_width, q_start, seq_lens, n_entries, n_tiles, n_heads, n_kv_heads, scale, window, error_flag,
+                                     keep_first, sink, gate, gate_row_stride, split_p, softcap, sinks, head_gate, head_gate_stride, 0,
+                                     nullptr, 0, 1.f, stream);
 }
 
 extern "C" int r2_attention_prefill(const void* q, int q_row_stride, void* out, int out_row_stride, const void* k_cache,

@@ -27,7 +27,7 @@ constexpr int MAX_EXPERTS = 1024;
 template <typename T>
 __global__ void __launch_bounds__(256)
 small_linear_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ w, const float* __restrict__ bias,
-                    float* __restrict__ out, int out_stride, int n_out, int width) {
+                    float* __restrict__ out, int out_stride, int n_out, int width, int act) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float row[];
@@ -40,7 +40,7 @@ small_linear_kernel(const T* __restrict__ h, int h_stride, const float* __restri
     float acc = 0.f;
     for (int k = lane; k < width; k += 32) acc = fmaf(row[k], wr[k], acc);
     acc = warp_sum(acc);
-    if (lane == 0) out[size_t(t) * out_stride + n] = acc + (bias != nullptr ? bias[n] : 0.f);
+    if (lane == 0) out[size_t(t) * out_stride + n] = activate(acc + (bias != nullptr ? bias[n] : 0.f), act);
   }
 }
 
@@ -222,11 +222,12 @@ route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restri
   }
 }
 
-constexpr int KIND_CLAMPED_SWISH = 0, KIND_RELU = 1, KIND_SILU = 2;
+constexpr int KIND_CLAMPED_SWISH = 0, KIND_RELU = 1, KIND_SILU = 2, KIND_GELU_TANH = 3;
 
 __device__ __forceinline__ float gated_unit(float g, float u, int kind, float limit, float alpha, float up_offset) {
   if (kind == KIND_RELU) return fmaxf(g, 0.f) * u;
   if (kind == KIND_SILU) return g / (1.f + expf(-g)) * u;
+  if (kind == KIND_GELU_TANH) return gelu_tanh(g) * u;
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-alpha * g)) * (u + up_offset);
@@ -260,16 +261,17 @@ expert_act_kernel(const T* __restrict__ gate_up, int in_stride, T* __restrict__ 
 }  // namespace
 
 extern "C" int r2_small_linear(const void* h, int h_stride, const float* w, const float* bias, float* out, int out_stride,
-                               int n_rows, int n_out, int width, int dtype, cudaStream_t stream) {
+                               int n_rows, int n_out, int width, int act, int dtype, cudaStream_t stream) {
   if (n_rows <= 0 || n_out <= 0) return R2_OK;
+  if (act < R2_ACT_NONE || act > R2_ACT_TANH) return R2_UNSUPPORTED;
   if (width < 1) return R2_BAD_SHAPE;
   const size_t smem = sizeof(float) * width;
   if (smem > 48 * 1024) return R2_UNSUPPORTED;
   const int threads = n_out >= 8 ? 256 : 32 * n_out;
   if (dtype == R2_F32) {
-    r2_launch(small_linear_kernel<float>, dim3(n_rows), dim3(threads), smem, stream, (const float*)h, h_stride, w, bias, out, out_stride, n_out, width);
+    r2_launch(small_linear_kernel<float>, dim3(n_rows), dim3(threads), smem, stream, (const float*)h, h_stride, w, bias, out, out_stride, n_out, width, act);
   } else if (dtype == R2_BF16) {
-    r2_launch(small_linear_kernel<bf16>, dim3(n_rows), dim3(threads), smem, stream, (const bf16*)h, h_stride, w, bias, out, out_stride, n_out, width);
+    r2_launch(small_linear_kernel<bf16>, dim3(n_rows), dim3(threads), smem, stream, (const bf16*)h, h_stride, w, bias, out, out_stride, n_out, width, act);
   } else {
     return R2_BAD_DTYPE;
   }

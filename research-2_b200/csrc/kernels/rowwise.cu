@@ -890,7 +890,8 @@ extern "C" int r2_pair_norm_add(const float* x, const float* a, const float* b, 
 }
 
 // ---- a sublayer's output, normalised, joins the stream (and the next sublayer's input leaves with it) --------------
-// out = x + y / rms(y) * w, all float; with `next_w` also h = out / rms(out) * next_w in the compute dtype: the norm after a
+// out = x + y / rms(y) * w, all float; with `next_w` also h = out / rms(out) * next_w in the compute dtype (with `next` alone h
+// is out itself in that dtype): the norm after a
 // sublayer, the residual sum and the norm before the next sublayer in one pass. One CTA per row; the row stays in
 // registers between the passes (ROWS_PER_THREAD elements a thread) where it fits, else it is read again.
 namespace {
@@ -935,6 +936,18 @@ norm_add_kernel(const float* __restrict__ x, const float* __restrict__ y, const 
     }
   }
   if (next == nullptr) return;
+  if (next_w == nullptr) {   // no second norm: the new rows themselves, rounded
+    if (fits) {
+#pragma unroll
+      for (int i = 0; i < NORM_ADD_KEEP; ++i) {
+        const int d = threadIdx.x + i * NORM_ADD_THREADS;
+        if (d < width) next[at + d] = from_float<O>(keep[i]);
+      }
+    } else {
+      for (int d = threadIdx.x; d < width; d += NORM_ADD_THREADS) next[at + d] = from_float<O>(out[at + d]);
+    }
+    return;
+  }
   const float inv_out = 1.f / sqrtf(block_sum(sq_out, scratch) / float(width) + next_eps);
   if (fits) {
 #pragma unroll
@@ -994,12 +1007,11 @@ xielu_vec8_kernel(const bf16* __restrict__ in, int in_stride, bf16* __restrict__
 }  // namespace
 
 // x, y, out float [n_rows, width] (out may be x); w float [width]. With next_w (float [width]) and next ([n_rows, width] in
-// `next_dtype`) the norm of the new stream rows is written too.
+// `next_dtype`) the norm of the new stream rows is written too; with next alone the new rows themselves in that dtype.
 extern "C" int r2_norm_add(const float* x, const float* y, const float* w, float* out, const float* next_w, void* next,
                            int n_rows, int width, float eps, float next_eps, int next_dtype, cudaStream_t stream) {
   if (n_rows <= 0) return R2_OK;
   if (width < 1) return R2_BAD_SHAPE;
-  if (next != nullptr && next_w == nullptr) return R2_BAD_SHAPE;
   if (next == nullptr || next_dtype == R2_F32) {
     r2_launch(norm_add_kernel<float>, dim3(n_rows), dim3(NORM_ADD_THREADS), size_t(0), stream, x, y, w, out, next_w, (float*)next, width, eps, next_eps);
   } else if (next_dtype == R2_BF16) {
@@ -1112,5 +1124,203 @@ extern "C" int r2_round_rows(const float* x, void* out, long long n, int dtype, 
   } else {
     return R2_BAD_DTYPE;
   }
+  return launch_status();
+}
+
+// ---- norms over whole query and key rows, with the cache write --------------------------------------------------------
+// A row of `buf` holds [q_width query numbers | ...], k_width key numbers from k_col on and the values from v_col on (v_col may
+// be k_col: the values are the keys as projected). Queries and keys are divided by the root mean square of ALL their heads at
+// once and multiplied by a gain per coordinate; queries in place, keys to column k_out_col of the row (< 0: nowhere, or k_col: in
+// place where the values lie elsewhere) and, with `slots`, keys and values to the row's cache slot. One CTA per row.
+namespace {
+template <typename T>
+__global__ void __launch_bounds__(256)
+row_norm_kernel(T* __restrict__ buf, int row_stride, int q_width, int k_col, int k_width, const float* __restrict__ w_q,
+                const float* __restrict__ w_k, float eps, int k_out_col, int v_col, int v_width, T* __restrict__ k_cache,
+                T* __restrict__ v_cache, const int32_t* __restrict__ slots, int head_dim, int v_head_dim, int page_size, int page_shift,
+                long long page_stride, int n_pages) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  T* row = buf + size_t(blockIdx.x) * row_stride;
+  float sq = 0.f, sk = 0.f;
+  for (int d = threadIdx.x; d < q_width; d += blockDim.x) {
+    const float v = to_float(row[d]);
+    sq = fmaf(v, v, sq);
+  }
+  for (int d = threadIdx.x; d < k_width; d += blockDim.x) {
+    const float v = to_float(row[k_col + d]);
+    sk = fmaf(v, v, sk);
+  }
+  const float inv_q = 1.f / sqrtf(block_sum(sq, scratch) / float(q_width) + eps);
+  const float inv_k = 1.f / sqrtf(block_sum(sk, scratch) / float(k_width) + eps);
+  for (int d = threadIdx.x; d < q_width; d += blockDim.x) row[d] = from_float<T>(to_float(row[d]) * inv_q * w_q[d]);
+  size_t k_page = 0;
+  int off = -1;
+  if (slots != nullptr) {
+    const int slot = slots[blockIdx.x];
+    const int page = slot < 0 ? -1 : page_index(slot, page_size, page_shift);
+    if (page > 0 && page < n_pages) {   // (rows of no entry point at the null page: nothing of them is kept)
+      k_page = size_t(page) * page_stride;
+      off = page_offset(slot, page_size, page_shift);
+    }
+  }
+  for (int d = threadIdx.x; d < v_width && off >= 0; d += blockDim.x)   // (before the keys: they may lie in the same columns)
+    v_cache[k_page + (size_t(d / v_head_dim) * page_size + off) * v_head_dim + d % v_head_dim] = row[v_col + d];
+  if (k_out_col == v_col && k_width > 0) __syncthreads();
+  for (int d = threadIdx.x; d < k_width; d += blockDim.x) {
+    const T k = from_float<T>(to_float(row[k_col + d]) * inv_k * w_k[d]);
+    if (k_out_col >= 0) row[k_out_col + d] = k;
+    if (off >= 0) k_cache[k_page + (size_t(d / head_dim) * page_size + off) * head_dim + d % head_dim] = k;
+  }
+}
+
+// The same for bfloat16 rows of up to 8 x 256 numbers a kind whose pieces of eight stay together: one 16-byte load and store each.
+__global__ void __launch_bounds__(256)
+row_norm_vec8_kernel(bf16* __restrict__ buf, int row_stride, int q_width, int k_col, int k_width, const float* __restrict__ w_q,
+                     const float* __restrict__ w_k, float eps, int k_out_col, int v_col, int v_width, bf16* __restrict__ k_cache,
+                     bf16* __restrict__ v_cache, const int32_t* __restrict__ slots, int head_dim, int v_head_dim, int page_size,
+                     int page_shift, long long page_stride, int n_pages) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float part[2][8];
+  bf16* row = buf + size_t(blockIdx.x) * row_stride;
+  const int d = 8 * int(threadIdx.x), lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  const bool has_q = d < q_width, has_k = d < k_width, has_v = d < v_width;
+  const uint4 none = {0u, 0u, 0u, 0u};
+  const uint4 qv = has_q ? *reinterpret_cast<const uint4*>(row + d) : none;
+  const uint4 kv = has_k ? *reinterpret_cast<const uint4*>(row + k_col + d) : none;
+  const uint4 vv = v_col == k_col ? kv : (has_v ? *reinterpret_cast<const uint4*>(row + v_col + d) : none);
+  float qf[8], kf[8], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 a = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&qv)[i]), b = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&kv)[i]);
+    qf[2 * i] = a.x; qf[2 * i + 1] = a.y; kf[2 * i] = b.x; kf[2 * i + 1] = b.y;
+    sq = fmaf(a.x, a.x, fmaf(a.y, a.y, sq));
+    sk = fmaf(b.x, b.x, fmaf(b.y, b.y, sk));
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) {
+    part[0][warp] = sq;
+    part[1][warp] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < n_warps; ++w) {
+    sq += part[0][w];
+    sk += part[1][w];
+  }
+  const float inv_q = 1.f / sqrtf(sq / float(q_width) + eps), inv_k = 1.f / sqrtf(sk / float(k_width) + eps);
+  auto times = [&](const float (&x)[8], float inv, const float* w) {
+    const float4 w0 = *reinterpret_cast<const float4*>(w + d), w1 = *reinterpret_cast<const float4*>(w + d + 4);
+    uint4 out;
+    __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&out);
+    o[0] = __floats2bfloat162_rn(x[0] * inv * w0.x, x[1] * inv * w0.y);
+    o[1] = __floats2bfloat162_rn(x[2] * inv * w0.z, x[3] * inv * w0.w);
+    o[2] = __floats2bfloat162_rn(x[4] * inv * w1.x, x[5] * inv * w1.y);
+    o[3] = __floats2bfloat162_rn(x[6] * inv * w1.z, x[7] * inv * w1.w);
+    return out;
+  };
+  if (has_q) *reinterpret_cast<uint4*>(row + d) = times(qf, inv_q, w_q);
+  size_t page_at = 0;
+  int off = -1;
+  if (slots != nullptr) {
+    const int slot = slots[blockIdx.x];
+    const int page = slot < 0 ? -1 : page_index(slot, page_size, page_shift);
+    if (page > 0 && page < n_pages) {
+      page_at = size_t(page) * page_stride;
+      off = page_offset(slot, page_size, page_shift);
+    }
+  }
+  if (has_k) {
+    const uint4 kn = times(kf, inv_k, w_k);
+    if (k_out_col >= 0) *reinterpret_cast<uint4*>(row + k_out_col + d) = kn;
+    if (off >= 0) *reinterpret_cast<uint4*>(k_cache + page_at + (size_t(d / head_dim) * page_size + off) * head_dim + d % head_dim) = kn;
+  }
+  if (has_v && off >= 0) *reinterpret_cast<uint4*>(v_cache + page_at + (size_t(d / v_head_dim) * page_size + off) * v_head_dim + d % v_head_dim) = vv;
+}
+}  // namespace
+
+extern "C" int r2_row_norm(void* buf, int row_stride, int n_rows, int q_width, int k_col, int k_width, const float* w_q, const float* w_k,
+                           float eps, int k_out_col, int v_col, int v_width, void* k_cache, void* v_cache, const int32_t* slots,
+                           int head_dim, int v_head_dim, int page_size, long long page_stride, int n_pages, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0) return R2_OK;
+  if (q_width < 1 || k_width < 1 || k_col < q_width || (k_out_col >= 0 && k_out_col < q_width)) return R2_BAD_SHAPE;
+  if (k_out_col >= 0 && k_out_col != k_col && k_out_col < k_col + k_width && k_out_col + k_width > k_col) return R2_BAD_SHAPE;
+  if (slots != nullptr && (head_dim < 1 || v_head_dim < 1 || page_size < 1 || k_cache == nullptr || v_cache == nullptr)) return R2_BAD_SHAPE;
+  if (slots == nullptr) v_width = 0, head_dim = v_head_dim = page_size = 1;
+  const int shift = page_shift_of(page_size);
+  const int widest = q_width > k_width ? (q_width > v_width ? q_width : v_width) : (k_width > v_width ? k_width : v_width);
+  const bool pieces = widest <= 2048 && row_stride % 8 == 0 && q_width % 8 == 0 && k_width % 8 == 0 && v_width % 8 == 0 && k_col % 8 == 0 &&
+                      v_col % 8 == 0 && (k_out_col < 0 || k_out_col % 8 == 0) && !(reinterpret_cast<uintptr_t>(buf) & 15) &&
+                      !(reinterpret_cast<uintptr_t>(w_q) & 15) && !(reinterpret_cast<uintptr_t>(w_k) & 15) &&
+                      (slots == nullptr || (head_dim % 8 == 0 && v_head_dim % 8 == 0 && page_stride % 8 == 0 &&
+                                            !(reinterpret_cast<uintptr_t>(k_cache) & 15) && !(reinterpret_cast<uintptr_t>(v_cache) & 15)));
+  if (dtype == R2_BF16 && pieces) {
+    r2_launch(row_norm_vec8_kernel, dim3(n_rows), dim3((widest / 8 + 31) / 32 * 32), size_t(0), stream, (bf16*)buf, row_stride, q_width, k_col,
+              k_width, w_q, w_k, eps, k_out_col, v_col, v_width, (bf16*)k_cache, (bf16*)v_cache, slots, head_dim, v_head_dim, page_size, shift,
+              page_stride, n_pages);
+  } else if (dtype == R2_F32) {
+    r2_launch(row_norm_kernel<float>, dim3(n_rows), dim3(256), size_t(0), stream, (float*)buf, row_stride, q_width, k_col, k_width, w_q, w_k, eps,
+              k_out_col, v_col, v_width, (float*)k_cache, (float*)v_cache, slots, head_dim, v_head_dim, page_size, shift, page_stride, n_pages);
+  } else if (dtype == R2_BF16) {
+    r2_launch(row_norm_kernel<bf16>, dim3(n_rows), dim3(256), size_t(0), stream, (bf16*)buf, row_stride, q_width, k_col, k_width, w_q, w_k, eps,
+              k_out_col, v_col, v_width, (bf16*)k_cache, (bf16*)v_cache, slots, head_dim, v_head_dim, page_size, shift, page_stride, n_pages);
+  } else {
+    return R2_BAD_DTYPE;
+  }
+  return launch_status();
+}
+
+// ---- a token's own row, gated: out[t] = gelu_tanh(gate[t]) * table[ids[t]] ----------------------------------------------
+namespace {
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_token_rows_kernel(const float* __restrict__ gate, int gate_stride, const int32_t* __restrict__ ids, const T* __restrict__ table,
+                        T* __restrict__ out, int n_rows, int dim, int n_table_rows) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long n = (long long)n_rows * dim;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const int t = int(i / dim), d = int(i % dim);
+    int id = ids[t];
+    id = (id < 0 || id >= n_table_rows) ? 0 : id;
+    out[i] = from_float<T>(gelu_tanh(gate[size_t(t) * gate_stride + d]) * to_float(table[size_t(id) * dim + d]));
+  }
+}
+
+__global__ void __launch_bounds__(256)
+soft_cap_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) x[i] = cap * tanhf(x[i] / cap);
+}
+}  // namespace
+
+extern "C" int r2_gated_token_rows(const float* gate, int gate_stride, const int32_t* ids, const void* table, void* out, int n_rows, int dim,
+                                   int n_table_rows, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0) return R2_OK;
+  if (dim < 1 || n_table_rows < 1) return R2_BAD_SHAPE;
+  const long long n = (long long)n_rows * dim;
+  const int blocks = int((n + 255) / 256 > 4096 ? 4096 : (n + 255) / 256);
+  if (dtype == R2_F32) {
+    r2_launch(gated_token_rows_kernel<float>, dim3(blocks), dim3(256), size_t(0), stream, gate, gate_stride, ids, (const float*)table,
+              (float*)out, n_rows, dim, n_table_rows);
+  } else if (dtype == R2_BF16) {
+    r2_launch(gated_token_rows_kernel<bf16>, dim3(blocks), dim3(256), size_t(0), stream, gate, gate_stride, ids, (const bf16*)table,
+              (bf16*)out, n_rows, dim, n_table_rows);
+  } else {
+    return R2_BAD_DTYPE;
+  }
+  return launch_status();
+}
+
+// x <- cap * tanh(x / cap), in place on n contiguous floats (logits).
+extern "C" int r2_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return R2_OK;
+  if (!(cap > 0.f)) return R2_BAD_SHAPE;
+  const int blocks = int((n + 1023) / 1024 > 4096 ? 4096 : (n + 1023) / 1024);
+  r2_launch(soft_cap_kernel, dim3(blocks), dim3(256), size_t(0), stream, x, n, cap);
   return launch_status();
 }

@@ -16,8 +16,9 @@ import torch
 from ..csrc.build import kernel_library
 
 F32, BF16 = 0, 1
-ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF = 0, 1, 2
-ACTIVATIONS = {None: ACT_NONE, "none": ACT_NONE, "gelu_new": ACT_GELU_TANH, "gelu": ACT_GELU_ERF}
+ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF, ACT_TANH = 0, 1, 2, 3
+# ("tanh" is taken by the CUDA-core products: a small matrix inside a gate, never a wide tensor-core product)
+ACTIVATIONS = {None: ACT_NONE, "none": ACT_NONE, "gelu_new": ACT_GELU_TANH, "gelu": ACT_GELU_ERF, "tanh": ACT_TANH}
 
 _STATUS = {-1: "unsupported dtype", -2: "bad shape", -3: "bad alignment", -4: "unsupported size or option"}
 
@@ -491,7 +492,8 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
                out: torch.Tensor | None = None, tail_gate: torch.Tensor | None = None) -> torch.Tensor:
     """The inner activation of gated feed-forwards whose projections lie side by side: a row of `gate_up` [T, 2 F] holds
     the gates of all F columns and then their ups. kind "relu": relu(g) * u. kind "clamped_swish": g' sigmoid(alpha g')
-    (u' + up_offset) with g' = min(g, limit), u' = clamp(u, -limit, limit). kind "silu": g sigmoid(g) * u. With `route` (float32 [T, n_experts], zero
+    (u' + up_offset) with g' = min(g, limit), u' = clamp(u, -limit, limit). kind "silu": g sigmoid(g) * u. kind "gelu_tanh": gelu(g) * u in gelu's
+    tanh form. With `route` (float32 [T, n_experts], zero
     for experts that a row does not use) the first n_experts * expert_width columns are the routed experts', each
     multiplied by the row's weight for its expert; the columns after them belong to an expert that every row uses
     (limit `tail_limit`), multiplied by sigmoid(tail_gate[row]) where `tail_gate` (float32 [T] or [T, 1], the gate's logit)
@@ -499,7 +501,7 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
     _need(gate_up, "gate_up", dim=2)
     if gate_up.shape[1] % 2:
         raise KernelError(f"expert_act: {tuple(gate_up.shape)} does not hold a gate and an up half")
-    kinds = {"clamped_swish": 0, "relu": 1, "silu": 2}
+    kinds = {"clamped_swish": 0, "relu": 1, "silu": 2, "gelu_tanh": 3}
     if kind not in kinds:
         raise KernelError(f"expert_act: unknown kind {kind!r}; known: {sorted(kinds)}")
     inner = gate_up.shape[1] // 2
@@ -525,9 +527,11 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
     return out
 
 
-def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, out: torch.Tensor | None = None,
+                 act: str | None = None) -> torch.Tensor:
     """h [T, K] (any compute dtype) times w [N, K] float32 (+ bias float32) -> float32 [T, N]: the few outputs per row
-    that must stay in 32-bit (gates of a recurrence, one gate per head, step sizes), each one warp's sum."""
+    that must stay in 32-bit (gates of a recurrence, one gate per head, step sizes), each one warp's sum; `act` (see
+    ACTIVATIONS) is applied to them."""
     _need(h, "h", dim=2)
     _need(w, "w", torch.float32, 2)
     if w.shape[1] != h.shape[1] or not w.is_contiguous():
@@ -539,7 +543,7 @@ def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = N
     if out is None:
         out = torch.empty(h.shape[0], w.shape[0], dtype=torch.float32, device=h.device)
     status = _lib("routing").r2_small_linear(_p(h), _rows(h, "h"), _p(w), _p(bias), _p(out), _rows(out, "out"), h.shape[0],
-                                            w.shape[0], h.shape[1], dtype_code(h.dtype), _stream())
+                                            w.shape[0], h.shape[1], ACTIVATIONS[act], dtype_code(h.dtype), _stream())
     _check(status, "small_linear")
     return out
 
@@ -615,10 +619,11 @@ def pair_norm_add(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor, w_a: torch.
 
 
 def norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, next_weight: torch.Tensor | None = None,
-             next_eps: float = 0.0, next_dtype: torch.dtype | None = None):
+             next_eps: float = 0.0, next_dtype: torch.dtype | None = None, rounded_dtype: torch.dtype | None = None):
     """x + y / rms(y) * weight, all float32 [T, D]: a sublayer's output is normalised and joins the stream. With
     `next_weight` the same launch also gives the norm of the new stream rows, rms_norm(x_new) * next_weight in `next_dtype`
-    (the next sublayer's input): -> (x_new, h_next); else -> x_new."""
+    (the next sublayer's input): -> (x_new, h_next); with `rounded_dtype` instead the new rows themselves in that dtype:
+    -> (x_new, rounded); else -> x_new."""
     for name, t in (("x", x), ("y", y)):
         _need(t, name, torch.float32, 2)
         if t.shape != x.shape or not t.is_contiguous():
@@ -633,6 +638,8 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
         if next_weight.shape[0] != x.shape[1]:
             raise KernelError(f"norm_add: next_weight {tuple(next_weight.shape)} does not fit the width {x.shape[1]}")
         nxt = torch.empty(x.shape, dtype=next_dtype or torch.float32, device=x.device)
+    elif rounded_dtype is not None:
+        nxt = torch.empty(x.shape, dtype=rounded_dtype, device=x.device)
     status = _lib("rowwise").r2_norm_add(_p(x), _p(y), _p(weight), _p(out), _p(next_weight), _p(nxt), x.shape[0], x.shape[1],
                                         C.c_float(eps), C.c_float(next_eps), dtype_code(nxt.dtype) if nxt is not None else F32, _stream())
     _check(status, "norm_add")
@@ -864,7 +871,7 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor | None, 
     """silu of a causal convolution per channel: x [T, C] (a slice of a projection), taps float32 [C, n_taps] whose last
     column is the current token's. Inputs before an entry's first row come from the request's state slot (float32
     [slots, floats]; at `conv_state_off` the inputs of the last n_taps - 1 positions, [n_taps - 1, C]), zeros before a
-    sequence's start. The slot is read only: `ssd_scan` renews it. -> [T, C] in x's dtype."""
+    sequence's start. The slot is read only: `ssd_scan` or `delta_scan` renews it. -> [T, C] in x's dtype."""
     _need(x, "x", dim=2)
     _need(taps, "taps", torch.float32, 2)
     _need(state, "state", torch.float32, 2)
@@ -921,8 +928,154 @@ def ssd_scan(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, steps: torch.Ten
     return out
 
 
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, step_bias: torch.Tensor, log_rate: torch.Tensor,
+               q_scale: float, unit_eps: float, state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor,
+               n_heads: int, n_groups: int, dim: int, vdim: int, conv_in: torch.Tensor | None = None, conv_taps: int = 1,
+               conv_state_off: int = 0) -> torch.Tensor:
+    """The gated delta rule for every entry of a batch, from and to the entries' state slots:
+
+        S' = g S, u = beta (v - S'^T k), S = S' + k u^T, o = S^T q
+        q, k made unit vectors (x / sqrt(sum x^2 + unit_eps)), q times q_scale; beta = sigmoid(gates[:, :H]);
+        g = exp(-exp(log_rate) softplus(gates[:, H:] + step_bias))
+
+    q, k [T, groups * dim], v [T, heads * vdim] (slices of a projection; head h uses the q and k of group h // (heads / groups));
+    gates float32 [T, 2 heads]; state float32 [slots, floats]: S [heads, dim, vdim] first, and with `conv_in` the convolution's last
+    inputs at `conv_state_off`, renewed as by `ssd_scan`. -> float32 [T, heads * vdim], the heads' outputs before their norm."""
+    n = _entries(q_start, state_slot, fresh)
+    if n_heads % n_groups:
+        raise KernelError(f"delta_scan: {n_heads} heads do not share {n_groups} groups of queries and keys")
+    for name, t, width in (("q", q, n_groups * dim), ("k", k, n_groups * dim), ("v", v, n_heads * vdim)):
+        _need(t, name, q.dtype, 2)
+        if t.shape[1] != width or t.shape[0] != q.shape[0]:
+            raise KernelError(f"delta_scan: {name} {tuple(t.shape)} is not [T, {width}]")
+    _need(gates, "gates", torch.float32, 2)
+    _need(state, "state", torch.float32, 2)
+    for name, t in (("step_bias", step_bias), ("log_rate", log_rate)):
+        _need(t, name, torch.float32, 1)
+        if t.shape[0] != n_heads:
+            raise KernelError(f"delta_scan: {name} {tuple(t.shape)} is not [{n_heads}]")
+    if gates.shape != (q.shape[0], 2 * n_heads) or state.shape[1] < n_heads * dim * vdim or not state.is_contiguous():
+        raise KernelError(f"delta_scan: gates {tuple(gates.shape)} / state {tuple(state.shape)} do not fit {n_heads} heads of {dim} x {vdim}")
+    channels = 0
+    if conv_in is not None:
+        _need(conv_in, "conv_in", q.dtype, 2)
+        channels = conv_in.shape[1]
+        if conv_state_off < n_heads * dim * vdim or conv_state_off + (conv_taps - 1) * channels > state.shape[1]:
+            raise KernelError("delta_scan: the convolution's state does not fit the slot")
+    out = torch.empty(q.shape[0], n_heads * vdim, dtype=torch.float32, device=q.device)
+    status = _lib("recurrent").r2_delta_scan(
+        _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(gates), _rows(gates, "gates"), _p(step_bias), _p(log_rate),
+        C.c_float(q_scale), C.c_float(unit_eps), _p(state), C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out),
+        _rows(out, "out"), n_heads, n_groups, dim, vdim, _p(conv_in), 0 if conv_in is None else _rows(conv_in, "conv_in"), channels,
+        conv_taps, C.c_longlong(conv_state_off), int(q.shape[0] <= n), dtype_code(q.dtype), _stream())
+    _check(status, "delta_scan")
+    return out
+
+
+def shift_mix(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, row_off: int, row_entry: torch.Tensor, q_start: torch.Tensor,
+              state_slot: torch.Tensor, fresh: torch.Tensor, float_last: bool = False):
+    """Mixes of every row with the row before it in its sequence: h + (h' - h) mu[s]. h [T, D]; mu float32 [n, D]; the row before an
+    entry's first comes from the request's state slot (float32 [slots, floats], at `row_off`; zeros before a sequence's start; the slot
+    is only read: `time_mix_scan` renews it). -> ([T, n, D] in h's dtype, None), or with `float_last` ([T, n - 1, D], the last mix
+    in float32 [T, D])."""
+    _need(h, "h", dim=2)
+    _need(mu, "mu", torch.float32, 2)
+    _need(state, "state", torch.float32, 2)
+    _need(row_entry, "row_entry", torch.int32, 1)
+    _entries(q_start, state_slot, fresh)
+    n, width = mu.shape
+    if width != h.shape[1] or not mu.is_contiguous() or row_off + width > state.shape[1]:
+        raise KernelError(f"shift_mix: h {tuple(h.shape)}, mu {tuple(mu.shape)}, state {tuple(state.shape)} do not fit")
+    n_mixes = n - 1 if float_last else n
+    out = torch.empty(h.shape[0], n_mixes, width, dtype=h.dtype, device=h.device)
+    last = torch.empty(h.shape[0], width, dtype=torch.float32, device=h.device) if float_last else None
+    status = _lib("recurrent").r2_shift_mix(
+        _p(h), _rows(h, "h"), _p(mu), n_mixes, _p(out), _p(last), h.shape[0], width, _p(state), C.c_longlong(state.shape[1]),
+        C.c_longlong(row_off), _p(row_entry), _p(q_start), _p(state_slot), _p(fresh), dtype_code(h.dtype), _stream())
+    _check(status, "shift_mix")
+    return out, last
+
+
+def time_mix_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_log: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor,
+                  q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor, n_heads: int, dim: int,
+                  row_in: torch.Tensor | None = None, row_state_off: int = 0) -> torch.Tensor:
+    """Time mixing with a decay per channel for every entry of a batch, from and to the entries' state slots:
+    o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, S_t = diag(exp(-exp(decay_log_t))) S_(t-1) + k_t v_t^T. r, k, v [T, heads * dim];
+    decay_log float32 [T, heads * dim]; bonus float32 [heads * dim]; state float32 [slots, floats]: S [heads, dim, dim] first, and with
+    `row_in` (this step's input rows [T, D]) the last position's input row at `row_state_off`, which is renewed.
+    -> float32 [T, heads * dim], the heads' outputs before their norm."""
+    n = _entries(q_start, state_slot, fresh)
+    width = n_heads * dim
+    for name, t in (("r", r), ("k", k), ("v", v)):
+        _need(t, name, r.dtype, 2)
+        if t.shape != (r.shape[0], width):
+            raise KernelError(f"time_mix_scan: {name} {tuple(t.shape)} is not [T, {width}]")
+    _need(decay_log, "decay_log", torch.float32, 2)
+    _need(bonus, "bonus", torch.float32)
+    _need(state, "state", torch.float32, 2)
+    if decay_log.shape != r.shape or bonus.numel() != width or not bonus.is_contiguous() or state.shape[1] < width * dim or not state.is_contiguous():
+        raise KernelError(f"time_mix_scan: decay_log {tuple(decay_log.shape)} / bonus {tuple(bonus.shape)} / state {tuple(state.shape)} do not fit {n_heads} heads of {dim}")
+    if row_in is not None:
+        _need(row_in, "row_in", r.dtype, 2)
+        if row_state_off < width * dim or row_state_off + row_in.shape[1] > state.shape[1]:
+            raise KernelError("time_mix_scan: the last input row does not fit the slot")
+    out = torch.empty(r.shape[0], width, dtype=torch.float32, device=r.device)
+    status = _lib("recurrent").r2_time_mix_scan(
+        _p(r), _rows(r, "r"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay_log), _rows(decay_log, "decay_log"), _p(bonus), _p(state),
+        C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out), _rows(out, "out"), n_heads, dim, _p(row_in),
+        0 if row_in is None else _rows(row_in, "row_in"), 0 if row_in is None else row_in.shape[1], C.c_longlong(row_state_off),
+        int(r.shape[0] <= n), dtype_code(r.dtype), _stream())
+    _check(status, "time_mix_scan")
+    return out
+
+
+def row_norm(buf: torch.Tensor, q_width: int, k_width: int, w_q: torch.Tensor, w_k: torch.Tensor, eps: float, k_out_col: int = -1,
+             kv: KvScatter | None = None, head_dim: int = 0) -> None:
+    """RMS norms over the WHOLE query row and the whole key row of a projection [q_width queries | k_width keys | ...] (all heads at
+    once), gains float32 [q_width], [k_width]: queries in place, keys to the row's columns from `k_out_col` on (-1: nowhere). With `kv`
+    (see `kv_scatter`: `col` the first value column, which may be the keys' own, values as they are before the norm; `head_dim` the
+    values' head size) the same launch puts the normed keys (heads of `head_dim`) and the values into the rows' cache slots."""
+    _need(buf, "buf", dim=2)
+    _need(w_q, "w_q", torch.float32, 1)
+    _need(w_k, "w_k", torch.float32, 1)
+    end = max(q_width + k_width, k_out_col + k_width if k_out_col >= 0 else 0, kv.col + kv.width if kv is not None else 0)
+    if w_q.shape[0] != q_width or w_k.shape[0] != k_width or buf.shape[1] < end:
+        raise KernelError(f"row_norm: rows of {buf.shape[1]} do not hold {q_width} queries and {k_width} keys (gains {tuple(w_q.shape)}, {tuple(w_k.shape)})")
+    if kv is not None and (head_dim < 1 or k_width % head_dim or kv.width % kv.head_dim or k_width // head_dim != kv.width // kv.head_dim):
+        raise KernelError("row_norm: the key and value heads do not fit each other")
+    cache = (C.c_void_p(kv.k_cache), C.c_void_p(kv.v_cache), C.c_void_p(kv.slots), head_dim, kv.head_dim, kv.page_size,
+             C.c_longlong(kv.page_stride), kv.n_pages) if kv is not None else (None, None, None, 0, 0, 0, C.c_longlong(0), 0)
+    status = _lib("rowwise").r2_row_norm(_p(buf), _rows(buf, "buf"), buf.shape[0], q_width, q_width, k_width, _p(w_q), _p(w_k), C.c_float(eps),
+                                        k_out_col, kv.col if kv is not None else q_width, kv.width if kv is not None else 0, *cache,
+                                        dtype_code(buf.dtype), _stream())
+    _check(status, "row_norm")
+
+
+def gated_token_rows(gate: torch.Tensor, ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    """gelu(gate[t]) * table[ids[t]] (gelu's tanh form): gate float32 [T, dim], table [rows, dim] -> [T, dim] in the table's dtype."""
+    _need(gate, "gate", torch.float32, 2)
+    _need(ids, "ids", torch.int32, 1)
+    _need(table, "table", dim=2)
+    if table.shape[1] != gate.shape[1] or not table.is_contiguous() or ids.shape[0] != gate.shape[0]:
+        raise KernelError(f"gated_token_rows: gate {tuple(gate.shape)}, ids {tuple(ids.shape)}, table {tuple(table.shape)} do not fit")
+    out = torch.empty(gate.shape, dtype=table.dtype, device=gate.device)
+    status = _lib("rowwise").r2_gated_token_rows(_p(gate), _rows(gate, "gate"), _p(ids), _p(table), _p(out), gate.shape[0], gate.shape[1],
+                                                table.shape[0], dtype_code(table.dtype), _stream())
+    _check(status, "gated_token_rows")
+    return out
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap * tanh(x / cap), in place, of contiguous float32 numbers (logits)."""
+    _need(x, "x", torch.float32)
+    if not x.is_contiguous() or cap <= 0:
+        raise KernelError("soft_cap: x must be contiguous and the cap positive")
+    _check(_lib("rowwise").r2_soft_cap(_p(x), C.c_longlong(x.numel()), C.c_float(cap), _stream()), "soft_cap")
+    return x
+
+
 def group_norm_gated(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor | None, n_groups: int, eps: float, gate_first,
-                     out_dtype: torch.dtype) -> torch.Tensor:
+                     out_dtype: torch.dtype, out: torch.Tensor | None = None) -> torch.Tensor:
     """RMS norm of float32 rows y [T, C] in n_groups equal parts, each by its own root mean square, times weight [C], with
     a gate [T, C] (a slice of a projection, in out_dtype): `gate_first`: y * silu(gate) is what is normalised; else the
     normalised, weighted result is multiplied by sigmoid(gate), or, with gate_first "silu_after", by silu(gate). `weight` None:
@@ -934,7 +1087,11 @@ def group_norm_gated(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor |
     if gate.shape != y.shape or (weight is not None and weight.shape[0] != y.shape[1]) or y.shape[1] % n_groups:
         raise KernelError(f"group_norm_gated: y {tuple(y.shape)}, gate {tuple(gate.shape)}, weight "
                           f"{None if weight is None else tuple(weight.shape)}, {n_groups} groups")
-    out = torch.empty(y.shape[0], y.shape[1], dtype=out_dtype, device=y.device)
+    if out is None:
+        out = torch.empty(y.shape[0], y.shape[1], dtype=out_dtype, device=y.device)
+    _need(out, "out", out_dtype, 2)
+    if out.shape != y.shape:
+        raise KernelError(f"group_norm_gated: out {tuple(out.shape)} is not {tuple(y.shape)}")
     status = _lib("recurrent").r2_group_norm_gated(
         _p(y), _rows(y, "y"), _p(gate), _rows(gate, "gate"), _p(weight), _p(out), _rows(out, "out"), y.shape[0], n_groups,
         y.shape[1] // n_groups, C.c_float(eps), 2 if gate_first == "silu_after" else int(bool(gate_first)), dtype_code(out_dtype), _stream())
@@ -1077,6 +1234,21 @@ def linear(a, w: torch.Tensor, bias: torch.Tensor | None = None, *, w_is_nk: boo
     return out
 
 
+def grouped_linear(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """Several products whose inputs lie side by side: a [T, n, K], w [n * N, K] (stored [out, in], the groups' matrices one after the
+    other) -> [T, n * N] whose columns s * N .. (s + 1) * N - 1 are a[:, s] @ w[s * N: (s + 1) * N]^T, in a's dtype."""
+    _need(a, "a", dim=3)
+    t, n, k = a.shape
+    if not a.is_contiguous() or w.shape[0] % n or w.shape[1] != k:
+        raise KernelError(f"grouped_linear: a {tuple(a.shape)} does not fit w {tuple(w.shape)}")
+    per = w.shape[0] // n
+    out = torch.empty(t, n * per, dtype=a.dtype, device=a.device)
+    flat = a.view(t, n * k)
+    for s in range(n):
+        linear(flat[:, s * k: (s + 1) * k], w[s * per: (s + 1) * per], None, w_is_nk=True, out=out[:, s * per: (s + 1) * per])
+    return out
+
+
 def _linear_kv(a: torch.Tensor, w: torch.Tensor, bias, w_is_nk: bool, out, kv: KvScatter):
     """The fused q/k/v product with keys and values written to the cache by the epilogue; None
     where the tensor-core kernel does not take the case."""
@@ -1122,6 +1294,16 @@ def kv_write(k_src: torch.Tensor, v_src: torch.Tensor, k_cache: torch.Tensor, v_
     _check(status, "kv_write")
 
 
+def _bias_len(dist_bias: torch.Tensor | None, n_heads: int) -> int:
+    """Entries per head of a bias by distance (0: none)."""
+    if dist_bias is None:
+        return 0
+    _need(dist_bias, "dist_bias", torch.float32, 2)
+    if dist_bias.shape[0] != n_heads or dist_bias.shape[1] < 1 or not dist_bias.is_contiguous():
+        raise KernelError(f"attention: dist_bias {tuple(dist_bias.shape)} is not [{n_heads}, distances]")
+    return dist_bias.shape[1]
+
+
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_stride: int, page_size: int,
                     n_pages: int, block_tables: torch.Tensor, row_entry: torch.Tensor, positions: torch.Tensor,
                     seq_lens: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
@@ -1129,7 +1311,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     max_context: int = 0, q_start: torch.Tensor | None = None, n_tiles: int = 0, v_head_dim: int = 0,
                     keep_first: int = 0, sink: bool = False, gate: torch.Tensor | None = None, softcap: float = 0.0,
                     sinks: torch.Tensor | None = None, head_gate: torch.Tensor | None = None,
-                    values_in_keys: bool = False) -> torch.Tensor:
+                    values_in_keys: bool = False, chunk: int = 0, dist_bias: torch.Tensor | None = None,
+                    out_scale: float = 1.0) -> torch.Tensor:
     """Causal attention of q [T, n_heads * head_dim] over the paged cache -> [T, n_heads * v_head_dim]
     (`v_head_dim` 0: the keys' head size). With a window, `keep_first` keeps a sequence's first keys visible;
     `sink` adds one to the softmax's denominator (an extra exp(0) term: the weights sum to less than one); `gate`
@@ -1140,6 +1323,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     `values_in_keys`: the cache holds key rows only and a key's first v_head_dim numbers are its value (a cache of
     latents; `v_cache` is not read); the general kernel takes it, and for bfloat16 with one key head and `q_start` the
     latent kernel, whose tiles hold all heads of a few tokens (it takes `sinks` as well).
+    `chunk` > 0 (without a window) limits a row at position p to the keys of its own chunk, [p // chunk * chunk, p]; `dist_bias`
+    (float32 [n_heads, n]) is added to the (scaled, capped) score of a key d positions back: column d, the last column for every
+    larger d; `out_scale` multiplies the output: taken by the general kernel, the mma.sync prefill kernel and the fused decode kernel.
     `decode_only` says that every row is an entry of its own (one new token each) and
     `max_context` bounds the rows' context lengths; `q_start` (int32 [R + 1]) with `n_tiles`, the
     sum over entries of ceil(rows / 64), lets the tensor-core prefill kernel take the batch. They
@@ -1168,7 +1354,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     # only the general kernel takes a value head size of its own or a head size that is no multiple of 16; kept
     # first keys, a sink and an output gate are taken by both prefill kernels and the fused decode kernel
     fits = v_head_dim == head_dim and head_dim % 16 == 0 and not values_in_keys
-    capped = softcap != 0.0 or sinks is not None or head_gate is not None   # what the tcgen05 kernel does not take
+    biased = chunk > 0 or dist_bias is not None or out_scale != 1.0
+    bias_len = _bias_len(dist_bias, n_heads)
+    capped = softcap != 0.0 or sinks is not None or head_gate is not None or biased   # what the tcgen05 kernel does not take
     head_gate_stride = 0
     if sinks is not None:
         _need(sinks, "sinks", torch.float32, 1)
@@ -1216,17 +1404,17 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0 and (gate is None or (gate_stride % 2 == 0 and gate.data_ptr() % 4 == 0))):
         _need(q_start, "q_start", torch.int32, 1)
         lib = _lib_for_head_dim("attention_prefill", head_dim)
-        status = lib.r2_attention_prefill_capped(
+        status = lib.r2_attention_prefill_biased(
             _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _p(k_cache), _p(v_cache), C.c_longlong(page_stride),
             page_size, n_pages, _p(block_tables), block_tables.shape[1], _p(q_start), _p(seq_lens),
             q_start.shape[0] - 1, n_tiles, n_heads, n_kv_heads, C.c_float(scale), window, _p(_workspace(q.device).error),
             keep_first, int(bool(sink)), _p(gate), gate_stride, int(_exact_weights and not plain), C.c_float(softcap), _p(sinks),
-            _p(head_gate), head_gate_stride, _stream())
+            _p(head_gate), head_gate_stride, chunk, _p(dist_bias), bias_len, C.c_float(out_scale), _stream())
         _check(status, "paged_attention (prefill)")
         _used("attention_prefill")
         return out
     if (values_in_keys and n_kv_heads == 1 and q.dtype == torch.bfloat16 and _fast_attention and q_start is not None and keep_first == 0
-            and not sink and gate is None and softcap == 0.0 and head_gate is None and head_dim <= 256 and v_head_dim <= head_dim):
+            and not sink and gate is None and softcap == 0.0 and head_gate is None and not biased and head_dim <= 256 and v_head_dim <= head_dim):
         # a cache of latents: every head reads the same rows, so a tile's rows are (token, head) pairs (mma.sync)
         _need(q_start, "q_start", torch.int32, 1)
         single_rows = decode_only and n == q_start.shape[0] - 1
@@ -1251,7 +1439,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         page_size, _p(block_tables), block_tables.shape[1], _p(row_entry), _p(positions), _p(seq_lens), n, n_heads,
         n_kv_heads, head_dim, v_head_dim, C.c_float(scale), window, keep_first, int(bool(sink)), _p(gate), gate_stride,
         n_pages, dtype_code(q.dtype), C.c_float(softcap), _p(sinks), _p(head_gate), head_gate_stride,
-        head_dim if values_in_keys else 0, _stream())
+        head_dim if values_in_keys else 0, chunk, _p(dist_bias), bias_len, C.c_float(out_scale), _stream())
     _check(status, "paged_attention")
     _used("attention_simt")
     return out
@@ -1263,13 +1451,15 @@ def decode_attention_fused(q: torch.Tensor, k_new: torch.Tensor | None, v_new: t
                            seq_lens: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                            window: int, max_context: int, keep_first: int = 0, sink: bool = False,
                            gate: torch.Tensor | None = None, exact_weights: bool = False, softcap: float = 0.0,
-                           sinks: torch.Tensor | None = None, head_gate: torch.Tensor | None = None) -> torch.Tensor | None:
+                           sinks: torch.Tensor | None = None, head_gate: torch.Tensor | None = None, chunk: int = 0,
+                           dist_bias: torch.Tensor | None = None, out_scale: float = 1.0,
+                           out: torch.Tensor | None = None) -> torch.Tensor | None:
     """Decode attention in ONE launch for a batch in which every row is an entry of its own: the
     kernel writes the new keys and values to their cache slots, and the slice that finishes last
     merges all slices of its row. Returns None when it does not take the case (the caller then writes
     the cache and calls `paged_attention`). With `k_new` None nothing is written: the rows read a cache that already holds
     their own position (a layer that reads the keys and values another layer wrote in this step).
-    `keep_first`, `sink`, `gate`, `softcap`, `sinks` and `head_gate` as in `paged_attention`;
+    `keep_first`, `sink`, `gate`, `softcap`, `sinks`, `head_gate`, `chunk`, `dist_bias` and `out_scale` as in `paged_attention`;
     `exact_weights` carries the softmax's weights into the second product as two bfloat16 terms."""
     group = n_heads // max(n_kv_heads, 1)
     if not (_fast_attention and _fused_decode and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16
@@ -1290,6 +1480,9 @@ def decode_attention_fused(q: torch.Tensor, k_new: torch.Tensor | None, v_new: t
         v_new = slot_mapping = None
     if window > 0:
         max_context = min(max_context, window + keep_first)   # what a row reads at most
+    elif chunk > 0:
+        max_context = min(max_context, chunk)
+    bias_len = _bias_len(dist_bias, n_heads)
     slices = decode_slices(n, n_kv_heads, max_context, q.device)
     lib = _lib_for_head_dim("attention_decode", head_dim)
     ws = _workspace(q.device)
@@ -1312,13 +1505,18 @@ def decode_attention_fused(q: torch.Tensor, k_new: torch.Tensor | None, v_new: t
         if head_gate.shape != (n, n_heads):
             raise KernelError(f"decode attention: head_gate {tuple(head_gate.shape)} is not [T, {n_heads}]")
         head_gate_stride = _rows(head_gate, "head_gate")
-    out = torch.empty(n, n_heads * head_dim, dtype=q.dtype, device=q.device)
-    status = lib.r2_attention_decode_fused_capped(
+    if out is None:
+        out = torch.empty(n, n_heads * head_dim, dtype=q.dtype, device=q.device)
+    _need(out, "out", q.dtype, 2)
+    if out.shape != (n, n_heads * head_dim):
+        raise KernelError(f"decode attention: out {tuple(out.shape)} is not [T, {n_heads} * {head_dim}]")
+    status = lib.r2_attention_decode_fused_biased(
         _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _p(k_cache), _p(v_cache), C.c_longlong(page_stride), page_size,
         n_pages, _p(block_tables), block_tables.shape[1], _p(row_entry), _p(positions), _p(seq_lens), n, n_heads,
         n_kv_heads, C.c_float(scale), window, slices, _p(k_new), _p(v_new), stride, _p(slot_mapping), _p(ws.floats),
         C.c_longlong(ws.floats.numel()), _p(ws.counters), ws.counters.numel(), keep_first, int(bool(sink)), _p(gate),
-        gate_stride, int(bool(exact_weights)), C.c_float(softcap), _p(sinks), _p(head_gate), head_gate_stride, _stream())
+        gate_stride, int(bool(exact_weights)), C.c_float(softcap), _p(sinks), _p(head_gate), head_gate_stride, chunk, _p(dist_bias), bias_len,
+        C.c_float(out_scale), _stream())
     if status == -4:
         return None
     _check(status, "decode attention (fused)")

@@ -43,6 +43,7 @@ class ModelSpec:
     final_norm: PartSpec
     schedule: tuple[ScheduleEntry, ...] = field(default=())
     embedding_scale: float = 1.0  # token table rows are multiplied by it
+    logit_softcap: float = 0.0  # > 0: logits are softcap * tanh(logits / softcap)
 
 
 def default_schedule(layers, mixers) -> tuple[ScheduleEntry, ...]:
@@ -73,6 +74,8 @@ class DecoderModel:
             block_cls = registry("block")[layer.block]
             post = {name: build_part("norm", spec, tensors, rt) for name, spec in
                     (("post_norm_1", layer.post_norm_1), ("post_norm_2", layer.post_norm_2)) if spec is not None}
+            if layer.token_side is not None:
+                post["token_side"] = build_part("token_side", layer.token_side, tensors, rt)
             self.blocks.append(block_cls(
                 build_part("norm", layer.norm_1, tensors, rt), mixer,
                 build_part("norm", layer.norm_2, tensors, rt) if layer.norm_2 is not None else None,
@@ -81,7 +84,7 @@ class DecoderModel:
         mixers = [b.mixer for b in self.blocks]
         self.schedule = spec.schedule or default_schedule(spec.layers, mixers)
         head_table = self.embedding.table if spec.head == spec.embedding else tensors[spec.head].to(rt.device, rt.dtype)
-        self.head = Head(build_part("norm", spec.final_norm, tensors, rt), head_table, rt.dtype)
+        self.head = Head(build_part("norm", spec.final_norm, tensors, rt), head_table, rt.dtype, spec.logit_softcap)
         self.cache_members, self.state_members = self._members(mixers)
         self._resident = None   # the one-kernel form of a decode step's layers, built at its first use
         self._resident_tried = False
@@ -143,8 +146,13 @@ class DecoderModel:
         add(self.embedding.table if self.head.table.data_ptr() != self.embedding.table.data_ptr() else None)
         add(self.head.table)
         for obj in [self.head.norm] + [p for b in self.blocks for p in (b.norm_1, b.mixer, b.norm_2, b.feed_forward,
-                                                                      getattr(b, "post_norm_1", None), getattr(b, "post_norm_2", None))]:
-            for v in (vars(obj).values() if obj is not None else ()):
-                if isinstance(v, torch.Tensor):
+                                                                      getattr(b, "post_norm_1", None), getattr(b, "post_norm_2", None),
+                                                                      getattr(b, "token_side", None))]:
+            for name, v in (vars(obj).items() if obj is not None else ()):
+                if isinstance(v, torch.Tensor) and name not in getattr(obj, "gathered", ()):
                     add(v)
+            for part in getattr(obj, "sides", ()):   # two mixers side by side
+                for v in vars(part).values():
+                    if isinstance(v, torch.Tensor):
+                        add(v)
         return total

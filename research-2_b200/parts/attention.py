@@ -9,6 +9,8 @@ output projection, whose epilogue adds the residual stream.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..kernels import ops
@@ -432,3 +434,130 @@ class LatentAttention:
 
     def forward(self, h, residual, ctx, cache, state=None, writes_cache: bool = True):
         return ops.linear(self._inner(h, ctx, cache, writes_cache), self.w_out, None, w_is_nk=True, residual=residual)
+
+
+def distance_buckets(n_distances: int, n_buckets: int, bias_max: int) -> list[int]:
+    """The row of a bias table of n_buckets rows for a key 0, 1, .., n_distances - 1 positions back: the first half of the rows are
+    distances of their own, the others divide the distances from there to bias_max into equal steps of the logarithm, and
+    everything farther has the last row."""
+    half = n_buckets // 2
+    if half < 1 or bias_max <= half:
+        raise ValueError(f"attention: {n_buckets} rows of bias do not reach to a distance of {bias_max}")
+    out = []
+    for n in range(n_distances):
+        if n < half:
+            out.append(n)
+        else:
+            out.append(min(n_buckets - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (n_buckets - half))))
+    return out
+
+
+@register_mixer("distance_bias_attention")
+class DistanceBiasAttention:
+    """Grouped causal attention over the paged cache whose scores get a learned bias by distance, with one RMS norm over the whole
+    query row and one over the whole key row. Positions enter only through the bias and the mask. Each chosen by a parameter or by
+    what the weights hold: chunks, a learned sink per head, biases on the projections, keys that are the values too.
+
+        q, k <- rms_norm over ALL heads at once, gains q_norm [H head_dim], k_norm [G head_dim]
+        s = (q . k) * scale + rel[bucket(i - j), head]          (buckets: `distance_buckets`)
+        position i sees the keys j <= i of its own chunk, i // chunk = j // chunk      (chunk 0: every key up to i)
+        weights = exp(s) / (sum over seen keys of exp(s) + exp(sink[head]))            (the sink has no key and no value)
+
+    Without `w_v` the values are the keys as projected, before their norm. Keys are cached after their norm. The bias table is spread
+    over distances once, when the layer is made. Norms, scores, bias, softmax and sink are computed in float32.
+
+    params: n_heads, n_kv_heads, head_dim, v_head_dim, scale, chunk, bias_max, qk_norm_eps, out_scale (default 1: a factor on the heads'
+    outputs, in float32 before they are rounded).
+    weights (matrices stored [out, in]): w_q [H head_dim, D], w_k [G head_dim, D], q_norm, k_norm, rel [buckets, H], w_out
+    [D, H v_head_dim]; optionally w_v [G v_head_dim, D], b_q, b_k, b_v, sink [H]."""
+
+    def __init__(self, params: dict, weights: dict, rt: Runtime):
+        self.n_heads, self.n_kv_heads = int(params["n_heads"]), int(params["n_kv_heads"])
+        self.head_dim, self.v_head_dim = int(params["head_dim"]), int(params["v_head_dim"])
+        self.scale, self.chunk = float(params["scale"]), int(params.get("chunk", 0))
+        self.norm_eps, self.out_scale = float(params["qk_norm_eps"]), float(params.get("out_scale", 1.0))
+        if self.n_heads % self.n_kv_heads != 0:
+            raise ValueError(f"attention: n_heads {self.n_heads} is not a multiple of n_kv_heads {self.n_kv_heads}")
+        if not (1 <= self.head_dim <= 1024 and 1 <= self.v_head_dim <= 1024):
+            raise ValueError(f"attention: head sizes lie in 1 .. 1024, got {self.head_dim} and {self.v_head_dim}")
+        self.q_width, self.k_width = self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim
+        self.v_width, self.inner_width = self.n_kv_heads * self.v_head_dim, self.n_heads * self.v_head_dim
+        self.own_values = weights.get("w_v") is not None
+        if not self.own_values and self.v_head_dim != self.head_dim:
+            raise ValueError(f"attention: values that are the keys have the keys' head size ({self.head_dim}), not {self.v_head_dim}")
+        stacked = [weights["w_q"], weights["w_k"]] + ([weights["w_v"]] if self.own_values else [])
+        want = [self.q_width, self.k_width, self.v_width][: len(stacked)]
+        if [w.shape[0] for w in stacked] != want or weights["w_out"].shape[1] != self.inner_width:
+            raise ValueError(f"attention: projections of {[tuple(w.shape) for w in stacked]} and an output of "
+                             f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads, {self.n_kv_heads} kv heads "
+                             f"of {self.head_dim} (values {self.v_head_dim})")
+        self.w_in = matrix(torch.cat(stacked, dim=0), rt)
+        biases = [weights.get(n) for n in ("b_q", "b_k", "b_v")[: len(stacked)]]
+        self.b_in = None
+        if any(b is not None for b in biases):
+            self.b_in = vector(torch.cat([torch.zeros(n) if b is None else b.to(torch.float32) for b, n in zip(biases, want)]), rt)
+        self.w_out = matrix(weights["w_out"], rt)
+        self.q_norm, self.k_norm = vector(weights["q_norm"], rt), vector(weights["k_norm"], rt)
+        self.sinks = vector(weights["sink"], rt) if weights.get("sink") is not None else None
+        rel = weights["rel"]
+        if rel.dim() != 2 or rel.shape[1] != self.n_heads:
+            raise ValueError(f"attention: a bias table {tuple(rel.shape)} does not fit {self.n_heads} heads")
+        # head h's bias for a key n positions back; beyond the last column it does not change (or no key is seen)
+        reach = int(params["bias_max"]) + 1
+        rows = distance_buckets(min(reach, self.chunk) if self.chunk > 0 else reach, rel.shape[0], int(params["bias_max"]))
+        self.dist_bias = vector(rel.to(torch.float32)[torch.tensor(rows)].T.contiguous(), rt)
+
+    def matrices(self):
+        return [self.w_in, self.w_out]
+
+    @property
+    def cache_spec(self) -> MemberSpec:
+        return MemberSpec(self.n_kv_heads, self.head_dim, 0, self.v_head_dim, 0, chunk=self.chunk)
+
+    state_spec = None
+    capturable = True
+
+    def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None):
+        """The heads' outputs [T, H v_head_dim] before w_out (into `out` where given)."""
+        if not writes_cache:
+            raise ValueError("attention: a layer with keys and values of its own writes them")
+        at = self.q_width + self.k_width
+        fused_decode = ctx.decode_only and self.v_head_dim == self.head_dim and self.head_dim <= 256
+        if self.own_values or not fused_decode:
+            proj = ops.linear(h, self.w_in, self.b_in, w_is_nk=True)
+            k_col = self.q_width
+        else:   # room for the normed keys beside the keys as projected, which are the values
+            proj = torch.empty(h.shape[0], at + self.k_width, dtype=h.dtype, device=h.device)
+            ops.linear(h, self.w_in, self.b_in, w_is_nk=True, out=proj[:, :at])
+            k_col = at
+        v_col = at if self.own_values else self.q_width
+        attend = dict(chunk=self.chunk, dist_bias=self.dist_bias, sinks=self.sinks, out_scale=self.out_scale, out=out)
+        if fused_decode:
+            ops.row_norm(proj, self.q_width, self.k_width, self.q_norm, self.k_norm, self.norm_eps, k_out_col=k_col)
+            q, k, v = proj[:, : self.q_width], proj[:, k_col: k_col + self.k_width], proj[:, v_col: v_col + self.v_width]
+            mixed = ops.decode_attention_fused(
+                q, k, v, ctx.slot_mapping[cache.group], cache.k, cache.v, cache.page_stride, cache.page_size, cache.n_pages,
+                ctx.block_tables[cache.group], ctx.row_entry, ctx.positions, ctx.seq_lens, self.n_heads, self.n_kv_heads, self.head_dim,
+                self.scale, 0, ctx.max_context, exact_weights=ops.exact_weights(), **attend)
+            if mixed is not None:
+                return mixed
+            ops.kv_write(k, v, cache.k, cache.v, ctx.slot_mapping[cache.group], self.n_kv_heads, self.head_dim,
+                         cache.page_size, cache.page_stride, cache.n_pages, v_head_dim=self.v_head_dim)
+        else:
+            # the norms' launch also puts the normed keys and the values into the rows' cache slots
+            scatter = ops.kv_scatter(ctx.slot_mapping[cache.group], cache.k, cache.v, cache.page_stride, cache.page_size,
+                                     cache.n_pages, v_col, self.v_width, self.v_head_dim)
+            ops.row_norm(proj, self.q_width, self.k_width, self.q_norm, self.k_norm, self.norm_eps, kv=scatter, head_dim=self.head_dim)
+            q = proj[:, : self.q_width]
+        return ops.paged_attention(
+            q, cache.k, cache.v, cache.page_stride, cache.page_size, cache.n_pages, ctx.block_tables[cache.group],
+            ctx.row_entry, ctx.positions, ctx.seq_lens, self.n_heads, self.n_kv_heads, self.head_dim, self.scale,
+            0, decode_only=ctx.decode_only, max_context=ctx.max_context, q_start=ctx.q_start,
+            n_tiles=ctx.n_attention_tiles, v_head_dim=self.v_head_dim, **attend)
+
+    def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
+        """The mixer's output [T, D] in float32, without the residual stream."""
+        return ops.linear(self.inner(h, ctx, cache, state, writes_cache), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
+
+    def forward(self, h, residual, ctx, cache, state=None, writes_cache: bool = True):
+        return ops.linear(self.inner(h, ctx, cache, state, writes_cache), self.w_out, None, w_is_nk=True, residual=residual)

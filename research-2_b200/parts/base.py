@@ -1,6 +1,6 @@
 """What a layer is made of, and how a part is found by its kind.
 
-A model is put together from five kinds of part, each of which takes its sizes and constants
+A model is put together from six kinds of part, each of which takes its sizes and constants
 as parameters and knows nothing about the model it is in:
 
   mixer          mixes information across positions; may keep a per-token cache (keys and
@@ -9,6 +9,7 @@ as parameters and knows nothing about the model it is in:
   norm           normalises rows
   positions      tells the model where a token is: added to the embedding, or applied to
                  queries and keys inside a mixer
+  token_side     adds something made from the token's own row of a table to the stream at a layer's end
   block          arranges norms, a mixer and a feed-forward around the residual stream
 
 Interfaces (duck-typed; `parts/attention.py`, `mlp.py`, `norm.py`, `positions.py`, `block.py`
@@ -21,6 +22,7 @@ are the GPT-2 ones):
   Norm.forward(x, out_dtype, rows=None)            -> normalised rows in out_dtype
   Positions.additive_table() -> Tensor | None      rows added to the token embedding
   Positions.rotate(q, k, ctx)                      in-place change of queries and keys (or no-op)
+  TokenSide.join(x, h, ctx, rounded_dtype)         -> (new x, its rows in rounded_dtype)
   Block.forward(x, ctx, cache, state, writes_cache) -> x
 
 The residual stream `x` is float32 in every mode; `h` has the compute dtype. Each kind has a
@@ -39,7 +41,7 @@ from ..cache.arena import MemberSpec
 
 __all__ = [
     "LayerSpec", "MemberSpec", "PartSpec", "Runtime", "StateSpec", "build_part", "register_block",
-    "register_feed_forward", "register_mixer", "register_norm", "register_positions", "registry",
+    "register_feed_forward", "register_mixer", "register_norm", "register_positions", "register_token_side", "registry",
 ]
 
 
@@ -73,11 +75,12 @@ class LayerSpec:
     norm_2: PartSpec | None = None  # None: an arrangement with one norm
     post_norm_1: PartSpec | None = None  # arrangements with a norm after each sublayer as well
     post_norm_2: PartSpec | None = None
+    token_side: PartSpec | None = None  # what joins the stream at the layer's end (arrangements that allow it)
     block_params: dict = field(default_factory=dict)  # constants of the arrangement itself (a factor on the stream, ...)
 
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Any]]] = {
-    "mixer": {}, "feed_forward": {}, "norm": {}, "positions": {}, "block": {},
+    "mixer": {}, "feed_forward": {}, "norm": {}, "positions": {}, "token_side": {}, "block": {},
 }
 
 
@@ -107,6 +110,10 @@ def register_norm(kind: str):
 
 def register_positions(kind: str):
     return _register("positions", kind)
+
+
+def register_token_side(kind: str):
+    return _register("token_side", kind)
 
 
 def register_block(kind: str):

@@ -121,12 +121,13 @@ class PostNormBlock:
     the stream itself (in the compute dtype) and hand over their output in float32 without it (`mix`); one launch scales the
     stream, adds the output, normalises the sum and writes the new rows twice: in float32 (the stream) and in the compute
     dtype (what the next sublayer's products read). The norms are RMS norms (`gain`, `eps`). A layer may have no feed-forward
-    (None; then no norm_2). `alpha` is the factor on the stream inside the sums.
+    (None; then no norm_2). `alpha` is the factor on the stream inside the sums. A layer may end with a `token_side` part, which adds
+    to the normalised stream what it makes from it and from the token's own row of a table.
 
     The compute-dtype copy of the rows that this block returns travels to the next block in `ctx.stream_rounded` as the pair
     (stream tensor, its copy); a block that is handed another tensor (the embedding's rows) makes the copy itself."""
 
-    def __init__(self, norm_1, mixer, norm_2, feed_forward, compute_dtype, alpha: float = 1.0):
+    def __init__(self, norm_1, mixer, norm_2, feed_forward, compute_dtype, alpha: float = 1.0, token_side=None):
         if feed_forward is not None and norm_2 is None:
             raise ValueError("a post-norm block needs a norm after every sublayer that it has")
         for part, what in ((mixer, "mixer"), (feed_forward, "feed-forward")):
@@ -136,7 +137,7 @@ class PostNormBlock:
             if norm is not None and not hasattr(norm, "gain"):
                 raise ValueError("a post-norm block's norms must be RMS norms")
         self.norm_1, self.mixer, self.norm_2, self.feed_forward = norm_1, mixer, norm_2, feed_forward
-        self.compute_dtype, self.alpha = compute_dtype, float(alpha)
+        self.compute_dtype, self.alpha, self.token_side = compute_dtype, float(alpha), token_side
         self.rounds = compute_dtype != torch.float32
 
     def _read(self, x, ctx):
@@ -159,5 +160,7 @@ class PostNormBlock:
         x, h = self._join(x, self.mixer.mix(h, ctx, cache, state, writes_cache), self.norm_1)
         if self.feed_forward is not None:
             x, h = self._join(x, self.feed_forward.mix(h, ctx), self.norm_2)
+        if self.token_side is not None:
+            x, h = self.token_side.join(x, h, ctx, self.compute_dtype if self.rounds else None)
         ctx.stream_rounded = (x, h)
         return x

@@ -25,12 +25,13 @@ class TokenEmbedding:
 
 
 class Head:
-    """logits[i] = norm(x[rows[i]]) @ table^T, float32."""
+    """logits[i] = norm(x[rows[i]]) @ table^T, float32; with `softcap` > 0 then softcap * tanh(logits / softcap)."""
 
-    def __init__(self, norm, table: torch.Tensor, compute_dtype: torch.dtype):
-        self.norm, self.table, self.compute_dtype = norm, table, compute_dtype
+    def __init__(self, norm, table: torch.Tensor, compute_dtype: torch.dtype, softcap: float = 0.0):
+        self.norm, self.table, self.compute_dtype, self.softcap = norm, table, compute_dtype, float(softcap)
 
     def forward(self, x, rows):
         lazy = getattr(self.norm, "can_be_lazy", False)
         last = self.norm.forward(x, self.compute_dtype, rows=rows, lazy=True) if lazy else self.norm.forward(x, self.compute_dtype, rows=rows)
-        return ops.linear(last, self.table, None, w_is_nk=True, out_dtype=torch.float32)
+        logits = ops.linear(last, self.table, None, w_is_nk=True, out_dtype=torch.float32)
+        return ops.soft_cap(logits, self.softcap) if self.softcap > 0.0 else logits

@@ -112,14 +112,21 @@ def _softplus(x: float) -> float:
 
 @register_feed_forward("gated_mlp")
 class GatedMLP:
-    """W_down (act(W_gate h) * (W_up h)) with act = relu. params: activation ("relu"). weights: w_gate [F, D], w_up
-    [F, D], w_down [D, F], stored [out, in], no biases. The two input projections run as one product."""
+    """W_down (act(W_gate h) * (W_up h)). params: activation ("relu", "silu" or "gelu_tanh"). weights: w_gate [F, D], w_up
+    [F, D], w_down [D, F], stored [out, in], and either no biases or all three: b_gate [F], b_up [F], b_down [D]. The two input
+    projections run as one product."""
 
     def __init__(self, params: dict, weights: dict, rt: Runtime):
         self.activation = params.get("activation", "relu")
-        if self.activation != "relu":
+        if self.activation not in ("relu", "silu", "gelu_tanh"):
             raise ValueError(f"gated feed-forward: unknown activation {self.activation!r}")
         gate, up, down = weights["w_gate"], weights["w_up"], weights["w_down"]
+        self.b_gate_up = self.b_down = None
+        if any(weights.get(n) is not None for n in ("b_gate", "b_up", "b_down")):
+            self.b_gate_up = vector(torch.cat([weights["b_gate"], weights["b_up"]]), rt)
+            self.b_down = vector(weights["b_down"], rt)
+            if self.b_gate_up.shape[0] != 2 * gate.shape[0] or self.b_down.shape[0] != down.shape[0]:
+                raise ValueError(f"gated feed-forward: biases {tuple(self.b_gate_up.shape)} and {tuple(self.b_down.shape)} do not fit")
         if gate.shape != up.shape or down.shape != (gate.shape[1], gate.shape[0]):
             raise ValueError(f"gated feed-forward: w_gate {tuple(gate.shape)}, w_up {tuple(up.shape)} and w_down {tuple(down.shape)} do not fit")
         self.w_gate_up = matrix(torch.cat([gate, up], dim=0), rt)
@@ -128,9 +135,15 @@ class GatedMLP:
     def matrices(self):
         return [self.w_gate_up, self.w_down]
 
+    def _inner(self, h):
+        return ops.expert_act(ops.linear(h, self.w_gate_up, self.b_gate_up, w_is_nk=True), self.activation)
+
+    def mix(self, h, ctx):
+        """The feed-forward's output [T, D] in float32, without the residual stream."""
+        return ops.linear(self._inner(h), self.w_down, self.b_down, w_is_nk=True, out_dtype=torch.float32)
+
     def forward(self, h, residual, ctx):
-        y = ops.expert_act(ops.linear(h, self.w_gate_up, None, w_is_nk=True), self.activation)
-        return ops.linear(y, self.w_down, None, w_is_nk=True, residual=residual)
+        return ops.linear(self._inner(h), self.w_down, self.b_down, w_is_nk=True, residual=residual)
 
 
 @register_feed_forward("routed_experts")

@@ -1,10 +1,11 @@
 """Mixers that carry a state of fixed size per request instead of a cache that grows with the sequence:
-a matrix memory with exponential gates (mLSTM), retention (linear attention with a fixed decay per head) and a
-state-space layer with a short causal convolution (the recurrence of Mamba-2). Their state lives in 32-bit floats in the request's state slot, starts at
+a matrix memory with exponential gates (mLSTM), retention (linear attention with a fixed decay per head), a
+state-space layer with a short causal convolution (the recurrence of Mamba-2), the gated delta rule behind short convolutions
+and time mixing with a decay per channel (RWKV's). Their state lives in 32-bit floats in the request's state slot, starts at
 zero with a sequence's first token and is carried from step to step; prompts, portions and single decoded
 tokens run through the same kernels (csrc/kernels/recurrent.cu), entry by entry, row by row.
 
-Both offer `mix(h, ctx, cache, state)`, the mixer's output [T, D] in float32 without the residual stream,
+All offer `mix(h, ctx, cache, state)`, the mixer's output [T, D] in float32 without the residual stream,
 for an arrangement that joins several mixers, beside the usual `forward`, whose last product adds the stream.
 """
 
@@ -200,31 +201,157 @@ class StateSpace:
         return ops.linear(self._inner(h, ctx, state), self.w_out, None, w_is_nk=True, residual=residual)
 
 
-@register_mixer("side_by_side")
-class SideBySide:
-    """Two mixers read the same input; each one's output is RMS-normed over the model width with a plain gain of its
-    own, and `share` times their sum joins the stream: x + share (norm(left(h)) w_left + norm(right(h)) w_right).
+@register_mixer("delta")
+class DeltaRule:
+    """The gated delta rule: a matrix per head that every row first lets decay, then asks for what it holds under the row's key, and
+    then corrects by a share of what is missing. Per head (head i uses the queries and keys of group i // (heads / groups)):
 
-    params: left, right: {"kind": mixer kind, "params": {...}}; eps; share (default 0.5).
-    weights: left_out, right_out [D], and each mixer's own weights under the prefixes "left." and "right.".
-    Either mixer may keep a per-token cache and either a per-request state, but only one of each."""
+        q, k, v = silu(conv(W_q h)), silu(conv(W_k h)), silu(conv(W_v h))     (a causal convolution per channel, last tap the current row)
+        q, k made unit vectors, x / sqrt(sum x^2 + unit_eps); q times head_dim^-1/2
+        beta = sigmoid(W_b h), g = exp(-exp(a_log) softplus(W_a h + dt_bias))
+        S' = g S, u = beta (v - S'^T k), S = S' + k u^T, o = S^T q            (S: [head_dim x v_head_dim], from zero)
+
+    Each head's o is divided by its root mean square, times `norm` [v_head_dim] (shared by the heads), times silu(W_g h); then W_o. The
+    state is S and the convolutions' last conv_taps - 1 inputs. The convolutions' outputs have the compute dtype; everything after
+    them is float32.
+
+    params: n_heads, n_groups, head_dim, v_head_dim, conv_taps, unit_eps, norm_eps.
+    weights (stored [out, in], no biases): w_q, w_k [groups head_dim, D], w_v, w_gate [H v_head_dim, D], w_out [D, H v_head_dim], conv_q,
+    conv_k [groups head_dim, taps], conv_v [H v_head_dim, taps], w_b, w_a [H, D], a_log, dt_bias [H], norm [v_head_dim].
+    The four wide projections run as one product, the strengths and step sizes as a 32-bit one, the three convolutions as one launch."""
 
     def __init__(self, params: dict, weights: dict, rt: Runtime):
+        self.n_heads, self.n_groups = int(params["n_heads"]), int(params["n_groups"])
+        self.head_dim, self.v_head_dim, self.conv_taps = int(params["head_dim"]), int(params["v_head_dim"]), int(params["conv_taps"])
+        self.unit_eps, self.norm_eps = float(params["unit_eps"]), float(params["norm_eps"])
+        self.qk_width, self.v_width = self.n_groups * self.head_dim, self.n_heads * self.v_head_dim
+        stacked = [weights["w_q"], weights["w_k"], weights["w_v"], weights["w_gate"]]
+        convs = [weights["conv_q"], weights["conv_k"], weights["conv_v"]]
+        if (self.n_heads % self.n_groups or [w.shape[0] for w in stacked] != [self.qk_width, self.qk_width, self.v_width, self.v_width]
+                or [tuple(c.shape) for c in convs] != [(n, self.conv_taps) for n in (self.qk_width, self.qk_width, self.v_width)]
+                or weights["w_out"].shape[1] != self.v_width or weights["norm"].shape[0] != self.v_head_dim):
+            raise ValueError(f"delta rule: projections {[tuple(w.shape) for w in stacked]}, convolutions {[tuple(c.shape) for c in convs]} and an output of "
+                             f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads, {self.n_groups} groups of {self.head_dim} x {self.v_head_dim}")
+        self.w_in = matrix(torch.cat(stacked, dim=0), rt)
+        self.w_out = matrix(weights["w_out"], rt)
+        self.conv = vector(torch.cat(convs, dim=0), rt)
+        self.channels = self.conv.shape[0]
+        self.w_gates = vector(torch.cat([weights["w_b"], weights["w_a"]], dim=0), rt)   # float32: they enter the recurrence
+        self.a_log, self.dt_bias = vector(weights["a_log"], rt), vector(weights["dt_bias"], rt)
+        self.norm = vector(weights["norm"].repeat(self.n_heads), rt)
+        self.conv_state_off = self.n_heads * self.head_dim * self.v_head_dim
+
+    cache_spec = None
+    capturable = True
+
+    def matrices(self):
+        return [self.w_in, self.w_out]
+
+    @property
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.conv_state_off + (self.conv_taps - 1) * self.channels,), torch.float32)
+
+    def _inner(self, h, ctx, state):
+        proj = ops.linear(h, self.w_in, None, w_is_nk=True)
+        gates = ops.small_linear(h, self.w_gates, None)
+        raw = proj[:, : self.channels]
+        mixed = ops.causal_conv(raw, self.conv, None, state, self.conv_state_off, ctx.row_entry, ctx.q_start, ctx.state_slot, ctx.fresh)
+        a, b = self.qk_width, 2 * self.qk_width
+        o = ops.delta_scan(mixed[:, :a], mixed[:, a:b], mixed[:, b:], gates, self.dt_bias, self.a_log, self.head_dim ** -0.5, self.unit_eps,
+                           state, ctx.q_start, ctx.state_slot, ctx.fresh, self.n_heads, self.n_groups, self.head_dim, self.v_head_dim,
+                           conv_in=raw, conv_taps=self.conv_taps, conv_state_off=self.conv_state_off)
+        return ops.group_norm_gated(o, proj[:, self.channels:], self.norm, self.n_heads, self.norm_eps, "silu_after", proj.dtype)
+
+    def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self._inner(h, ctx, state), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
+
+    def forward(self, h, residual, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self._inner(h, ctx, state), self.w_out, None, w_is_nk=True, residual=residual)
+
+
+@register_mixer("time_mix")
+class TimeMix:
+    """Time mixing with a decay per channel that depends on the input. h' is the row before h in its sequence (zeros before the first);
+    each of r, k, v, g and w reads a mix of its own, mix_s = h + (h' - h) mu_s:
+
+        r, k, v = W_r mix_r, W_k mix_k, W_v mix_v (heads of head_dim); gate = silu(W_g mix_g)
+        w = exp(-exp(W_w2 tanh(W_w1 mix_w) + w0))                                   (per head and key channel)
+        o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T     (S from zero)
+
+    Each head's o is divided by its root mean square, the heads are concatenated, times `norm`, times the gate; then W_o. The state is S
+    and the last row h. The way to the decays (mix_w, both small products, the exponentials) is float32 throughout.
+
+    params: n_heads, head_dim, norm_eps, out_scale (default 1: a factor on the gated outputs, folded into the norm's gains).
+    weights (stored [out, in], no biases): w_r, w_k, w_v, w_gate [H head_dim, D], mu_r, mu_k, mu_v, mu_g, mu_w [D], w1 [rank, D], w2 [H head_dim,
+    rank], w0 [H head_dim], bonus [H, head_dim], norm [H head_dim], w_out [D, H head_dim]."""
+
+    def __init__(self, params: dict, weights: dict, rt: Runtime):
+        self.n_heads, self.head_dim, self.norm_eps = int(params["n_heads"]), int(params["head_dim"]), float(params["norm_eps"])
+        self.inner_width = self.n_heads * self.head_dim
+        stacked = [weights[n] for n in ("w_r", "w_k", "w_v", "w_gate")]
+        self.width = stacked[0].shape[1]
+        w1, w2 = weights["w1"], weights["w2"]
+        if (any(tuple(w.shape) != (self.inner_width, self.width) for w in stacked) or w1.shape[1] != self.width or w1.shape[0] != w2.shape[1]
+                or w2.shape[0] != self.inner_width or weights["w_out"].shape[1] != self.inner_width or weights["bonus"].numel() != self.inner_width):
+            raise ValueError(f"time mixing: projections {[tuple(w.shape) for w in stacked]}, decay {tuple(w1.shape)} and {tuple(w2.shape)} and an output of "
+                             f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads of {self.head_dim}")
+        self.w_in = matrix(torch.cat(stacked, dim=0), rt)      # [4 H head_dim, D], the rows of each kind read a mix of their own
+        self.w_out = matrix(weights["w_out"], rt)
+        self.mu = vector(torch.stack([weights["mu_" + s] for s in "rkvgw"]), rt)
+        self.w1, self.w2, self.w0 = vector(w1, rt), vector(w2, rt), vector(weights["w0"], rt)
+        self.bonus = vector(weights["bonus"].reshape(-1), rt)
+        self.norm = vector(weights["norm"], rt) * float(params.get("out_scale", 1.0))
+        self.row_state_off = self.inner_width * self.head_dim
+
+    cache_spec = None
+    capturable = True
+
+    def matrices(self):
+        return [self.w_in, self.w_out]
+
+    @property
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.row_state_off + self.width,), torch.float32)
+
+    def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None):
+        """The gated heads' outputs [T, H head_dim] before w_out (into `out` where given)."""
+        mixes, mix_w = ops.shift_mix(h, self.mu, state, self.row_state_off, ctx.row_entry, ctx.q_start, ctx.state_slot, ctx.fresh, float_last=True)
+        n = self.inner_width
+        proj = ops.grouped_linear(mixes, self.w_in)
+        if h.dtype == torch.bfloat16 and h.shape[0] <= 64:   # a warp per output; many rows share the matrices in tiles
+            low = ops.small_linear(mix_w, self.w1, None, act="tanh")
+            decay_log = ops.small_linear(low, self.w2, self.w0)
+        else:
+            low = ops.linear(mix_w, self.w1, None, w_is_nk=True, act="tanh")
+            decay_log = ops.linear(low, self.w2, self.w0, w_is_nk=True)
+        o = ops.time_mix_scan(proj[:, :n], proj[:, n: 2 * n], proj[:, 2 * n: 3 * n], decay_log, self.bonus, state, ctx.q_start, ctx.state_slot,
+                              ctx.fresh, self.n_heads, self.head_dim, row_in=h, row_state_off=self.row_state_off)
+        return ops.group_norm_gated(o, proj[:, 3 * n:], self.norm, self.n_heads, self.norm_eps, "silu_after", proj.dtype, out=out)
+
+    def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self.inner(h, ctx, cache, state), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
+
+    def forward(self, h, residual, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self.inner(h, ctx, cache, state), self.w_out, None, w_is_nk=True, residual=residual)
+
+
+class _TwoMixers:
+    """Two mixers that read the same input; either may keep a per-token cache and either a per-request state, but only one of each."""
+
+    def _make_sides(self, params: dict, weights: dict, rt: Runtime, ask: str, extra=({}, {})):
         from .base import registry
 
-        self.eps, self.share = float(params["eps"]), float(params.get("share", 0.5))
         self.sides = []
-        for side in ("left", "right"):
+        for side, more in zip(("left", "right"), extra):
             spec = params[side]
             own = {name[len(side) + 1:]: t for name, t in weights.items() if name.startswith(side + ".")}
-            part = registry("mixer")[spec["kind"]](spec["params"], own, rt)
-            if not hasattr(part, "mix"):
-                raise ValueError(f"side_by_side: a mixer of kind {spec['kind']!r} has no `mix` (its output without the stream)")
+            part = registry("mixer")[spec["kind"]]({**spec["params"], **more}, own, rt)
+            if not hasattr(part, ask):
+                raise ValueError(f"two mixers side by side: a mixer of kind {spec['kind']!r} has no `{ask}` (its output without the stream)")
             self.sides.append(part)
-        self.w_left, self.w_right = vector(weights["left_out"], rt), vector(weights["right_out"], rt)
         for what in ("cache_spec", "state_spec"):
             if sum(getattr(p, what, None) is not None for p in self.sides) > 1:
-                raise ValueError(f"side_by_side: both mixers have a {what}; a layer has one cache member and one state member")
+                raise ValueError(f"two mixers side by side: both have a {what}; a layer has one cache member and one state member")
         self.capturable = all(getattr(p, "capturable", False) for p in self.sides)
 
     def _of(self, what):
@@ -237,6 +364,55 @@ class SideBySide:
     @property
     def state_spec(self):
         return self._of("state_spec")
+
+
+@register_mixer("side_by_side_sum")
+class SideBySideSum(_TwoMixers):
+    """left_scale left(h) + right_scale right(h): two mixers read the same input and their scaled outputs are summed. Each mixer hands over
+    what it has before its last product (`inner`, with its scale inside, in float32 before it is rounded), side by side in
+    one buffer, and ONE product over both output matrices makes the sum.
+
+    params: left, right: {"kind": mixer kind, "params": {...}} (mixers that take `out_scale` and offer `inner`); left_scale, right_scale.
+    weights: each mixer's own under the prefixes "left." and "right."."""
+
+    def __init__(self, params: dict, weights: dict, rt: Runtime):
+        self._make_sides(params, weights, rt, "inner", ({"out_scale": float(params["left_scale"])}, {"out_scale": float(params["right_scale"])}))
+        self.w_out = torch.cat([p.w_out for p in self.sides], dim=1).contiguous()
+        at = 0
+        for p in self.sides:   # the parts keep views into the joint matrix
+            p.w_out, at = self.w_out[:, at: at + p.inner_width], at + p.inner_width
+
+    def matrices(self):
+        return [self.sides[0].w_in, self.sides[1].w_in, self.w_out]
+
+    def _inner(self, h, ctx, cache, state, writes_cache):
+        both = torch.empty(h.shape[0], self.w_out.shape[1], dtype=h.dtype, device=h.device)
+        at = 0
+        for p in self.sides:
+            p.inner(h, ctx, cache, state, writes_cache, out=both[:, at: at + p.inner_width])
+            at += p.inner_width
+        return both
+
+    def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self._inner(h, ctx, cache, state, writes_cache), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
+
+    def forward(self, h, residual, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self._inner(h, ctx, cache, state, writes_cache), self.w_out, None, w_is_nk=True, residual=residual)
+
+
+@register_mixer("side_by_side")
+class SideBySide(_TwoMixers):
+    """Two mixers read the same input; each one's output is RMS-normed over the model width with a plain gain of its
+    own, and `share` times their sum joins the stream: x + share (norm(left(h)) w_left + norm(right(h)) w_right).
+
+    params: left, right: {"kind": mixer kind, "params": {...}}; eps; share (default 0.5).
+    weights: left_out, right_out [D], and each mixer's own weights under the prefixes "left." and "right.".
+    Either mixer may keep a per-token cache and either a per-request state, but only one of each."""
+
+    def __init__(self, params: dict, weights: dict, rt: Runtime):
+        self.eps, self.share = float(params["eps"]), float(params.get("share", 0.5))
+        self._make_sides(params, weights, rt, "mix")
+        self.w_left, self.w_right = vector(weights["left_out"], rt), vector(weights["right_out"], rt)
 
     def matrices(self):
         return [m for p in self.sides for m in p.matrices()]

@@ -34,8 +34,11 @@ class WeightError(ValueError):
 
 @dataclass(frozen=True)
 class TensorSpec:
+    """A size in `shape` is a number, or a name for one that the configuration leaves to the checkpoint: any size does, the same
+    wherever the name stands."""
+
     name: str
-    shape: tuple[int, ...]
+    shape: tuple[int | str, ...]
     integer: bool = False
 
 
@@ -49,12 +52,25 @@ class WeightSpec:
     tied: tuple[tuple[str, str], ...] = field(default=())
 
 
+def _fits(have: tuple[int, ...], want: tuple, sizes: dict[str, int]) -> bool:
+    """Whether a tensor has the shape that a spec asks for; names not met before take the size that they find here."""
+    if len(have) != len(want) or any(not isinstance(w, str) and w != h for h, w in zip(have, want)):
+        return False
+    found = dict(sizes)
+    for h, w in zip(have, want):
+        if isinstance(w, str) and found.setdefault(w, h) != h:
+            return False
+    sizes.update(found)
+    return True
+
+
 def check_and_select(found: dict[str, torch.Tensor], spec: WeightSpec, where: str = "checkpoint") -> dict[str, torch.Tensor]:
     """Pick the spec's tensors out of `found` (bare names in the result) or raise WeightError."""
     missing: list[str] = []
     wrong: list[str] = []
     used: set[str] = set()
     out: dict[str, torch.Tensor] = {}
+    sizes: dict[str, int] = {}   # what the named sizes turned out to be
     for ts in spec.tensors:
         spellings = [p + ts.name for p in spec.prefixes]
         key = next((s for s in spellings if s in found), None)
@@ -63,8 +79,9 @@ def check_and_select(found: dict[str, torch.Tensor], spec: WeightSpec, where: st
             continue
         used.add(key)
         tensor = found[key]
-        if tuple(tensor.shape) != tuple(ts.shape):
-            wrong.append(f"{key}: expected shape {tuple(ts.shape)}, got {tuple(tensor.shape)}")
+        if not _fits(tuple(tensor.shape), ts.shape, sizes):
+            expected = tuple(sizes.get(d, d) if isinstance(d, str) else d for d in ts.shape)
+            wrong.append(f"{key}: expected shape {expected}, got {tuple(tensor.shape)}")
             continue
         if ts.integer:
             if tensor.dtype not in INT_DTYPES:
