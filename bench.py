@@ -21,7 +21,8 @@ A "step" is one decode step. The default run decodes a batch of 8 requests whose
 
 `--design bosenex` prints the same points for a Bosenex model beside a Zirunex model of equal layer sizes, and the
 design's kernels one by one; `--design zudalorn` a Zudalorn model beside a Bosenex model of equal layer sizes, likewise;
-`--design pidodra` a Pidodra model beside a Zudalorn model of equal layer sizes whose layers are all latent attention. `--design zirunex` prints, instead, the same decode and prefill points for Zirunex models with the layer sizes
+`--design pidodra` a Pidodra model beside a Zudalorn model of equal layer sizes whose layers are all latent attention;
+`--design lagelorn` a Lagelorn model beside a Bosenex model of equal layer sizes with dense feed-forwards. `--design zirunex` prints, instead, the same decode and prefill points for Zirunex models with the layer sizes
 of `--model` beside GPT-2's, and the design's kernels one by one beside their likes.
 
 `--model gpt2-355M` and `--model gpt2-1.5B` run the same at those sizes (the 1.5B decode workload has
@@ -236,6 +237,8 @@ class DecodeLoop:
         total = 0.0
         for m in model.cache_members:   # a member with a window reads its window and its kept first tokens only
             seen = min(ctx, m.window + m.keep_first) if m.window > 0 else ctx
+            if m.chunk > 0:                 # one with chunks, the keys of the position's own chunk
+                seen = sum((PROMPT_LEN + first_step + i) % m.chunk + 1 for i in range(n)) / n
             total += m.n_kv_heads * (m.head_dim + m.value_dim) * size * seen
         return self.batch * total
 
@@ -286,6 +289,8 @@ def prefill_point(model, cfg, pk: dict) -> dict:
         flops = zudalorn_flops(cfg, n_req, length)
     elif type(cfg).__name__ == "PidodraConfig":
         flops = pidodra_flops(cfg, n_req, length)
+    elif type(cfg).__name__ == "LagelornConfig":
+        flops = lagelorn_flops(cfg, n_req, length)
     else:
         flops = gated_design_flops(cfg, n_req, length)
     return {"value": t / (ms / 1e3), "tokens": t, "ms": ms, "frac": flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12)}
@@ -318,7 +323,7 @@ def gated_design_flops(cfg, n_req: int, length: int) -> float:
     return total + 2 * n_req * cfg.width * cfg.vocab_size
 
 
-def build_gated_design(data: dict, dtype: str = "bfloat16"):
+def build_gated_design(data: dict, dtype: str = "bfloat16", **init_options):
     import torch
     from research_2_b200 import models  # noqa: F401
     from research_2_b200.config.registry import architecture_of
@@ -327,7 +332,7 @@ def build_gated_design(data: dict, dtype: str = "bfloat16"):
 
     arch = architecture_of(data)
     cfg = arch.parse_config(data)
-    tensors = {k: v.to(torch.bfloat16) for k, v in arch.random_weights(cfg, SEED, std=0.02).items()}
+    tensors = {k: v.to(torch.bfloat16) for k, v in arch.random_weights(cfg, SEED, std=0.02, **init_options).items()}
     return arch.build(cfg, tensors, Runtime(torch.device("cuda:0"), compute_dtype(dtype))), cfg
 
 
@@ -965,6 +970,237 @@ def pidodra_points(args, pk: dict) -> dict:
     return out
 
 
+def half_heads_for(h: int) -> int:
+    """The largest divisor of h up to h / 2: the delta rule's heads of queries and keys."""
+    return max(k for k in range(1, max(1, h // 2) + 1) if h % k == 0)
+
+
+def lagelorn_config(size: str, n_layer: int) -> dict:
+    """A Lagelorn configuration with the width, heads, head size, layers and vocabulary of a GPT-2 size, laid out like the Bosenex
+    configuration beside it: of every three layers two are the gated delta rule (as many value heads as the size has heads, half as
+    many of queries and keys) and one is attention by chunks of 256 (four query heads a key head) beside time mixing; the feed-forward's
+    inner width is the dense Bosenex layer's; 64 numbers per token and layer from the side table."""
+    g = SIZES[size]
+    d, h = g["n_embd"], g["n_head"]
+    hd = d // h
+    ff = max(128, round(2 * g["n_inner"] / 3 / 128) * 128)
+    delta = {"heads": h, "kv_heads": half_heads_for(h), "dim": hd, "vdim": hd, "conv": 4}
+    pair = {"left": {"heads": h, "kv_heads": kv_heads_for(h), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "bias_max": 128, "mask": {"size": 256}},
+            "left_scale": 1.2, "right": {"heads": h, "dim": hd}, "right_scale": 0.8}
+    layers = [{"type": "parallel" if i % 3 == 2 else "delta", "mixer": pair if i % 3 == 2 else delta, "mlp": {"kind": "dense", "ff": ff}}
+              for i in range(n_layer)]
+    return {"architecture": "Lagelorn", "vocab": g["vocab_size"], "width": d, "norm": {"eps": 1e-5}, "max_positions": CONTEXT, "postln_alpha": 2.0,
+            "token_side": {"dim": 64}, "logit_softcap": 30.0, "layers": layers}
+
+
+def bosenex_dense_config(size: str, n_layer: int) -> dict:
+    """The closest of the other models at equal layer sizes: the Bosenex configuration with its dense feed-forward in every layer."""
+    data = bosenex_config(size, n_layer)
+    dense = next(layer["mlp"] for layer in data["layers"] if layer["mlp"]["kind"] == "dense")
+    for layer in data["layers"]:
+        layer["mlp"] = dense
+    return data
+
+
+def lagelorn_flops(cfg, n_req: int, length: int) -> float:
+    """Flops that one prefill step of n_req prompts of `length` tokens NEEDS in a Lagelorn configuration: products with the weights,
+    the recurrences, and the attention's seen pairs (the side input's and the decays' small matrices counted as products)."""
+    from research_2_b200.config.lagelorn import DeltaMixer
+
+    t, d, total = n_req * length, cfg.width, 0.0
+    for layer in cfg.layers:
+        m = layer.mixer
+        if isinstance(m, DeltaMixer):
+            qk, v = m.kv_heads * m.dim, m.heads * m.vdim
+            total += 2 * t * d * (2 * qk + 2 * v + 2 * m.heads) + 2 * t * v * d + t * m.heads * 8 * m.dim * m.vdim
+        else:
+            a, r = m.left, m.right
+            q, k, n = a.heads * a.dim, a.kv_heads * a.dim, r.heads * r.dim
+            total += 2 * t * d * (q + k) + 2 * t * q * d + n_req * 4 * q * sum(i % (a.chunk or length) + 1 for i in range(length))
+            total += 2 * t * d * 4 * n + 2 * t * n * d + t * r.heads * 6 * r.dim * r.dim + 2 * t * DECAY_RANK * (d + n)
+        if layer.mlp is not None:
+            total += 2 * t * d * 3 * layer.mlp.ff
+        total += 4 * t * d * cfg.side_dim
+    return total + 2 * n_req * d * cfg.vocab_size
+
+
+DECAY_RANK = 64   # inner width of the decays' two small matrices in a Lagelorn model here
+
+
+def lagelorn_points(args, pk: dict) -> dict:
+    """`--design lagelorn`: prefill and decode throughput of a Lagelorn model with the layer sizes of `--model`, beside a Bosenex
+    model of that size with dense feed-forwards (the closest of the other models: recurrences with a state per request, and attention
+    beside a recurrence in one layer) through the same loops, and the design's kernels one by one beside their likes."""
+    import torch
+    from research_2_b200.kernels import ops
+    from research_2_b200.profiling import kernel_cases
+
+    g = SIZES[args.model]
+    d, h = g["n_embd"], g["n_head"]
+    hd = d // h
+    variants = {"bosenex, dense feed-forwards": bosenex_dense_config(args.model, args.layers), "lagelorn": lagelorn_config(args.model, args.layers)}
+    out = {"design": "lagelorn", "sizes_of": args.model, "layers": args.layers, "prompt_len": PROMPT_LEN, "models": {}}
+    for name, data in variants.items():
+        model, cfg = build_gated_design(data, **({"bias_rows": 32, "decay_rank": DECAY_RANK} if name == "lagelorn" else {}))
+        point = {}
+        for batch in (8, 64):
+            steps = min(args.steps, 96)
+            value, ms, loop, kv_bytes = decode_point(model, batch, steps, args.warmup)
+            state_bytes = 2 * batch * sum(4 * int(torch.tensor(spec.shape).prod()) for spec in model.state_members)   # read and written
+            achieved = (model.weight_bytes_per_step() + kv_bytes + state_bytes) / (ms / 1e3) / 1e9
+            point[f"decode_b{batch}"] = {"tokens/s": round(value), "ms_per_step": round(ms, 4), "kernels_per_step": loop.graph.kernels,
+                                         "hbm_frac": round(achieved / pk["hbm_gbs"], 3)}
+            del loop
+            torch.cuda.empty_cache()
+        pre = prefill_point(model, cfg, pk)
+        point["prefill_2x1024"] = {"tokens/s": round(pre["value"]), "ms": round(pre["ms"], 3), "bf16_frac": round(pre["frac"], 3)}
+        out["models"][name] = point
+        del model
+        torch.cuda.empty_cache()
+
+    # the design's kernels one by one, at a prompt step (2 x 1,024 rows) and at decode steps (8 and 64 rows at position 1,023)
+    table = {}
+
+    def add(name, fn, n_bytes=0, flops=0):
+        us = kernel_cases.time_in_graph(fn)
+        entry = {"us": round(us, 2)}
+        if n_bytes:
+            entry.update(frac=round(n_bytes / us / 1e3 / pk["hbm_gbs"], 3), of="copy bandwidth")
+        if flops:
+            entry.update(flops_frac=round(flops / us / 1e6 / pk["bf16_tflops"], 4))
+        table[name] = entry
+
+    dev, bf = "cuda:0", torch.bfloat16
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)  # noqa: E731
+    page, length, chunk = PAGE, 1024, 256
+    for label, n_entries, rows_each in (("2 x 1,024 rows", 2, 1024), ("8 decoded rows", 8, 1), ("64 decoded rows", 64, 1)):
+        t = n_entries * rows_each
+        q_start = i32([i * rows_each for i in range(n_entries + 1)])
+        slots, fresh = i32(list(range(n_entries))), i32([0] * n_entries)
+        row_entry = i32([e for e in range(n_entries) for _ in range(rows_each)])
+        positions = i32([length - 1 if rows_each == 1 else p for _ in range(n_entries) for p in range(rows_each)])
+        seq_lens = i32([length] * n_entries)
+        slot_map = i32([e * length + p for e, p in zip(row_entry.tolist(), positions.tolist())])
+        x32, y32 = torch.randn(t, d, device=dev), torch.randn(t, d, device=dev)
+        hrow = torch.randn(t, d, device=dev).to(bf)
+        gain = torch.ones(d, device=dev)
+        # the delta rule beside the matrix memory and the state-space layer
+        kvh, taps = half_heads_for(h), 4
+        channels = 2 * kvh * hd + d
+        raw = torch.randn(t, channels + d, device=dev).to(bf)
+        conv_w, conv_b = torch.randn(channels, taps, device=dev) * 0.3, torch.zeros(channels, device=dev)
+        off = h * hd * hd
+        state = torch.zeros(n_entries, off + (taps - 1) * channels, device=dev)
+        gates, per_head, w_gates = torch.randn(t, 2 * h, device=dev), torch.zeros(h, device=dev), torch.randn(2 * h, d, device=dev) * 0.02
+        prepare = lambda: ops.delta_prepare(raw[:, :channels], hrow, conv_w, w_gates, per_head, per_head, hd ** -0.5, 1e-6, h, kvh, hd, hd, state, off,  # noqa: E731
+                                            row_entry, q_start, slots, fresh)
+        qk_f, v_f, numbers = prepare()
+        add(f"delta rule: convolutions + silu of {channels:,} channels, unit vectors, strengths and decays, {label}", prepare,
+            n_bytes=t * (channels * 6 + d * 2 + h * 16) + w_gates.numel() * 4)
+        add(f"its like: convolution + silu alone, {channels:,} channels (Bosenex), {label}",
+            lambda: ops.causal_conv(raw[:, :channels], conv_w, conv_b, state, off, row_entry, q_start, slots, fresh), n_bytes=t * channels * 4)
+        add(f"its like: gates in 32-bit alone, {2 * h} outputs (Bosenex), {label}", lambda: ops.small_linear(hrow, w_gates, None), n_bytes=t * d * 2 + w_gates.numel() * 4)
+        add(f"delta rule: recurrence, {h} heads of {hd} x {hd}, {label}",
+            lambda: ops.delta_scan(qk_f, v_f, numbers, hd, state, q_start, slots, fresh, conv_in=raw[:, :channels], conv_taps=taps, conv_state_off=off),
+            n_bytes=t * (channels * 4 + h * 16 + d * 4) + 2 * state.numel() * 4)
+        dk = hd // 2
+        proj = torch.randn(t, 2 * h * dk + 2 * d, device=dev).to(bf)
+        mstate = torch.zeros(n_entries, h * ops.mlstm_state_floats(dk, hd), device=dev)
+        add(f"its like: matrix memory's recurrence, {h} heads of {dk} x {hd} (Bosenex), {label}",
+            lambda: ops.mlstm_scan(proj[:, : h * dk], proj[:, h * dk: 2 * h * dk], proj[:, 2 * h * dk: 2 * h * dk + d], gates, 15.0, dk ** -0.5,
+                                   mstate, q_start, slots, fresh, h, dk, hd), n_bytes=t * (2 * h * dk + d) * 2 + t * d * 4 + 2 * mstate.numel() * 4)
+        sh, n_state = 2 * h, 64
+        inner = sh * hd
+        xbc = torch.randn(t, inner + 2 * n_state, device=dev).to(bf)
+        soff = sh * n_state * hd
+        sstate = torch.zeros(n_entries, soff + (taps - 1) * xbc.shape[1], device=dev)
+        steps_in, sper_head = torch.randn(t, sh, device=dev), torch.zeros(sh, device=dev)
+        add(f"its like: state-space recurrence, {sh} heads of {n_state} x {hd} (Bosenex), {label}",
+            lambda: ops.ssd_scan(xbc[:, :inner], xbc[:, inner: inner + n_state], xbc[:, inner + n_state:], steps_in, sper_head, sper_head, sper_head,
+                                 sstate, q_start, slots, fresh, sh, 1, n_state, hd, conv_in=xbc, conv_taps=taps, conv_state_off=soff),
+            n_bytes=t * xbc.shape[1] * 2 + t * inner * 4 + 2 * sstate.numel() * 4)
+        # time mixing
+        toff = h * hd * hd
+        tstate = torch.zeros(n_entries, toff + d, device=dev)
+        mu = torch.rand(5, d, device=dev)
+        w1, w2t, w0 = torch.randn(DECAY_RANK, d, device=dev) * 0.02, torch.randn(DECAY_RANK, d, device=dev) * 0.1, torch.zeros(d, device=dev)
+        prepare = lambda: ops.time_mix_prepare(hrow, mu, w1, w2t, w0, tstate, toff, row_entry, q_start, slots, fresh)  # noqa: E731
+        mixes, decay = prepare()
+        add(f"time mixing: a row's mixes with the row before it, decays through an inner width of {DECAY_RANK} in 32-bit, {label}", prepare,
+            n_bytes=t * d * (2 + 8 + 4) + 8 * d * DECAY_RANK)
+        w_in = (torch.randn(4 * d, d, device=dev) * 0.02).to(bf)
+        add(f"time mixing: four products of {d} x {d} on their mixes, {label}", lambda: ops.grouped_linear(mixes, w_in),
+            n_bytes=t * d * 16 + 8 * d * d, flops=8 * t * d * d)
+        add(f"its like: one product of {d} x {4 * d:,} (any model), {label}", lambda: ops.linear(hrow, w_in, None, w_is_nk=True),
+            n_bytes=t * d * 10 + 8 * d * d, flops=8 * t * d * d)
+        rkvg = ops.grouped_linear(mixes, w_in)
+        bonus = torch.zeros(d, device=dev)
+        scan = lambda: ops.time_mix_scan(rkvg[:, :d], rkvg[:, d: 2 * d], rkvg[:, 2 * d: 3 * d], decay, bonus, tstate, q_start, slots, fresh, h, hd,  # noqa: E731
+                                         row_in=hrow, row_state_off=toff)
+        o32 = scan()
+        add(f"time mixing: recurrence, {h} heads of {hd} x {hd}, {label}", scan, n_bytes=t * d * (6 + 4 + 4) + 2 * tstate.numel() * 4)
+        add(f"heads' norm and silu gate (both recurrences), {label}", lambda: ops.group_norm_gated(o32, rkvg[:, 3 * d:], gain, h, 1e-5, "silu_after", bf), n_bytes=t * d * 8)
+        add(f"its like: heads' norm and sigmoid gate (Bosenex), {label}", lambda: ops.group_norm_gated(o32, rkvg[:, 3 * d:], gain, h, 1e-5, False, bf), n_bytes=t * d * 8)
+        # attention by chunks
+        kvh = kv_heads_for(h)
+        qk = torch.randn(t, (h + 2 * kvh) * hd, device=dev).to(bf)
+        gq, gk = torch.ones(h * hd, device=dev), torch.ones(kvh * hd, device=dev)
+        pages_each = length // page
+        tables = torch.arange(n_entries * pages_each, dtype=torch.int32, device=dev).view(n_entries, pages_each).contiguous()
+        stride = 2 * kvh * page * hd
+        pool = torch.randn(n_entries * pages_each, stride, device=dev).to(bf).view(-1)
+        scatter = ops.kv_scatter(slot_map, pool, pool[kvh * page * hd:], stride, page, n_entries * pages_each, h * hd, kvh * hd, hd)
+        norm_bytes = t * (h + kvh) * hd * 4 + t * kvh * hd * 4
+        add(f"attention: norms over whole query and key rows, cache write, {label}",
+            lambda: ops.row_norm(qk, h * hd, kvh * hd, gq, gk, 1e-5, kv=scatter, head_dim=hd), n_bytes=norm_bytes)
+        head_w = torch.ones(hd, device=dev)
+        scatter2 = ops.kv_scatter(slot_map, pool, pool[kvh * page * hd:], stride, page, n_entries * pages_each, (h + kvh) * hd, kvh * hd, hd)
+        add(f"its like: heads' norms and cache write (Zirunex), {label}", lambda: ops.head_norm(qk, h, kvh, hd, head_w, head_w, 1e-5, kv=scatter2), n_bytes=norm_bytes)
+        bias, sinks, att_out = torch.randn(h, 129, device=dev), torch.randn(h, device=dev), torch.empty(t, h * hd, device=dev, dtype=bf)
+        seen = sum(p % chunk + 1 for p in positions.tolist())
+        windowed = sum(min(p + 1, chunk) for p in positions.tolist())
+        if rows_each > 1:
+            attend = lambda **kw: ops.paged_attention(qk[:, : h * hd], pool, pool[kvh * page * hd:], stride, page, n_entries * pages_each, tables, row_entry,  # noqa: E731
+                                                      positions, seq_lens, h, kvh, hd, hd ** -0.5, out=att_out, max_context=length, q_start=q_start,
+                                                      n_tiles=n_entries * -(-rows_each // 64), sinks=sinks, **kw)
+            keys = n_entries * length
+        else:
+            attend = lambda **kw: ops.decode_attention_fused(  # noqa: E731
+                qk[:, : h * hd], qk[:, h * hd: (h + kvh) * hd], qk[:, (h + kvh) * hd:], slot_map, pool, pool[kvh * page * hd:], stride, page, n_entries * pages_each,
+                tables, row_entry, positions, seq_lens, h, kvh, hd, hd ** -0.5, max_context=length, exact_weights=ops.exact_weights(), sinks=sinks, **kw)
+            keys = n_entries * chunk
+        size = dict(n_bytes=t * h * hd * 4 + keys * 2 * kvh * hd * 2)
+        add(f"attention by chunks of {chunk} with a bias by distance and sinks, {h} heads of {hd} over {kvh}, {label}",
+            lambda: attend(window=0, chunk=chunk, dist_bias=bias, out_scale=1.2), flops=4 * seen * h * hd, **size)
+        add(f"its like: window of {chunk}, capped scores, sinks (Bosenex), {label}", lambda: attend(window=chunk, softcap=30.0), flops=4 * windowed * h * hd, **size)
+        # the rest of a layer and the head
+        ff = max(128, round(2 * g["n_inner"] / 3 / 128) * 128)
+        gu = torch.randn(t, 2 * ff, device=dev).to(bf)
+        add(f"gated gelu unit, {ff:,} columns, {label}", lambda: ops.expert_act(gu, "gelu_tanh"), n_bytes=t * ff * 6)
+        add(f"its like: gated relu unit (Bosenex), {label}", lambda: ops.expert_act(gu, "relu"), n_bytes=t * ff * 6)
+        side = 64
+        from research_2_b200.parts import Runtime
+        from research_2_b200.parts.token_side import GatedTokenRows
+        part = GatedTokenRows({"column": 0, "dim": side, "eps": 1e-5}, {
+            "table": torch.randn(4096, side), "gate": torch.randn(side, d) * 0.02, "proj": torch.randn(d, side) * 0.1, "norm": torch.ones(d)},
+            Runtime(torch.device(dev), bf))
+        ids = torch.randint(0, 4096, (t,), device=dev, dtype=torch.int32)
+
+        class Ctx:
+            input_ids = ids
+
+        add(f"token's own row: gate, product, norm into the stream (all launches), {label}", lambda: part.join(x32, hrow, Ctx, bf),
+            n_bytes=t * d * (2 + 4 + 4 + 2) + 4 * side * d)
+        add(f"its like: a sublayer's output normed into the stream + the next norm (Zudalorn), {label}",
+            lambda: ops.norm_add(x32, y32, gain, 1e-5, gain, 1e-5, bf), n_bytes=t * d * 14)
+        add(f"the norm after a sum (as Pidodra's), {label}", lambda: ops.add_norm(x32, y32, 2.0, gain, 1e-5, bf), n_bytes=t * d * 14)
+        if rows_each == 1:
+            logits = torch.randn(t, g["vocab_size"], device=dev)
+            add(f"capped logits, {g['vocab_size']:,} columns, {label}", lambda: ops.soft_cap(logits, 30.0), n_bytes=t * g["vocab_size"] * 8)
+    out["kernels"] = table
+    return out
+
+
 def e2e_point(model, batch: int, steps: int, warmup: int) -> dict:
     """Through the Python entry point: submit prompts (host token lists), step, poll tokens."""
     import torch
@@ -1138,7 +1374,7 @@ def main() -> int:
     ap.add_argument("--phases", action="store_true", help="print where a layer's time goes inside the resident decode kernel at --batch rows, and stop")
     ap.add_argument("--logits-ctas", action="store_true", help="print when each CTA of a decode step's logits product starts and ends (its waves), and stop")
     ap.add_argument("--prefill", action="store_true", help="print the prefill point (2 x 1,024 tokens in one step) alone, and stop")
-    ap.add_argument("--design", default=None, choices=("zirunex", "bosenex", "zudalorn", "pidodra"),
+    ap.add_argument("--design", default=None, choices=("zirunex", "bosenex", "zudalorn", "pidodra", "lagelorn"),
                     help="print prefill and decode throughput of that design at the layer sizes of --model beside GPT-2's, "
                          "and its kernels beside their likes, and stop (the default workload is GPT-2's)")
     args = ap.parse_args()
@@ -1173,7 +1409,7 @@ def main() -> int:
 
     pk, pk_source = peaks()
     if args.design:
-        points = {"bosenex": bosenex_points, "zudalorn": zudalorn_points, "pidodra": pidodra_points}.get(args.design, design_points)
+        points = {"bosenex": bosenex_points, "zudalorn": zudalorn_points, "pidodra": pidodra_points, "lagelorn": lagelorn_points}.get(args.design, design_points)
         print(json.dumps(points(args, pk)))
         return 0
     model, cfg = build_model(args.layers, size=args.model)

@@ -57,7 +57,6 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 #define R2_ACT_NONE 0
 #define R2_ACT_GELU_TANH 1
 #define R2_ACT_GELU_ERF 2
-#define R2_ACT_TANH 3
 
 __device__ __forceinline__ float gelu_tanh(float x) {
   const float k = 0.7978845608028654f;  // sqrt(2 / pi)
@@ -82,7 +81,6 @@ __device__ __forceinline__ float gelu_erf(float x) {
 __device__ __forceinline__ float activate(float x, int act) {
   if (act == R2_ACT_GELU_TANH) return gelu_tanh(x);
   if (act == R2_ACT_GELU_ERF) return gelu_erf(x);
-  if (act == R2_ACT_TANH) return tanhf(x);
   return x;
 }
 

@@ -107,7 +107,7 @@ extern "C" int r2_gemm_simt(const void* a, int lda, const void* w, int ldw, int 
                             int in_dtype, int out_dtype, cudaStream_t stream) {
   if (m <= 0 || n <= 0) return R2_OK;
   if (k < 1) return R2_BAD_SHAPE;
-  if (act < R2_ACT_NONE || act > R2_ACT_TANH) return R2_UNSUPPORTED;
+  if (act < R2_ACT_NONE || act > R2_ACT_GELU_ERF) return R2_UNSUPPORTED;
   if (in_dtype == R2_F32 && out_dtype == R2_F32)
     return launch<float, float, float>(a, lda, w, ldw, w_is_nk, bias, residual, ldr, out, ldo, m, n, k, act, stream);
   if (in_dtype == R2_BF16 && out_dtype == R2_F32)

@@ -98,6 +98,9 @@ struct GemmParams {
   bf16* kv_v;
   long long kv_page_stride;
   int kv_page_size, kv_page_shift, kv_n_pages, kv_col, kv_width, kv_head_dim, kv_head_shift;
+  // Several products side by side: the features [s * group_n, (s + 1) * group_n) read the tokens' columns from s * group_k on
+  // (0: one product). No tile straddles two groups. A K tail reads on into the next group's columns against zeros of the weight.
+  int group_n, group_k;
   // Profiling hook, normally null: six times of the nanosecond clock per CTA of the single-CTA forms (its start,
   // before and after the wait on the kernel before, tokens ready (the form with the norm inside), products
   // complete, end), [CTA][6], for the first `cta_stamps_cap` CTAs: shows how many CTAs an SM really holds.
@@ -702,11 +705,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
       }
     }
   };
+  const int token_k = p.group_n > 0 ? (TRANSPOSED ? a0 : b0) / p.group_n * p.group_k : 0;
   auto load_tokens = [&](int k0, uint32_t a_dst, uint32_t b_dst, uint32_t bar) {
     if (TRANSPOSED) {
-      tma_load_2d(b_dst, &map_b, k0, b0, bar);  // tokens are K-major
+      tma_load_2d(b_dst, &map_b, token_k + k0, b0, bar);  // tokens are K-major
     } else {
-      tma_load_2d(a_dst, &map_a, k0, a0, bar);
+      tma_load_2d(a_dst, &map_a, token_k + k0, a0, bar);
     }
   };
   const int first = min(n_kb, p.stages);
@@ -1131,6 +1135,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     for (int tile = pair; tile < p.n_tiles && ok; tile += n_pairs) {
       const int a0 = ((tile / p.col_tiles) * 2 + int(rank)) * BM;
       const int b0 = (tile % p.col_tiles) * p.bn + int(rank) * half;
+      const int token_k = p.group_n > 0 ? (tile % p.col_tiles) * p.bn / p.group_n * p.group_k : 0;
       for (int kb = 0; kb < n_kb; ++kb) {
         if (!mbar_wait(empty_base + uint32_t(stage) * 8u, parity ^ 1u)) {
           if (lane == 0) atomicMax(p.error_flag, R2_ERR_TIMEOUT_EMPTY);
@@ -1151,7 +1156,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         if (waited) {
           if (elect_one()) {
             load_weights();
-            tma_load_2d_pair(a_dst, &map_a, k0, a0, bar);
+            tma_load_2d_pair(a_dst, &map_a, token_k + k0, a0, bar);
           }
         } else {
           // the weights of the first k-block go on their way; the tokens may have been written by
@@ -1159,7 +1164,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           if (elect_one()) load_weights();
           pdl_wait();
           waited = true;
-          if (elect_one()) tma_load_2d_pair(a_dst, &map_a, k0, a0, bar);
+          if (elect_one()) tma_load_2d_pair(a_dst, &map_a, token_k + k0, a0, bar);
         }
         __syncwarp();
         a_dst += a_bytes;
@@ -1562,12 +1567,17 @@ extern "C" int r2_gemm_tc_plan(int m, int n, int k, int w_is_nk, int* bn_out, in
 // With ln_x != null the tokens are LayerNorm(ln_x[ln_rows[i]] or ln_x[i]) computed inside the kernel
 // (`x` is then ignored); this form takes at most 16 tokens and k <= 1024, else R2_UNSUPPORTED.
 // `prefetch` (may be null) names memory, typically the next product's weight, that the kernel asks into L2.
-extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_is_nk, const float* bias,
+namespace {
+int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, const float* bias,
                           const float* residual, int ldr, void* out, int ldo, int m, int n, int k, int act,
                           int out_dtype, int* error_flag, const float* ln_x, int ln_ldx, const int32_t* ln_rows,
                           const float* ln_gamma, const float* ln_beta, float ln_eps, const void* prefetch,
-                          long long prefetch_bytes, const R2KvScatter* kv, cudaStream_t stream) {
+                          long long prefetch_bytes, const R2KvScatter* kv, int n_groups, cudaStream_t stream) {
   if (m <= 0 || n <= 0) return R2_OK;
+  // (n_groups > 1: x [m, n_groups * k], the features' n / n_groups of group s on x's columns from s * k on)
+  const int group_n = n_groups > 1 ? n / n_groups : 0;
+  const uint64_t x_cols = uint64_t(k) * uint64_t(n_groups > 1 ? n_groups : 1);
+  if (n_groups > 1 && (n % n_groups != 0 || group_n % BM != 0 || ln_x != nullptr || kv != nullptr)) return R2_UNSUPPORTED;
   const bool fused_ln = ln_x != nullptr;
   if (fused_ln) {
     if (m > LN_MAX_TOKENS || k > LN_MAX_K || k % 8 != 0 || ln_ldx % 4 != 0 || ln_gamma == nullptr) return R2_UNSUPPORTED;
@@ -1614,6 +1624,9 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
     p.kv_head_dim = kv->head_dim;
     p.kv_head_shift = (kv->head_dim & (kv->head_dim - 1)) == 0 ? page_shift_of(kv->head_dim) : -1;
   }
+  p.group_n = group_n;
+  p.group_k = k;
+  if (group_n > 0 && !pl.swapped && group_n % pl.bn != 0) return R2_UNSUPPORTED;
   p.cta_stamps = g_cta_stamps;
   p.cta_stamps_cap = g_cta_stamps_cap;
   p.a_total = pl.a_total;
@@ -1638,7 +1651,7 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
 
   if (!pl.swapped && !fused_ln && g_pair_form != 0) {
     const PairPlan pp = make_pair_plan(m, n, k, w_is_nk, g_pair_form == 2);
-    if (pp.use) {
+    if (pp.use && (group_n == 0 || group_n % pp.bn == 0)) {
       p.bn = pp.bn;
       p.stages = pp.stages;
       p.splits = 1;
@@ -1646,7 +1659,7 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
       p.n_tiles = pp.n_tiles;
       p.col_tiles = pp.col_tiles;
       CUtensorMap pa, pb;
-      bool maps = make_map(&pa, x, uint64_t(k), uint64_t(m), uint64_t(lda), BK, BM);
+      bool maps = make_map(&pa, x, x_cols, uint64_t(m), uint64_t(lda), BK, BM);
       if (w_is_nk) {
         maps = maps && make_map(&pb, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, uint32_t(pp.bn / 2));
         if (maps) return launch_pair<false>(pa, pb, p, pp, stream);
@@ -1666,7 +1679,7 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
   bool ok;
   if (!pl.swapped) {
     // a side: tokens [m, k] K-major; b side: the weight
-    ok = make_map(&ma, x, uint64_t(k), uint64_t(m), uint64_t(lda), BK, BM);
+    ok = make_map(&ma, x, x_cols, uint64_t(m), uint64_t(lda), BK, BM);
     if (w_is_nk) {
       ok = ok && make_map(&mb, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, uint32_t(bn));
       if (!ok) return R2_UNSUPPORTED;
@@ -1678,7 +1691,7 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
   }
   // swapped: a side = the weight's features, b side = tokens [m, k] K-major
   ok = fused_ln ? make_map(&mb, w, 64, 64, 64, BK, 16)  // a placeholder map: the kernel never uses it
-                : make_map(&mb, x, uint64_t(k), uint64_t(m), uint64_t(lda), BK, uint32_t(bn));
+                : make_map(&mb, x, x_cols, uint64_t(m), uint64_t(lda), BK, uint32_t(bn));
   if (w_is_nk) {
     ok = ok && make_map(&ma, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, BM);
     if (!ok) return R2_UNSUPPORTED;
@@ -1689,4 +1702,24 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
   if (!ok) return R2_UNSUPPORTED;
   return fused_ln ? launch<true, false, true, true>(ma, mb, p, grid, smem, stream)
                   : launch<true, false, true>(ma, mb, p, grid, smem, stream);
+}
+}  // namespace
+
+extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_is_nk, const float* bias,
+                          const float* residual, int ldr, void* out, int ldo, int m, int n, int k, int act,
+                          int out_dtype, int* error_flag, const float* ln_x, int ln_ldx, const int32_t* ln_rows,
+                          const float* ln_gamma, const float* ln_beta, float ln_eps, const void* prefetch,
+                          long long prefetch_bytes, const R2KvScatter* kv, cudaStream_t stream) {
+  return gemm_tc_run(x, lda, w, ldw, w_is_nk, bias, residual, ldr, out, ldo, m, n, k, act, out_dtype, error_flag, ln_x, ln_ldx, ln_rows,
+                     ln_gamma, ln_beta, ln_eps, prefetch, prefetch_bytes, kv, 1, stream);
+}
+
+// n_groups products in one launch: x [m, n_groups * k], w [n_groups * n, k] (the groups' matrices one after the other, stored
+// [out, in]), out [m, n_groups * n]: out's columns of group s are x's columns of group s times w's rows of group s. Groups of a
+// multiple of 128 features; else R2_UNSUPPORTED (the caller then runs one product a group).
+extern "C" int r2_gemm_tc_grouped(const void* x, int lda, const void* w, int ldw, void* out, int ldo, int m, int n, int k, int n_groups,
+                                  int out_dtype, int* error_flag, cudaStream_t stream) {
+  if (n_groups < 1) return R2_BAD_SHAPE;
+  return gemm_tc_run(x, lda, w, ldw, 1, nullptr, nullptr, 0, out, ldo, m, n * n_groups, k, R2_ACT_NONE, out_dtype, error_flag, nullptr, 0,
+                     nullptr, nullptr, nullptr, 0.f, nullptr, 0, nullptr, n_groups, stream);
 }

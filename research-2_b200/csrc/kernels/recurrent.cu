@@ -1,14 +1,12 @@
 // Mixers that carry a state of fixed size from token to token instead of a cache that grows: a matrix
-// memory with exponential gates (mLSTM), a state-space layer (Mamba-2's recurrence), retention (linear attention
+// memory with exponential gates (mLSTM), a state-space layer (Mamba-2's recurrence) and retention (linear attention
 // with one fixed decay per head, keep_t = decay and take_t = 1; its queries and keys are rotated by position on their way
-// into shared memory, in float, so what enters the recurrence is never rounded to 16 bits) and time mixing with a decay per
-// channel (keep_t = diag(w_t); the read-out sees the state BEFORE the row's write, and the row's own write times a bonus per
-// channel), all of the form
+// into shared memory, in float, so what enters the recurrence is never rounded to 16 bits), all of the form
 //
 //     S_t = keep_t * S_(t-1) + take_t * w_t v_t^T        S: [rows x columns] per head, float
 //     y_t = S_t^T r_t  (+ what the layer adds)
 //
-// with a write vector w (keys; B), a read vector r (queries; C) and values v. One kernel serves them all and
+// with a write vector w (keys; B), a read vector r (queries; C) and values v. One kernel serves both and
 // serves prompts, portions and single decoded tokens alike: a CTA owns one (entry, head, slice of the
 // value columns), takes the state from the request's slot (or zeros for a sequence's first rows), walks the
 // entry's rows in order and puts the state back. A thread keeps RPT rows of one column in registers; the
@@ -18,10 +16,8 @@
 // The order of operations depends on the row's position alone, so a row's result is the same bits however
 // its prompt was cut into steps.
 //
-// Beside it: the gated delta rule, whose write depends on what the state holds already (a kernel of its own below, with the
-// same division of a head's state); the short causal convolution in front of the state-space recurrence and of the delta
-// rule (its last inputs are state too); the mixes of a row with the row before it in front of time mixing (that row is state
-// too); and the norm over groups of columns with a gate that follows all of them.
+// Beside it: the short causal convolution in front of the state-space recurrence (its last inputs are
+// state too), and the norm over groups of columns with a gate that follows both mixers.
 #include <math.h>
 
 #include "common.cuh"
@@ -33,7 +29,7 @@ namespace {
 constexpr int MAX_TILE = 32, SMALL_TILE = 4;
 constexpr int NORM_COPIES = 8;  // copies of a matrix memory's normaliser and maximum: one per slice of the columns at most
 
-constexpr int MODE_MLSTM = 0, MODE_SSD = 1, MODE_DECAY = 2, MODE_CHANNEL = 3;
+constexpr int MODE_MLSTM = 0, MODE_SSD = 1, MODE_DECAY = 2;
 
 __device__ __forceinline__ float soft_cap(float x, float cap) { return cap > 0.f ? cap * tanhf(x / cap) : x; }
 __device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
@@ -45,9 +41,8 @@ struct ScanArgs {
   const void* value; int value_stride;   // v: [T, heads * cols]
   const float* gates; int gates_stride;  // mLSTM: [T, 2 heads] input gates then forget gates, before the cap
                                          // state space: [T, heads] step sizes before bias and softplus
-                                         // delta rule: [T, 2 heads] write strengths before the sigmoid, then step sizes
-  const float* step_bias;                // state space and delta rule, per head
-  const float* log_rate;                 // state space and delta rule, per head: the decay is exp(-exp(log_rate) * step)
+  const float* step_bias;                // state space, per head
+  const float* log_rate;                 // state space, per head: the decay is exp(-exp(log_rate) * step)
   const float* skip;                     // state space, per head: y += skip * v
   float cap;                             // mLSTM: gates are cap * tanh(x / cap); 0 = no cap
   float read_scale;                      // r is multiplied by it
@@ -55,35 +50,15 @@ struct ScanArgs {
   const float* decay;                    // retention, per head: keep
   const float* inv_freq; int rot_half;   // retention: of r and w the first 2 * rot_half dimensions turn, dimension i with
   const int32_t* positions;              // i + rot_half, by the angle positions[row] * inv_freq[i] (rot_half 0: no rotation)
-  const float* channel_log; int channel_log_stride;  // decay per channel: [T, heads * rows], the decay is exp(-exp(channel_log))
-  const float* bonus;                    // decay per channel: [heads * rows], the factor on the row's own write in its read-out
-  float unit_eps;                        // delta rule: q and k are divided by sqrt(sum of squares + unit_eps)
   float* state; long long slot_stride;   // per request slot; per head: S [rows][cols] (+ mLSTM: NORM_COPIES times n [rows], m)
   int head_stride;
   const int32_t* q_start; const int32_t* state_slot; const int32_t* fresh;
   float* out; int out_stride;            // [T, heads * cols] float
   int heads_per_group, rows, cols, G, cv;
   int single_rows;                       // a hint: no entry has more than one row (a decode step)
-  // the last conv_taps - 1 input rows of the convolution (of the mixes: 2 taps), kept by the CTA of (entry, head 0, slice 0)
+  // state space: the convolution's last inputs, renewed by the entry's CTAs together
   const void* conv_in; int conv_in_stride; int conv_channels, conv_taps; long long conv_state_off;
 };
-
-// The inputs of the convolution's last taps - 1 positions: this step's newest rows, and before them what the slot held
-// (each channel is one thread's: it reads a place before it writes over it).
-template <typename T>
-__device__ __forceinline__ void keep_conv_inputs(const ScanArgs& a, int e, int row0, int row1, bool is_fresh) {
-  const T* in = static_cast<const T*>(a.conv_in);
-  float* cs = a.state + size_t(a.state_slot[e]) * a.slot_stride + a.conv_state_off;
-  const int keep = a.conv_taps - 1, n = row1 - row0;
-  for (int c = threadIdx.x; c < a.conv_channels; c += blockDim.x)
-    for (int s = 0; s < keep; ++s) {
-      const int l = n - keep + s;
-      float val = 0.f;
-      if (l >= 0) val = to_float(in[size_t(row0 + l) * a.conv_in_stride + c]);
-      else if (!is_fresh) val = cs[size_t(s + n) * a.conv_channels + c];
-      cs[size_t(s) * a.conv_channels + c] = val;
-    }
-}
 
 template <typename T, int RPT, int MODE, int TILE>
 __global__ void __launch_bounds__(256)
@@ -102,7 +77,6 @@ outer_scan_kernel(const ScanArgs a) {
   float* g0 = vs + TILE * cv;             // [TILE] log input gate, then take | step
   float* g1 = g0 + TILE;                  // [TILE] log forget gate, then keep | decay
   float* g2 = g1 + TILE;                  // [TILE] running maximum after the row
-  float* ds = g2 + TILE;                  // [TILE][padded] decay per channel (that mode only); g2 holds the own write's bonus
   // a thread has the rows g * RPT .. g * RPT + RPT - 1 of column j; the G threads of a column are neighbouring lanes
   const int tid = threadIdx.x, g = tid % G, jl = tid / G;
   const int j = blockIdx.z * cv + jl;
@@ -112,8 +86,22 @@ outer_scan_kernel(const ScanArgs a) {
   // copies z, z + slices, z + 2 slices, ..., so that every copy is current whatever the number of slices of a launch
   float* norm_state = head_state + size_t(rows) * cols;
 
-  if ((MODE == MODE_SSD || MODE == MODE_CHANNEL) && a.conv_in != nullptr && h == 0 && blockIdx.z == 0)
-    keep_conv_inputs<T>(a, e, row0, row1, is_fresh);
+  if (MODE == MODE_SSD && a.conv_in != nullptr) {
+    // the inputs of the convolution's last taps - 1 positions: this step's newest rows, and before them what the
+    // slot held (each channel is one thread's: it reads a place before it writes over it), spread over the entry's CTAs
+    const int part = h * gridDim.z + blockIdx.z, n_parts = gridDim.y * gridDim.z;
+    const T* in = static_cast<const T*>(a.conv_in);
+    float* cs = a.state + size_t(a.state_slot[e]) * a.slot_stride + a.conv_state_off;
+    const int keep = a.conv_taps - 1, n = row1 - row0;
+    for (int c = part * blockDim.x + tid; c < a.conv_channels; c += n_parts * blockDim.x)
+      for (int s = 0; s < keep; ++s) {
+        const int l = n - keep + s;
+        float val = 0.f;
+        if (l >= 0) val = to_float(in[size_t(row0 + l) * a.conv_in_stride + c]);
+        else if (!is_fresh) val = cs[size_t(s + n) * a.conv_channels + c];
+        cs[size_t(s) * a.conv_channels + c] = val;
+      }
+  }
 
   float S[RPT], nrm[RPT], m = 0.f;
 #pragma unroll
@@ -134,7 +122,7 @@ outer_scan_kernel(const ScanArgs a) {
     __syncthreads();  // the last rows' vectors have been used
     // (loads in batches of eight before their stores: a loop of load-then-store would wait for every load in turn)
     for (int base = 0; base < nt * padded; base += 8 * blockDim.x) {
-      float tr[8], tw[8], td[8];
+      float tr[8], tw[8];
 #pragma unroll
       for (int u = 0; u < 8; ++u) {
         const int idx = base + u * blockDim.x + tid;
@@ -143,7 +131,6 @@ outer_scan_kernel(const ScanArgs a) {
         const size_t row = size_t(t0 + tt);
         tr[u] = live ? to_float(read[row * a.read_stride + i]) : 0.f;
         tw[u] = live ? to_float(write[row * a.write_stride + i]) : 0.f;
-        if (MODE == MODE_CHANNEL) td[u] = live ? a.channel_log[row * a.channel_log_stride + size_t(h) * rows + i] : 0.f;
         if (MODE == MODE_DECAY && live && i < 2 * a.rot_half) {
           // the pair (u, v) = (x[i], x[i + half]) becomes (u cos - v sin, v cos + u sin); position and angle are float
           const bool low = i < a.rot_half;
@@ -161,7 +148,6 @@ outer_scan_kernel(const ScanArgs a) {
         if (idx < nt * padded) {
           rs[idx] = tr[u] * a.read_scale;
           ws[idx] = MODE == MODE_DECAY ? tw[u] * a.write_scale : tw[u];
-          if (MODE == MODE_CHANNEL) ds[idx] = expf(-expf(td[u]));
         }
       }
     }
@@ -179,9 +165,7 @@ outer_scan_kernel(const ScanArgs a) {
         if (idx < nt * cv) vs[idx] = tv[u];
       }
     }
-    if (MODE == MODE_CHANNEL) {
-      // nothing per row: the decays are per channel
-    } else if (MODE == MODE_DECAY) {
+    if (MODE == MODE_DECAY) {
       if (tid < nt) {
         g0[tid] = 1.f;
         g1[tid] = a.decay[h];
@@ -231,17 +215,6 @@ outer_scan_kernel(const ScanArgs a) {
       __syncthreads();
       m = g2[nt - 1];
     }
-    if (MODE == MODE_CHANNEL) {
-      // the read-out of a row's own write: (sum over channels of r * bonus * k) times its value; a warp per row
-      const int lane = tid & 31;
-      for (int tt = tid >> 5; tt < nt; tt += blockDim.x >> 5) {
-        float sum = 0.f;
-        for (int i = lane; i < rows; i += 32) sum = fmaf(rs[tt * padded + i] * a.bonus[size_t(h) * rows + i], ws[tt * padded + i], sum);
-        sum = warp_sum(sum);
-        if (lane == 0) g2[tt] = sum;
-      }
-      __syncthreads();
-    }
     float num[TILE], nq[TILE];
 #pragma unroll
     for (int tt = 0; tt < TILE; ++tt) {
@@ -249,9 +222,8 @@ outer_scan_kernel(const ScanArgs a) {
       num[tt] = 0.f;
       nq[tt] = 0.f;
       {
-        const float take = MODE == MODE_CHANNEL ? 1.f : g0[tt], keep = MODE == MODE_CHANNEL ? 1.f : g1[tt];
+        const float take = g0[tt], keep = g1[tt];
         const float tv = take * vs[tt * cv + jl];
-        const float4* dr = reinterpret_cast<const float4*>(ds + tt * padded + g * RPT);
         const float4* wr = reinterpret_cast<const float4*>(ws + tt * padded + g * RPT);
         const float4* rr = reinterpret_cast<const float4*>(rs + tt * padded + g * RPT);
         float acc = 0.f, acc_n = 0.f;
@@ -259,19 +231,9 @@ outer_scan_kernel(const ScanArgs a) {
         for (int r4 = 0; r4 < RPT / 4; ++r4) {
           const float4 w4 = wr[r4], q4 = rr[r4];
           const float w[4] = {w4.x, w4.y, w4.z, w4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
-          float d[4] = {0.f, 0.f, 0.f, 0.f};
-          if (MODE == MODE_CHANNEL) {
-            const float4 d4 = dr[r4];
-            d[0] = d4.x; d[1] = d4.y; d[2] = d4.z; d[3] = d4.w;
-          }
 #pragma unroll
           for (int u = 0; u < 4; ++u) {
             const int r = r4 * 4 + u;
-            if (MODE == MODE_CHANNEL) {
-              acc = fmaf(S[r], q[u], acc);          // the state before this row's write
-              S[r] = fmaf(d[u], S[r], w[u] * tv);
-              continue;
-            }
             S[r] = fmaf(keep, S[r], w[u] * tv);
             acc = fmaf(S[r], q[u], acc);
             if (MODE == MODE_MLSTM) {
@@ -302,7 +264,7 @@ outer_scan_kernel(const ScanArgs a) {
         {
           float y;
           if (MODE == MODE_MLSTM) y = num[tt] / (fmaxf(fabsf(nq[tt]), expf(-g2[tt])) + 1e-6f);
-          else y = fmaf(MODE == MODE_CHANNEL ? g2[tt] : skip, vs[tt * cv + jl], num[tt]);
+          else y = fmaf(skip, vs[tt * cv + jl], num[tt]);
           a.out[size_t(t0 + tt) * a.out_stride + size_t(h) * cols + j] = y;
         }
       }
@@ -349,14 +311,6 @@ ScanShape scan_shape(int rows, int cols, int pairs) {
   return s;
 }
 
-// Launches of more than the default 48 KB of shared memory ask for it once per kernel and device.
-template <typename... A>
-bool room_for(void (*kernel)(A...), size_t smem) {
-  if (smem <= 48 * 1024) return true;
-  if (smem > 227 * 1024) return false;
-  return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) == cudaSuccess;
-}
-
 template <typename T, int MODE>
 int launch_scan(const ScanArgs& in, int n_entries, int n_heads, cudaStream_t stream) {
   ScanArgs a = in;
@@ -367,13 +321,10 @@ int launch_scan(const ScanArgs& in, int n_entries, int n_heads, cudaStream_t str
   a.cv = s.cv;
   const bool single_rows = a.single_rows != 0;
   const int tile = single_rows ? SMALL_TILE : (rpt <= 16 ? MAX_TILE : 16);
-  const size_t smem = sizeof(float) * (size_t(tile) * ((MODE == MODE_CHANNEL ? 3 : 2) * rpt * G + a.cv) + 3 * tile);
+  const size_t smem = sizeof(float) * (size_t(tile) * (2 * rpt * G + a.cv) + 3 * tile);
+  if (smem > 48 * 1024) return R2_UNSUPPORTED;
   dim3 grid(n_entries, n_heads, splits);
-#define R2_SCAN(RPT_, TILE_)                                                                  \
-  do {                                                                                        \
-    if (!room_for(outer_scan_kernel<T, RPT_, MODE, TILE_>, smem)) return R2_UNSUPPORTED;      \
-    r2_launch(outer_scan_kernel<T, RPT_, MODE, TILE_>, grid, dim3(threads), smem, stream, a); \
-  } while (0)
+#define R2_SCAN(RPT_, TILE_) r2_launch(outer_scan_kernel<T, RPT_, MODE, TILE_>, grid, dim3(threads), smem, stream, a)
   switch (rpt) {
     case 4: if (single_rows) R2_SCAN(4, SMALL_TILE); else R2_SCAN(4, MAX_TILE); break;
     case 8: if (single_rows) R2_SCAN(8, SMALL_TILE); else R2_SCAN(8, MAX_TILE); break;
@@ -382,214 +333,6 @@ int launch_scan(const ScanArgs& in, int n_entries, int n_heads, cudaStream_t str
   }
 #undef R2_SCAN
   return launch_status();
-}
-
-// ---- the gated delta rule -----------------------------------------------------------------------
-// Per head, with unit vectors q, k (q times a scale), a decay g and a write strength beta per row:
-//
-//     S' = g S,   u = beta (v - S'^T k),   S = S' + k u^T,   o = S^T q = S'^T q + (k . q) u
-//
-// The write needs what the state returns for the row's key, so every row costs a sum over the state's rows before the next can
-// begin; S'^T k and S'^T q are summed side by side (the second form of o), which leaves one round of shuffles a row on the
-// chain. q and k stay as they came in shared memory: their lengths and their product are numbers per row that are multiplied
-// in where a sum or a write uses them. The state's division and the staging are the outer products' kernel's.
-template <typename T, int RPT, int TILE>
-__global__ void __launch_bounds__(256)
-delta_scan_kernel(const ScanArgs a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  extern __shared__ __align__(16) float smem[];
-  const int e = blockIdx.x, h = blockIdx.y;
-  const int row0 = a.q_start[e], row1 = a.q_start[e + 1];
-  if (row1 <= row0) return;
-  const int G = a.G, cv = a.cv, rows = a.rows, cols = a.cols;
-  const int padded = RPT * G;
-  float* qs = smem;                      // [TILE][padded]
-  float* ks = qs + TILE * padded;        // [TILE][padded]
-  float* vs = ks + TILE * padded;        // [TILE][cv]
-  float* per_row = vs + TILE * cv;       // [TILE][8]: g, beta, 1 / |k|, scale / |q|, k . q of the unit vectors
-  const int tid = threadIdx.x, g = tid % G, jl = tid / G, lane = tid & 31;
-  const int j = blockIdx.z * cv + jl;
-  const bool is_fresh = a.fresh[e] != 0;
-  float* head_state = a.state + size_t(a.state_slot[e]) * a.slot_stride + size_t(h) * a.head_stride;
-  if (a.conv_in != nullptr && h == 0 && blockIdx.z == 0) keep_conv_inputs<T>(a, e, row0, row1, is_fresh);
-
-  float S[RPT];
-#pragma unroll
-  for (int r = 0; r < RPT; ++r) {
-    const int i = g * RPT + r;
-    S[r] = (!is_fresh && i < rows && j < cols) ? head_state[size_t(i) * cols + j] : 0.f;
-  }
-  const T* read = static_cast<const T*>(a.read) + size_t(h / a.heads_per_group) * rows;
-  const T* write = static_cast<const T*>(a.write) + size_t(h / a.heads_per_group) * rows;
-  const T* value = static_cast<const T*>(a.value) + size_t(h) * cols + size_t(blockIdx.z) * cv;
-
-  for (int t0 = row0; t0 < row1; t0 += TILE) {
-    const int nt = row1 - t0 < TILE ? row1 - t0 : TILE;
-    __syncthreads();
-    for (int base = 0; base < nt * padded; base += 8 * blockDim.x) {
-      float tq[8], tk[8];
-#pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const int idx = base + u * blockDim.x + tid;
-        const int tt = idx / padded, i = idx - tt * padded;
-        const bool live = idx < nt * padded && i < rows;
-        const size_t row = size_t(t0 + tt);
-        tq[u] = live ? to_float(read[row * a.read_stride + i]) : 0.f;
-        tk[u] = live ? to_float(write[row * a.write_stride + i]) : 0.f;
-      }
-#pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const int idx = base + u * blockDim.x + tid;
-        if (idx < nt * padded) {
-          qs[idx] = tq[u];
-          ks[idx] = tk[u];
-        }
-      }
-    }
-    for (int base = 0; base < nt * cv; base += 4 * blockDim.x) {
-      float tv[4];
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int idx = base + u * blockDim.x + tid;
-        const int tt = idx / cv, c = idx - tt * cv;
-        tv[u] = (idx < nt * cv && blockIdx.z * cv + c < cols) ? to_float(value[size_t(t0 + tt) * a.value_stride + c]) : 0.f;
-      }
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int idx = base + u * blockDim.x + tid;
-        if (idx < nt * cv) vs[idx] = tv[u];
-      }
-    }
-    if (tid < nt) {
-      const float* gr = a.gates + size_t(t0 + tid) * a.gates_stride;
-      const float step = softplus(gr[gridDim.y + h] + a.step_bias[h]);
-      per_row[tid * 8 + 0] = expf(-expf(a.log_rate[h]) * step);
-      per_row[tid * 8 + 1] = 1.f / (1.f + expf(-gr[h]));
-    }
-    __syncthreads();
-    for (int tt = tid >> 5; tt < nt; tt += blockDim.x >> 5) {   // a warp per row: lengths and product of q and k
-      float qq = 0.f, kk = 0.f, kq = 0.f;
-      for (int i = lane; i < rows; i += 32) {
-        const float q = qs[tt * padded + i], k = ks[tt * padded + i];
-        qq = fmaf(q, q, qq);
-        kk = fmaf(k, k, kk);
-        kq = fmaf(k, q, kq);
-      }
-      qq = warp_sum(qq);
-      kk = warp_sum(kk);
-      kq = warp_sum(kq);
-      if (lane == 0) {
-        const float qn = a.read_scale / sqrtf(qq + a.unit_eps), kn = 1.f / sqrtf(kk + a.unit_eps);
-        per_row[tt * 8 + 2] = kn;
-        per_row[tt * 8 + 3] = qn;
-        per_row[tt * 8 + 4] = kq * kn * qn;
-      }
-    }
-    __syncthreads();
-    float out[TILE];
-#pragma unroll
-    for (int tt = 0; tt < TILE; ++tt) {
-      if (tt >= nt) break;
-      const float4 n4 = *reinterpret_cast<const float4*>(per_row + tt * 8);   // g, beta, 1 / |k|, scale / |q|
-      const float kq = per_row[tt * 8 + 4];
-      const float4* kr = reinterpret_cast<const float4*>(ks + tt * padded + g * RPT);
-      const float4* qr = reinterpret_cast<const float4*>(qs + tt * padded + g * RPT);
-      float ak[4] = {0.f, 0.f, 0.f, 0.f}, aq[4] = {0.f, 0.f, 0.f, 0.f};
-      float4 k4[RPT / 4];
-#pragma unroll
-      for (int r4 = 0; r4 < RPT / 4; ++r4) {
-        k4[r4] = kr[r4];
-        const float4 q4 = qr[r4];
-        const float k[4] = {k4[r4].x, k4[r4].y, k4[r4].z, k4[r4].w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          S[r4 * 4 + u] *= n4.x;
-          ak[u] = fmaf(S[r4 * 4 + u], k[u], ak[u]);
-          aq[u] = fmaf(S[r4 * 4 + u], q[u], aq[u]);
-        }
-      }
-      float sk = (ak[0] + ak[1]) + (ak[2] + ak[3]), sq = (aq[0] + aq[1]) + (aq[2] + aq[3]);
-      for (int o = G >> 1; o > 0; o >>= 1) {
-        sk += __shfl_xor_sync(0xffffffffu, sk, o);
-        sq += __shfl_xor_sync(0xffffffffu, sq, o);
-      }
-      const float u_row = n4.y * (vs[tt * cv + jl] - n4.z * sk);
-      out[tt] = fmaf(kq, u_row, n4.w * sq);
-      const float ku = n4.z * u_row;
-#pragma unroll
-      for (int r4 = 0; r4 < RPT / 4; ++r4) {
-        const float k[4] = {k4[r4].x, k4[r4].y, k4[r4].z, k4[r4].w};
-#pragma unroll
-        for (int u = 0; u < 4; ++u) S[r4 * 4 + u] = fmaf(ku, k[u], S[r4 * 4 + u]);
-      }
-    }
-    if (g == 0 && j < cols) {
-#pragma unroll
-      for (int tt = 0; tt < TILE; ++tt) {
-        if (tt >= nt) break;
-        a.out[size_t(t0 + tt) * a.out_stride + size_t(h) * cols + j] = out[tt];
-      }
-    }
-  }
-#pragma unroll
-  for (int r = 0; r < RPT; ++r) {
-    const int i = g * RPT + r;
-    if (i < rows && j < cols) head_state[size_t(i) * cols + j] = S[r];
-  }
-}
-
-template <typename T>
-int launch_delta(const ScanArgs& in, int n_entries, int n_heads, cudaStream_t stream) {
-  ScanArgs a = in;
-  const ScanShape s = scan_shape(a.rows, a.cols, n_entries * n_heads);
-  if (s.G > 32 || s.threads > 256) return R2_UNSUPPORTED;
-  a.G = s.G;
-  a.cv = s.cv;
-  const bool single_rows = a.single_rows != 0;
-  const int tile = single_rows ? SMALL_TILE : (s.rpt <= 16 ? MAX_TILE : 16);
-  const size_t smem = sizeof(float) * (size_t(tile) * (2 * s.rpt * s.G + a.cv) + 8 * tile);
-  dim3 grid(n_entries, n_heads, s.splits);
-#define R2_DELTA(RPT_, TILE_)                                                                   \
-  do {                                                                                          \
-    if (!room_for(delta_scan_kernel<T, RPT_, TILE_>, smem)) return R2_UNSUPPORTED;              \
-    r2_launch(delta_scan_kernel<T, RPT_, TILE_>, grid, dim3(s.threads), smem, stream, a);       \
-  } while (0)
-  switch (s.rpt) {
-    case 4: if (single_rows) R2_DELTA(4, SMALL_TILE); else R2_DELTA(4, MAX_TILE); break;
-    case 8: if (single_rows) R2_DELTA(8, SMALL_TILE); else R2_DELTA(8, MAX_TILE); break;
-    case 16: if (single_rows) R2_DELTA(16, SMALL_TILE); else R2_DELTA(16, MAX_TILE); break;
-    default: if (single_rows) R2_DELTA(32, SMALL_TILE); else R2_DELTA(32, 16); break;
-  }
-#undef R2_DELTA
-  return launch_status();
-}
-
-// ---- a row mixed with the row before it ---------------------------------------------------------
-// Mix s of row t: h + (h' - h) * mu[s], h' the row before it in its sequence: the row above inside the entry, the slot's row for
-// an entry's first (zeros for a sequence's first). Mixes 0 .. n_mixes - 1 go to out [T][n_mixes][width] in the rows' dtype; one
-// more, mu[n_mixes], to out_float [T][width] in float (null: none). The slot is only read: the recurrence's kernel renews it.
-template <typename T>
-__global__ void __launch_bounds__(256)
-shift_mix_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ mu, int n_mixes, T* __restrict__ out,
-                 float* __restrict__ out_float, int width, const float* __restrict__ state, long long slot_stride, long long row_off,
-                 const int32_t* __restrict__ row_entry, const int32_t* __restrict__ q_start, const int32_t* __restrict__ state_slot,
-                 const int32_t* __restrict__ fresh) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int t = blockIdx.x, e = row_entry[t];
-  const bool first = e >= 0 && t == q_start[e];
-  const float* kept = (first && fresh[e] == 0) ? state + size_t(state_slot[e]) * slot_stride + row_off : nullptr;
-  const T* hr = h + size_t(t) * h_stride;
-  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
-    const float now = e >= 0 ? to_float(hr[c]) : 0.f;
-    float before = 0.f;
-    if (e >= 0 && !first) before = to_float(hr[c - (long long)h_stride]);
-    else if (kept != nullptr) before = kept[c];
-    const float step = before - now;
-    for (int s = 0; s < n_mixes; ++s) out[(size_t(t) * n_mixes + s) * width + c] = from_float<T>(fmaf(step, mu[size_t(s) * width + c], now));
-    if (out_float != nullptr) out_float[size_t(t) * width + c] = fmaf(step, mu[size_t(n_mixes) * width + c], now);
-  }
 }
 
 // ---- the short causal convolution --------------------------------------------------------------
@@ -777,74 +520,6 @@ extern "C" int r2_ssd_scan(const void* x, int x_stride, const void* b, int b_str
   if (dtype == R2_F32) return launch_scan<float, MODE_SSD>(a, n_entries, n_heads, stream);
   if (dtype == R2_BF16) return launch_scan<bf16, MODE_SSD>(a, n_entries, n_heads, stream);
   return R2_BAD_DTYPE;
-}
-
-// The gated delta rule. q, k [T, groups * dim], v [T, heads * vdim] (after convolution and silu, before their unit norms); gates
-// float [T, 2 * heads]: write strengths before the sigmoid, then step sizes before bias and softplus; per head step_bias and
-// log_rate (the decay is exp(-exp(log_rate) * softplus(step + step_bias))). State per slot: S [heads][dim][vdim] and, at
-// conv_state_off, the convolution's last inputs, renewed from conv_in as by r2_ssd_scan. out [T, heads * vdim] float.
-extern "C" int r2_delta_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
-                             const float* gates, int gates_stride, const float* step_bias, const float* log_rate, float q_scale,
-                             float unit_eps, float* state, long long slot_stride, const int32_t* q_start, const int32_t* state_slot,
-                             const int32_t* fresh, int n_entries, float* out, int out_stride, int n_heads, int n_groups, int dim,
-                             int vdim, const void* conv_in, int conv_in_stride, int conv_channels, int conv_taps,
-                             long long conv_state_off, int single_rows, int dtype, cudaStream_t stream) {
-  if (n_entries <= 0) return R2_OK;
-  if (n_heads < 1 || n_groups < 1 || n_heads % n_groups != 0 || dim < 1 || vdim < 1) return R2_BAD_SHAPE;
-  ScanArgs a = {};
-  a.read = q; a.read_stride = q_stride; a.write = k; a.write_stride = k_stride; a.value = v; a.value_stride = v_stride;
-  a.gates = gates; a.gates_stride = gates_stride; a.step_bias = step_bias; a.log_rate = log_rate;
-  a.read_scale = q_scale; a.unit_eps = unit_eps; a.state = state; a.slot_stride = slot_stride; a.head_stride = dim * vdim;
-  a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh; a.out = out; a.out_stride = out_stride;
-  a.heads_per_group = n_heads / n_groups; a.rows = dim; a.cols = vdim; a.single_rows = single_rows;
-  a.conv_in = conv_taps > 1 ? conv_in : nullptr; a.conv_in_stride = conv_in_stride; a.conv_channels = conv_channels;
-  a.conv_taps = conv_taps; a.conv_state_off = conv_state_off;
-  if (dtype == R2_F32) return launch_delta<float>(a, n_entries, n_heads, stream);
-  if (dtype == R2_BF16) return launch_delta<bf16>(a, n_entries, n_heads, stream);
-  return R2_BAD_DTYPE;
-}
-
-// Time mixing with a decay per channel: o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T
-// with w = exp(-exp(decay_log)). r, k, v [T, heads * dim]; decay_log float [T, heads * dim]; bonus float [heads * dim]. State per
-// slot: S [heads][dim][dim] and, at row_state_off, the input row of the sequence's last position [row_width], which this kernel
-// renews from row_in (this step's input rows). out [T, heads * dim] float.
-extern "C" int r2_time_mix_scan(const void* r, int r_stride, const void* k, int k_stride, const void* v, int v_stride,
-                                const float* decay_log, int decay_stride, const float* bonus, float* state, long long slot_stride,
-                                const int32_t* q_start, const int32_t* state_slot, const int32_t* fresh, int n_entries, float* out,
-                                int out_stride, int n_heads, int dim, const void* row_in, int row_in_stride, int row_width,
-                                long long row_state_off, int single_rows, int dtype, cudaStream_t stream) {
-  if (n_entries <= 0) return R2_OK;
-  if (n_heads < 1 || dim < 1) return R2_BAD_SHAPE;
-  ScanArgs a = {};
-  a.read = r; a.read_stride = r_stride; a.write = k; a.write_stride = k_stride; a.value = v; a.value_stride = v_stride;
-  a.channel_log = decay_log; a.channel_log_stride = decay_stride; a.bonus = bonus; a.read_scale = 1.f;
-  a.state = state; a.slot_stride = slot_stride; a.head_stride = dim * dim;
-  a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh; a.out = out; a.out_stride = out_stride;
-  a.heads_per_group = 1; a.rows = dim; a.cols = dim; a.single_rows = single_rows;
-  a.conv_in = row_in; a.conv_in_stride = row_in_stride; a.conv_channels = row_width; a.conv_taps = 2; a.conv_state_off = row_state_off;
-  if (dtype == R2_F32) return launch_scan<float, MODE_CHANNEL>(a, n_entries, n_heads, stream);
-  if (dtype == R2_BF16) return launch_scan<bf16, MODE_CHANNEL>(a, n_entries, n_heads, stream);
-  return R2_BAD_DTYPE;
-}
-
-// h [T, width]; mu float [n_mixes (+ 1 with out_float)][width]; out [T][n_mixes][width]; out_float [T][width] or null; state: the row
-// before an entry's first at row_off of its slot.
-extern "C" int r2_shift_mix(const void* h, int h_stride, const float* mu, int n_mixes, void* out, float* out_float, int n_rows, int width,
-                            const float* state, long long slot_stride, long long row_off, const int32_t* row_entry,
-                            const int32_t* q_start, const int32_t* state_slot, const int32_t* fresh, int dtype, cudaStream_t stream) {
-  if (n_rows <= 0) return R2_OK;
-  if (width < 1 || n_mixes < 0) return R2_BAD_SHAPE;
-  dim3 grid(n_rows, (width + 1023) / 1024);
-  if (dtype == R2_F32) {
-    r2_launch(shift_mix_kernel<float>, grid, dim3(256), size_t(0), stream, (const float*)h, h_stride, mu, n_mixes, (float*)out, out_float,
-              width, state, slot_stride, row_off, row_entry, q_start, state_slot, fresh);
-  } else if (dtype == R2_BF16) {
-    r2_launch(shift_mix_kernel<bf16>, grid, dim3(256), size_t(0), stream, (const bf16*)h, h_stride, mu, n_mixes, (bf16*)out, out_float,
-              width, state, slot_stride, row_off, row_entry, q_start, state_slot, fresh);
-  } else {
-    return R2_BAD_DTYPE;
-  }
-  return launch_status();
 }
 
 extern "C" int r2_causal_conv(const void* in, int in_stride, void* out, int out_stride, const float* taps, const float* bias,

@@ -16,9 +16,8 @@ import torch
 from ..csrc.build import kernel_library
 
 F32, BF16 = 0, 1
-ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF, ACT_TANH = 0, 1, 2, 3
-# ("tanh" is taken by the CUDA-core products: a small matrix inside a gate, never a wide tensor-core product)
-ACTIVATIONS = {None: ACT_NONE, "none": ACT_NONE, "gelu_new": ACT_GELU_TANH, "gelu": ACT_GELU_ERF, "tanh": ACT_TANH}
+ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF = 0, 1, 2
+ACTIVATIONS = {None: ACT_NONE, "none": ACT_NONE, "gelu_new": ACT_GELU_TANH, "gelu": ACT_GELU_ERF}
 
 _STATUS = {-1: "unsupported dtype", -2: "bad shape", -3: "bad alignment", -4: "unsupported size or option"}
 
@@ -144,7 +143,7 @@ def _lib(source: str) -> C.CDLL:
 def build_all(head_dims=()) -> None:
     """Compile every kernel library that does not depend on a model, and the attention kernels
     for the given head sizes (a model compiles its own head size at first use otherwise)."""
-    for source in ("rowwise", "recurrent", "routing", "gemm_simt", "gemm_tc", "attention_simt", "attention_prefill_tc", "latent_attention",
+    for source in ("rowwise", "recurrent", "state_scan", "routing", "gemm_simt", "gemm_tc", "attention_simt", "attention_prefill_tc", "latent_attention",
                    "sampling", "wait_selftest"):
         _lib(source)
     kernel_library("sfu_probe")  # (profiling/sfu_probe.py: a measurement, no part of a step)
@@ -527,11 +526,9 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
     return out
 
 
-def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, out: torch.Tensor | None = None,
-                 act: str | None = None) -> torch.Tensor:
+def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
     """h [T, K] (any compute dtype) times w [N, K] float32 (+ bias float32) -> float32 [T, N]: the few outputs per row
-    that must stay in 32-bit (gates of a recurrence, one gate per head, step sizes), each one warp's sum; `act` (see
-    ACTIVATIONS) is applied to them."""
+    that must stay in 32-bit (gates of a recurrence, one gate per head, step sizes), each one warp's sum."""
     _need(h, "h", dim=2)
     _need(w, "w", torch.float32, 2)
     if w.shape[1] != h.shape[1] or not w.is_contiguous():
@@ -543,7 +540,7 @@ def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = N
     if out is None:
         out = torch.empty(h.shape[0], w.shape[0], dtype=torch.float32, device=h.device)
     status = _lib("routing").r2_small_linear(_p(h), _rows(h, "h"), _p(w), _p(bias), _p(out), _rows(out, "out"), h.shape[0],
-                                            w.shape[0], h.shape[1], ACTIVATIONS[act], dtype_code(h.dtype), _stream())
+                                            w.shape[0], h.shape[1], dtype_code(h.dtype), _stream())
     _check(status, "small_linear")
     return out
 
@@ -871,7 +868,7 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor | None, 
     """silu of a causal convolution per channel: x [T, C] (a slice of a projection), taps float32 [C, n_taps] whose last
     column is the current token's. Inputs before an entry's first row come from the request's state slot (float32
     [slots, floats]; at `conv_state_off` the inputs of the last n_taps - 1 positions, [n_taps - 1, C]), zeros before a
-    sequence's start. The slot is read only: `ssd_scan` or `delta_scan` renews it. -> [T, C] in x's dtype."""
+    sequence's start. The slot is read only: `ssd_scan` renews it. -> [T, C] in x's dtype."""
     _need(x, "x", dim=2)
     _need(taps, "taps", torch.float32, 2)
     _need(state, "state", torch.float32, 2)
@@ -928,80 +925,110 @@ def ssd_scan(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, steps: torch.Ten
     return out
 
 
-def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, step_bias: torch.Tensor, log_rate: torch.Tensor,
-               q_scale: float, unit_eps: float, state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor,
-               n_heads: int, n_groups: int, dim: int, vdim: int, conv_in: torch.Tensor | None = None, conv_taps: int = 1,
-               conv_state_off: int = 0) -> torch.Tensor:
-    """The gated delta rule for every entry of a batch, from and to the entries' state slots:
+def delta_prepare(raw: torch.Tensor, h: torch.Tensor, taps: torch.Tensor, w_gates: torch.Tensor, step_bias: torch.Tensor, log_rate: torch.Tensor,
+                  q_scale: float, unit_eps: float, n_heads: int, n_groups: int, dim: int, vdim: int, state: torch.Tensor, conv_off: int,
+                  row_entry: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor):
+    """What the gated delta rule walks over, in one launch and in float32. raw [T, 2 groups dim + heads vdim]: the projections of q, k and v;
+    h [T, D]: the layer's input. The causal convolution per channel (taps float32 [channels, n], the last column the current row's;
+    inputs before an entry's first row from the request's state slot at `conv_off`, zeros before a sequence's start; the slot is
+    only read) and silu; q and k made unit vectors, x / sqrt(sum x^2 + unit_eps), q times q_scale; with (b, a) = w_gates h (float32 [2 heads, D])
+    beta = sigmoid(b), g = exp(-exp(log_rate) softplus(a + step_bias)).
+    -> (qk float32 [T, groups, 2, dim rounded up to 4], v float32 [T, heads * vdim], numbers float32 [T, heads, 4]: g, beta, k . q, 0)."""
+    _entries(q_start, state_slot, fresh)
+    channels, n_taps = taps.shape
+    for name, t, dim_ in (("taps", taps, 2), ("w_gates", w_gates, 2), ("step_bias", step_bias, 1), ("log_rate", log_rate, 1), ("state", state, 2)):
+        _need(t, name, torch.float32, dim_)
+        if not t.is_contiguous():
+            raise KernelError(f"delta_prepare: {name} must be contiguous")
+    _need(raw, "raw", dim=2)
+    _need(h, "h", raw.dtype, 2)
+    _need(row_entry, "row_entry", torch.int32, 1)
+    if (n_heads % n_groups or channels != 2 * n_groups * dim + n_heads * vdim or raw.shape[1] != channels or h.shape[0] != raw.shape[0]
+            or tuple(w_gates.shape) != (2 * n_heads, h.shape[1]) or step_bias.shape[0] != n_heads or log_rate.shape[0] != n_heads
+            or row_entry.shape[0] < raw.shape[0] or conv_off + (n_taps - 1) * channels > state.shape[1]):
+        raise KernelError(f"delta_prepare: raw {tuple(raw.shape)}, taps {tuple(taps.shape)}, w_gates {tuple(w_gates.shape)}, state {tuple(state.shape)} do not "
+                          f"fit {n_heads} heads, {n_groups} groups of {dim} x {vdim}")
+    t, dim4 = raw.shape[0], -(-dim // 4) * 4
+    qk = torch.empty(t, n_groups, 2, dim4, dtype=torch.float32, device=raw.device)
+    v = torch.empty(t, n_heads * vdim, dtype=torch.float32, device=raw.device)
+    numbers = torch.empty(t, n_heads, 4, dtype=torch.float32, device=raw.device)
+    status = _lib("state_scan").r2_delta_prepare(
+        _p(raw), _rows(raw, "raw"), _p(h), _rows(h, "h"), h.shape[1], _p(taps), n_taps, _p(w_gates), _p(step_bias), _p(log_rate), C.c_float(q_scale),
+        C.c_float(unit_eps), n_heads, n_groups, dim, vdim, t, _p(qk), _p(v), _p(numbers), _p(state), C.c_longlong(state.shape[1]),
+        C.c_longlong(conv_off), _p(row_entry), _p(q_start), _p(state_slot), _p(fresh), sm_count(raw.device), dtype_code(raw.dtype), _stream())
+    _check(status, "delta_prepare")
+    return qk, v, numbers
+
+
+def delta_scan(qk: torch.Tensor, v: torch.Tensor, numbers: torch.Tensor, dim: int, state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor,
+               fresh: torch.Tensor, conv_in: torch.Tensor | None = None, conv_taps: int = 1, conv_state_off: int = 0) -> torch.Tensor:
+    """The gated delta rule over what `delta_prepare` made, for every entry of a batch, from and to the entries' state slots:
 
         S' = g S, u = beta (v - S'^T k), S = S' + k u^T, o = S^T q
-        q, k made unit vectors (x / sqrt(sum x^2 + unit_eps)), q times q_scale; beta = sigmoid(gates[:, :H]);
-        g = exp(-exp(log_rate) softplus(gates[:, H:] + step_bias))
 
-    q, k [T, groups * dim], v [T, heads * vdim] (slices of a projection; head h uses the q and k of group h // (heads / groups));
-    gates float32 [T, 2 heads]; state float32 [slots, floats]: S [heads, dim, vdim] first, and with `conv_in` the convolution's last
-    inputs at `conv_state_off`, renewed as by `ssd_scan`. -> float32 [T, heads * vdim], the heads' outputs before their norm."""
+    state float32 [slots, floats]: S [heads, dim, vdim] first, and with `conv_in` ([T, channels], this step's inputs of the convolution) the
+    last conv_taps - 1 inputs at `conv_state_off`, which are renewed. Head h uses the q and k of group h // (heads / groups).
+    -> float32 [T, heads * vdim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
-    if n_heads % n_groups:
-        raise KernelError(f"delta_scan: {n_heads} heads do not share {n_groups} groups of queries and keys")
-    for name, t, width in (("q", q, n_groups * dim), ("k", k, n_groups * dim), ("v", v, n_heads * vdim)):
-        _need(t, name, q.dtype, 2)
-        if t.shape[1] != width or t.shape[0] != q.shape[0]:
-            raise KernelError(f"delta_scan: {name} {tuple(t.shape)} is not [T, {width}]")
-    _need(gates, "gates", torch.float32, 2)
-    _need(state, "state", torch.float32, 2)
-    for name, t in (("step_bias", step_bias), ("log_rate", log_rate)):
-        _need(t, name, torch.float32, 1)
-        if t.shape[0] != n_heads:
-            raise KernelError(f"delta_scan: {name} {tuple(t.shape)} is not [{n_heads}]")
-    if gates.shape != (q.shape[0], 2 * n_heads) or state.shape[1] < n_heads * dim * vdim or not state.is_contiguous():
-        raise KernelError(f"delta_scan: gates {tuple(gates.shape)} / state {tuple(state.shape)} do not fit {n_heads} heads of {dim} x {vdim}")
-    channels = 0
+    for name, t, dims in (("qk", qk, 4), ("v", v, 2), ("numbers", numbers, 3), ("state", state, 2)):
+        _need(t, name, torch.float32, dims)
+        if not t.is_contiguous():
+            raise KernelError(f"delta_scan: {name} must be contiguous")
+    t, groups, heads = qk.shape[0], qk.shape[1], numbers.shape[1]
+    vdim = v.shape[1] // heads
+    if (qk.shape[2] != 2 or qk.shape[3] != -(-dim // 4) * 4 or heads % groups or v.shape != (t, heads * vdim) or numbers.shape != (t, heads, 4)
+            or state.shape[1] < heads * dim * vdim):
+        raise KernelError(f"delta_scan: qk {tuple(qk.shape)}, v {tuple(v.shape)}, numbers {tuple(numbers.shape)}, state {tuple(state.shape)} do not fit each other")
+    channels, in_dtype = 0, F32
     if conv_in is not None:
-        _need(conv_in, "conv_in", q.dtype, 2)
-        channels = conv_in.shape[1]
-        if conv_state_off < n_heads * dim * vdim or conv_state_off + (conv_taps - 1) * channels > state.shape[1]:
+        _need(conv_in, "conv_in", dim=2)
+        channels, in_dtype = conv_in.shape[1], dtype_code(conv_in.dtype)
+        if conv_state_off < heads * dim * vdim or conv_state_off + (conv_taps - 1) * channels > state.shape[1]:
             raise KernelError("delta_scan: the convolution's state does not fit the slot")
-    out = torch.empty(q.shape[0], n_heads * vdim, dtype=torch.float32, device=q.device)
-    status = _lib("recurrent").r2_delta_scan(
-        _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(gates), _rows(gates, "gates"), _p(step_bias), _p(log_rate),
-        C.c_float(q_scale), C.c_float(unit_eps), _p(state), C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out),
-        _rows(out, "out"), n_heads, n_groups, dim, vdim, _p(conv_in), 0 if conv_in is None else _rows(conv_in, "conv_in"), channels,
-        conv_taps, C.c_longlong(conv_state_off), int(q.shape[0] <= n), dtype_code(q.dtype), _stream())
+    out = torch.empty(t, heads * vdim, dtype=torch.float32, device=qk.device)
+    status = _lib("state_scan").r2_delta_scan(
+        _p(qk), _p(v), _p(numbers), _p(state), C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out), _rows(out, "out"),
+        heads, groups, dim, vdim, _p(conv_in), 0 if conv_in is None else _rows(conv_in, "conv_in"), channels, conv_taps, C.c_longlong(conv_state_off),
+        in_dtype, int(t <= n), sm_count(qk.device), _stream())
     _check(status, "delta_scan")
     return out
 
 
-def shift_mix(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, row_off: int, row_entry: torch.Tensor, q_start: torch.Tensor,
-              state_slot: torch.Tensor, fresh: torch.Tensor, float_last: bool = False):
-    """Mixes of every row with the row before it in its sequence: h + (h' - h) mu[s]. h [T, D]; mu float32 [n, D]; the row before an
-    entry's first comes from the request's state slot (float32 [slots, floats], at `row_off`; zeros before a sequence's start; the slot
-    is only read: `time_mix_scan` renews it). -> ([T, n, D] in h's dtype, None), or with `float_last` ([T, n - 1, D], the last mix
-    in float32 [T, D])."""
+def time_mix_prepare(h: torch.Tensor, mu: torch.Tensor, w1: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, state: torch.Tensor, row_off: int,
+                     row_entry: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor):
+    """Mixes of every row with the row before it in its sequence, mix_s = h + (h' - h) mu[s], and the decays made from the last of
+    them: decay = exp(-exp(w0 + W2 tanh(W1 mix_last))). h [T, D]; mu float32 [n, D]; w1 float32 [rank, D], w2t float32 [rank, N] (W2 transposed), w0
+    float32 [N]. The row before an entry's first comes from the request's state slot (float32 [slots, floats], at `row_off`; zeros
+    before a sequence's start; the slot is only read: `time_mix_scan` renews it). The decays' way is float32 throughout.
+    -> (the other mixes [T, n - 1, D] in h's dtype, decay float32 [T, N])."""
     _need(h, "h", dim=2)
-    _need(mu, "mu", torch.float32, 2)
-    _need(state, "state", torch.float32, 2)
+    for name, t, dim in (("mu", mu, 2), ("w1", w1, 2), ("w2t", w2t, 2), ("w0", w0, 1), ("state", state, 2)):
+        _need(t, name, torch.float32, dim)
+        if not t.is_contiguous():
+            raise KernelError(f"time_mix_prepare: {name} must be contiguous")
     _need(row_entry, "row_entry", torch.int32, 1)
     _entries(q_start, state_slot, fresh)
     n, width = mu.shape
-    if width != h.shape[1] or not mu.is_contiguous() or row_off + width > state.shape[1]:
-        raise KernelError(f"shift_mix: h {tuple(h.shape)}, mu {tuple(mu.shape)}, state {tuple(state.shape)} do not fit")
-    n_mixes = n - 1 if float_last else n
-    out = torch.empty(h.shape[0], n_mixes, width, dtype=h.dtype, device=h.device)
-    last = torch.empty(h.shape[0], width, dtype=torch.float32, device=h.device) if float_last else None
-    status = _lib("recurrent").r2_shift_mix(
-        _p(h), _rows(h, "h"), _p(mu), n_mixes, _p(out), _p(last), h.shape[0], width, _p(state), C.c_longlong(state.shape[1]),
-        C.c_longlong(row_off), _p(row_entry), _p(q_start), _p(state_slot), _p(fresh), dtype_code(h.dtype), _stream())
-    _check(status, "shift_mix")
-    return out, last
+    rank, n_out = w2t.shape
+    if n < 1 or width != h.shape[1] or tuple(w1.shape) != (rank, width) or w0.shape[0] != n_out or row_off + width > state.shape[1] or row_entry.shape[0] < h.shape[0]:
+        raise KernelError(f"time_mix_prepare: h {tuple(h.shape)}, mu {tuple(mu.shape)}, w1 {tuple(w1.shape)}, w2t {tuple(w2t.shape)}, w0 {tuple(w0.shape)}, "
+                          f"state {tuple(state.shape)} do not fit")
+    out = torch.empty(h.shape[0], n - 1, width, dtype=h.dtype, device=h.device)
+    decay = torch.empty(h.shape[0], n_out, dtype=torch.float32, device=h.device)
+    status = _lib("state_scan").r2_time_mix_prepare(
+        _p(h), _rows(h, "h"), _p(mu), n - 1, _p(out), h.shape[0], width, _p(w1), _p(w2t), _p(w0), rank, n_out, _p(decay), _p(state),
+        C.c_longlong(state.shape[1]), C.c_longlong(row_off), _p(row_entry), _p(q_start), _p(state_slot), _p(fresh), sm_count(h.device),
+        dtype_code(h.dtype), _stream())
+    _check(status, "time_mix_prepare")
+    return out, decay
 
 
-def time_mix_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_log: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor,
+def time_mix_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor,
                   q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor, n_heads: int, dim: int,
                   row_in: torch.Tensor | None = None, row_state_off: int = 0) -> torch.Tensor:
     """Time mixing with a decay per channel for every entry of a batch, from and to the entries' state slots:
-    o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, S_t = diag(exp(-exp(decay_log_t))) S_(t-1) + k_t v_t^T. r, k, v [T, heads * dim];
-    decay_log float32 [T, heads * dim]; bonus float32 [heads * dim]; state float32 [slots, floats]: S [heads, dim, dim] first, and with
+    o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, S_t = diag(decay_t) S_(t-1) + k_t v_t^T. r, k, v [T, heads * dim];
+    decay float32 [T, heads * dim]; bonus float32 [heads * dim]; state float32 [slots, floats]: S [heads, dim, dim] first, and with
     `row_in` (this step's input rows [T, D]) the last position's input row at `row_state_off`, which is renewed.
     -> float32 [T, heads * dim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
@@ -1010,21 +1037,21 @@ def time_mix_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_log: 
         _need(t, name, r.dtype, 2)
         if t.shape != (r.shape[0], width):
             raise KernelError(f"time_mix_scan: {name} {tuple(t.shape)} is not [T, {width}]")
-    _need(decay_log, "decay_log", torch.float32, 2)
+    _need(decay, "decay", torch.float32, 2)
     _need(bonus, "bonus", torch.float32)
     _need(state, "state", torch.float32, 2)
-    if decay_log.shape != r.shape or bonus.numel() != width or not bonus.is_contiguous() or state.shape[1] < width * dim or not state.is_contiguous():
-        raise KernelError(f"time_mix_scan: decay_log {tuple(decay_log.shape)} / bonus {tuple(bonus.shape)} / state {tuple(state.shape)} do not fit {n_heads} heads of {dim}")
+    if decay.shape != r.shape or bonus.numel() != width or not bonus.is_contiguous() or state.shape[1] < width * dim or not state.is_contiguous():
+        raise KernelError(f"time_mix_scan: decay {tuple(decay.shape)} / bonus {tuple(bonus.shape)} / state {tuple(state.shape)} do not fit {n_heads} heads of {dim}")
     if row_in is not None:
         _need(row_in, "row_in", r.dtype, 2)
         if row_state_off < width * dim or row_state_off + row_in.shape[1] > state.shape[1]:
             raise KernelError("time_mix_scan: the last input row does not fit the slot")
     out = torch.empty(r.shape[0], width, dtype=torch.float32, device=r.device)
-    status = _lib("recurrent").r2_time_mix_scan(
-        _p(r), _rows(r, "r"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay_log), _rows(decay_log, "decay_log"), _p(bonus), _p(state),
+    status = _lib("state_scan").r2_time_mix_scan(
+        _p(r), _rows(r, "r"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), _rows(decay, "decay"), _p(bonus), _p(state),
         C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out), _rows(out, "out"), n_heads, dim, _p(row_in),
         0 if row_in is None else _rows(row_in, "row_in"), 0 if row_in is None else row_in.shape[1], C.c_longlong(row_state_off),
-        int(r.shape[0] <= n), dtype_code(r.dtype), _stream())
+        int(r.shape[0] <= n), sm_count(r.device), dtype_code(r.dtype), _stream())
     _check(status, "time_mix_scan")
     return out
 
@@ -1236,7 +1263,7 @@ def linear(a, w: torch.Tensor, bias: torch.Tensor | None = None, *, w_is_nk: boo
 
 def grouped_linear(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """Several products whose inputs lie side by side: a [T, n, K], w [n * N, K] (stored [out, in], the groups' matrices one after the
-    other) -> [T, n * N] whose columns s * N .. (s + 1) * N - 1 are a[:, s] @ w[s * N: (s + 1) * N]^T, in a's dtype."""
+    other) -> [T, n * N] in one launch where the groups are multiples of a tile, whose columns s * N .. (s + 1) * N - 1 are a[:, s] @ w[s * N: (s + 1) * N]^T, in a's dtype."""
     _need(a, "a", dim=3)
     t, n, k = a.shape
     if not a.is_contiguous() or w.shape[0] % n or w.shape[1] != k:
@@ -1244,7 +1271,14 @@ def grouped_linear(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     per = w.shape[0] // n
     out = torch.empty(t, n * per, dtype=a.dtype, device=a.device)
     flat = a.view(t, n * k)
-    for s in range(n):
+    if a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and _tensor_core_gemm and n > 1:
+        _need(w, "w", dim=2)
+        status = _lib("gemm_tc").r2_gemm_tc_grouped(_p(flat), n * k, _p(w), _rows(w, "w"), _p(out), n * per, t, per, k, n, BF16,
+                                                    _p(_workspace(a.device).error), _stream())
+        if status != -4:
+            _check(status, "grouped_linear (tensor cores)")
+            return out
+    for s in range(n):   # (groups that are no multiple of a tile, and the CUDA-core products)
         linear(flat[:, s * k: (s + 1) * k], w[s * per: (s + 1) * per], None, w_is_nk=True, out=out[:, s * per: (s + 1) * per])
     return out
 

@@ -3,7 +3,7 @@ a matrix memory with exponential gates (mLSTM), retention (linear attention with
 state-space layer with a short causal convolution (the recurrence of Mamba-2), the gated delta rule behind short convolutions
 and time mixing with a decay per channel (RWKV's). Their state lives in 32-bit floats in the request's state slot, starts at
 zero with a sequence's first token and is carried from step to step; prompts, portions and single decoded
-tokens run through the same kernels (csrc/kernels/recurrent.cu), entry by entry, row by row.
+tokens run through the same kernels (csrc/kernels/recurrent.cu, state_scan.cu), entry by entry, row by row.
 
 All offer `mix(h, ctx, cache, state)`, the mixer's output [T, D] in float32 without the residual stream,
 for an arrangement that joins several mixers, beside the usual `forward`, whose last product adds the stream.
@@ -212,13 +212,13 @@ class DeltaRule:
         S' = g S, u = beta (v - S'^T k), S = S' + k u^T, o = S^T q            (S: [head_dim x v_head_dim], from zero)
 
     Each head's o is divided by its root mean square, times `norm` [v_head_dim] (shared by the heads), times silu(W_g h); then W_o. The
-    state is S and the convolutions' last conv_taps - 1 inputs. The convolutions' outputs have the compute dtype; everything after
-    them is float32.
+    state is S and the convolutions' last conv_taps - 1 inputs. Everything after the
+    projections is float32.
 
     params: n_heads, n_groups, head_dim, v_head_dim, conv_taps, unit_eps, norm_eps.
     weights (stored [out, in], no biases): w_q, w_k [groups head_dim, D], w_v, w_gate [H v_head_dim, D], w_out [D, H v_head_dim], conv_q,
     conv_k [groups head_dim, taps], conv_v [H v_head_dim, taps], w_b, w_a [H, D], a_log, dt_bias [H], norm [v_head_dim].
-    The four wide projections run as one product, the strengths and step sizes as a 32-bit one, the three convolutions as one launch."""
+    The four wide projections run as one product; one launch prepares what the recurrence walks over."""
 
     def __init__(self, params: dict, weights: dict, rt: Runtime):
         self.n_heads, self.n_groups = int(params["n_heads"]), int(params["n_groups"])
@@ -253,13 +253,12 @@ class DeltaRule:
 
     def _inner(self, h, ctx, state):
         proj = ops.linear(h, self.w_in, None, w_is_nk=True)
-        gates = ops.small_linear(h, self.w_gates, None)
         raw = proj[:, : self.channels]
-        mixed = ops.causal_conv(raw, self.conv, None, state, self.conv_state_off, ctx.row_entry, ctx.q_start, ctx.state_slot, ctx.fresh)
-        a, b = self.qk_width, 2 * self.qk_width
-        o = ops.delta_scan(mixed[:, :a], mixed[:, a:b], mixed[:, b:], gates, self.dt_bias, self.a_log, self.head_dim ** -0.5, self.unit_eps,
-                           state, ctx.q_start, ctx.state_slot, ctx.fresh, self.n_heads, self.n_groups, self.head_dim, self.v_head_dim,
-                           conv_in=raw, conv_taps=self.conv_taps, conv_state_off=self.conv_state_off)
+        qk, v, numbers = ops.delta_prepare(raw, h, self.conv, self.w_gates, self.dt_bias, self.a_log, self.head_dim ** -0.5, self.unit_eps, self.n_heads,
+                                           self.n_groups, self.head_dim, self.v_head_dim, state, self.conv_state_off, ctx.row_entry, ctx.q_start,
+                                           ctx.state_slot, ctx.fresh)
+        o = ops.delta_scan(qk, v, numbers, self.head_dim, state, ctx.q_start, ctx.state_slot, ctx.fresh, conv_in=raw, conv_taps=self.conv_taps,
+                           conv_state_off=self.conv_state_off)
         return ops.group_norm_gated(o, proj[:, self.channels:], self.norm, self.n_heads, self.norm_eps, "silu_after", proj.dtype)
 
     def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
@@ -298,7 +297,7 @@ class TimeMix:
         self.w_in = matrix(torch.cat(stacked, dim=0), rt)      # [4 H head_dim, D], the rows of each kind read a mix of their own
         self.w_out = matrix(weights["w_out"], rt)
         self.mu = vector(torch.stack([weights["mu_" + s] for s in "rkvgw"]), rt)
-        self.w1, self.w2, self.w0 = vector(w1, rt), vector(w2, rt), vector(weights["w0"], rt)
+        self.w1, self.w2t, self.w0 = vector(w1, rt), vector(w2.to(torch.float32).T.contiguous(), rt), vector(weights["w0"], rt)
         self.bonus = vector(weights["bonus"].reshape(-1), rt)
         self.norm = vector(weights["norm"], rt) * float(params.get("out_scale", 1.0))
         self.row_state_off = self.inner_width * self.head_dim
@@ -315,16 +314,11 @@ class TimeMix:
 
     def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None):
         """The gated heads' outputs [T, H head_dim] before w_out (into `out` where given)."""
-        mixes, mix_w = ops.shift_mix(h, self.mu, state, self.row_state_off, ctx.row_entry, ctx.q_start, ctx.state_slot, ctx.fresh, float_last=True)
+        mixes, decay = ops.time_mix_prepare(h, self.mu, self.w1, self.w2t, self.w0, state, self.row_state_off, ctx.row_entry, ctx.q_start,
+                                                ctx.state_slot, ctx.fresh)
         n = self.inner_width
         proj = ops.grouped_linear(mixes, self.w_in)
-        if h.dtype == torch.bfloat16 and h.shape[0] <= 64:   # a warp per output; many rows share the matrices in tiles
-            low = ops.small_linear(mix_w, self.w1, None, act="tanh")
-            decay_log = ops.small_linear(low, self.w2, self.w0)
-        else:
-            low = ops.linear(mix_w, self.w1, None, w_is_nk=True, act="tanh")
-            decay_log = ops.linear(low, self.w2, self.w0, w_is_nk=True)
-        o = ops.time_mix_scan(proj[:, :n], proj[:, n: 2 * n], proj[:, 2 * n: 3 * n], decay_log, self.bonus, state, ctx.q_start, ctx.state_slot,
+        o = ops.time_mix_scan(proj[:, :n], proj[:, n: 2 * n], proj[:, 2 * n: 3 * n], decay, self.bonus, state, ctx.q_start, ctx.state_slot,
                               ctx.fresh, self.n_heads, self.head_dim, row_in=h, row_state_off=self.row_state_off)
         return ops.group_norm_gated(o, proj[:, 3 * n:], self.norm, self.n_heads, self.norm_eps, "silu_after", proj.dtype, out=out)
 
