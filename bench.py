@@ -1091,15 +1091,16 @@ def lagelorn_points(args, pk: dict) -> dict:
         conv_w, conv_b = torch.randn(channels, taps, device=dev) * 0.3, torch.zeros(channels, device=dev)
         off = h * hd * hd
         state = torch.zeros(n_entries, off + (taps - 1) * channels, device=dev)
-        gates, per_head, w_gates = torch.randn(t, 2 * h, device=dev), torch.zeros(h, device=dev), torch.randn(2 * h, d, device=dev) * 0.02
+        gates, per_head, w_gates = torch.randn(t, 2 * h, device=dev), torch.zeros(h, device=dev), (torch.randn(2 * h, d, device=dev) * 0.02).to(bf)
+        w_gates_32 = w_gates.float()
         prepare = lambda: ops.delta_prepare(raw[:, :channels], hrow, conv_w, w_gates, per_head, per_head, hd ** -0.5, 1e-6, h, kvh, hd, hd, state, off,  # noqa: E731
                                             row_entry, q_start, slots, fresh)
         qk_f, v_f, numbers = prepare()
         add(f"delta rule: convolutions + silu of {channels:,} channels, unit vectors, strengths and decays, {label}", prepare,
-            n_bytes=t * (channels * 6 + d * 2 + h * 16) + w_gates.numel() * 4)
+            n_bytes=t * (channels * 6 + d * 2 + h * 16) + w_gates.numel() * 2)
         add(f"its like: convolution + silu alone, {channels:,} channels (Bosenex), {label}",
             lambda: ops.causal_conv(raw[:, :channels], conv_w, conv_b, state, off, row_entry, q_start, slots, fresh), n_bytes=t * channels * 4)
-        add(f"its like: gates in 32-bit alone, {2 * h} outputs (Bosenex), {label}", lambda: ops.small_linear(hrow, w_gates, None), n_bytes=t * d * 2 + w_gates.numel() * 4)
+        add(f"its like: gates in 32-bit alone, {2 * h} outputs (Bosenex), {label}", lambda: ops.small_linear(hrow, w_gates_32, None), n_bytes=t * d * 2 + w_gates.numel() * 4)
         add(f"delta rule: recurrence, {h} heads of {hd} x {hd}, {label}",
             lambda: ops.delta_scan(qk_f, v_f, numbers, hd, state, q_start, slots, fresh, conv_in=raw[:, :channels], conv_taps=taps, conv_state_off=off),
             n_bytes=t * (channels * 4 + h * 16 + d * 4) + 2 * state.numel() * 4)
@@ -1123,11 +1124,12 @@ def lagelorn_points(args, pk: dict) -> dict:
         toff = h * hd * hd
         tstate = torch.zeros(n_entries, toff + d, device=dev)
         mu = torch.rand(5, d, device=dev)
-        w1, w2t, w0 = torch.randn(DECAY_RANK, d, device=dev) * 0.02, torch.randn(DECAY_RANK, d, device=dev) * 0.1, torch.zeros(d, device=dev)
+        w1, w2t = (torch.randn(DECAY_RANK, d, device=dev) * 0.02).to(bf), (torch.randn(DECAY_RANK, d, device=dev) * 0.1).to(bf)
+        w0 = torch.zeros(d, device=dev)
         prepare = lambda: ops.time_mix_prepare(hrow, mu, w1, w2t, w0, tstate, toff, row_entry, q_start, slots, fresh)  # noqa: E731
         mixes, decay = prepare()
         add(f"time mixing: a row's mixes with the row before it, decays through an inner width of {DECAY_RANK} in 32-bit, {label}", prepare,
-            n_bytes=t * d * (2 + 8 + 4) + 8 * d * DECAY_RANK)
+            n_bytes=t * d * (2 + 8 + 4) + 4 * d * DECAY_RANK)
         w_in = (torch.randn(4 * d, d, device=dev) * 0.02).to(bf)
         add(f"time mixing: four products of {d} x {d} on their mixes, {label}", lambda: ops.grouped_linear(mixes, w_in),
             n_bytes=t * d * 16 + 8 * d * d, flops=8 * t * d * d)

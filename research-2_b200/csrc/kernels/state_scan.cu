@@ -4,7 +4,7 @@
 //   delta rule       S' = g S,  u = beta (v - S'^T k),  S = S' + k u^T,  o = S^T q         (q, k unit vectors, q scaled; g, beta per row)
 //   time mixing      o = (S + diag(bonus) k v^T)^T r,   S <- diag(w) S + k v^T             (w per row and channel)
 //
-// S is [rows x cols] per head, float, in the request's slot. A CTA owns one (entry, head, slice of the columns), takes the state from
+// S is [rows x cols] per head, float, in the request's slot, stored in pieces of four rows: [rows / 4][cols][4]. A CTA owns one (entry, head, slice of the columns), takes the state from
 // the slot (or zeros for a sequence's first rows), walks the entry's rows in order and puts the state back. A thread keeps RPT
 // rows of one column in registers, a column's rows are spread over G neighbouring lanes in pieces of four. The rows' vectors come
 // through shared memory in tiles, copied asynchronously one tile ahead. The delta rule's write needs what the state returns for
@@ -63,13 +63,6 @@ __device__ __forceinline__ void stage_rows(T* dst, int dst_stride, const T* src,
   }
 }
 
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-  const uint2 raw = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-
 // The newest keep_rows input rows of an entry: this step's, and before them what the slot held. Channel c is one thread's: it reads
 // a place before it writes over it.
 template <typename T>
@@ -87,8 +80,9 @@ __device__ __forceinline__ void keep_inputs(const StateScanArgs& a, float* slot,
     }
 }
 
-template <typename T, int RPT, int MODE>
-__global__ void __launch_bounds__(256)
+// GL: the lanes of a column where they are fixed (8, 16, 32); 0: a.G of them.
+template <typename T, int RPT, int GL, int MODE>
+__global__ void __launch_bounds__(256, 1)
 state_scan_kernel(const StateScanArgs a) {
   pdl_launch_dependents();
   // q_start, slots and fresh flags belong to the batch, which no kernel writes
@@ -103,7 +97,7 @@ state_scan_kernel(const StateScanArgs a) {
   float* head_state = slot + size_t(h) * a.head_stride;
   extern __shared__ __align__(16) uint8_t scan_smem[];
   constexpr int Q = RPT / 4;
-  const int G = a.G, cv = a.cv, rows = a.rows, cols = a.cols, tile = a.tile;
+  const int G = GL > 0 ? GL : a.G, cv = a.cv, rows = a.rows, cols = a.cols, tile = a.tile;
   const int padded = RPT * G, cvp = (cv + 7) & ~7;
   // a stage: read vectors, write vectors, values, then decays (time mixing) or row numbers (delta rule)
   const int stage_bytes = tile * ((2 * padded + cvp) * int(sizeof(T)) + (MODE == MODE_CHANNEL ? padded : 4) * 4);
@@ -143,10 +137,13 @@ state_scan_kernel(const StateScanArgs a) {
 
   // this thread's rows of its column: pieces of four, piece r4 starts at row (r4 * G + g) * 4
   float S[RPT];
+  const int n_pieces = (rows + 3) >> 2;
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) {
-    const int i = ((r >> 2) * G + g) * 4 + (r & 3);
-    S[r] = (!is_fresh && i < rows && j < cols) ? head_state[size_t(i) * cols + j] : 0.f;
+  for (int r4 = 0; r4 < Q; ++r4) {
+    const int piece = r4 * G + g;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (!is_fresh && piece < n_pieces && j < cols) v = load4(head_state + (size_t(piece) * cols + j) * 4);
+    S[r4 * 4] = v.x; S[r4 * 4 + 1] = v.y; S[r4 * 4 + 2] = v.z; S[r4 * 4 + 3] = v.w;
   }
   float bonus[MODE == MODE_CHANNEL ? RPT : 1];
   if (MODE == MODE_CHANNEL) {
@@ -182,6 +179,7 @@ state_scan_kernel(const StateScanArgs a) {
         k4[r4] = load4(ws + (r4 * G + g) * 4);
         q4[r4] = load4(rs + (r4 * G + g) * 4);
       }
+#pragma unroll 2
       for (int tt = 0; tt < nt; ++tt) {
         const int next = tt + 1 < nt ? tt + 1 : tt;
         num_n = load4(fs + next * 4);
@@ -203,6 +201,7 @@ state_scan_kernel(const StateScanArgs a) {
           }
         }
         float sk = (ak[0] + ak[1]) + (ak[2] + ak[3]), sq = (aq[0] + aq[1]) + (aq[2] + aq[3]);
+#pragma unroll
         for (int o = G >> 1; o > 0; o >>= 1) {
           sk += __shfl_xor_sync(0xffffffffu, sk, o);
           sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -244,6 +243,7 @@ state_scan_kernel(const StateScanArgs a) {
         float y[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) y[i] = one_row(tt + i);
+#pragma unroll
         for (int o = G >> 1; o > 0; o >>= 1) {
 #pragma unroll
           for (int i = 0; i < 4; ++i) y[i] += __shfl_xor_sync(0xffffffffu, y[i], o);
@@ -262,9 +262,116 @@ state_scan_kernel(const StateScanArgs a) {
     __syncthreads();  // the stage may be filled again
   }
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) {
-    const int i = ((r >> 2) * G + g) * 4 + (r & 3);
-    if (i < rows && j < cols) head_state[size_t(i) * cols + j] = S[r];
+  for (int r4 = 0; r4 < Q; ++r4) {
+    const int piece = r4 * G + g;
+    if (piece < n_pieces && j < cols)
+      *reinterpret_cast<float4*>(head_state + (size_t(piece) * cols + j) * 4) = make_float4(S[r4 * 4], S[r4 * 4 + 1], S[r4 * 4 + 2], S[r4 * 4 + 3]);
+  }
+}
+
+// The same for launches in which (nearly) every entry is one row, a decode step: nothing is staged, every thread asks for its part
+// of the state and of the row at once. The arithmetic and its order are the walk's.
+template <typename T, int RPT, int GL, int MODE>
+__global__ void __launch_bounds__(256)
+state_step_kernel(const StateScanArgs a) {
+  pdl_launch_dependents();
+  const int e = blockIdx.x, h = blockIdx.y;
+  const int row0 = a.q_start[e], row1 = a.q_start[e + 1];
+  if (row1 <= row0) {
+    pdl_wait();
+    return;
+  }
+  const bool is_fresh = a.fresh[e] != 0;
+  float* slot = a.state + size_t(a.state_slot[e]) * a.slot_stride;
+  float* head_state = slot + size_t(h) * a.head_stride;
+  constexpr int Q = RPT / 4;
+  const int G = GL > 0 ? GL : a.G, cv = a.cv, rows = a.rows, cols = a.cols;
+  const int tid = threadIdx.x, g = tid % G, j = blockIdx.z * cv + tid / G;
+  const int n_pieces = (rows + 3) >> 2, group = h / a.heads_per_group;
+  const bool has_column = j < cols;
+  pdl_wait();
+  float S[RPT];
+#pragma unroll
+  for (int r4 = 0; r4 < Q; ++r4) {
+    const int piece = r4 * G + g;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (!is_fresh && piece < n_pieces && has_column) v = load4(head_state + (size_t(piece) * cols + j) * 4);
+    S[r4 * 4] = v.x; S[r4 * 4 + 1] = v.y; S[r4 * 4 + 2] = v.z; S[r4 * 4 + 3] = v.w;
+  }
+  // four numbers of a row from dimension i on, zeros after the last
+  auto row4 = [&](const auto* p, int i) {
+    if (a.pieces) return i < rows ? load4(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    return make_float4(i < rows ? to_float(p[i]) : 0.f, i + 1 < rows ? to_float(p[i + 1]) : 0.f, i + 2 < rows ? to_float(p[i + 2]) : 0.f,
+                       i + 3 < rows ? to_float(p[i + 3]) : 0.f);
+  };
+  for (int t = row0; t < row1; ++t) {
+    const T* read = static_cast<const T*>(a.read) + size_t(t) * a.read_stride + size_t(group) * a.read_group;
+    const T* write = static_cast<const T*>(a.write) + size_t(t) * a.write_stride + size_t(group) * a.write_group;
+    const float v = has_column ? to_float(static_cast<const T*>(a.value)[size_t(t) * a.value_stride + size_t(h) * cols + j]) : 0.f;
+    float y;
+    if (MODE == MODE_DELTA) {
+      const float4 num = a.row_numbers[size_t(t) * gridDim.y + h];
+      float ak[4] = {0.f, 0.f, 0.f, 0.f}, aq[4] = {0.f, 0.f, 0.f, 0.f};
+      float4 k4[Q];
+#pragma unroll
+      for (int r4 = 0; r4 < Q; ++r4) {
+        k4[r4] = row4(write, (r4 * G + g) * 4);
+        const float4 q4 = row4(read, (r4 * G + g) * 4);
+        const float k[4] = {k4[r4].x, k4[r4].y, k4[r4].z, k4[r4].w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          S[r4 * 4 + u] *= num.x;
+          ak[u] = fmaf(S[r4 * 4 + u], k[u], ak[u]);
+          aq[u] = fmaf(S[r4 * 4 + u], q[u], aq[u]);
+        }
+      }
+      float sk = (ak[0] + ak[1]) + (ak[2] + ak[3]), sq = (aq[0] + aq[1]) + (aq[2] + aq[3]);
+#pragma unroll
+      for (int o = G >> 1; o > 0; o >>= 1) {
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      }
+      const float u_row = num.y * (v - sk);
+      y = fmaf(num.z, u_row, sq);
+#pragma unroll
+      for (int r4 = 0; r4 < Q; ++r4) {
+        const float k[4] = {k4[r4].x, k4[r4].y, k4[r4].z, k4[r4].w};
+#pragma unroll
+        for (int u = 0; u < 4; ++u) S[r4 * 4 + u] = fmaf(u_row, k[u], S[r4 * 4 + u]);
+      }
+    } else {
+      const float* decay = a.decay + size_t(t) * a.decay_stride + size_t(h) * rows;
+      const float* bonus = a.bonus + size_t(h) * rows;
+      float acc[2] = {0.f, 0.f}, own[2] = {0.f, 0.f};
+#pragma unroll
+      for (int r4 = 0; r4 < Q; ++r4) {
+        const int i = (r4 * G + g) * 4;
+        const float4 q4 = row4(read, i), k4 = row4(write, i), w4 = row4(decay, i);
+        const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, w[4] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const int r = r4 * 4 + u;
+          acc[u & 1] = fmaf(S[r], q[u], acc[u & 1]);
+          own[u & 1] = fmaf((i + u < rows ? bonus[i + u] : 0.f) * k[u], q[u], own[u & 1]);
+          S[r] = fmaf(w[u], S[r], k[u] * v);
+        }
+      }
+      y = fmaf(own[0] + own[1], v, acc[0] + acc[1]);
+#pragma unroll
+      for (int o = G >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    }
+    if (g == 0 && has_column) a.out[size_t(t) * a.out_stride + size_t(h) * cols + j] = y;
+  }
+#pragma unroll
+  for (int r4 = 0; r4 < Q; ++r4) {
+    const int piece = r4 * G + g;
+    if (piece < n_pieces && has_column)
+      *reinterpret_cast<float4*>(head_state + (size_t(piece) * cols + j) * 4) = make_float4(S[r4 * 4], S[r4 * 4 + 1], S[r4 * 4 + 2], S[r4 * 4 + 3]);
+  }
+  if (a.keep_in != nullptr) {
+    const int part = h * gridDim.z + blockIdx.z, n_parts = gridDim.y * gridDim.z;
+    if (a.keep_is_bf16) keep_inputs<bf16>(a, slot, row0, row1, is_fresh, part, n_parts);
+    else keep_inputs<float>(a, slot, row0, row1, is_fresh, part, n_parts);
   }
 }
 
@@ -291,22 +398,27 @@ int launch_state_scan(const StateScanArgs& in, int n_entries, int n_heads, int s
   const int threads = a.cv * a.G;
   const int padded = rpt * a.G, cvp = (a.cv + 7) & ~7;
   const size_t per_row = size_t(2 * padded + cvp) * sizeof(T) + size_t(MODE == MODE_CHANNEL ? padded : 4) * 4;
-  int tile = single_rows ? 1 : 32;
+  int tile = 32;
   while (tile > 1 && SCAN_STAGES * tile * per_row > 100 * 1024) tile /= 2;
   a.tile = tile;
   const size_t smem = SCAN_STAGES * tile * per_row;
   dim3 grid(n_entries, n_heads, splits);
-#define R2_STATE_SCAN(RPT_)                                                                    \
+#define R2_STATE_SCAN(RPT_, GL_)                                                               \
   do {                                                                                         \
-    if (!room_for(state_scan_kernel<T, RPT_, MODE>, smem)) return R2_UNSUPPORTED;              \
-    r2_launch(state_scan_kernel<T, RPT_, MODE>, grid, dim3(threads), smem, stream, a);         \
+    if (single_rows) {                                                                         \
+      r2_launch(state_step_kernel<T, RPT_, GL_, MODE>, grid, dim3(threads), 0, stream, a);     \
+    } else {                                                                                   \
+      if (!room_for(state_scan_kernel<T, RPT_, GL_, MODE>, smem)) return R2_UNSUPPORTED;       \
+      r2_launch(state_scan_kernel<T, RPT_, GL_, MODE>, grid, dim3(threads), smem, stream, a);  \
+    }                                                                                          \
   } while (0)
-  switch (rpt) {
-    case 4: R2_STATE_SCAN(4); break;
-    case 8: R2_STATE_SCAN(8); break;
-    case 16: R2_STATE_SCAN(16); break;
-    default: R2_STATE_SCAN(32); break;
-  }
+  if (rpt == 4 && a.G == 8) R2_STATE_SCAN(4, 8);
+  else if (rpt == 4) R2_STATE_SCAN(4, 0);
+  else if (rpt == 8) R2_STATE_SCAN(8, 8);
+  else if (rpt == 16 && a.G == 8) R2_STATE_SCAN(16, 8);
+  else if (rpt == 16 && a.G == 16) R2_STATE_SCAN(16, 16);
+  else if (rpt == 16) R2_STATE_SCAN(16, 32);
+  else R2_STATE_SCAN(32, 32);
 #undef R2_STATE_SCAN
   return launch_status();
 }
@@ -322,7 +434,7 @@ struct DeltaPrepareArgs {
   const void* in; int in_stride;              // [T, 2 groups dim + heads vdim]: the projections of q, k, v
   const void* h; int h_stride, width;         // [T, width]: the layer's input
   const float* taps; int n_taps;              // [channels][n_taps]
-  const float* w_gates;                       // [2 heads][width]: write strengths, then step sizes
+  const void* w_gates;                        // [2 heads][width] (dtype): write strengths, then step sizes
   const float* step_bias; const float* log_rate;
   float q_scale, unit_eps;
   int heads, groups, dim, vdim, n_rows;
@@ -359,11 +471,24 @@ delta_prepare_kernel(const DeltaPrepareArgs a) {
     const int r = i / wpad, c = i - r * wpad;
     rows_h[i] = (c < a.width && entry_row[r] >= 0) ? to_float(h[size_t(t0 + r) * a.h_stride + c]) : 0.f;
   }
+  // four taps and rows that all lie inside one entry behind its first three: every input is a row of this step
+  const bool inside = ROWS > 1 && a.n_taps == 4 && entry_row[0] >= 3 && entry_row[ROWS - 1] == entry_row[0] + ROWS - 1;
   for (int c = threadIdx.x; c < channels; c += PREP_THREADS) {
     float acc[ROWS];
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
-    for (int d = 0; d < a.n_taps; ++d) {
+    if (inside) {
+      float x[ROWS + 3];
+#pragma unroll
+      for (int r = 0; r < ROWS + 3; ++r) x[r] = to_float(in[size_t(t0 + r - 3) * a.in_stride + c]);
+      float tap[4];
+#pragma unroll
+      for (int d = 0; d < 4; ++d) tap[d] = a.taps[size_t(c) * 4 + d];
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+        for (int d = 0; d < 4; ++d) acc[r] = fmaf(tap[d], x[r + d], acc[r]);
+    } else for (int d = 0; d < a.n_taps; ++d) {
       const float tap = a.taps[size_t(c) * a.n_taps + d];
       const int back = a.n_taps - 1 - d;
 #pragma unroll
@@ -385,7 +510,7 @@ delta_prepare_kernel(const DeltaPrepareArgs a) {
     }
   }
   __syncthreads();
-  rows_times_matrix<ROWS, 2>(rows_h, wpad, a.w_gates, a.width, 2 * a.heads, [&](int r, int n, float sum) { gates[r * 2 * a.heads + n] = sum; });
+  rows_times_matrix<ROWS, (ROWS > 1 ? 2 : 1)>(rows_h, wpad, static_cast<const T*>(a.w_gates), a.width, 2 * a.heads, [&](int r, int n, float sum) { gates[r * 2 * a.heads + n] = sum; });
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, dim4 = (a.dim + 3) & ~3;
   for (int unit = warp; unit < ROWS * a.groups; unit += PREP_THREADS / 32) {   // a warp per row and group
     const int r = unit / a.groups, grp = unit - r * a.groups;
@@ -426,14 +551,14 @@ delta_prepare_kernel(const DeltaPrepareArgs a) {
 // an entry's first (zeros for a sequence's first). Mixes 0 .. n_mixes - 1 go to out [T][n_mixes][width] in the rows' dtype. One
 // more, with mu[n_mixes], stays in float in shared memory and becomes the row's decays on the spot:
 //
-//     decay[t] = exp(-exp(w0 + W2 tanh(W1 mix)))       W1 [rank][width], W2 stored transposed [rank][n_out], all float
+//     decay[t] = exp(-exp(w0 + W2 tanh(W1 mix)))       W1 [rank][width], W2 stored transposed [rank][n_out], sums in float
 //
 // A CTA takes ROWS rows, so that the two small matrices come out of L2 once for all of them; in the second product a thread has one
 // column of every row. A row's sums are made in the same order whatever ROWS is. The slot is only read.
 struct TimeMixPrepareArgs {
   const void* h; int h_stride, width, n_rows;
   const float* mu; int n_mixes; void* out;
-  const float* w1; const float* w2t; const float* w0; int rank, n_out; float* decay;
+  const void* w1; const void* w2t; const float* w0; int rank, n_out; float* decay;   // both matrices in the dtype
   const float* state; long long slot_stride, row_off;
   const int32_t* row_entry; const int32_t* q_start; const int32_t* state_slot; const int32_t* fresh;
 };
@@ -460,6 +585,8 @@ time_mix_prepare_kernel(const TimeMixPrepareArgs a) {
   __syncthreads();
   const T* h = static_cast<const T*>(a.h);
   T* out = static_cast<T*>(a.out);
+  // (with few rows several CTAs share them: each makes the whole inner row, and its share of the mixes and of the columns)
+  const int share = blockIdx.y, n_shares = gridDim.y;
   for (int c = threadIdx.x; c < wpad; c += PREP_THREADS) {
     const bool inside = c < width;
     float now[ROWS + 1], step[ROWS];   // now[r + 1]: row t0 + r; now[0]: the row above the first
@@ -468,7 +595,7 @@ time_mix_prepare_kernel(const TimeMixPrepareArgs a) {
     for (int r = 0; r < ROWS; ++r) now[r + 1] = (inside && kind[r] != 0) ? to_float(h[size_t(t0 + r) * a.h_stride + c]) : 0.f;
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) step[r] = (kind[r] == 1 ? now[r] : ((inside && kind[r] == 3) ? kept_row[r][c] : 0.f)) - now[r + 1];
-    for (int s = 0; s < a.n_mixes; ++s) {
+    for (int s = share; s < a.n_mixes; s += n_shares) {
       const float m = inside ? a.mu[size_t(s) * width + c] : 0.f;
 #pragma unroll
       for (int r = 0; r < ROWS; ++r)
@@ -479,18 +606,19 @@ time_mix_prepare_kernel(const TimeMixPrepareArgs a) {
     for (int r = 0; r < ROWS; ++r) mix[r * wpad + c] = fmaf(step[r], m, now[r + 1]);
   }
   __syncthreads();
-  rows_times_matrix<ROWS, 4>(mix, wpad, a.w1, width, a.rank, [&](int r, int n, float sum) { low[r * rpad + n] = tanhf(sum); });
+  rows_times_matrix<ROWS, 4>(mix, wpad, static_cast<const T*>(a.w1), width, a.rank, [&](int r, int n, float sum) { low[r * rpad + n] = tanhf(sum); });
   __syncthreads();
-  for (int n = threadIdx.x; n < a.n_out; n += PREP_THREADS) {
+  for (int n = share * PREP_THREADS + threadIdx.x; n < a.n_out; n += n_shares * PREP_THREADS) {
     float acc[ROWS];
+    const T* w2t = static_cast<const T*>(a.w2t);
     const float start = a.w0[n];
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) acc[r] = start;
-#pragma unroll 4
+#pragma unroll (ROWS == 1 ? 16 : 4)
     for (int i = 0; i < rpad; i += 4) {
       float w[4];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) w[u] = i + u < a.rank ? a.w2t[size_t(i + u) * a.n_out + n] : 0.f;
+      for (int u = 0; u < 4; ++u) w[u] = i + u < a.rank ? to_float(w2t[size_t(i + u) * a.n_out + n]) : 0.f;
 #pragma unroll
       for (int r = 0; r < ROWS; ++r) {
         const float4 l = *reinterpret_cast<const float4*>(low + r * rpad + i);
@@ -510,23 +638,23 @@ int rows_per_cta(int n_rows, int n_sms, size_t per_row) {
   return rows;
 }
 
-#define R2_PREPARE(KERNEL_, T_, ROWS_)                                                                             \
-  do {                                                                                                             \
-    if (!room_for(KERNEL_<T_, ROWS_>, per_row * ROWS_)) return R2_UNSUPPORTED;                                     \
-    r2_launch(KERNEL_<T_, ROWS_>, dim3((a.n_rows + ROWS_ - 1) / ROWS_), dim3(PREP_THREADS), per_row * ROWS_, stream, a); \
+#define R2_PREPARE(KERNEL_, T_, ROWS_)                                                                                                  \
+  do {                                                                                                                                  \
+    if (!room_for(KERNEL_<T_, ROWS_>, per_row * ROWS_)) return R2_UNSUPPORTED;                                                          \
+    r2_launch(KERNEL_<T_, ROWS_>, dim3((a.n_rows + ROWS_ - 1) / ROWS_, shares), dim3(PREP_THREADS), per_row * ROWS_, stream, a);        \
   } while (0)
-#define R2_PREPARE_ROWS(KERNEL_, T_)            \
-  do {                                          \
-    if (rows == 8) R2_PREPARE(KERNEL_, T_, 8);  \
+#define R2_PREPARE_ROWS(KERNEL_, T_)                \
+  do {                                              \
+    if (rows == 8) R2_PREPARE(KERNEL_, T_, 8);      \
     else if (rows == 4) R2_PREPARE(KERNEL_, T_, 4); \
-    else R2_PREPARE(KERNEL_, T_, 1);            \
+    else R2_PREPARE(KERNEL_, T_, 1);                \
   } while (0)
 
 }  // namespace
 
-// in [T, 2 groups dim + heads vdim], h [T, width] (dtype); everything else float: see DeltaPrepareArgs.
+// in [T, 2 groups dim + heads vdim], h [T, width], w_gates [2 heads, width] (dtype); everything else float: see DeltaPrepareArgs.
 extern "C" int r2_delta_prepare(const void* in, int in_stride, const void* h, int h_stride, int width, const float* taps, int n_taps,
-                                const float* w_gates, const float* step_bias, const float* log_rate, float q_scale, float unit_eps, int n_heads,
+                                const void* w_gates, const float* step_bias, const float* log_rate, float q_scale, float unit_eps, int n_heads,
                                 int n_groups, int dim, int vdim, int n_rows, float* qk, float* v_out, float* numbers, const float* state,
                                 long long slot_stride, long long conv_off, const int32_t* row_entry, const int32_t* q_start,
                                 const int32_t* state_slot, const int32_t* fresh, int n_sms, int dtype, cudaStream_t stream) {
@@ -540,14 +668,14 @@ extern "C" int r2_delta_prepare(const void* in, int in_stride, const void* h, in
   a.state = state; a.slot_stride = slot_stride; a.conv_off = conv_off;
   a.row_entry = row_entry; a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh;
   const size_t per_row = sizeof(float) * (size_t((width + 3) & ~3) + size_t(2) * n_groups * dim + 2 * n_heads + n_groups);
-  const int rows = rows_per_cta(n_rows, n_sms, per_row);
+  const int rows = rows_per_cta(n_rows, n_sms, per_row), shares = 1;
   if (dtype == R2_F32) R2_PREPARE_ROWS(delta_prepare_kernel, float);
   else if (dtype == R2_BF16) R2_PREPARE_ROWS(delta_prepare_kernel, bf16);
   else return R2_BAD_DTYPE;
   return launch_status();
 }
 
-// The delta rule over what r2_delta_prepare made. State per slot: S [heads][dim][vdim] and, at conv_off, the convolution's last
+// The delta rule over what r2_delta_prepare made. State per slot: S [heads][dim / 4 rounded up][vdim][4] and, at conv_off, the convolution's last
 // n_taps - 1 inputs, renewed here from conv_in [T, channels] (in_dtype). out [T, heads * vdim] float, the heads' outputs before their norm.
 extern "C" int r2_delta_scan(const float* qk, const float* v, const float* numbers, float* state, long long slot_stride, const int32_t* q_start,
                              const int32_t* state_slot, const int32_t* fresh, int n_entries, float* out, int out_stride, int n_heads, int n_groups,
@@ -556,13 +684,13 @@ extern "C" int r2_delta_scan(const float* qk, const float* v, const float* numbe
   if (n_entries <= 0) return R2_OK;
   if (n_heads < 1 || n_groups < 1 || n_heads % n_groups != 0 || dim < 1 || vdim < 1 || n_sms < 1) return R2_BAD_SHAPE;
   if (in_dtype != R2_F32 && in_dtype != R2_BF16) return R2_BAD_DTYPE;
-  if (!aligned16(qk) || !aligned16(numbers)) return R2_BAD_ALIGN;
+  if (!aligned16(qk) || !aligned16(numbers) || !aligned16(state) || slot_stride % 4 != 0) return R2_BAD_ALIGN;
   const int dim4 = (dim + 3) & ~3;
   StateScanArgs a = {};
   a.read = qk; a.read_stride = (long long)n_groups * 2 * dim4; a.read_group = 2 * dim4;
   a.write = qk + dim4; a.write_stride = a.read_stride; a.write_group = 2 * dim4;
   a.value = v; a.value_stride = (long long)n_heads * vdim; a.row_numbers = reinterpret_cast<const float4*>(numbers);
-  a.state = state; a.slot_stride = slot_stride; a.head_stride = dim * vdim; a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh;
+  a.state = state; a.slot_stride = slot_stride; a.head_stride = dim4 * vdim; a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh;
   a.out = out; a.out_stride = out_stride; a.heads_per_group = n_heads / n_groups; a.rows = dim; a.cols = vdim;
   a.pieces = dim % 4 == 0 && vdim % 4 == 0 && aligned16(v);
   a.keep_in = n_taps > 1 ? conv_in : nullptr; a.keep_in_stride = conv_in_stride; a.keep_width = conv_channels; a.keep_rows = n_taps - 1;
@@ -570,9 +698,9 @@ extern "C" int r2_delta_scan(const float* qk, const float* v, const float* numbe
   return launch_state_scan<float, MODE_DELTA>(a, n_entries, n_heads, single_rows, n_sms, stream);
 }
 
-// h [T, width]; mu float [n_mixes + 1][width]; out [T][n_mixes][width]; decay float [T][n_out]: see TimeMixPrepareArgs.
-extern "C" int r2_time_mix_prepare(const void* h, int h_stride, const float* mu, int n_mixes, void* out, int n_rows, int width, const float* w1,
-                                   const float* w2t, const float* w0, int rank, int n_out, float* decay, const float* state,
+// h [T, width], w1, w2t, out [T][n_mixes][width] (dtype); mu float [n_mixes + 1][width]; decay float [T][n_out]: see TimeMixPrepareArgs.
+extern "C" int r2_time_mix_prepare(const void* h, int h_stride, const float* mu, int n_mixes, void* out, int n_rows, int width, const void* w1,
+                                   const void* w2t, const float* w0, int rank, int n_out, float* decay, const float* state,
                                    long long slot_stride, long long row_off, const int32_t* row_entry, const int32_t* q_start,
                                    const int32_t* state_slot, const int32_t* fresh, int n_sms, int dtype, cudaStream_t stream) {
   if (n_rows <= 0) return R2_OK;
@@ -582,7 +710,8 @@ extern "C" int r2_time_mix_prepare(const void* h, int h_stride, const float* mu,
   a.w1 = w1; a.w2t = w2t; a.w0 = w0; a.rank = rank; a.n_out = n_out; a.decay = decay; a.state = state; a.slot_stride = slot_stride;
   a.row_off = row_off; a.row_entry = row_entry; a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh;
   const size_t per_row = sizeof(float) * (size_t((width + 3) & ~3) + ((rank + 3) & ~3));
-  const int rows = rows_per_cta(n_rows, n_sms, per_row);
+  const int rows = rows_per_cta(n_rows, n_sms, per_row), column_blocks = (n_out + PREP_THREADS - 1) / PREP_THREADS;
+  const int shares = 2 * n_rows > n_sms ? 1 : (column_blocks < 4 ? column_blocks : 4);
   if (dtype == R2_F32) R2_PREPARE_ROWS(time_mix_prepare_kernel, float);
   else if (dtype == R2_BF16) R2_PREPARE_ROWS(time_mix_prepare_kernel, bf16);
   else return R2_BAD_DTYPE;
@@ -590,7 +719,7 @@ extern "C" int r2_time_mix_prepare(const void* h, int h_stride, const float* mu,
 }
 
 // Time mixing: o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, S_t = diag(decay_t) S_(t-1) + k_t v_t^T. r, k, v [T, heads * dim] (dtype, row
-// strides); decay float [T, heads * dim]; bonus float [heads * dim]. State per slot: S [heads][dim][dim] and, at row_off, the input row of
+// strides); decay float [T, heads * dim]; bonus float [heads * dim]. State per slot: S [heads][dim / 4 rounded up][dim][4] and, at row_off, the input row of
 // the sequence's last position [row_width], renewed here from row_in [T, row_width] (dtype). out [T, heads * dim] float.
 extern "C" int r2_time_mix_scan(const void* r, int r_stride, const void* k, int k_stride, const void* v, int v_stride, const float* decay,
                                 int decay_stride, const float* bonus, float* state, long long slot_stride, const int32_t* q_start,
@@ -600,11 +729,12 @@ extern "C" int r2_time_mix_scan(const void* r, int r_stride, const void* k, int 
   if (n_entries <= 0) return R2_OK;
   if (n_heads < 1 || dim < 1 || n_sms < 1) return R2_BAD_SHAPE;
   if (dtype != R2_F32 && dtype != R2_BF16) return R2_BAD_DTYPE;
+  if (!aligned16(state) || slot_stride % 4 != 0) return R2_BAD_ALIGN;
   const int per = dtype == R2_BF16 ? 8 : 4;
   StateScanArgs a = {};
   a.read = r; a.read_stride = r_stride; a.read_group = dim; a.write = k; a.write_stride = k_stride; a.write_group = dim;
   a.value = v; a.value_stride = v_stride; a.decay = decay; a.decay_stride = decay_stride; a.bonus = bonus;
-  a.state = state; a.slot_stride = slot_stride; a.head_stride = dim * dim; a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh;
+  a.state = state; a.slot_stride = slot_stride; a.head_stride = ((dim + 3) & ~3) * dim; a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh;
   a.out = out; a.out_stride = out_stride; a.heads_per_group = 1; a.rows = dim; a.cols = dim;
   a.pieces = dim % per == 0 && r_stride % per == 0 && k_stride % per == 0 && v_stride % per == 0 && decay_stride % 4 == 0 && aligned16(r) &&
              aligned16(k) && aligned16(v) && aligned16(decay);

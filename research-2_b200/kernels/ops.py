@@ -931,13 +931,13 @@ def delta_prepare(raw: torch.Tensor, h: torch.Tensor, taps: torch.Tensor, w_gate
     """What the gated delta rule walks over, in one launch and in float32. raw [T, 2 groups dim + heads vdim]: the projections of q, k and v;
     h [T, D]: the layer's input. The causal convolution per channel (taps float32 [channels, n], the last column the current row's;
     inputs before an entry's first row from the request's state slot at `conv_off`, zeros before a sequence's start; the slot is
-    only read) and silu; q and k made unit vectors, x / sqrt(sum x^2 + unit_eps), q times q_scale; with (b, a) = w_gates h (float32 [2 heads, D])
+    only read) and silu; q and k made unit vectors, x / sqrt(sum x^2 + unit_eps), q times q_scale; with (b, a) = w_gates h ([2 heads, D] in h's dtype)
     beta = sigmoid(b), g = exp(-exp(log_rate) softplus(a + step_bias)).
     -> (qk float32 [T, groups, 2, dim rounded up to 4], v float32 [T, heads * vdim], numbers float32 [T, heads, 4]: g, beta, k . q, 0)."""
     _entries(q_start, state_slot, fresh)
     channels, n_taps = taps.shape
     for name, t, dim_ in (("taps", taps, 2), ("w_gates", w_gates, 2), ("step_bias", step_bias, 1), ("log_rate", log_rate, 1), ("state", state, 2)):
-        _need(t, name, torch.float32, dim_)
+        _need(t, name, raw.dtype if name == "w_gates" else torch.float32, dim_)
         if not t.is_contiguous():
             raise KernelError(f"delta_prepare: {name} must be contiguous")
     _need(raw, "raw", dim=2)
@@ -960,13 +960,19 @@ def delta_prepare(raw: torch.Tensor, h: torch.Tensor, taps: torch.Tensor, w_gate
     return qk, v, numbers
 
 
+def scan_state_floats(dim: int, vdim: int) -> int:
+    """Floats of one head's matrix in a request's slot, as `delta_scan` and `time_mix_scan` keep it: [dim / 4 rounded up][vdim][4]. (A slot
+    holds a multiple of four floats.)"""
+    return -(-dim // 4) * 4 * vdim
+
+
 def delta_scan(qk: torch.Tensor, v: torch.Tensor, numbers: torch.Tensor, dim: int, state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor,
                fresh: torch.Tensor, conv_in: torch.Tensor | None = None, conv_taps: int = 1, conv_state_off: int = 0) -> torch.Tensor:
     """The gated delta rule over what `delta_prepare` made, for every entry of a batch, from and to the entries' state slots:
 
         S' = g S, u = beta (v - S'^T k), S = S' + k u^T, o = S^T q
 
-    state float32 [slots, floats]: S [heads, dim, vdim] first, and with `conv_in` ([T, channels], this step's inputs of the convolution) the
+    state float32 [slots, floats]: the heads' matrices first (`scan_state_floats` each), and with `conv_in` ([T, channels], this step's inputs of the convolution) the
     last conv_taps - 1 inputs at `conv_state_off`, which are renewed. Head h uses the q and k of group h // (heads / groups).
     -> float32 [T, heads * vdim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
@@ -977,13 +983,13 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, numbers: torch.Tensor, dim: in
     t, groups, heads = qk.shape[0], qk.shape[1], numbers.shape[1]
     vdim = v.shape[1] // heads
     if (qk.shape[2] != 2 or qk.shape[3] != -(-dim // 4) * 4 or heads % groups or v.shape != (t, heads * vdim) or numbers.shape != (t, heads, 4)
-            or state.shape[1] < heads * dim * vdim):
+            or state.shape[1] < heads * scan_state_floats(dim, vdim)):
         raise KernelError(f"delta_scan: qk {tuple(qk.shape)}, v {tuple(v.shape)}, numbers {tuple(numbers.shape)}, state {tuple(state.shape)} do not fit each other")
     channels, in_dtype = 0, F32
     if conv_in is not None:
         _need(conv_in, "conv_in", dim=2)
         channels, in_dtype = conv_in.shape[1], dtype_code(conv_in.dtype)
-        if conv_state_off < heads * dim * vdim or conv_state_off + (conv_taps - 1) * channels > state.shape[1]:
+        if conv_state_off < heads * scan_state_floats(dim, vdim) or conv_state_off + (conv_taps - 1) * channels > state.shape[1]:
             raise KernelError("delta_scan: the convolution's state does not fit the slot")
     out = torch.empty(t, heads * vdim, dtype=torch.float32, device=qk.device)
     status = _lib("state_scan").r2_delta_scan(
@@ -997,13 +1003,13 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, numbers: torch.Tensor, dim: in
 def time_mix_prepare(h: torch.Tensor, mu: torch.Tensor, w1: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, state: torch.Tensor, row_off: int,
                      row_entry: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor):
     """Mixes of every row with the row before it in its sequence, mix_s = h + (h' - h) mu[s], and the decays made from the last of
-    them: decay = exp(-exp(w0 + W2 tanh(W1 mix_last))). h [T, D]; mu float32 [n, D]; w1 float32 [rank, D], w2t float32 [rank, N] (W2 transposed), w0
+    them: decay = exp(-exp(w0 + W2 tanh(W1 mix_last))). h [T, D]; mu float32 [n, D]; w1 [rank, D], w2t [rank, N] (W2 transposed) in h's dtype, w0
     float32 [N]. The row before an entry's first comes from the request's state slot (float32 [slots, floats], at `row_off`; zeros
-    before a sequence's start; the slot is only read: `time_mix_scan` renews it). The decays' way is float32 throughout.
+    before a sequence's start; the slot is only read: `time_mix_scan` renews it). The decays' way is float32 but for the stored matrices.
     -> (the other mixes [T, n - 1, D] in h's dtype, decay float32 [T, N])."""
     _need(h, "h", dim=2)
     for name, t, dim in (("mu", mu, 2), ("w1", w1, 2), ("w2t", w2t, 2), ("w0", w0, 1), ("state", state, 2)):
-        _need(t, name, torch.float32, dim)
+        _need(t, name, h.dtype if name in ("w1", "w2t") else torch.float32, dim)
         if not t.is_contiguous():
             raise KernelError(f"time_mix_prepare: {name} must be contiguous")
     _need(row_entry, "row_entry", torch.int32, 1)
@@ -1028,7 +1034,7 @@ def time_mix_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torc
                   row_in: torch.Tensor | None = None, row_state_off: int = 0) -> torch.Tensor:
     """Time mixing with a decay per channel for every entry of a batch, from and to the entries' state slots:
     o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, S_t = diag(decay_t) S_(t-1) + k_t v_t^T. r, k, v [T, heads * dim];
-    decay float32 [T, heads * dim]; bonus float32 [heads * dim]; state float32 [slots, floats]: S [heads, dim, dim] first, and with
+    decay float32 [T, heads * dim]; bonus float32 [heads * dim]; state float32 [slots, floats]: the heads' matrices first (`scan_state_floats` each), and with
     `row_in` (this step's input rows [T, D]) the last position's input row at `row_state_off`, which is renewed.
     -> float32 [T, heads * dim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
@@ -1040,11 +1046,11 @@ def time_mix_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torc
     _need(decay, "decay", torch.float32, 2)
     _need(bonus, "bonus", torch.float32)
     _need(state, "state", torch.float32, 2)
-    if decay.shape != r.shape or bonus.numel() != width or not bonus.is_contiguous() or state.shape[1] < width * dim or not state.is_contiguous():
+    if decay.shape != r.shape or bonus.numel() != width or not bonus.is_contiguous() or state.shape[1] < n_heads * scan_state_floats(dim, dim) or not state.is_contiguous():
         raise KernelError(f"time_mix_scan: decay {tuple(decay.shape)} / bonus {tuple(bonus.shape)} / state {tuple(state.shape)} do not fit {n_heads} heads of {dim}")
     if row_in is not None:
         _need(row_in, "row_in", r.dtype, 2)
-        if row_state_off < width * dim or row_state_off + row_in.shape[1] > state.shape[1]:
+        if row_state_off < n_heads * scan_state_floats(dim, dim) or row_state_off + row_in.shape[1] > state.shape[1]:
             raise KernelError("time_mix_scan: the last input row does not fit the slot")
     out = torch.empty(r.shape[0], width, dtype=torch.float32, device=r.device)
     status = _lib("state_scan").r2_time_mix_scan(

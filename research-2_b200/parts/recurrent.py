@@ -236,10 +236,10 @@ class DeltaRule:
         self.w_out = matrix(weights["w_out"], rt)
         self.conv = vector(torch.cat(convs, dim=0), rt)
         self.channels = self.conv.shape[0]
-        self.w_gates = vector(torch.cat([weights["w_b"], weights["w_a"]], dim=0), rt)   # float32: they enter the recurrence
+        self.w_gates = matrix(torch.cat([weights["w_b"], weights["w_a"]], dim=0), rt)   # (the products with it are float32 sums)
         self.a_log, self.dt_bias = vector(weights["a_log"], rt), vector(weights["dt_bias"], rt)
         self.norm = vector(weights["norm"].repeat(self.n_heads), rt)
-        self.conv_state_off = self.n_heads * self.head_dim * self.v_head_dim
+        self.conv_state_off = self.n_heads * ops.scan_state_floats(self.head_dim, self.v_head_dim)
 
     cache_spec = None
     capturable = True
@@ -249,7 +249,7 @@ class DeltaRule:
 
     @property
     def state_spec(self) -> StateSpec:
-        return StateSpec((self.conv_state_off + (self.conv_taps - 1) * self.channels,), torch.float32)
+        return StateSpec((-(-(self.conv_state_off + (self.conv_taps - 1) * self.channels) // 4) * 4,), torch.float32)   # (whole 16-byte pieces)
 
     def _inner(self, h, ctx, state):
         proj = ops.linear(h, self.w_in, None, w_is_nk=True)
@@ -278,7 +278,7 @@ class TimeMix:
         o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T     (S from zero)
 
     Each head's o is divided by its root mean square, the heads are concatenated, times `norm`, times the gate; then W_o. The state is S
-    and the last row h. The way to the decays (mix_w, both small products, the exponentials) is float32 throughout.
+    and the last row h. The way to the decays (mix_w, the sums of both small products, tanh, the exponentials) is float32.
 
     params: n_heads, head_dim, norm_eps, out_scale (default 1: a factor on the gated outputs, folded into the norm's gains).
     weights (stored [out, in], no biases): w_r, w_k, w_v, w_gate [H head_dim, D], mu_r, mu_k, mu_v, mu_g, mu_w [D], w1 [rank, D], w2 [H head_dim,
@@ -297,10 +297,10 @@ class TimeMix:
         self.w_in = matrix(torch.cat(stacked, dim=0), rt)      # [4 H head_dim, D], the rows of each kind read a mix of their own
         self.w_out = matrix(weights["w_out"], rt)
         self.mu = vector(torch.stack([weights["mu_" + s] for s in "rkvgw"]), rt)
-        self.w1, self.w2t, self.w0 = vector(w1, rt), vector(w2.to(torch.float32).T.contiguous(), rt), vector(weights["w0"], rt)
+        self.w1, self.w2t, self.w0 = matrix(w1, rt), matrix(w2.T, rt), vector(weights["w0"], rt)
         self.bonus = vector(weights["bonus"].reshape(-1), rt)
         self.norm = vector(weights["norm"], rt) * float(params.get("out_scale", 1.0))
-        self.row_state_off = self.inner_width * self.head_dim
+        self.row_state_off = self.n_heads * ops.scan_state_floats(self.head_dim, self.head_dim)
 
     cache_spec = None
     capturable = True
@@ -310,7 +310,7 @@ class TimeMix:
 
     @property
     def state_spec(self) -> StateSpec:
-        return StateSpec((self.row_state_off + self.width,), torch.float32)
+        return StateSpec((-(-(self.row_state_off + self.width) // 4) * 4,), torch.float32)
 
     def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None):
         """The gated heads' outputs [T, H head_dim] before w_out (into `out` where given)."""
