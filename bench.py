@@ -986,11 +986,11 @@ def lagelorn_config(size: str, n_layer: int) -> dict:
     ff = max(128, round(2 * g["n_inner"] / 3 / 128) * 128)
     delta = {"heads": h, "kv_heads": half_heads_for(h), "dim": hd, "vdim": hd, "conv": 4}
     pair = {"left": {"heads": h, "kv_heads": kv_heads_for(h), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "bias_max": 128, "mask": {"size": 256}},
-            "left_scale": 1.2, "right": {"heads": h, "dim": hd}, "right_scale": 0.8}
+            "left_scale": 1.5, "right": {"heads": h, "dim": hd}, "right_scale": 0.8}
     layers = [{"type": "parallel" if i % 3 == 2 else "delta", "mixer": pair if i % 3 == 2 else delta, "mlp": {"kind": "dense", "ff": ff}}
               for i in range(n_layer)]
     return {"architecture": "Lagelorn", "vocab": g["vocab_size"], "width": d, "norm": {"eps": 1e-5}, "max_positions": CONTEXT, "postln_alpha": 2.0,
-            "token_side": {"dim": 64}, "logit_softcap": 30.0, "layers": layers}
+            "token_side": {"dim": 64}, "logit_softcap": 25.0, "layers": layers}
 
 
 def bosenex_dense_config(size: str, n_layer: int) -> dict:
@@ -1173,7 +1173,7 @@ def lagelorn_points(args, pk: dict) -> dict:
             keys = n_entries * chunk
         size = dict(n_bytes=t * h * hd * 4 + keys * 2 * kvh * hd * 2)
         add(f"attention by chunks of {chunk} with a bias by distance and sinks, {h} heads of {hd} over {kvh}, {label}",
-            lambda: attend(window=0, chunk=chunk, dist_bias=bias, out_scale=1.2), flops=4 * seen * h * hd, **size)
+            lambda: attend(window=0, chunk=chunk, dist_bias=bias, out_scale=1.5), flops=4 * seen * h * hd, **size)
         add(f"its like: window of {chunk}, capped scores, sinks (Bosenex), {label}", lambda: attend(window=chunk, softcap=30.0), flops=4 * windowed * h * hd, **size)
         # the rest of a layer and the head
         ff = max(128, round(2 * g["n_inner"] / 3 / 128) * 128)

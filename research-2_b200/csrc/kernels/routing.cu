@@ -19,29 +19,29 @@
 #include <math.h>
 
 #include "common.cuh"
-#include "small_products.cuh"
 
 namespace {
 
 constexpr int MAX_EXPERTS = 1024;
 
-// A CTA takes ROWS rows: the matrix comes out of L2 once for all of them.
-template <typename T, int ROWS>
+template <typename T>
 __global__ void __launch_bounds__(256)
 small_linear_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ w, const float* __restrict__ bias,
-                    float* __restrict__ out, int out_stride, int n_rows, int n_out, int width) {
+                    float* __restrict__ out, int out_stride, int n_out, int width) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ __align__(16) float rows[];
-  const int t0 = blockIdx.x * ROWS, wpad = (width + 3) & ~3;
-  for (int i = threadIdx.x; i < ROWS * wpad; i += blockDim.x) {
-    const int r = i / wpad, k = i - r * wpad;
-    rows[i] = (k < width && t0 + r < n_rows) ? to_float(h[size_t(t0 + r) * h_stride + k]) : 0.f;
-  }
+  extern __shared__ float row[];
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  const T* hr = h + size_t(t) * h_stride;
+  for (int k = threadIdx.x; k < width; k += blockDim.x) row[k] = to_float(hr[k]);
   __syncthreads();
-  rows_times_matrix<ROWS, ROWS == 1 ? 1 : 2>(rows, wpad, w, width, n_out, [&](int r, int n, float sum) {
-    if (t0 + r < n_rows) out[size_t(t0 + r) * out_stride + n] = sum + (bias != nullptr ? bias[n] : 0.f);
-  });
+  for (int n = warp; n < n_out; n += n_warps) {
+    const float* wr = w + size_t(n) * width;
+    float acc = 0.f;
+    for (int k = lane; k < width; k += 32) acc = fmaf(row[k], wr[k], acc);
+    acc = warp_sum(acc);
+    if (lane == 0) out[size_t(t) * out_stride + n] = acc + (bias != nullptr ? bias[n] : 0.f);
+  }
 }
 
 template <typename T>
@@ -264,27 +264,16 @@ extern "C" int r2_small_linear(const void* h, int h_stride, const float* w, cons
                                int n_rows, int n_out, int width, int dtype, cudaStream_t stream) {
   if (n_rows <= 0 || n_out <= 0) return R2_OK;
   if (width < 1) return R2_BAD_SHAPE;
-  const size_t per_row = sizeof(float) * ((width + 3) & ~3);
-  int rows = n_rows > 512 ? 8 : (n_rows > 128 ? 4 : 1);
-  while (rows > 1 && per_row * rows > 100 * 1024) rows = rows == 8 ? 4 : 1;
-#define R2_SMALL(T_, ROWS_)                                                                                                \
-  do {                                                                                                                     \
-    if (!room_for(small_linear_kernel<T_, ROWS_>, per_row * ROWS_)) return R2_UNSUPPORTED;                                 \
-    r2_launch(small_linear_kernel<T_, ROWS_>, dim3((n_rows + ROWS_ - 1) / ROWS_), dim3(256), per_row * ROWS_, stream,      \
-              (const T_*)h, h_stride, w, bias, out, out_stride, n_rows, n_out, width);                                     \
-  } while (0)
+  const size_t smem = sizeof(float) * width;
+  if (smem > 48 * 1024) return R2_UNSUPPORTED;
+  const int threads = n_out >= 8 ? 256 : 32 * n_out;
   if (dtype == R2_F32) {
-    if (rows == 8) R2_SMALL(float, 8);
-    else if (rows == 4) R2_SMALL(float, 4);
-    else R2_SMALL(float, 1);
+    r2_launch(small_linear_kernel<float>, dim3(n_rows), dim3(threads), smem, stream, (const float*)h, h_stride, w, bias, out, out_stride, n_out, width);
   } else if (dtype == R2_BF16) {
-    if (rows == 8) R2_SMALL(bf16, 8);
-    else if (rows == 4) R2_SMALL(bf16, 4);
-    else R2_SMALL(bf16, 1);
+    r2_launch(small_linear_kernel<bf16>, dim3(n_rows), dim3(threads), smem, stream, (const bf16*)h, h_stride, w, bias, out, out_stride, n_out, width);
   } else {
     return R2_BAD_DTYPE;
   }
-#undef R2_SMALL
   return launch_status();
 }
 

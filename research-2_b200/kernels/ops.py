@@ -1441,7 +1441,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             _used("attention_prefill_tc")
             return out
     if (fits and q.dtype == torch.bfloat16 and _fast_attention and q_start is not None and n_tiles > 0 and head_dim <= 128
-            and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0 and (gate is None or (gate_stride % 2 == 0 and gate.data_ptr() % 4 == 0))):
+            and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0 and _rows(out, "out") % 2 == 0 and out.data_ptr() % 4 == 0 and (gate is None or (gate_stride % 2 == 0 and gate.data_ptr() % 4 == 0))):
         _need(q_start, "q_start", torch.int32, 1)
         lib = _lib_for_head_dim("attention_prefill", head_dim)
         status = lib.r2_attention_prefill_biased(

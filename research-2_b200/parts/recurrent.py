@@ -380,7 +380,8 @@ class SideBySideSum(_TwoMixers):
         return [self.sides[0].w_in, self.sides[1].w_in, self.w_out]
 
     def _inner(self, h, ctx, cache, state, writes_cache):
-        both = torch.empty(h.shape[0], self.w_out.shape[1], dtype=h.dtype, device=h.device)
+        # (rows a multiple of eight numbers apart: the attention kernels write pairs, the product reads 16-byte pieces)
+        both = torch.empty(h.shape[0], -(-self.w_out.shape[1] // 8) * 8, dtype=h.dtype, device=h.device)[:, : self.w_out.shape[1]]
         at = 0
         for p in self.sides:
             p.inner(h, ctx, cache, state, writes_cache, out=both[:, at: at + p.inner_width])
