@@ -1130,19 +1130,21 @@ def lagelorn_points(args, pk: dict) -> dict:
         mixes, decay = prepare()
         add(f"time mixing: a row's mixes with the row before it, decays through an inner width of {DECAY_RANK} in 32-bit, {label}", prepare,
             n_bytes=t * d * (2 + 8 + 4) + 4 * d * DECAY_RANK)
-        w_in = (torch.randn(4 * d, d, device=dev) * 0.02).to(bf)
+        group = -(-d // 128) * 128     # a group's features, padded to whole tiles as the layer pads them
+        w_in, w_like = ((torch.randn(4 * n, d, device=dev) * 0.02).to(bf) for n in (group, d))
         add(f"time mixing: four products of {d} x {d} on their mixes, {label}", lambda: ops.grouped_linear(mixes, w_in),
             n_bytes=t * d * 16 + 8 * d * d, flops=8 * t * d * d)
-        add(f"its like: one product of {d} x {4 * d:,} (any model), {label}", lambda: ops.linear(hrow, w_in, None, w_is_nk=True),
+        add(f"its like: one product of {d} x {4 * d:,} (any model), {label}", lambda: ops.linear(hrow, w_like, None, w_is_nk=True),
             n_bytes=t * d * 10 + 8 * d * d, flops=8 * t * d * d)
         rkvg = ops.grouped_linear(mixes, w_in)
         bonus = torch.zeros(d, device=dev)
-        scan = lambda: ops.time_mix_scan(rkvg[:, :d], rkvg[:, d: 2 * d], rkvg[:, 2 * d: 3 * d], decay, bonus, tstate, q_start, slots, fresh, h, hd,  # noqa: E731
+        r_, k_, v_, gate = (rkvg[:, i * group: i * group + d] for i in range(4))
+        scan = lambda: ops.time_mix_scan(r_, k_, v_, decay, bonus, tstate, q_start, slots, fresh, h, hd,  # noqa: E731
                                          row_in=hrow, row_state_off=toff)
         o32 = scan()
         add(f"time mixing: recurrence, {h} heads of {hd} x {hd}, {label}", scan, n_bytes=t * d * (6 + 4 + 4) + 2 * tstate.numel() * 4)
-        add(f"heads' norm and silu gate (both recurrences), {label}", lambda: ops.group_norm_gated(o32, rkvg[:, 3 * d:], gain, h, 1e-5, "silu_after", bf), n_bytes=t * d * 8)
-        add(f"its like: heads' norm and sigmoid gate (Bosenex), {label}", lambda: ops.group_norm_gated(o32, rkvg[:, 3 * d:], gain, h, 1e-5, False, bf), n_bytes=t * d * 8)
+        add(f"heads' norm and silu gate (both recurrences), {label}", lambda: ops.group_norm_gated(o32, gate, gain, h, 1e-5, "silu_after", bf), n_bytes=t * d * 8)
+        add(f"its like: heads' norm and sigmoid gate (Bosenex), {label}", lambda: ops.group_norm_gated(o32, gate, gain, h, 1e-5, False, bf), n_bytes=t * d * 8)
         # attention by chunks
         kvh = kv_heads_for(h)
         qk = torch.randn(t, (h + 2 * kvh) * hd, device=dev).to(bf)

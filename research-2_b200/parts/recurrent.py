@@ -294,7 +294,10 @@ class TimeMix:
                 or w2.shape[0] != self.inner_width or weights["w_out"].shape[1] != self.inner_width or weights["bonus"].numel() != self.inner_width):
             raise ValueError(f"time mixing: projections {[tuple(w.shape) for w in stacked]}, decay {tuple(w1.shape)} and {tuple(w2.shape)} and an output of "
                              f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads of {self.head_dim}")
-        self.w_in = matrix(torch.cat(stacked, dim=0), rt)      # [4 H head_dim, D], the rows of each kind read a mix of their own
+        # [4 groups of H head_dim rows, D]: the rows of each kind read a mix of their own; for the tensor cores a group is padded with
+        # zeros to whole tiles, so that the four products are one launch
+        self.group = -(-self.inner_width // 128) * 128 if rt.dtype == torch.bfloat16 else self.inner_width
+        self.w_in = matrix(torch.cat([torch.nn.functional.pad(w, (0, 0, 0, self.group - self.inner_width)) for w in stacked], dim=0), rt)
         self.w_out = matrix(weights["w_out"], rt)
         self.mu = vector(torch.stack([weights["mu_" + s] for s in "rkvgw"]), rt)
         self.w1, self.w2t, self.w0 = matrix(w1, rt), matrix(w2.T, rt), vector(weights["w0"], rt)
@@ -316,11 +319,11 @@ class TimeMix:
         """The gated heads' outputs [T, H head_dim] before w_out (into `out` where given)."""
         mixes, decay = ops.time_mix_prepare(h, self.mu, self.w1, self.w2t, self.w0, state, self.row_state_off, ctx.row_entry, ctx.q_start,
                                                 ctx.state_slot, ctx.fresh)
-        n = self.inner_width
         proj = ops.grouped_linear(mixes, self.w_in)
-        o = ops.time_mix_scan(proj[:, :n], proj[:, n: 2 * n], proj[:, 2 * n: 3 * n], decay, self.bonus, state, ctx.q_start, ctx.state_slot,
-                              ctx.fresh, self.n_heads, self.head_dim, row_in=h, row_state_off=self.row_state_off)
-        return ops.group_norm_gated(o, proj[:, 3 * n:], self.norm, self.n_heads, self.norm_eps, "silu_after", proj.dtype, out=out)
+        r, k, v, gate = (proj[:, i * self.group: i * self.group + self.inner_width] for i in range(4))
+        o = ops.time_mix_scan(r, k, v, decay, self.bonus, state, ctx.q_start, ctx.state_slot, ctx.fresh, self.n_heads, self.head_dim,
+                              row_in=h, row_state_off=self.row_state_off)
+        return ops.group_norm_gated(o, gate, self.norm, self.n_heads, self.norm_eps, "silu_after", proj.dtype, out=out)
 
     def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
         return ops.linear(self.inner(h, ctx, cache, state), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
