@@ -33,6 +33,7 @@ constexpr int MODE_MLSTM = 0, MODE_SSD = 1, MODE_DECAY = 2;
 
 __device__ __forceinline__ float soft_cap(float x, float cap) { return cap > 0.f ? cap * tanhf(x / cap) : x; }
 __device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 struct ScanArgs {
@@ -50,6 +51,7 @@ struct ScanArgs {
   const float* decay;                    // retention, per head: keep
   const float* inv_freq; int rot_half;   // retention: of r and w the first 2 * rot_half dimensions turn, dimension i with
   const int32_t* positions;              // i + rot_half, by the angle positions[row] * inv_freq[i] (rot_half 0: no rotation)
+  int silu_in;                           // retention: r, w and v pass silu on their way in
   float* state; long long slot_stride;   // per request slot; per head: S [rows][cols] (+ mLSTM: NORM_COPIES times n [rows], m)
   int head_stride;
   const int32_t* q_start; const int32_t* state_slot; const int32_t* fresh;
@@ -141,6 +143,10 @@ outer_scan_kernel(const ScanArgs a) {
           tr[u] = fmaf(tr[u], cs, to_float(read[row * a.read_stride + other]) * sn);
           tw[u] = fmaf(tw[u], cs, to_float(write[row * a.write_stride + other]) * sn);
         }
+        if (MODE == MODE_DECAY && a.silu_in) {
+          tr[u] = silu(tr[u]);
+          tw[u] = silu(tw[u]);
+        }
       }
 #pragma unroll
       for (int u = 0; u < 8; ++u) {
@@ -162,7 +168,7 @@ outer_scan_kernel(const ScanArgs a) {
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
         const int idx = base + u * blockDim.x + tid;
-        if (idx < nt * cv) vs[idx] = tv[u];
+        if (idx < nt * cv) vs[idx] = (MODE == MODE_DECAY && a.silu_in) ? silu(tv[u]) : tv[u];
       }
     }
     if (MODE == MODE_DECAY) {
@@ -475,19 +481,20 @@ extern "C" int r2_mlstm_scan(const void* q, int q_stride, const void* k, int k_s
 
 // Retention: S <- decay[h] S + k v^T, o = S^T q per head, with q and k rotated by position (the first rot_dims dimensions
 // of a head, dimension i with i + rot_dims / 2, angle positions[t] * inv_freq[i]; rot_dims 0: none) and k multiplied by
-// k_scale after the rotation. q, k [T, heads * dim], v [T, heads * vdim] (slices of a projection); decay float [heads];
+// k_scale after the rotation. silu_in: q, k and v pass silu on their way in (then without a rotation). q, k [T, heads * dim], v [T, heads * vdim] (slices of a projection); decay float [heads];
 // state float [slots][heads][dim][vdim]; out [T, heads * vdim] float, before the heads' norm.
 extern "C" int r2_retention_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
                                  const float* decay, float k_scale, const float* inv_freq, int rot_dims, const int32_t* positions,
                                  float* state, long long slot_stride, const int32_t* q_start, const int32_t* state_slot,
                                  const int32_t* fresh, int n_entries, float* out, int out_stride, int n_heads, int dim, int vdim,
-                                 int single_rows, int dtype, cudaStream_t stream) {
+                                 int single_rows, int silu_in, int dtype, cudaStream_t stream) {
   if (n_entries <= 0) return R2_OK;
+  if (silu_in && rot_dims > 0) return R2_BAD_SHAPE;
   if (n_heads < 1 || dim < 1 || vdim < 1 || rot_dims < 0 || rot_dims % 2 != 0 || rot_dims > dim) return R2_BAD_SHAPE;
   if (rot_dims > 0 && (inv_freq == nullptr || positions == nullptr)) return R2_BAD_SHAPE;
   ScanArgs a = {};
   a.read = q; a.read_stride = q_stride; a.write = k; a.write_stride = k_stride; a.value = v; a.value_stride = v_stride;
-  a.read_scale = 1.f; a.write_scale = k_scale; a.decay = decay; a.inv_freq = inv_freq; a.rot_half = rot_dims / 2; a.positions = positions;
+  a.read_scale = 1.f; a.write_scale = k_scale; a.decay = decay; a.inv_freq = inv_freq; a.rot_half = rot_dims / 2; a.positions = positions; a.silu_in = silu_in;
   a.state = state; a.slot_stride = slot_stride; a.head_stride = dim * vdim;
   a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh; a.out = out; a.out_stride = out_stride;
   a.heads_per_group = 1; a.rows = dim; a.cols = vdim; a.single_rows = single_rows;

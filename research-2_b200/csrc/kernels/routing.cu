@@ -16,6 +16,10 @@
 //                     (and of one more expert that every row uses) lie side by side in one row; each expert's
 //                     columns are multiplied by the row's weight for that expert, so that ONE down product over the
 //                     stacked matrices is the weighted sum of the experts' outputs.
+//   r2_expert_unit    the same for experts without gates.
+//
+// In r2_route_scored the last outputs of the router may stand for no expert but for the row itself (identity outputs): the launch
+// then also gives the row times their weights' sum, which joins the experts' sum as that product's addend.
 #include <math.h>
 
 #include "common.cuh"
@@ -107,16 +111,20 @@ route_top_k_kernel(const T* __restrict__ h, int h_stride, const float* __restric
 // can be chosen (the lower index wins a tie, among groups and among experts). The `top` largest choice scores are chosen; a
 // chosen expert's weight is its s over the sum of the chosen s (+ 1e-20).
 // softmax_scores: s = softmax of the logits over all experts instead of their sigmoids. mark_best_only: a group's mark is its
-// largest choice score alone. normalise = 0: a chosen expert's weight is s * weight_scale.
+// largest choice score alone. normalise = 0: the chosen s are not divided by their sum. The weights are multiplied by weight_scale.
+// n_identity: the last of the n_experts outputs stand for no expert but for the input row itself: carried[t] = their weights' sum
+// * h[t] (+ base[t] where given), float.
 template <typename T>
 __global__ void __launch_bounds__(256)
 route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ w, const float* __restrict__ correction,
                     float* __restrict__ dense, int32_t* __restrict__ chosen, float* __restrict__ chosen_weight,
                     float* __restrict__ extra, int n_experts, int n_extra, int top, int n_groups, int keep, int width,
-                    int softmax_scores, int mark_best_only, int normalise, float weight_scale) {
+                    int softmax_scores, int mark_best_only, int normalise, float weight_scale, int n_identity,
+                    const float* __restrict__ base, float* __restrict__ carried) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float smem[];
+  __shared__ float identity_weight;
   float* row = smem;                    // [width]
   float* score = smem + width;          // [n_experts] sigmoid of the logit
   float* choice = score + n_experts;    // [n_experts] score + correction; -inf once picked or outside the kept groups
@@ -142,84 +150,97 @@ route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restri
   }
   for (int n = threadIdx.x; n < n_experts; n += blockDim.x) dense[size_t(t) * n_experts + n] = 0.f;
   __syncthreads();
-  if (warp != 0) return;
-  if (softmax_scores) {
-    // s = exp(z - max) / sum over all experts, one warp, sums in a fixed order
-    float top_z = -INFINITY;
-    for (int n = lane; n < n_experts; n += 32) top_z = fmaxf(top_z, score[n]);
-    for (int o = 16; o > 0; o >>= 1) top_z = fmaxf(top_z, __shfl_xor_sync(0xffffffffu, top_z, o));
-    float total = 0.f;
-    for (int n = lane; n < n_experts; n += 32) {
-      const float e = expf(score[n] - top_z);
-      score[n] = e;
-      total += e;
-    }
-    total = warp_sum(total);
-    const float inv_total = 1.f / total;
-    for (int n = lane; n < n_experts; n += 32) {
-      const float s = score[n] * inv_total;
-      score[n] = s;
-      choice[n] = s + (correction != nullptr ? correction[n] : 0.f);
-    }
-    __syncwarp();
-  }
-  const int size = n_experts / n_groups;
-  if (keep < n_groups) {
-    for (int g = lane; g < n_groups; g += 32) {
-      float a = -INFINITY, b = -INFINITY;   // the group's largest and second largest
-      for (int n = g * size; n < (g + 1) * size; ++n) {
-        const float c = choice[n];
-        if (c > a) { b = a; a = c; }
-        else if (c > b) b = c;
+  if (warp == 0) {
+    if (softmax_scores) {
+      // s = exp(z - max) / sum over all experts, one warp, sums in a fixed order
+      float top_z = -INFINITY;
+      for (int n = lane; n < n_experts; n += 32) top_z = fmaxf(top_z, score[n]);
+      for (int o = 16; o > 0; o >>= 1) top_z = fmaxf(top_z, __shfl_xor_sync(0xffffffffu, top_z, o));
+      float total = 0.f;
+      for (int n = lane; n < n_experts; n += 32) {
+        const float e = expf(score[n] - top_z);
+        score[n] = e;
+        total += e;
       }
-      mark[g] = (size > 1 && !mark_best_only) ? a + b : a;
+      total = warp_sum(total);
+      const float inv_total = 1.f / total;
+      for (int n = lane; n < n_experts; n += 32) {
+        const float s = score[n] * inv_total;
+        score[n] = s;
+        choice[n] = s + (correction != nullptr ? correction[n] : 0.f);
+      }
+      __syncwarp();
     }
-    __syncwarp();
-    // the kept groups: `keep` times the largest mark; a kept group's mark becomes +inf, and what is not +inf at the end is out
-    for (int c = 0; c < keep; ++c) {
+    const int size = n_experts / n_groups;
+    if (keep < n_groups) {
+      for (int g = lane; g < n_groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;   // the group's largest and second largest
+        for (int n = g * size; n < (g + 1) * size; ++n) {
+          const float c = choice[n];
+          if (c > a) { b = a; a = c; }
+          else if (c > b) b = c;
+        }
+        mark[g] = (size > 1 && !mark_best_only) ? a + b : a;
+      }
+      __syncwarp();
+      // the kept groups: `keep` times the largest mark; a kept group's mark becomes +inf, and what is not +inf at the end is out
+      for (int c = 0; c < keep; ++c) {
+        float v = -INFINITY;
+        int at = n_groups;
+        for (int g = lane; g < n_groups; g += 32)
+          if (mark[g] != INFINITY && (mark[g] > v || at == n_groups)) { v = mark[g]; at = g; }
+        for (int o = 16; o > 0; o >>= 1) {
+          const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+          const int oat = __shfl_xor_sync(0xffffffffu, at, o);
+          if (oat < n_groups && (at == n_groups || ov > v || (ov == v && oat < at))) { v = ov; at = oat; }
+        }
+        if (lane == 0 && at < n_groups) mark[at] = INFINITY;
+        __syncwarp();
+      }
+      for (int n = lane; n < n_experts; n += 32)
+        if (mark[n / size] != INFINITY) choice[n] = -INFINITY;
+      __syncwarp();
+    }
+    float sum = 0.f;
+    for (int c = 0; c < top; ++c) {
       float v = -INFINITY;
-      int at = n_groups;
-      for (int g = lane; g < n_groups; g += 32)
-        if (mark[g] != INFINITY && (mark[g] > v || at == n_groups)) { v = mark[g]; at = g; }
+      int at = n_experts;
+      for (int n = lane; n < n_experts; n += 32)
+        if (choice[n] > v) { v = choice[n]; at = n; }
       for (int o = 16; o > 0; o >>= 1) {
         const float ov = __shfl_xor_sync(0xffffffffu, v, o);
         const int oat = __shfl_xor_sync(0xffffffffu, at, o);
-        if (oat < n_groups && (at == n_groups || ov > v || (ov == v && oat < at))) { v = ov; at = oat; }
+        if (ov > v || (ov == v && oat < at)) { v = ov; at = oat; }
       }
-      if (lane == 0 && at < n_groups) mark[at] = INFINITY;
+      if (at >= n_experts) at = c;   // scores that are not numbers: no index may leave the row
+      const float s = score[at];
+      sum += s;
+      if (lane == 0) {
+        chosen[size_t(t) * top + c] = at;
+        chosen_weight[size_t(t) * top + c] = s;
+        choice[at] = -INFINITY;
+      }
       __syncwarp();
     }
-    for (int n = lane; n < n_experts; n += 32)
-      if (mark[n / size] != INFINITY) choice[n] = -INFINITY;
-    __syncwarp();
-  }
-  float sum = 0.f;
-  for (int c = 0; c < top; ++c) {
-    float v = -INFINITY;
-    int at = n_experts;
-    for (int n = lane; n < n_experts; n += 32)
-      if (choice[n] > v) { v = choice[n]; at = n; }
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-      const int oat = __shfl_xor_sync(0xffffffffu, at, o);
-      if (ov > v || (ov == v && oat < at)) { v = ov; at = oat; }
+    const float inv = (normalise ? 1.f / (sum + 1e-20f) : 1.f) * weight_scale;
+    for (int c = lane; c < top; c += 32) {
+      const float p = chosen_weight[size_t(t) * top + c] * inv;
+      chosen_weight[size_t(t) * top + c] = p;
+      dense[size_t(t) * n_experts + chosen[size_t(t) * top + c]] = p;
     }
-    if (at >= n_experts) at = c;   // scores that are not numbers: no index may leave the row
-    const float s = score[at];
-    sum += s;
-    if (lane == 0) {
-      chosen[size_t(t) * top + c] = at;
-      chosen_weight[size_t(t) * top + c] = s;
-      choice[at] = -INFINITY;
+    if (n_identity > 0) {
+      __syncwarp();   // (the warp's writes to the row of weights are seen by its lanes)
+      float c = 0.f;
+      for (int n = n_experts - n_identity + lane; n < n_experts; n += 32) c += dense[size_t(t) * n_experts + n];
+      c = warp_sum(c);
+      if (lane == 0) identity_weight = c;
     }
-    __syncwarp();
   }
-  const float inv = normalise ? 1.f / (sum + 1e-20f) : weight_scale;
-  for (int c = lane; c < top; c += 32) {
-    const float p = chosen_weight[size_t(t) * top + c] * inv;
-    chosen_weight[size_t(t) * top + c] = p;
-    dense[size_t(t) * n_experts + chosen[size_t(t) * top + c]] = p;
-  }
+  if (n_identity == 0) return;
+  __syncthreads();
+  const float share = identity_weight;
+  for (int k = threadIdx.x; k < width; k += blockDim.x)
+    carried[size_t(t) * width + k] = share * row[k] + (base != nullptr ? base[size_t(t) * width + k] : 0.f);
 }
 
 constexpr int KIND_CLAMPED_SWISH = 0, KIND_RELU = 1, KIND_SILU = 2, KIND_GELU_TANH = 3;
@@ -240,7 +261,7 @@ __device__ __forceinline__ float gated_unit(float g, float u, int kind, float li
 template <typename T>
 __global__ void __launch_bounds__(256)
 expert_act_kernel(const T* __restrict__ gate_up, int in_stride, T* __restrict__ out, int out_stride, int inner, int kind,
-                  float limit, float alpha, float up_offset, const float* __restrict__ route, int n_experts, int expert_width,
+                  float limit, float alpha, float up_offset, const float* __restrict__ route, int route_stride, int n_experts, int expert_width,
                   float tail_limit, const float* __restrict__ tail_gate, int tail_gate_stride) {
   pdl_launch_dependents();
   pdl_wait();
@@ -251,10 +272,45 @@ expert_act_kernel(const T* __restrict__ gate_up, int in_stride, T* __restrict__ 
   const int routed = n_experts * expert_width;
   for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < inner; f += gridDim.y * blockDim.x) {
     const bool tail = f >= routed;
-    const float weight = tail ? tail_weight : route[size_t(blockIdx.x) * n_experts + f / expert_width];
+    const float weight = tail ? tail_weight : route[size_t(blockIdx.x) * route_stride + f / expert_width];
     float y = 0.f;
     if (weight != 0.f) y = weight * gated_unit(to_float(in[f]), to_float(in[inner + f]), kind, tail ? tail_limit : limit, alpha, up_offset);
     o[f] = from_float<T>(y);
+  }
+}
+
+// Experts without gates: a row of `up` holds the experts' inner values side by side; act(up) times the row's weight for the column's
+// expert. (`route` rows are route_stride numbers apart.) With `vec` eight neighbouring columns, all of one expert, are one 16-byte piece.
+template <typename T>
+__global__ void __launch_bounds__(256)
+expert_unit_kernel(const T* __restrict__ up, int in_stride, T* __restrict__ out, int out_stride, int inner, int act,
+                   const float* __restrict__ route, int route_stride, int expert_width, int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const T* in = up + size_t(blockIdx.x) * in_stride;
+  T* o = out + size_t(blockIdx.x) * out_stride;
+  const float* weights = route + size_t(blockIdx.x) * route_stride;
+  if (sizeof(T) == 2 && vec) {
+    for (int f = 8 * (blockIdx.y * blockDim.x + threadIdx.x); f < inner; f += 8 * gridDim.y * blockDim.x) {
+      const float weight = weights[f / expert_width];
+      uint4 yq = make_uint4(0u, 0u, 0u, 0u);
+      if (weight != 0.f) {
+        const uint4 zq = *reinterpret_cast<const uint4*>(in + f);
+        const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&zq);
+        __nv_bfloat162* y2 = reinterpret_cast<__nv_bfloat162*>(&yq);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 z = __bfloat1622float2(z2[i]);
+          y2[i] = __floats2bfloat162_rn(weight * activate(z.x, act), weight * activate(z.y, act));
+        }
+      }
+      *reinterpret_cast<uint4*>(o + f) = yq;
+    }
+    return;
+  }
+  for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < inner; f += gridDim.y * blockDim.x) {
+    const float weight = weights[f / expert_width];
+    o[f] = from_float<T>(weight != 0.f ? weight * activate(to_float(in[f]), act) : 0.f);
   }
 }
 
@@ -294,23 +350,25 @@ extern "C" int r2_route_top_k(const void* h, int h_stride, const float* w, const
 }
 
 // w float [n_experts + n_extra, width]; correction float [n_experts] (may be null); dense [T, n_experts], chosen / chosen_weight
-// [T, top], extra [T, n_extra] (the further rows' logits; null when n_extra is 0). softmax_scores, mark_best_only, normalise and
+// [T, top], extra [T, n_extra] (the further rows' logits; null when n_extra is 0); carried float [T, width] where n_identity > 0 (base
+// likewise, or null). softmax_scores, mark_best_only, normalise and
 // weight_scale choose the router's form (see the kernel).
 extern "C" int r2_route_scored(const void* h, int h_stride, const float* w, const float* correction, float* dense, int32_t* chosen,
                                float* chosen_weight, float* extra, int n_rows, int n_experts, int n_extra, int top, int n_groups,
                                int keep, int width, int softmax_scores, int mark_best_only, int normalise, float weight_scale,
-                               int dtype, cudaStream_t stream) {
+                               int n_identity, const float* base, float* carried, int dtype, cudaStream_t stream) {
   if (n_rows <= 0) return R2_OK;
   if (width < 1 || n_experts < 1 || n_experts > MAX_EXPERTS || top < 1 || n_groups < 1 || n_experts % n_groups != 0 || keep < 1 ||
-      keep > n_groups || top > n_experts / n_groups * keep || n_extra < 0 || (n_extra > 0 && extra == nullptr)) return R2_BAD_SHAPE;
+      keep > n_groups || top > n_experts / n_groups * keep || n_extra < 0 || (n_extra > 0 && extra == nullptr) ||
+      n_identity < 0 || n_identity > n_experts || (n_identity > 0 && carried == nullptr)) return R2_BAD_SHAPE;
   const size_t smem = sizeof(float) * (size_t(width) + 2 * n_experts + n_groups);
   if (smem > 48 * 1024) return R2_UNSUPPORTED;
   if (dtype == R2_F32) {
     r2_launch(route_scored_kernel<float>, dim3(n_rows), dim3(256), smem, stream, (const float*)h, h_stride, w, correction, dense, chosen,
-              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale);
+              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried);
   } else if (dtype == R2_BF16) {
     r2_launch(route_scored_kernel<bf16>, dim3(n_rows), dim3(256), smem, stream, (const bf16*)h, h_stride, w, correction, dense, chosen,
-              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale);
+              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried);
   } else {
     return R2_BAD_DTYPE;
   }
@@ -318,18 +376,37 @@ extern "C" int r2_route_scored(const void* h, int h_stride, const float* w, cons
 }
 
 extern "C" int r2_expert_act(const void* gate_up, int in_stride, void* out, int out_stride, int n_rows, int inner, int kind,
-                             float limit, float alpha, float up_offset, const float* route, int n_experts, int expert_width,
+                             float limit, float alpha, float up_offset, const float* route, int route_stride, int n_experts, int expert_width,
                              float tail_limit, const float* tail_gate, int tail_gate_stride, int dtype, cudaStream_t stream) {
   if (n_rows <= 0) return R2_OK;
-  if (inner < 1 || n_experts < 0 || (n_experts > 0 && (expert_width < 1 || route == nullptr || n_experts * expert_width > inner))) return R2_BAD_SHAPE;
+  if (inner < 1 || n_experts < 0 || (n_experts > 0 && (expert_width < 1 || route == nullptr || route_stride < n_experts || n_experts * expert_width > inner))) return R2_BAD_SHAPE;
   if (n_experts == 0) expert_width = 1;
   dim3 grid(n_rows, (inner + 1023) / 1024);
   if (dtype == R2_F32) {
     r2_launch(expert_act_kernel<float>, grid, dim3(256), size_t(0), stream, (const float*)gate_up, in_stride, (float*)out, out_stride, inner, kind,
-              limit, alpha, up_offset, route, n_experts, expert_width, tail_limit, tail_gate, tail_gate_stride);
+              limit, alpha, up_offset, route, route_stride, n_experts, expert_width, tail_limit, tail_gate, tail_gate_stride);
   } else if (dtype == R2_BF16) {
     r2_launch(expert_act_kernel<bf16>, grid, dim3(256), size_t(0), stream, (const bf16*)gate_up, in_stride, (bf16*)out, out_stride, inner, kind,
-              limit, alpha, up_offset, route, n_experts, expert_width, tail_limit, tail_gate, tail_gate_stride);
+              limit, alpha, up_offset, route, route_stride, n_experts, expert_width, tail_limit, tail_gate, tail_gate_stride);
+  } else {
+    return R2_BAD_DTYPE;
+  }
+  return launch_status();
+}
+
+// up and out [n_rows, inner] with inner = experts * expert_width; act one of the feed-forward activations; route float [n_rows, >= experts].
+extern "C" int r2_expert_unit(const void* up, int in_stride, void* out, int out_stride, int n_rows, int inner, int act, const float* route,
+                              int route_stride, int expert_width, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0) return R2_OK;
+  if (inner < 1 || expert_width < 1 || inner % expert_width != 0 || route == nullptr || route_stride < inner / expert_width) return R2_BAD_SHAPE;
+  if (act < R2_ACT_NONE || act > R2_ACT_GELU_ERF) return R2_UNSUPPORTED;
+  if (dtype == R2_F32) {
+    r2_launch(expert_unit_kernel<float>, dim3(n_rows, (inner + 1023) / 1024), dim3(256), size_t(0), stream, (const float*)up, in_stride, (float*)out,
+              out_stride, inner, act, route, route_stride, expert_width, 0);
+  } else if (dtype == R2_BF16) {
+    const bool vec = expert_width % 8 == 0 && in_stride % 8 == 0 && out_stride % 8 == 0 && !((reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out)) & 15);
+    r2_launch(expert_unit_kernel<bf16>, dim3(n_rows, vec ? (inner + 2047) / 2048 : (inner + 1023) / 1024), dim3(256), size_t(0), stream, (const bf16*)up,
+              in_stride, (bf16*)out, out_stride, inner, act, route, route_stride, expert_width, int(vec));
   } else {
     return R2_BAD_DTYPE;
   }

@@ -316,13 +316,22 @@ extern "C" int r2_rms_norm(const float* x, const int32_t* rows, const float* wei
 // values, shared by all heads of their kind). One warp per (row, head), sums in float.
 // With a cache (k_cache not null) the same launch also puts the row's normed key heads and its value
 // heads (n_k_heads heads of v_head_dim values from column v_col on) into the row's cache slot, so that
-// no second kernel reads the projection again.
+// no second kernel reads the projection again. A temperature multiplies the normed query heads by a factor of the row's position.
+struct QueryTemp {
+  const int32_t* positions;   // null: no temperature
+  float coef;                 // the factor at position p is 1 + coef ln(floor((p + 1) / every) + 1)
+  int every;
+};
+__device__ __forceinline__ float query_factor(const QueryTemp& q, int row) {
+  return q.positions == nullptr ? 1.f : 1.f + q.coef * logf(float((q.positions[row] + 1) / q.every + 1));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_kernel(T* __restrict__ buf, int row_stride, int n_rows, int n_q_heads, int n_k_heads, int head_dim,
                  const float* __restrict__ w_q, const float* __restrict__ w_k, float eps, float offset,
                  T* __restrict__ k_cache, T* __restrict__ v_cache, const int32_t* __restrict__ slot_mapping, int v_col,
-                 int v_head_dim, int page_size, long long page_stride, int n_pages) {
+                 int v_head_dim, int page_size, long long page_stride, int n_pages, QueryTemp temp) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -356,7 +365,7 @@ head_norm_kernel(T* __restrict__ buf, int row_stride, int n_rows, int n_q_heads,
     float v = to_float(p[d]);
     sq = fmaf(v, v, sq);
   }
-  const float inv = 1.f / sqrtf(warp_sum(sq) / float(head_dim) + eps);
+  const float inv = 1.f / sqrtf(warp_sum(sq) / float(head_dim) + eps) * (h < n_q_heads ? query_factor(temp, r) : 1.f);
   T* dst = nullptr;
   if (cached) dst = k_cache + page_base + (size_t(h - n_q_heads) * page_size + off) * head_dim;
   for (int d = lane; d < head_dim; d += 32) {
@@ -373,7 +382,7 @@ __global__ void __launch_bounds__(128)
 head_norm_pair_kernel(T* __restrict__ buf, int row_stride, int n_rows, int n_q_heads, int n_k_heads, int head_dim,
                       const float* __restrict__ w_q, const float* __restrict__ w_k, float eps, float offset,
                       T* __restrict__ k_cache, T* __restrict__ v_cache, const int32_t* __restrict__ slot_mapping, int v_col,
-                      int v_head_dim, int page_size, long long page_stride, int n_pages) {
+                      int v_head_dim, int page_size, long long page_stride, int n_pages, QueryTemp temp) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -413,7 +422,7 @@ head_norm_pair_kernel(T* __restrict__ buf, int row_stride, int n_rows, int n_q_h
     v[i] = d < head_dim ? load2(p + d) : make_float2(0.f, 0.f);
     sq += v[i].x * v[i].x + v[i].y * v[i].y;
   }
-  const float inv = 1.f / sqrtf(warp_sum(sq) / float(head_dim) + eps);
+  const float inv = 1.f / sqrtf(warp_sum(sq) / float(head_dim) + eps) * (h < n_q_heads ? query_factor(temp, r) : 1.f);
   T* dst = cached ? k_cache + page_base + (size_t(h - n_q_heads) * page_size + off) * head_dim : nullptr;
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
@@ -435,7 +444,7 @@ __global__ void __launch_bounds__(128)
 head_norm_vec8_kernel(bf16* __restrict__ buf, int row_stride, int n_rows, int n_q_heads, int n_k_heads, int head_dim,
                       const float* __restrict__ w_q, const float* __restrict__ w_k, float eps, float offset,
                       bf16* __restrict__ k_cache, bf16* __restrict__ v_cache, const int32_t* __restrict__ slot_mapping, int v_col,
-                      int v_head_dim, int page_size, long long page_stride, int n_pages) {
+                      int v_head_dim, int page_size, long long page_stride, int n_pages, QueryTemp temp) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -485,7 +494,7 @@ head_norm_vec8_kernel(bf16* __restrict__ buf, int row_stride, int n_rows, int n_
   const int first_lane = (lane / lanes_qk) * lanes_qk;
   for (int j = 0; j < lanes_qk; ++j) total += __shfl_sync(0xffffffffu, sq, (first_lane + j) & 31);
   if (!mine) return;
-  const float inv = 1.f / sqrtf(total / float(head_dim) + eps);
+  const float inv = 1.f / sqrtf(total / float(head_dim) + eps) * (h < n_q_heads ? query_factor(temp, r) : 1.f);
   const float* gain = (h < n_q_heads ? w_q : w_k) + e;
   const float4 g0 = *reinterpret_cast<const float4*>(gain), g1 = *reinterpret_cast<const float4*>(gain + 4);
   uint4 y;
@@ -503,10 +512,12 @@ head_norm_vec8_kernel(bf16* __restrict__ buf, int row_stride, int n_rows, int n_
 extern "C" int r2_head_norm(void* buf, int row_stride, int n_rows, int n_q_heads, int n_k_heads, int head_dim,
                             const float* w_q, const float* w_k, float eps, float offset, void* k_cache, void* v_cache,
                             const int32_t* slot_mapping, int v_col, int v_head_dim, int page_size, long long page_stride,
-                            int n_pages, int dtype, cudaStream_t stream) {
+                            int n_pages, const int32_t* positions, float temp_coef, int temp_every, int dtype, cudaStream_t stream) {
   if (n_rows <= 0) return R2_OK;
   if (n_q_heads < 0 || n_k_heads < 0 || n_q_heads + n_k_heads < 1 || head_dim < 1) return R2_BAD_SHAPE;
   if (k_cache != nullptr && (v_cache == nullptr || slot_mapping == nullptr || v_head_dim < 1 || page_size < 1 || n_pages < 1)) return R2_BAD_SHAPE;
+  if (positions != nullptr && temp_every < 1) return R2_BAD_SHAPE;
+  const QueryTemp temp = {positions, temp_coef, temp_every};
   const long long items = (long long)n_rows * (n_q_heads + n_k_heads + (k_cache != nullptr ? n_k_heads : 0));
   dim3 grid((unsigned)((items + 3) / 4));
   const size_t esize = dtype == R2_F32 ? 4 : 2;
@@ -525,25 +536,25 @@ extern "C" int r2_head_norm(void* buf, int row_stride, int n_rows, int n_q_heads
     }
     const long long warps = (long long)n_rows * slabs;
     r2_launch(head_norm_vec8_kernel, dim3((unsigned)((warps + 3) / 4)), dim3(128), size_t(0), stream, (bf16*)buf, row_stride, n_rows, n_q_heads, n_k_heads,
-              head_dim, w_q, w_k, eps, offset, (bf16*)k_cache, (bf16*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages);
+              head_dim, w_q, w_k, eps, offset, (bf16*)k_cache, (bf16*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages, temp);
     return launch_status();
   }
   if (pairs && dtype == R2_F32) {
     r2_launch(head_norm_pair_kernel<float>, grid, dim3(128), size_t(0), stream, (float*)buf, row_stride, n_rows, n_q_heads, n_k_heads, head_dim, w_q, w_k, eps, offset,
-              (float*)k_cache, (float*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages);
+              (float*)k_cache, (float*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages, temp);
     return launch_status();
   }
   if (pairs && dtype == R2_BF16) {
     r2_launch(head_norm_pair_kernel<bf16>, grid, dim3(128), size_t(0), stream, (bf16*)buf, row_stride, n_rows, n_q_heads, n_k_heads, head_dim, w_q, w_k, eps, offset,
-              (bf16*)k_cache, (bf16*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages);
+              (bf16*)k_cache, (bf16*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages, temp);
     return launch_status();
   }
   if (dtype == R2_F32) {
     r2_launch(head_norm_kernel<float>, grid, dim3(128), size_t(0), stream, (float*)buf, row_stride, n_rows, n_q_heads, n_k_heads, head_dim, w_q, w_k, eps, offset,
-              (float*)k_cache, (float*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages);
+              (float*)k_cache, (float*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages, temp);
   } else if (dtype == R2_BF16) {
     r2_launch(head_norm_kernel<bf16>, grid, dim3(128), size_t(0), stream, (bf16*)buf, row_stride, n_rows, n_q_heads, n_k_heads, head_dim, w_q, w_k, eps, offset,
-              (bf16*)k_cache, (bf16*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages);
+              (bf16*)k_cache, (bf16*)v_cache, slot_mapping, v_col, v_head_dim, page_size, page_stride, n_pages, temp);
   } else {
     return R2_BAD_DTYPE;
   }
@@ -688,7 +699,8 @@ rotate_half_kernel(T* __restrict__ buf, int row_stride, int n_heads, int head_di
 // all in float and rounded once on the way out. One warp per unit of work and eight units a CTA (grid: rows x ceil(units / 8)),
 // so that a decode step's few rows still spread over many SMs: units 0 .. n_heads - 1 are the heads (the first n_q_heads take the
 // gain q_w, the others k_w; null: no norm), and a key head's warp also puts the turned key into the row's cache slot; with a
-// cache, units n_heads .. n_heads + n_kv_heads - 1 copy the value heads to the slot. The row's cosines and sines are made once
+// cache, units n_heads .. n_heads + n_kv_heads - 1 copy the value heads to the slot. `interleaved`: dimension 2i turns with 2i + 1
+// instead of i with i + half. The row's cosines and sines are made once
 // a CTA, in shared memory, for all its heads. `vec`: neighbouring pairs of elements may go as one access (even sizes and strides).
 constexpr int NORM_ROTATE_MAX_DIM = 512, NORM_ROTATE_WARPS = 8;
 template <typename T>
@@ -697,7 +709,7 @@ norm_rotate_half_kernel(T* __restrict__ buf, int row_stride, int n_heads, int n_
                         float magnitude, const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                         const int32_t* __restrict__ positions, T* __restrict__ k_cache, T* __restrict__ v_cache,
                         const int32_t* __restrict__ slot_mapping, int k_col, int v_col, int n_kv_heads, int v_head_dim, int page_size,
-                        long long page_stride, int n_pages, int vec) {
+                        long long page_stride, int n_pages, int vec, int interleaved) {
   pdl_launch_dependents();
   __shared__ float stage[NORM_ROTATE_WARPS][NORM_ROTATE_MAX_DIM];
   __shared__ float cs_s[NORM_ROTATE_MAX_DIM / 2], sn_s[NORM_ROTATE_MAX_DIM / 2];
@@ -771,6 +783,29 @@ norm_rotate_half_kernel(T* __restrict__ buf, int row_stride, int n_heads, int n_
   __syncwarp();
   // the value at dimension d after its norm
   auto normed = [&](int d) { return w != nullptr ? mine[d] * inv * w[d] : mine[d]; };
+  if (interleaved) {   // a lane has whole pairs: dimensions d and d + 1
+    for (int d = 2 * lane; d < head_dim; d += 64) {
+      const bool two = d + 1 < head_dim;
+      float a0 = normed(d), a1 = two ? normed(d + 1) : 0.f;
+      if (d < 2 * half) {
+        const float u = a0, v = a1, cs = cs_s[d >> 1], sn = sn_s[d >> 1];
+        a0 = u * cs - v * sn;
+        a1 = v * cs + u * sn;
+      }
+      if (vec) {
+        store2(x + d, a0, a1);
+        if (kdst != nullptr) store2(kdst + d, a0, a1);
+      } else {
+        x[d] = from_float<T>(a0);
+        if (two) x[d + 1] = from_float<T>(a1);
+        if (kdst != nullptr) {
+          kdst[d] = from_float<T>(a0);
+          if (two) kdst[d + 1] = from_float<T>(a1);
+        }
+      }
+    }
+    continue;
+  }
   if (vec) {   // half and head_dim are even: two neighbouring pairs (or two passing dimensions) a step
     for (int i = 2 * lane; i < head_dim - half; i += 64) {
       if (i < half) {
@@ -831,18 +866,19 @@ pair_norm_add_kernel(const float* __restrict__ x, const float* __restrict__ a, c
 // With k_cache (may be null) the launch also writes the row's keys (columns k_col .., n_kv_heads heads of head_dim, after
 // their rotation) and values (columns v_col .., heads of v_head_dim) to the row's slot of the paged cache.
 // With q_norm_w / k_norm_w (float [head_dim]; both or neither) every head is RMS-normed before its rotation: the first
-// n_q_heads heads with q_norm_w, the others with k_norm_w. `magnitude` multiplies cos and sin.
+// n_q_heads heads with q_norm_w, the others with k_norm_w. `magnitude` multiplies cos and sin. `interleaved`: the pairs are
+// dimensions 2i and 2i + 1.
 extern "C" int r2_rotate_half(void* buf, int row_stride, int n_rows, int n_heads, int head_dim, int rot_dims, const float* inv_freq,
                               const int32_t* positions, void* k_cache, void* v_cache, const int32_t* slot_mapping, int k_col, int v_col,
                               int n_kv_heads, int v_head_dim, int page_size, long long page_stride, int n_pages,
-                              const float* q_norm_w, const float* k_norm_w, int n_q_heads, float norm_eps, float magnitude, int dtype,
+                              const float* q_norm_w, const float* k_norm_w, int n_q_heads, float norm_eps, float magnitude, int interleaved, int dtype,
                               cudaStream_t stream) {
   const bool normed = q_norm_w != nullptr || k_norm_w != nullptr;
   if (n_rows <= 0 || (rot_dims == 0 && k_cache == nullptr && !normed)) return R2_OK;
   if (n_heads < 1 || rot_dims < 0 || rot_dims % 2 != 0 || rot_dims > head_dim) return R2_BAD_SHAPE;
   if (k_cache != nullptr && (v_cache == nullptr || slot_mapping == nullptr || n_kv_heads < 1 || v_head_dim < 1 || page_size < 1)) return R2_BAD_SHAPE;
   const int half = rot_dims / 2;
-  if (normed || magnitude != 1.f) {
+  if (normed || magnitude != 1.f || interleaved) {
     if (head_dim > NORM_ROTATE_MAX_DIM || n_q_heads < 0 || n_q_heads > n_heads) return R2_BAD_SHAPE;
     if ((n_q_heads > 0 && normed && q_norm_w == nullptr) || (n_q_heads < n_heads && normed && k_norm_w == nullptr)) return R2_BAD_SHAPE;
     // few rows (a decode step): a row's units spread over several CTAs; a prompt step's rows: one CTA a row, its cosines and sines made
@@ -851,18 +887,18 @@ extern "C" int r2_rotate_half(void* buf, int row_stride, int n_rows, int n_heads
     const bool one_cta_a_row = n_rows >= 512 && n_rows < 16384;
     const dim3 grid2(n_rows, one_cta_a_row ? 1 : (n_heads + (k_cache != nullptr ? n_kv_heads : 0) + NORM_ROTATE_WARPS - 1) / NORM_ROTATE_WARPS);
     // neighbouring elements as one access: every size, stride and column that an address is made of is even
-    const bool pairs_ok = head_dim % 2 == 0 && half % 2 == 0 && row_stride % 2 == 0 &&
+    const bool pairs_ok = head_dim % 2 == 0 && (interleaved || half % 2 == 0) && row_stride % 2 == 0 &&
                           (k_cache == nullptr || (k_col % 2 == 0 && v_col % 2 == 0 && v_head_dim % 2 == 0 && page_stride % 2 == 0));
     if (dtype == R2_F32) {
       const bool vec = pairs_ok && pair_aligned((const float*)buf) && (k_cache == nullptr || (pair_aligned((const float*)k_cache) && pair_aligned((const float*)v_cache)));
       r2_launch(norm_rotate_half_kernel<float>, grid2, dim3(NORM_ROTATE_WARPS * 32), size_t(0), stream, (float*)buf, row_stride, n_heads, n_q_heads, head_dim,
                 half, inv_freq, magnitude, q_norm_w, k_norm_w, norm_eps, positions, (float*)k_cache, (float*)v_cache, slot_mapping, k_col, v_col,
-                n_kv_heads, v_head_dim, page_size, page_stride, n_pages, int(vec));
+                n_kv_heads, v_head_dim, page_size, page_stride, n_pages, int(vec), interleaved);
     } else if (dtype == R2_BF16) {
       const bool vec = pairs_ok && pair_aligned((const bf16*)buf) && (k_cache == nullptr || (pair_aligned((const bf16*)k_cache) && pair_aligned((const bf16*)v_cache)));
       r2_launch(norm_rotate_half_kernel<bf16>, grid2, dim3(NORM_ROTATE_WARPS * 32), size_t(0), stream, (bf16*)buf, row_stride, n_heads, n_q_heads, head_dim,
                 half, inv_freq, magnitude, q_norm_w, k_norm_w, norm_eps, positions, (bf16*)k_cache, (bf16*)v_cache, slot_mapping, k_col, v_col,
-                n_kv_heads, v_head_dim, page_size, page_stride, n_pages, int(vec));
+                n_kv_heads, v_head_dim, page_size, page_stride, n_pages, int(vec), interleaved);
     } else {
       return R2_BAD_DTYPE;
     }

@@ -143,7 +143,7 @@ def _lib(source: str) -> C.CDLL:
 def build_all(head_dims=()) -> None:
     """Compile every kernel library that does not depend on a model, and the attention kernels
     for the given head sizes (a model compiles its own head size at first use otherwise)."""
-    for source in ("rowwise", "recurrent", "state_scan", "routing", "gemm_simt", "gemm_tc", "attention_simt", "attention_prefill_tc", "latent_attention",
+    for source in ("rowwise", "recurrent", "state_scan", "streams", "routing", "gemm_simt", "gemm_tc", "attention_simt", "attention_prefill_tc", "latent_attention",
                    "sampling", "wait_selftest"):
         _lib(source)
     kernel_library("sfu_probe")  # (profiling/sfu_probe.py: a measurement, no part of a step)
@@ -449,15 +449,21 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch
 
 
 def head_norm(buf: torch.Tensor, n_q_heads: int, n_k_heads: int, head_dim: int, w_q: torch.Tensor, w_k: torch.Tensor,
-              eps: float, unit_offset: bool = False, kv: KvScatter | None = None) -> None:
+              eps: float, unit_offset: bool = False, kv: KvScatter | None = None, temperature: tuple | None = None) -> None:
     """RMS norm, in place, of each of the first n_q_heads + n_k_heads heads of every row of `buf` (a fused
     projection whose first columns are the query heads and then the key heads); the query heads take the
     gain `w_q`, the key heads `w_k` (float32 [head_dim], shared by the heads of a kind). With `kv` (see
     `kv_scatter`; `col` the first value column, `width` the values' width, `head_dim` the values' head size)
-    the same launch puts the normed keys and the values into the rows' cache slots."""
+    the same launch puts the normed keys and the values into the rows' cache slots. `temperature` (positions int32 [T], coef,
+    every): the normed query heads are multiplied by 1 + coef ln(floor((position + 1) / every) + 1)."""
     _need(buf, "buf", dim=2)
     _need(w_q, "w_q", torch.float32, 1)
     _need(w_k, "w_k", torch.float32, 1)
+    positions, temp_coef, temp_every = temperature if temperature is not None else (None, 0.0, 1)
+    if positions is not None:
+        _need(positions, "positions", torch.int32, 1)
+        if positions.shape[0] < buf.shape[0] or temp_every < 1:
+            raise KernelError("head_norm: a temperature needs a position for every row and a period of at least one")
     if w_q.shape[0] != head_dim or w_k.shape[0] != head_dim or buf.shape[1] < (n_q_heads + n_k_heads) * head_dim:
         raise KernelError(f"head_norm: buf {tuple(buf.shape)} does not hold {n_q_heads} + {n_k_heads} heads of {head_dim}")
     if kv is not None and (kv.width != n_k_heads * kv.head_dim or kv.col + kv.width > buf.shape[1]):
@@ -466,7 +472,7 @@ def head_norm(buf: torch.Tensor, n_q_heads: int, n_k_heads: int, head_dim: int, 
              C.c_longlong(kv.page_stride), kv.n_pages) if kv is not None else (None, None, None, 0, 0, 0, C.c_longlong(0), 0)
     status = _lib("rowwise").r2_head_norm(_p(buf), _rows(buf, "buf"), buf.shape[0], n_q_heads, n_k_heads, head_dim, _p(w_q),
                                          _p(w_k), C.c_float(eps), C.c_float(1.0 if unit_offset else 0.0), *cache,
-                                         dtype_code(buf.dtype), _stream())
+                                         _p(positions), C.c_float(temp_coef), int(temp_every), dtype_code(buf.dtype), _stream())
     _check(status, "head_norm")
 
 
@@ -492,7 +498,7 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
     """The inner activation of gated feed-forwards whose projections lie side by side: a row of `gate_up` [T, 2 F] holds
     the gates of all F columns and then their ups. kind "relu": relu(g) * u. kind "clamped_swish": g' sigmoid(alpha g')
     (u' + up_offset) with g' = min(g, limit), u' = clamp(u, -limit, limit). kind "silu": g sigmoid(g) * u. kind "gelu_tanh": gelu(g) * u in gelu's
-    tanh form. With `route` (float32 [T, n_experts], zero
+    tanh form. With `route` (float32 [T, >= n_experts], zero
     for experts that a row does not use) the first n_experts * expert_width columns are the routed experts', each
     multiplied by the row's weight for its expert; the columns after them belong to an expert that every row uses
     (limit `tail_limit`), multiplied by sigmoid(tail_gate[row]) where `tail_gate` (float32 [T] or [T, 1], the gate's logit)
@@ -506,7 +512,7 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
     inner = gate_up.shape[1] // 2
     if route is not None:
         _need(route, "route", torch.float32, 2)
-        if route.shape != (gate_up.shape[0], n_experts) or not route.is_contiguous() or n_experts * expert_width > inner:
+        if route.shape[0] != gate_up.shape[0] or route.shape[1] < n_experts or not route.is_contiguous() or n_experts * expert_width > inner:
             raise KernelError(f"expert_act: route {tuple(route.shape)} does not fit {n_experts} experts of {expert_width} in {inner} columns")
     else:
         n_experts = 0
@@ -520,10 +526,57 @@ def expert_act(gate_up: torch.Tensor, kind: str, limit: float = 0.0, alpha: floa
         out = torch.empty(gate_up.shape[0], inner, dtype=gate_up.dtype, device=gate_up.device)
     status = _lib("routing").r2_expert_act(
         _p(gate_up), _rows(gate_up, "gate_up"), _p(out), _rows(out, "out"), gate_up.shape[0], inner, kinds[kind],
-        C.c_float(limit), C.c_float(alpha), C.c_float(up_offset), _p(route), n_experts, expert_width,
+        C.c_float(limit), C.c_float(alpha), C.c_float(up_offset), _p(route), 0 if route is None else route.shape[1], n_experts, expert_width,
         C.c_float(limit if tail_limit is None else tail_limit), _p(tail_gate), tail_gate_stride, dtype_code(gate_up.dtype), _stream())
     _check(status, "expert_act")
     return out
+
+
+def expert_unit(up: torch.Tensor, act: str, route: torch.Tensor, expert_width: int, out: torch.Tensor | None = None) -> torch.Tensor:
+    """act(up) times the row's weight for the column's expert: the inner activation of experts without gates, whose values lie side by
+    side in a row of `up` [T, experts * expert_width]; route float32 [T, >= experts]. -> [T, F] in the same dtype."""
+    _need(up, "up", dim=2)
+    _need(route, "route", torch.float32, 2)
+    if act not in ACTIVATIONS or expert_width < 1 or up.shape[1] % expert_width or route.shape[0] != up.shape[0] or route.shape[1] < up.shape[1] // expert_width:
+        raise KernelError(f"expert_unit: up {tuple(up.shape)}, experts of {expert_width}, route {tuple(route.shape)}, activation {act!r} do not fit")
+    if out is None:
+        out = torch.empty(up.shape, dtype=up.dtype, device=up.device)
+    status = _lib("routing").r2_expert_unit(_p(up), _rows(up, "up"), _p(out), _rows(out, "out"), up.shape[0], up.shape[1], ACTIVATIONS[act], _p(route),
+                                           _rows(route, "route"), expert_width, dtype_code(up.dtype), _stream())
+    _check(status, "expert_unit")
+    return out
+
+
+def stream_join(x: torch.Tensor, read: torch.Tensor, gain: torch.Tensor | None = None, eps: float = 0.0, dtype: torch.dtype = torch.float32,
+                y: torch.Tensor | None = None, mix: torch.Tensor | None = None, join: torch.Tensor | None = None, keep: bool = True):
+    """Several residual streams side by side: x float32 [T, S, D], or [T, D] for streams that all hold that row (S is then the length of
+    `read`). With `y` (float32 [T, D]) the streams take a sublayer's output, x_b <- sum_a mix[a, b] x_a + join[b] y (mix float32 [S, S],
+    [from, to]; join float32 [S]), all of them at once; then u = sum_a read[a] x_a of the new streams. With `gain` (float32 [D])
+    u leaves as rms_norm(u) * gain in `dtype`, else as it is in float32. The new streams are written over x where x holds them all;
+    `keep` False: they are not needed. -> (the streams float32 [T, S, D] or None, u [T, D])."""
+    _need(x, "x", torch.float32)
+    _need(read, "read", torch.float32, 1)
+    s, t, d = read.shape[0], x.shape[0], x.shape[-1]
+    spread = x.dim() == 2
+    if not x.is_contiguous() or x.dim() not in (2, 3) or (not spread and x.shape[1] != s):
+        raise KernelError(f"stream_join: x {tuple(x.shape)} does not hold {s} streams")
+    if gain is not None:
+        _need(gain, "gain", torch.float32, 1)
+        if gain.shape[0] != d:
+            raise KernelError(f"stream_join: gain {tuple(gain.shape)} does not fit the width {d}")
+    streams = None
+    if y is not None:
+        for name, w, shape in (("y", y, (t, d)), ("mix", mix, (s, s)), ("join", join, (s,))):
+            _need(w, name, torch.float32)
+            if tuple(w.shape) != shape or not w.is_contiguous():
+                raise KernelError(f"stream_join: {name} {tuple(w.shape)} is not a contiguous {shape}")
+        if keep:
+            streams = torch.empty(t, s, d, dtype=torch.float32, device=x.device) if spread else x
+    u = torch.empty(t, d, dtype=dtype if gain is not None else torch.float32, device=x.device)
+    status = _lib("streams").r2_stream_join(_p(x), int(spread), _p(y), _p(mix), _p(join), _p(read), _p(streams), _p(gain), C.c_float(eps), _p(u), t, s, d,
+                                           dtype_code(u.dtype), _stream())
+    _check(status, "stream_join")
+    return (streams if y is not None else x), u
 
 
 def small_linear(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
@@ -567,14 +620,16 @@ def route_top_k(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, top
 
 def rotate_half(buf: torch.Tensor, n_heads: int, head_dim: int, rot_dims: int, inv_freq: torch.Tensor, positions: torch.Tensor,
                 kv: KvScatter | None = None, n_kv_heads: int = 0, k_col: int = 0, *, q_norm: torch.Tensor | None = None,
-                k_norm: torch.Tensor | None = None, n_q_heads: int = 0, norm_eps: float = 0.0, magnitude: float = 1.0) -> None:
+                k_norm: torch.Tensor | None = None, n_q_heads: int = 0, norm_eps: float = 0.0, magnitude: float = 1.0,
+                interleaved: bool = False) -> None:
     """Rotation by position, in place, of the first `n_heads` heads of every row of `buf` (a stacked projection whose
     first columns are the query heads and then the key heads): of each head the first rot_dims dimensions, dimension i
     paired with i + rot_dims / 2, by the angle position * inv_freq[i] (float32 [rot_dims / 2]). With `kv` (see
     `kv_scatter`: `col` the first value column, `head_dim` the values' head size) the same launch puts the rotated keys
     (n_kv_heads heads from column `k_col`) and the values into the rows' cache slots. With `q_norm` / `k_norm` (float32
     [head_dim]) every head is RMS-normed before its rotation, in float32 and in the same launch: the first `n_q_heads` heads with
-    the gain q_norm, the others with k_norm, eps `norm_eps`. `magnitude` multiplies cos and sin."""
+    the gain q_norm, the others with k_norm, eps `norm_eps`. `magnitude` multiplies cos and sin. `interleaved`: the pairs are dimensions
+    2i and 2i + 1 instead."""
     _need(buf, "buf", dim=2)
     _need(inv_freq, "inv_freq", torch.float32, 1)
     for name, t in (("q_norm", q_norm), ("k_norm", k_norm)):
@@ -593,7 +648,7 @@ def rotate_half(buf: torch.Tensor, n_heads: int, head_dim: int, rot_dims: int, i
              C.c_longlong(kv.page_stride), kv.n_pages) if kv is not None else (None, None, None, 0, 0, 0, 0, 0, C.c_longlong(0), 0)
     status = _lib("rowwise").r2_rotate_half(_p(buf), _rows(buf, "buf"), buf.shape[0], n_heads, head_dim, rot_dims, _p(inv_freq),
                                            _p(positions), *cache, _p(q_norm), _p(k_norm), n_q_heads, C.c_float(norm_eps),
-                                           C.c_float(magnitude), dtype_code(buf.dtype), _stream())
+                                           C.c_float(magnitude), int(bool(interleaved)), dtype_code(buf.dtype), _stream())
     _check(status, "rotate_half")
 
 
@@ -685,14 +740,16 @@ def xielu(z: torch.Tensor, a_pos: float, a_neg: float, out: torch.Tensor | None 
 
 
 def route_scored(h: torch.Tensor, w: torch.Tensor, correction: torch.Tensor | None, top: int, n_groups: int = 1, keep_groups: int = 1,
-                 n_extra: int = 0, scoring: str = "sigmoid", group_mark: str = "two_best", normalise: bool = True, weight_scale: float = 1.0):
+                 n_extra: int = 0, scoring: str = "sigmoid", group_mark: str = "two_best", normalise: bool = True, weight_scale: float = 1.0,
+                 n_identity: int = 0, base: torch.Tensor | None = None):
     """Router with sigmoid scores: logits h @ w^T in float32 (w float32 [experts + n_extra, K]); an expert is chosen by
     sigmoid(logit) + correction, only inside the `keep_groups` best of `n_groups` equal groups of neighbouring experts (a
     group counts by the sum of its two largest choice scores; the lower index wins ties), the `top` largest; the chosen
     experts' weights are their sigmoids over the sum of the chosen sigmoids (+ 1e-20). The last n_extra rows of w are further
     gates: their logits come back as they are. `scoring` "softmax": the scores are the softmax of the logits over all experts
-    instead of their sigmoids. `group_mark` "best": a group counts by its largest choice score alone. `normalise` False: a chosen
-    expert's weight is its score times `weight_scale` (the weights are not made to sum to one).
+    instead of their sigmoids. `group_mark` "best": a group counts by its largest choice score alone. `normalise` False: the chosen
+    scores are not made to sum to one. The weights are multiplied by `weight_scale`. `n_identity` > 0: the last of the experts stand for
+    the row h itself, and a fifth result is h times their weights' sum (+ `base` [T, K] where given), float32 [T, K].
     -> (dense float32 [T, experts]: a row's weights, zero where not chosen; chosen
     int32 [T, top]; their weights float32 [T, top]; extra float32 [T, n_extra] or None)."""
     if scoring not in ("sigmoid", "softmax") or group_mark not in ("two_best", "best"):
@@ -712,20 +769,26 @@ def route_scored(h: torch.Tensor, w: torch.Tensor, correction: torch.Tensor | No
     chosen = torch.empty(n, top, dtype=torch.int32, device=h.device)
     weight = torch.empty(n, top, dtype=torch.float32, device=h.device)
     extra = torch.empty(n, n_extra, dtype=torch.float32, device=h.device) if n_extra else None
+    carried = torch.empty(n, h.shape[1], dtype=torch.float32, device=h.device) if n_identity else None
+    if base is not None:
+        _need(base, "base", torch.float32, 2)
+        if not n_identity or base.shape != h.shape or not base.is_contiguous():
+            raise KernelError(f"route_scored: base {tuple(base.shape)} does not fit h {tuple(h.shape)} (or nothing is to be carried)")
     status = _lib("routing").r2_route_scored(_p(h), _rows(h, "h"), _p(w), _p(correction), _p(dense), _p(chosen), _p(weight), _p(extra),
                                             n, e, n_extra, top, n_groups, keep_groups, h.shape[1], int(scoring == "softmax"),
-                                            int(group_mark == "best"), int(bool(normalise)), C.c_float(weight_scale), dtype_code(h.dtype), _stream())
+                                            int(group_mark == "best"), int(bool(normalise)), C.c_float(weight_scale), int(n_identity), _p(base), _p(carried),
+                                            dtype_code(h.dtype), _stream())
     _check(status, "route_scored")
-    return dense, chosen, weight, extra
+    return (dense, chosen, weight, extra, carried) if n_identity else (dense, chosen, weight, extra)
 
 
 def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, k_scale: float,
                    inv_freq: torch.Tensor | None, rot_dims: int, positions: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor,
-                   state_slot: torch.Tensor, fresh: torch.Tensor, n_heads: int, dim: int, vdim: int) -> torch.Tensor:
+                   state_slot: torch.Tensor, fresh: torch.Tensor, n_heads: int, dim: int, vdim: int, silu: bool = False) -> torch.Tensor:
     """Retention's recurrence S <- decay[h] S + k v^T, o = S^T q for every entry of a batch, from and to the entries' state
     slots. q, k [T, heads * dim], v [T, heads * vdim] (slices of a projection); the kernel rotates q and k by position on their
     way in (of each head the first rot_dims dimensions, i with i + rot_dims / 2, angle positions[t] * inv_freq[i], in float32)
-    and multiplies k by k_scale after that. decay float32 [heads]; state float32 [slots, heads * dim * vdim].
+    and multiplies k by k_scale after that. `silu`: q, k and v pass silu on their way in (float32, instead of a rotation). decay float32 [heads]; state float32 [slots, heads * dim * vdim].
     -> float32 [T, heads * vdim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
     for name, t, width in (("q", q, n_heads * dim), ("k", k, n_heads * dim), ("v", v, n_heads * vdim)):
@@ -745,7 +808,7 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     status = _lib("recurrent").r2_retention_scan(
         _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), C.c_float(k_scale), _p(inv_freq if rot_dims else None),
         rot_dims, _p(positions), _p(state), C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out),
-        _rows(out, "out"), n_heads, dim, vdim, int(q.shape[0] <= n), dtype_code(q.dtype), _stream())
+        _rows(out, "out"), n_heads, dim, vdim, int(q.shape[0] <= n), int(bool(silu)), dtype_code(q.dtype), _stream())
     _check(status, "retention_scan")
     return out
 
@@ -1352,7 +1415,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     keep_first: int = 0, sink: bool = False, gate: torch.Tensor | None = None, softcap: float = 0.0,
                     sinks: torch.Tensor | None = None, head_gate: torch.Tensor | None = None,
                     values_in_keys: bool = False, chunk: int = 0, dist_bias: torch.Tensor | None = None,
-                    out_scale: float = 1.0) -> torch.Tensor:
+                    out_scale: float = 1.0, exact: bool = False) -> torch.Tensor:
     """Causal attention of q [T, n_heads * head_dim] over the paged cache -> [T, n_heads * v_head_dim]
     (`v_head_dim` 0: the keys' head size). With a window, `keep_first` keeps a sequence's first keys visible;
     `sink` adds one to the softmax's denominator (an extra exp(0) term: the weights sum to less than one); `gate`
@@ -1369,7 +1432,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     `decode_only` says that every row is an entry of its own (one new token each) and
     `max_context` bounds the rows' context lengths; `q_start` (int32 [R + 1]) with `n_tiles`, the
     sum over entries of ceil(rows / 64), lets the tensor-core prefill kernel take the batch. They
-    only choose the kernel and its slicing."""
+    only choose the kernel and its slicing. `exact`: attention without any of the extras also carries its softmax weights into the
+    tensor cores' second product as two terms (see `use_exact_weights`)."""
     _need(q, "q", dim=2)
     for name, t in (("row_entry", row_entry), ("positions", positions), ("seq_lens", seq_lens)):
         _need(t, name, torch.int32, 1)
@@ -1408,7 +1472,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             raise KernelError(f"attention: head_gate {tuple(head_gate.shape)} is not [T, {n_heads}]")
         head_gate_stride = _rows(head_gate, "head_gate")
     plain = fits and keep_first == 0 and not sink and gate is None and not capped
-    if plain and q.dtype == torch.bfloat16 and decode_only and _fast_attention and group in (1, 2, 4, 8):
+    if plain and not exact and q.dtype == torch.bfloat16 and decode_only and _fast_attention and group in (1, 2, 4, 8):
         lib = _lib_for_head_dim("attention_decode", head_dim)
         n_slices = decode_slices(n, n_kv_heads, max_context, q.device)
         ws = _workspace(q.device)
@@ -1435,7 +1499,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             _p(q), _rows(q, "q"), n, _p(out), _rows(out, "out"), _p(k_cache), _p(v_cache), C.c_longlong(page_stride),
             page_size, n_pages, _p(block_tables), block_tables.shape[1], _p(q_start), _p(seq_lens), n_entries,
             (n_tiles + n_entries + 1) // 2, n_heads, n_kv_heads, C.c_float(scale), window, _p(_workspace(q.device).error),
-            keep_first, int(bool(sink)), _p(gate), gate_stride, int(_exact_weights and not plain), _stream())
+            keep_first, int(bool(sink)), _p(gate), gate_stride, int(_exact_weights and (exact or not plain)), _stream())
         if status != -4:
             _check(status, "paged_attention (prefill, tcgen05)")
             _used("attention_prefill_tc")
@@ -1448,7 +1512,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _p(k_cache), _p(v_cache), C.c_longlong(page_stride),
             page_size, n_pages, _p(block_tables), block_tables.shape[1], _p(q_start), _p(seq_lens),
             q_start.shape[0] - 1, n_tiles, n_heads, n_kv_heads, C.c_float(scale), window, _p(_workspace(q.device).error),
-            keep_first, int(bool(sink)), _p(gate), gate_stride, int(_exact_weights and not plain), C.c_float(softcap), _p(sinks),
+            keep_first, int(bool(sink)), _p(gate), gate_stride, int(_exact_weights and (exact or not plain)), C.c_float(softcap), _p(sinks),
             _p(head_gate), head_gate_stride, chunk, _p(dist_bias), bias_len, C.c_float(out_scale), _stream())
         _check(status, "paged_attention (prefill)")
         _used("attention_prefill")

@@ -76,6 +76,8 @@ class DecoderModel:
                     (("post_norm_1", layer.post_norm_1), ("post_norm_2", layer.post_norm_2)) if spec is not None}
             if layer.token_side is not None:
                 post["token_side"] = build_part("token_side", layer.token_side, tensors, rt)
+            if layer.block_weights:
+                post["weights"] = {own: tensors[name].to(rt.device, torch.float32) for own, name in layer.block_weights.items()}
             self.blocks.append(block_cls(
                 build_part("norm", layer.norm_1, tensors, rt), mixer,
                 build_part("norm", layer.norm_2, tensors, rt) if layer.norm_2 is not None else None,
@@ -129,10 +131,13 @@ class DecoderModel:
                 self._resident = ResidentLayers.build(self.blocks, self.schedule, self.rt)
             if self._resident is not None and self._resident.forward(x, ctx, cache_members) is not None:
                 return self.head.forward(x, ctx.logit_rows)
-        for entry in self.schedule:
+        for i, entry in enumerate(self.schedule):
             cache = cache_members[entry.cache] if entry.cache is not None else None
             state = state_tensors[entry.state] if entry.state is not None else None
-            x = self.blocks[entry.layer].forward(x, ctx, cache, state, entry.writes_cache)
+            block, ahead = self.blocks[entry.layer], {}
+            if getattr(block, "looks_ahead", False):   # its last launch also prepares what the next block reads
+                ahead["upcoming"] = self.blocks[self.schedule[i + 1].layer] if i + 1 < len(self.schedule) else None
+            x = block.forward(x, ctx, cache, state, entry.writes_cache, **ahead)
         return self.head.forward(x, ctx.logit_rows)
 
     def weight_bytes_per_step(self) -> int:
@@ -151,8 +156,8 @@ class DecoderModel:
             for name, v in (vars(obj).items() if obj is not None else ()):
                 if isinstance(v, torch.Tensor) and name not in getattr(obj, "gathered", ()):
                     add(v)
-            for part in getattr(obj, "sides", ()):   # two mixers side by side
+            for part in getattr(obj, "sides", ()):   # two mixers side by side (their views of a joint matrix are counted with it)
                 for v in vars(part).values():
-                    if isinstance(v, torch.Tensor):
+                    if isinstance(v, torch.Tensor) and not v._is_view():
                         add(v)
         return total

@@ -18,6 +18,15 @@ from .base import MemberSpec, Runtime, register_mixer
 from .util import matrix, vector
 
 
+def _stacked_bias(parts: list, widths: list[int], rt: Runtime) -> torch.Tensor | None:
+    """The biases of projections that run as one product, zeros for those without; None where no projection has one."""
+    if all(b is None for b in parts):
+        return None
+    if any(b is not None and tuple(b.shape) != (n,) for b, n in zip(parts, widths)):
+        raise ValueError(f"attention: biases {[None if b is None else tuple(b.shape) for b in parts]} do not fit projections of {widths} rows")
+    return vector(torch.cat([torch.zeros(n) if b is None else b.to(torch.float32) for b, n in zip(parts, widths)]), rt)
+
+
 @register_mixer("attention")
 class PagedAttention:
     """params: n_heads, n_kv_heads, head_dim, scale, window (0 = none).
@@ -208,15 +217,18 @@ class RotaryWindowAttention:
         head's output * sigmoid(w_gate h)[head], then w_out
 
     With `qk_norm_eps` every query and key head is RMS-normed before its rotation (weights q_norm, k_norm [head_dim], plain
-    gains shared by the heads of a kind), in the rotation's launch. The rotation's frequencies are rot_base^(-2 i / rot_dims), or
+    gains shared by the heads of a kind; without these weights gains of one, and then it makes no difference which of norm and rotation
+    comes first, a rotation keeps a head's length), in the rotation's launch. `rot_layout` "interleaved" pairs dimension 2i with 2i + 1
+    instead. `exact_weights`: the softmax's weights go into the second product with 16 bits of mantissa also where none of cap, sink
+    and gate is there. The rotation's frequencies are rot_base^(-2 i / rot_dims), or
     the list `rot_freqs` (stretched ones, made by the caller), with cos and sin times `rot_magnitude`. A layer without w_k and
     w_v has no keys and values of its own: it reads a cache member that another layer writes (keys as that layer cached
     them, after norm and rotation) and must be scheduled with `writes_cache=False`.
 
-    params: n_heads, n_kv_heads, head_dim, v_head_dim, scale, softcap, window, rot_dims, rot_base | rot_freqs, rot_magnitude,
-    qk_norm_eps.
-    weights (matrices stored [out, in], no biases): w_q [H * head_dim, D], w_k [G * head_dim, D], w_v [G * v_head_dim, D],
-    w_out [D, H * v_head_dim], and optionally sink [H], w_gate [H, D], q_norm [head_dim], k_norm [head_dim].
+    params: n_heads, n_kv_heads, head_dim, v_head_dim, scale, softcap, window, rot_dims, rot_base | rot_freqs, rot_magnitude, rot_layout
+    ("half" | "interleaved"), qk_norm_eps, exact_weights (default false).
+    weights (matrices stored [out, in]): w_q [H * head_dim, D], w_k [G * head_dim, D], w_v [G * v_head_dim, D],
+    w_out [D, H * v_head_dim], and optionally sink [H], w_gate [H, D], q_norm [head_dim], k_norm [head_dim], b_q, b_k, b_v, b_out.
     Keys are cached after their rotation. Norms, angles, scores, softmax, sink and gate are computed in float32."""
 
     def __init__(self, params: dict, weights: dict, rt: Runtime):
@@ -241,19 +253,26 @@ class RotaryWindowAttention:
                              f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads, {self.n_kv_heads} kv heads "
                              f"of {self.head_dim} (values {self.v_head_dim})")
         self.w_in = matrix(torch.cat(stacked, dim=0), rt)
+        self.b_in = _stacked_bias([weights.get(n) for n in ("b_q", "b_k", "b_v")[: len(stacked)]], want, rt)
         self.w_out = matrix(weights["w_out"], rt)
+        self.b_out = vector(weights["b_out"], rt) if weights.get("b_out") is not None else None
+        self.exact = bool(params.get("exact_weights", False))
         self.sinks = vector(weights["sink"], rt) if weights.get("sink") is not None else None
         self.w_gate = vector(weights["w_gate"], rt) if weights.get("w_gate") is not None else None   # float32: one gate per head
         self.norm_eps = float(params["qk_norm_eps"]) if params.get("qk_norm_eps") is not None else None
         self.q_norm = self.k_norm = None
         if self.norm_eps is not None:
-            self.q_norm = vector(weights["q_norm"], rt)
-            self.k_norm = vector(weights["k_norm"], rt) if self.own_kv else None
+            one = torch.ones(self.head_dim)
+            self.q_norm = vector(weights.get("q_norm", one), rt)
+            self.k_norm = vector(weights.get("k_norm", one), rt) if self.own_kv else None
             if any(w is not None and tuple(w.shape) != (self.head_dim,) for w in (self.q_norm, self.k_norm)):
                 raise ValueError(f"attention: the query and key norms' weights must be [{self.head_dim}]")
         # the rotation's frequencies: exact in float64, then rounded once to float32
         half = self.rot_dims // 2
         self.rot_magnitude = float(params.get("rot_magnitude", 1.0))
+        if params.get("rot_layout", "half") not in ("half", "interleaved"):
+            raise ValueError(f"attention: unknown rotation layout {params['rot_layout']!r}")
+        self.interleaved = params.get("rot_layout", "half") == "interleaved"
         if params.get("rot_freqs") is not None:
             freqs = [float(f) for f in params["rot_freqs"]]
             if len(freqs) != half:
@@ -275,14 +294,14 @@ class RotaryWindowAttention:
     def _inner(self, h, ctx, cache, writes_cache):
         if writes_cache and not self.own_kv:
             raise ValueError("attention: a layer without keys and values of its own reads a cache member that another layer writes")
-        proj = ops.linear(h, self.w_in, None, w_is_nk=True)
+        proj = ops.linear(h, self.w_in, self.b_in, w_is_nk=True)
         gate = ops.small_linear(h, self.w_gate, None) if self.w_gate is not None else None
         at = self.q_width + self.k_width
         q, k, v = proj[:, : self.q_width], proj[:, self.q_width: at], proj[:, at:]
         fused_decode = ctx.decode_only and self.v_head_dim == self.head_dim
         turned = self.n_heads + (self.n_kv_heads if self.own_kv else 0)    # the heads that are normed and rotated
         norms = dict(q_norm=self.q_norm, k_norm=self.k_norm, n_q_heads=self.n_heads, norm_eps=self.norm_eps or 0.0,
-                     magnitude=self.rot_magnitude)
+                     magnitude=self.rot_magnitude, interleaved=self.interleaved)
         if writes_cache and not fused_decode:
             # the rotation's launch also puts the rotated keys and the values into the rows' cache slots
             scatter = ops.kv_scatter(ctx.slot_mapping[cache.group], cache.k, cache.v, cache.page_stride, cache.page_size,
@@ -308,14 +327,14 @@ class RotaryWindowAttention:
             q, cache.k, cache.v, cache.page_stride, cache.page_size, cache.n_pages, ctx.block_tables[cache.group],
             ctx.row_entry, ctx.positions, ctx.seq_lens, self.n_heads, self.n_kv_heads, self.head_dim, self.scale,
             self.window, decode_only=ctx.decode_only, max_context=ctx.max_context, q_start=ctx.q_start,
-            n_tiles=ctx.n_attention_tiles, v_head_dim=self.v_head_dim, softcap=self.softcap, sinks=self.sinks, head_gate=gate)
+            n_tiles=ctx.n_attention_tiles, v_head_dim=self.v_head_dim, softcap=self.softcap, sinks=self.sinks, head_gate=gate, exact=self.exact)
 
     def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
         """The mixer's output [T, D] in float32, without the residual stream."""
-        return ops.linear(self._inner(h, ctx, cache, writes_cache), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
+        return ops.linear(self._inner(h, ctx, cache, writes_cache), self.w_out, self.b_out, w_is_nk=True, out_dtype=torch.float32)
 
     def forward(self, h, residual, ctx, cache, state=None, writes_cache: bool = True):
-        return ops.linear(self._inner(h, ctx, cache, writes_cache), self.w_out, None, w_is_nk=True, residual=residual)
+        return ops.linear(self._inner(h, ctx, cache, writes_cache), self.w_out, self.b_out, w_is_nk=True, residual=residual)
 
 
 @register_mixer("latent_attention")
@@ -454,11 +473,13 @@ def distance_buckets(n_distances: int, n_buckets: int, bias_max: int) -> list[in
 
 @register_mixer("distance_bias_attention")
 class DistanceBiasAttention:
-    """Grouped causal attention over the paged cache whose scores get a learned bias by distance, with one RMS norm over the whole
-    query row and one over the whole key row. Positions enter only through the bias and the mask. Each chosen by a parameter or by
-    what the weights hold: chunks, a learned sink per head, biases on the projections, keys that are the values too.
+    """Grouped causal attention over the paged cache whose scores get a learned bias by distance, with RMS norms of queries and
+    keys. Positions enter only through the bias, the mask and the queries' temperature. Each chosen by a parameter or by
+    what the weights hold: chunks, a learned sink per head, biases on the projections, keys that are the values too, a temperature.
 
-        q, k <- rms_norm over ALL heads at once, gains q_norm [H head_dim], k_norm [G head_dim]
+        q, k <- rms_norm over ALL heads at once, gains q_norm [H head_dim], k_norm [G head_dim] (qk_norm_over "row"), or head by head,
+                gains [head_dim] shared by the heads of a kind ("head"; then the layer has values of its own)
+        q <- q (1 + q_temp_coef ln(floor((i + 1) / q_temp_every) + 1)) at position i      ("head" norms; q_temp_coef 0: as it is)
         s = (q . k) * scale + rel[bucket(i - j), head]          (buckets: `distance_buckets`)
         position i sees the keys j <= i of its own chunk, i // chunk = j // chunk      (chunk 0: every key up to i)
         weights = exp(s) / (sum over seen keys of exp(s) + exp(sink[head]))            (the sink has no key and no value)
@@ -466,8 +487,8 @@ class DistanceBiasAttention:
     Without `w_v` the values are the keys as projected, before their norm. Keys are cached after their norm. The bias table is spread
     over distances once, when the layer is made. Norms, scores, bias, softmax and sink are computed in float32.
 
-    params: n_heads, n_kv_heads, head_dim, v_head_dim, scale, chunk, bias_max, qk_norm_eps, out_scale (default 1: a factor on the heads'
-    outputs, in float32 before they are rounded).
+    params: n_heads, n_kv_heads, head_dim, v_head_dim, scale, chunk, bias_max, qk_norm_eps, qk_norm_over (default "row"), q_temp_coef
+    (default 0), q_temp_every, out_scale (default 1: a factor on the heads' outputs, in float32 before they are rounded).
     weights (matrices stored [out, in]): w_q [H head_dim, D], w_k [G head_dim, D], q_norm, k_norm, rel [buckets, H], w_out
     [D, H v_head_dim]; optionally w_v [G v_head_dim, D], b_q, b_k, b_v, sink [H]."""
 
@@ -492,12 +513,19 @@ class DistanceBiasAttention:
                              f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads, {self.n_kv_heads} kv heads "
                              f"of {self.head_dim} (values {self.v_head_dim})")
         self.w_in = matrix(torch.cat(stacked, dim=0), rt)
-        biases = [weights.get(n) for n in ("b_q", "b_k", "b_v")[: len(stacked)]]
-        self.b_in = None
-        if any(b is not None for b in biases):
-            self.b_in = vector(torch.cat([torch.zeros(n) if b is None else b.to(torch.float32) for b, n in zip(biases, want)]), rt)
+        self.b_in = _stacked_bias([weights.get(n) for n in ("b_q", "b_k", "b_v")[: len(stacked)]], want, rt)
         self.w_out = matrix(weights["w_out"], rt)
         self.q_norm, self.k_norm = vector(weights["q_norm"], rt), vector(weights["k_norm"], rt)
+        norm_over = params.get("qk_norm_over", "row")
+        if norm_over not in ("row", "head"):
+            raise ValueError(f"attention: norms over {norm_over!r} are not known")
+        self.norm_heads = norm_over == "head"
+        self.temperature = (float(params.get("q_temp_coef", 0.0)), int(params.get("q_temp_every", 1)))
+        if not self.norm_heads and self.temperature[0] != 0.0 or self.norm_heads and not self.own_values:
+            raise ValueError("attention: a temperature needs norms head by head, and those need values of the layer's own")
+        gains = (self.head_dim, self.head_dim) if self.norm_heads else (self.q_width, self.k_width)
+        if (tuple(self.q_norm.shape), tuple(self.k_norm.shape)) != ((gains[0],), (gains[1],)):
+            raise ValueError(f"attention: the norms' gains {tuple(self.q_norm.shape)} and {tuple(self.k_norm.shape)} are not {gains}")
         self.sinks = vector(weights["sink"], rt) if weights.get("sink") is not None else None
         rel = weights["rel"]
         if rel.dim() != 2 or rel.shape[1] != self.n_heads:
@@ -517,13 +545,21 @@ class DistanceBiasAttention:
     state_spec = None
     capturable = True
 
-    def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None):
-        """The heads' outputs [T, H v_head_dim] before w_out (into `out` where given)."""
+    def input_matrix(self):
+        """The stacked projections of the input, [q; k; v] x D stored [out, in], where they may run beside another mixer's as one
+        product and come back as `proj`; else None."""
+        return self.w_in if self.own_values and self.b_in is None else None
+
+    def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None, proj=None):
+        """The heads' outputs [T, H v_head_dim] before w_out (into `out` where given). `proj`: the input's projections, where they are
+        there already (worked on in place)."""
         if not writes_cache:
             raise ValueError("attention: a layer with keys and values of its own writes them")
         at = self.q_width + self.k_width
         fused_decode = ctx.decode_only and self.v_head_dim == self.head_dim and self.head_dim <= 256
-        if self.own_values or not fused_decode:
+        if proj is not None:
+            k_col = self.q_width
+        elif self.own_values or not fused_decode:
             proj = ops.linear(h, self.w_in, self.b_in, w_is_nk=True)
             k_col = self.q_width
         else:   # room for the normed keys beside the keys as projected, which are the values
@@ -533,7 +569,10 @@ class DistanceBiasAttention:
         v_col = at if self.own_values else self.q_width
         attend = dict(chunk=self.chunk, dist_bias=self.dist_bias, sinks=self.sinks, out_scale=self.out_scale, out=out)
         if fused_decode:
-            ops.row_norm(proj, self.q_width, self.k_width, self.q_norm, self.k_norm, self.norm_eps, k_out_col=k_col)
+            if self.norm_heads:
+                self._norm(proj, ctx)
+            else:
+                ops.row_norm(proj, self.q_width, self.k_width, self.q_norm, self.k_norm, self.norm_eps, k_out_col=k_col)
             q, k, v = proj[:, : self.q_width], proj[:, k_col: k_col + self.k_width], proj[:, v_col: v_col + self.v_width]
             mixed = ops.decode_attention_fused(
                 q, k, v, ctx.slot_mapping[cache.group], cache.k, cache.v, cache.page_stride, cache.page_size, cache.n_pages,
@@ -547,13 +586,20 @@ class DistanceBiasAttention:
             # the norms' launch also puts the normed keys and the values into the rows' cache slots
             scatter = ops.kv_scatter(ctx.slot_mapping[cache.group], cache.k, cache.v, cache.page_stride, cache.page_size,
                                      cache.n_pages, v_col, self.v_width, self.v_head_dim)
-            ops.row_norm(proj, self.q_width, self.k_width, self.q_norm, self.k_norm, self.norm_eps, kv=scatter, head_dim=self.head_dim)
+            if self.norm_heads:
+                self._norm(proj, ctx, scatter)
+            else:
+                ops.row_norm(proj, self.q_width, self.k_width, self.q_norm, self.k_norm, self.norm_eps, kv=scatter, head_dim=self.head_dim)
             q = proj[:, : self.q_width]
         return ops.paged_attention(
             q, cache.k, cache.v, cache.page_stride, cache.page_size, cache.n_pages, ctx.block_tables[cache.group],
             ctx.row_entry, ctx.positions, ctx.seq_lens, self.n_heads, self.n_kv_heads, self.head_dim, self.scale,
             0, decode_only=ctx.decode_only, max_context=ctx.max_context, q_start=ctx.q_start,
             n_tiles=ctx.n_attention_tiles, v_head_dim=self.v_head_dim, **attend)
+
+    def _norm(self, proj, ctx, scatter=None):
+        ops.head_norm(proj, self.n_heads, self.n_kv_heads, self.head_dim, self.q_norm, self.k_norm, self.norm_eps, kv=scatter,
+                      temperature=(ctx.positions, *self.temperature) if self.temperature[0] != 0.0 else None)
 
     def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
         """The mixer's output [T, D] in float32, without the residual stream."""

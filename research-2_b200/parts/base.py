@@ -23,7 +23,8 @@ are the GPT-2 ones):
   Positions.additive_table() -> Tensor | None      rows added to the token embedding
   Positions.rotate(q, k, ctx)                      in-place change of queries and keys (or no-op)
   TokenSide.join(x, h, ctx, rounded_dtype)         -> (new x, its rows in rounded_dtype)
-  Block.forward(x, ctx, cache, state, writes_cache) -> x
+  Block.forward(x, ctx, cache, state, writes_cache) -> x    (a block that says `looks_ahead` is also told `upcoming`, the block
+                                                   that runs after it, None for the last)
 
 The residual stream `x` is float32 in every mode; `h` has the compute dtype. Each kind has a
 registry from a name to a constructor `cls(params: dict, weights: dict, rt: Runtime)`; a
@@ -77,6 +78,7 @@ class LayerSpec:
     post_norm_2: PartSpec | None = None
     token_side: PartSpec | None = None  # what joins the stream at the layer's end (arrangements that allow it)
     block_params: dict = field(default_factory=dict)  # constants of the arrangement itself (a factor on the stream, ...)
+    block_weights: dict = field(default_factory=dict)  # the arrangement's own weights: its name -> checkpoint tensor name
 
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Any]]] = {

@@ -164,3 +164,74 @@ class PostNormBlock:
             x, h = self.token_side.join(x, h, ctx, self.compute_dtype if self.rounds else None)
         ctx.stream_rounded = (x, h)
         return x
+
+
+@register_block("streams")
+class StreamsBlock:
+    """Hyper-connections: the residual stream runs in S copies side by side. A sublayer q (1: mixer, 2: feed-forward) reads
+    u = sum_s in_q[s] x_s through its norm, and its output y joins all streams at once from the old ones,
+
+        x_t <- sum_s mix_q[s, t] x_s + factor out_q[t] y                    (mix: [from, to])
+
+    All streams start as the embedding's output; at the end the stream is their sum. A block without weights of its own is the plain
+    residual sum x + factor y(norm x). A layer may have no feed-forward (None; then no norm_2).
+
+    The sublayers hand over y in float32 without the stream (`mix`); one launch between two sublayers renews the streams and gives the
+    next one's normed input, the next block's too: the block is told which one follows (`upcoming`) and hands its input on in
+    `ctx.stream_input` as the pair (streams, input). The last block returns the streams' sum [T, D] instead of the streams [T, S, D]; a
+    block that is handed [T, D] takes it as what all its streams hold.
+
+    weights: in_1, out_1 [S], mix_1 [S, S], with a feed-forward in_2, out_2, mix_2, float32; or none. params: factor (default 1)."""
+
+    looks_ahead = True
+
+    def __init__(self, norm_1, mixer, norm_2, feed_forward, compute_dtype, factor: float = 1.0, weights: dict | None = None):
+        if feed_forward is not None and norm_2 is None:
+            raise ValueError("a block of streams needs a norm before every sublayer that it has")
+        for part, what in ((mixer, "mixer"), (feed_forward, "feed-forward")):
+            if part is not None and not hasattr(part, "mix"):
+                raise ValueError(f"a streams block's {what} must offer `mix` (its output without the stream)")
+        for norm in (norm_1, norm_2):
+            if norm is not None and not hasattr(norm, "gain"):
+                raise ValueError("a streams block's norms must be RMS norms")
+        self.norm_1, self.mixer, self.norm_2, self.feed_forward = norm_1, mixer, norm_2, feed_forward
+        self.compute_dtype = compute_dtype
+        one = torch.ones(1, device=norm_1.gain.device)
+        self.ways = []   # per sublayer: (in [S], mix [S, S], factor * out [S])
+        for q in (1, 2) if feed_forward is not None else (1,):
+            if weights:
+                read, join, mix = (weights[f"{name}_{q}"].to(torch.float32).contiguous() for name in ("in", "out", "mix"))
+            else:
+                read, join, mix = one, one, one.reshape(1, 1)
+            n = read.shape[0]
+            if read.dim() != 1 or tuple(join.shape) != (n,) or tuple(mix.shape) != (n, n) or n != (self.ways[0][0].shape[0] if self.ways else n):
+                raise ValueError(f"streams: in {tuple(read.shape)}, out {tuple(join.shape)} and mix {tuple(mix.shape)} do not fit each other")
+            self.ways.append((read, mix, join * float(factor)))
+        self.sum = torch.ones_like(self.ways[0][0])
+
+    @property
+    def n_streams(self) -> int:
+        return self.sum.shape[0]
+
+    def _join(self, x, y, way, read, norm):
+        return ops.stream_join(x, read, norm.gain if norm is not None else None, norm.eps if norm is not None else 0.0, self.compute_dtype,
+                               y=y, mix=way[1], join=way[2], keep=norm is not None)
+
+    def forward(self, x, ctx, cache=None, state=None, writes_cache: bool = True, upcoming=None):
+        carried = getattr(ctx, "stream_input", None)
+        if carried is not None and carried[0] is x:
+            h = carried[1]
+        else:
+            _, h = ops.stream_join(x, self.ways[0][0], self.norm_1.gain, self.norm_1.eps, self.compute_dtype)
+        ctx.stream_input = None
+        follows = isinstance(upcoming, StreamsBlock) and upcoming.n_streams == self.n_streams
+        after = (upcoming.ways[0][0], upcoming.norm_1) if follows else (self.sum, None)
+        y = self.mixer.mix(h, ctx, cache, state, writes_cache)
+        if self.feed_forward is not None:
+            x, h = self._join(x, y, self.ways[0], self.ways[1][0], self.norm_2)
+            y = self.feed_forward.mix(h, ctx)
+        x, h = self._join(x, y, self.ways[-1], *after)
+        if not follows:
+            return h
+        ctx.stream_input = (x, h)
+        return x

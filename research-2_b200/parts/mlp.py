@@ -148,7 +148,7 @@ class GatedMLP:
 
 @register_feed_forward("routed_experts")
 class RoutedExperts:
-    """A mixture of small gated feed-forwards, of which each row uses `top`, and optionally one more that every row uses.
+    """A mixture of small feed-forwards, gated or not, of which each row uses `top`, and optionally one more that every row uses.
 
         z = W_router h + b_router (float32); the `top` largest logits are chosen (the lower index wins a tie) and their
         weights are the softmax over the chosen logits only
@@ -161,25 +161,29 @@ class RoutedExperts:
     "silu" an expert is W_down (g sigmoid(g) u) without clamps. With `shared.w_sg` [1, D] the expert that every row uses is
     multiplied by sigmoid(w_sg h), one number per row. With `scoring` "softmax" the scores s are the softmax of the logits over
     ALL experts, chosen inside the best groups as with "sigmoid". `group_mark` "best": a group counts by its largest score alone.
-    `normalise` false: the weights are the chosen experts' scores times `route_scale` and are not made to sum to one.
+    `normalise` false: the chosen experts' scores are not made to sum to one. The weights are multiplied by `route_scale`.
+    With `gated` false an expert is W_down act(W_up h), `activation` "gelu" (the erf form), without a gate. The last `n_identity` of the
+    router's outputs stand for no expert but for the row itself: chosen, they add h times their weight.
 
-    params: n_experts, top, limit, alpha, up_offset, shared_limit (None: no shared expert); scoring ("softmax_top" | "sigmoid" |
+    params: n_experts, n_identity, top, limit, alpha, up_offset, shared_limit (None: no shared expert); scoring ("softmax_top" | "sigmoid" |
     "softmax"), n_groups, keep_groups, group_mark ("two_best" | "best"), normalise, route_scale, activation ("clamped_swish" |
-    "silu"), shared (true: a shared expert, for activations without a limit).
-    weights: router [E, D], router_b [E] or correction [E], e<i>.w_gate / e<i>.w_up [F, D], e<i>.w_down [D, F] for every expert,
+    "silu", without gates "gelu"), gated (default true), shared (true: a shared expert, for activations without a limit).
+    weights: router [E + identities, D], router_b [E] or correction [E + identities], e<i>.w_gate / e<i>.w_up [F, D], e<i>.w_down [D, F] for every expert,
     and optionally shared.w_gate / shared.w_up [Fs, D], shared.w_down [D, Fs], shared.w_sg [1, D].
 
     All experts' input projections are stacked into one matrix ([gates of every expert; shared gate; ups of every expert;
     shared up]) and their down matrices side by side into another, so that a layer is two dense products: the
     activation between them multiplies an expert's columns by the row's weight for that expert (zero where it was not
-    chosen), and the second product's sum over all columns is the weighted sum over experts. Every step reads all
+    chosen), and the second product's sum over all columns is the weighted sum over experts (the identities' part, made in the router's
+    launch, is its addend). Every step reads all
     experts' weights; a form that reads only the chosen ones for a few rows is not built."""
 
     def __init__(self, params: dict, weights: dict, rt: Runtime):
         self.n_experts, self.top = int(params["n_experts"]), int(params["top"])
         self.activation = params.get("activation", "clamped_swish")
         self.scoring = params.get("scoring", "softmax_top")
-        if self.activation not in ("clamped_swish", "silu") or self.scoring not in ("softmax_top", "sigmoid", "softmax"):
+        self.n_identity, self.gated = int(params.get("n_identity", 0)), bool(params.get("gated", True))
+        if self.activation not in (("clamped_swish", "silu") if self.gated else ("gelu",)) or self.scoring not in ("softmax_top", "sigmoid", "softmax"):
             raise ValueError(f"routed experts: unknown activation {self.activation!r} or scoring {self.scoring!r}")
         self.n_groups, self.keep_groups = int(params.get("n_groups", 1)), int(params.get("keep_groups", 1))
         self.group_mark, self.normalise = params.get("group_mark", "two_best"), bool(params.get("normalise", True))
@@ -188,19 +192,21 @@ class RoutedExperts:
         self.limit, self.alpha, self.up_offset = (float(params[k]) if clamped else 0.0 for k in ("limit", "alpha", "up_offset"))
         self.shared = params.get("shared_limit") is not None or bool(params.get("shared", False))
         self.shared_limit = float(params["shared_limit"]) if params.get("shared_limit") is not None else self.limit
-        gates = [weights[f"e{i}.w_gate"] for i in range(self.n_experts)]
+        if not self.gated and self.shared or self.n_identity and self.scoring == "softmax_top":
+            raise ValueError("routed experts: a shared expert needs gates, and identity outputs need scores over all outputs")
         ups = [weights[f"e{i}.w_up"] for i in range(self.n_experts)]
         downs = [weights[f"e{i}.w_down"] for i in range(self.n_experts)]
-        self.expert_width = gates[0].shape[0]
-        if any(g.shape != gates[0].shape or u.shape != gates[0].shape or d.shape != (g.shape[1], g.shape[0]) for g, u, d in zip(gates, ups, downs)):
+        gates = [weights[f"e{i}.w_gate"] for i in range(self.n_experts)] if self.gated else []
+        self.expert_width = ups[0].shape[0]
+        if any(w.shape != ups[0].shape for w in gates + ups) or any(d.shape != (u.shape[1], u.shape[0]) for u, d in zip(ups, downs)):
             raise ValueError("routed experts: the experts' matrices differ in shape or do not fit each other")
         if self.shared:
             gates.append(weights["shared.w_gate"]); ups.append(weights["shared.w_up"]); downs.append(weights["shared.w_down"])
-        self.w_gate_up = matrix(torch.cat(gates + ups, dim=0), rt)
+        self.w_gate_up = matrix(torch.cat(gates + ups, dim=0), rt)   # (without gates the ups alone)
         self.w_down = matrix(torch.cat(downs, dim=1), rt)
         router = weights["router"]
-        if router.shape[0] != self.n_experts or not 1 <= self.top <= self.n_experts:
-            raise ValueError(f"routed experts: router {tuple(router.shape)}, top {self.top}, {self.n_experts} experts")
+        if router.shape[0] != self.n_experts + self.n_identity or not 1 <= self.top <= router.shape[0]:
+            raise ValueError(f"routed experts: router {tuple(router.shape)}, top {self.top}, {self.n_experts} experts and {self.n_identity} identity outputs")
         # a gate on the shared expert is one more row of the router's matrix: its logit comes out of the router's launch
         self.shared_gate = self.shared and weights.get("shared.w_sg") is not None
         if self.shared_gate:
@@ -214,21 +220,30 @@ class RoutedExperts:
     def matrices(self):
         return [self.w_gate_up, self.w_down]
 
-    def _inner(self, h):
-        gate = None
+    def _inner(self, h, residual=None):
+        """-> (the experts' weighted inner activations [T, columns], what the down product adds: the residual stream, the identity
+        outputs' part, or both; None: nothing)."""
+        gate, addend = None, residual
         if self.scoring != "softmax_top":
-            route, _, _, gate = ops.route_scored(h, self.router, self.correction, self.top, self.n_groups, self.keep_groups,
-                                                 n_extra=int(self.shared_gate), scoring=self.scoring, group_mark=self.group_mark,
-                                                 normalise=self.normalise, weight_scale=self.route_scale)
+            route, _, _, gate, *carried = ops.route_scored(
+                h, self.router, self.correction, self.top, self.n_groups, self.keep_groups, n_extra=int(self.shared_gate), scoring=self.scoring,
+                group_mark=self.group_mark, normalise=self.normalise, weight_scale=self.route_scale, n_identity=self.n_identity,
+                base=residual if self.n_identity else None)
+            if self.n_identity:
+                addend = carried[0]
         else:
             route, _, _ = ops.route_top_k(h, self.router, self.router_b, self.top)
+        if not self.gated:
+            return ops.expert_unit(ops.linear(h, self.w_gate_up, None, w_is_nk=True), self.activation, route, self.expert_width), addend
         return ops.expert_act(ops.linear(h, self.w_gate_up, None, w_is_nk=True), self.activation, self.limit, self.alpha,
                               self.up_offset, route=route, n_experts=self.n_experts, expert_width=self.expert_width,
-                              tail_limit=self.shared_limit, tail_gate=gate)
+                              tail_limit=self.shared_limit, tail_gate=gate), addend
 
     def mix(self, h, ctx):
         """The feed-forward's output [T, D] in float32, without the residual stream."""
-        return ops.linear(self._inner(h), self.w_down, None, w_is_nk=True, out_dtype=torch.float32)
+        inner, addend = self._inner(h)
+        return ops.linear(inner, self.w_down, None, w_is_nk=True, residual=addend, out_dtype=torch.float32)
 
     def forward(self, h, residual, ctx):
-        return ops.linear(self._inner(h), self.w_down, None, w_is_nk=True, residual=residual)
+        inner, addend = self._inner(h, residual)
+        return ops.linear(inner, self.w_down, None, w_is_nk=True, residual=addend)

@@ -1,5 +1,5 @@
 """Mixers that carry a state of fixed size per request instead of a cache that grows with the sequence:
-a matrix memory with exponential gates (mLSTM), retention (linear attention with a fixed decay per head), a
+a matrix memory with exponential gates (mLSTM), retention and decay attention (linear attention with a fixed decay per head), a
 state-space layer with a short causal convolution (the recurrence of Mamba-2), the gated delta rule behind short convolutions
 and time mixing with a decay per channel (RWKV's). Their state lives in 32-bit floats in the request's state slot, starts at
 zero with a sequence's first token and is carried from step to step; prompts, portions and single decoded
@@ -134,6 +134,67 @@ class Retention:
 
     def forward(self, h, residual, ctx, cache=None, state=None, writes_cache: bool = True):
         return ops.linear(self._inner(h, ctx, state), self.w_out, None, w_is_nk=True, residual=residual)
+
+
+@register_mixer("decay_attention")
+class DecayAttention:
+    """Linear attention with one fixed decay per head and silu on queries, keys and values, all heads normed together. Per head:
+
+        S' = decay S + k v^T   (S: [head_dim x v_head_dim], from zero),   o = S'^T q
+        q = silu(W_q h), k = silu(W_k h), v = silu(W_v h)
+
+    The concatenated heads are RMS-normed as one row, times `norm`, times sigmoid(W_g h), and projected by W_o. silu and the
+    recurrence run in one kernel in float32: what enters the recurrence is the projections' values and nothing rounded after them.
+
+    params: n_heads, head_dim, v_head_dim, decay (one number per head), norm_eps, out_scale (default 1: a factor on the gated outputs,
+    folded into the norm's gains).
+    weights (stored [out, in], no biases): w_q, w_k [H head_dim, D], w_v, w_gate [H v_head_dim, D], norm [H v_head_dim], w_out
+    [D, H v_head_dim]."""
+
+    def __init__(self, params: dict, weights: dict, rt: Runtime):
+        self.n_heads, self.head_dim, self.v_head_dim = int(params["n_heads"]), int(params["head_dim"]), int(params["v_head_dim"])
+        self.norm_eps, decay = float(params["norm_eps"]), [float(x) for x in params["decay"]]
+        self.qk_width, self.inner_width = self.n_heads * self.head_dim, self.n_heads * self.v_head_dim
+        stacked = [weights["w_q"], weights["w_k"], weights["w_v"], weights["w_gate"]]
+        if (len(decay) != self.n_heads or [w.shape[0] for w in stacked] != [self.qk_width, self.qk_width, self.inner_width, self.inner_width]
+                or weights["w_out"].shape[1] != self.inner_width or weights["norm"].shape[0] != self.inner_width):
+            raise ValueError(f"decay attention: {len(decay)} decays, projections {[tuple(w.shape) for w in stacked]} and an output of "
+                             f"{tuple(weights['w_out'].shape)} do not fit {self.n_heads} heads of {self.head_dim} x {self.v_head_dim}")
+        self.w_in = matrix(torch.cat(stacked, dim=0), rt)
+        self.w_out = matrix(weights["w_out"], rt)
+        self.norm = vector(weights["norm"], rt) * float(params.get("out_scale", 1.0))
+        # decays: exact in float64, rounded once to float32
+        self.decay = torch.tensor(decay, dtype=torch.float64).to(torch.float32).to(rt.device)
+
+    cache_spec = None
+    capturable = True
+
+    def matrices(self):
+        return [self.w_in, self.w_out]
+
+    @property
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.n_heads * self.head_dim * self.v_head_dim,), torch.float32)
+
+    def input_matrix(self):
+        """The stacked projections of the input, [q; k; v; gate] x D stored [out, in], which may run beside another mixer's as one
+        product and come back as `proj`."""
+        return self.w_in
+
+    def inner(self, h, ctx, cache=None, state=None, writes_cache: bool = True, out=None, proj=None):
+        """The gated heads' outputs [T, H v_head_dim] before w_out (into `out` where given)."""
+        if proj is None:
+            proj = ops.linear(h, self.w_in, None, w_is_nk=True)
+        a, b = self.qk_width, 2 * self.qk_width
+        o = ops.retention_scan(proj[:, :a], proj[:, a:b], proj[:, b: b + self.inner_width], self.decay, 1.0, None, 0, ctx.positions, state,
+                               ctx.q_start, ctx.state_slot, ctx.fresh, self.n_heads, self.head_dim, self.v_head_dim, silu=True)
+        return ops.group_norm_gated(o, proj[:, b + self.inner_width:], self.norm, 1, self.norm_eps, False, proj.dtype, out=out)
+
+    def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self.inner(h, ctx, cache, state), self.w_out, None, w_is_nk=True, out_dtype=torch.float32)
+
+    def forward(self, h, residual, ctx, cache=None, state=None, writes_cache: bool = True):
+        return ops.linear(self.inner(h, ctx, cache, state), self.w_out, None, w_is_nk=True, residual=residual)
 
 
 @register_mixer("ssd")
@@ -367,7 +428,8 @@ class _TwoMixers:
 class SideBySideSum(_TwoMixers):
     """left_scale left(h) + right_scale right(h): two mixers read the same input and their scaled outputs are summed. Each mixer hands over
     what it has before its last product (`inner`, with its scale inside, in float32 before it is rounded), side by side in
-    one buffer, and ONE product over both output matrices makes the sum.
+    one buffer, and ONE product over both output matrices makes the sum. Where both mixers begin with plain products of the input
+    (`input_matrix`), those run as one too.
 
     params: left, right: {"kind": mixer kind, "params": {...}} (mixers that take `out_scale` and offer `inner`); left_scale, right_scale.
     weights: each mixer's own under the prefixes "left." and "right."."""
@@ -378,16 +440,26 @@ class SideBySideSum(_TwoMixers):
         at = 0
         for p in self.sides:   # the parts keep views into the joint matrix
             p.w_out, at = self.w_out[:, at: at + p.inner_width], at + p.inner_width
+        self.w_in = None
+        asked = [getattr(p, "input_matrix", lambda: None)() for p in self.sides]
+        if all(m is not None for m in asked):
+            self.w_in, self.split = torch.cat(asked, dim=0), asked[0].shape[0]
+            self.sides[0].w_in, self.sides[1].w_in = self.w_in[: self.split], self.w_in[self.split:]
 
     def matrices(self):
-        return [self.sides[0].w_in, self.sides[1].w_in, self.w_out]
+        return ([self.sides[0].w_in, self.sides[1].w_in] if self.w_in is None else [self.w_in]) + [self.w_out]
 
     def _inner(self, h, ctx, cache, state, writes_cache):
         # (rows a multiple of eight numbers apart: the attention kernels write pairs, the product reads 16-byte pieces)
         both = torch.empty(h.shape[0], -(-self.w_out.shape[1] // 8) * 8, dtype=h.dtype, device=h.device)[:, : self.w_out.shape[1]]
+        projected = ({}, {})
+        if self.w_in is not None:   # (rows a multiple of eight numbers apart, as above)
+            proj = torch.empty(h.shape[0], -(-self.w_in.shape[0] // 8) * 8, dtype=h.dtype, device=h.device)[:, : self.w_in.shape[0]]
+            ops.linear(h, self.w_in, None, w_is_nk=True, out=proj)
+            projected = ({"proj": proj[:, : self.split]}, {"proj": proj[:, self.split:]})
         at = 0
-        for p in self.sides:
-            p.inner(h, ctx, cache, state, writes_cache, out=both[:, at: at + p.inner_width])
+        for p, more in zip(self.sides, projected):
+            p.inner(h, ctx, cache, state, writes_cache, out=both[:, at: at + p.inner_width], **more)
             at += p.inner_width
         return both
 
