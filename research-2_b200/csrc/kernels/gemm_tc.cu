@@ -80,6 +80,10 @@ struct GemmParams {
   int out_is_bf16;
   int act;
   int* error_flag;
+  // Weights by token and block of route_width neighbouring features (a mixture's experts side by side): the activated value is
+  // multiplied by route[token * route_stride + feature / route_width]. Null: none.
+  const float* route;
+  int route_stride, route_width;
   // LayerNorm of the tokens fused in front of the product (swapped form only): the token operand
   // is built in shared memory from float rows instead of being loaded by TMA.
   const float* ln_x;       // [*, k] float rows, or null: no fused norm
@@ -387,8 +391,22 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
                                                  int row0, int col0, int c_begin, int c_end, int lane, bool have_acc) {
   const int rows = min(32, p.a_total - row0);        // rows of this slab that exist
   const int sub = lane >> 3, piece = lane & 7;       // step (2): the row within four, the 16-byte piece of it
-  // 32 columns from c on, given their accumulators: + bias, activated
-  auto finish_values = [&](int c, const uint32_t (&r)[32], float (&v)[32]) {
+  // the weights of this lane's row for the 32 columns from c on, which lie in at most two blocks: the first one's, the second one's,
+  // and how many of the columns are the first one's (asked for before the accumulators are waited for)
+  struct RouteAt { float first, second; int n_first; };
+  auto route_at = [&](int c) {
+    RouteAt at = {1.f, 1.f, 32};
+    if (p.route != nullptr) {
+      const int block = (col0 + c) / p.route_width, last = p.b_total / p.route_width - 1;
+      const float* weights = p.route + size_t(min(row0 + lane, p.a_total - 1)) * p.route_stride;
+      at.n_first = (block + 1) * p.route_width - (col0 + c);
+      at.first = weights[min(block, last)];
+      at.second = weights[min(block + 1, last)];
+    }
+    return at;
+  };
+  // 32 columns from c on, given their accumulators: + bias, activated, times their weight
+  auto finish_values = [&](int c, const uint32_t (&r)[32], float (&v)[32], const RouteAt& at) {
     const float4* b4 = reinterpret_cast<const float4*>(bias_s + (c & (BIAS_SLOTS - 1)));
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -410,16 +428,21 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
 #pragma unroll
       for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
     }
+    if (p.route != nullptr) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) v[j] *= j < at.n_first ? at.first : at.second;
+    }
   };
   auto row_values = [&](int c, float (&v)[32]) {     // the same, reading the accumulators first
     uint32_t r[32];
+    const RouteAt at = route_at(c);
     if (have_acc) {
       tmem_load32(lane_addr + uint32_t(c), r);
     } else {
 #pragma unroll
       for (int j = 0; j < 32; ++j) r[j] = 0u;
     }
-    finish_values(c, r, v);
+    finish_values(c, r, v, at);
   };
   const bool inside = rows == 32 && col0 + c_end <= p.b_total;  // the whole slab lies inside the output
   if (p.out_is_bf16 && p.residual == nullptr) {
@@ -441,6 +464,7 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
       {
         // both halves' accumulators are asked for before either is waited for
         const bool two = c0 + 32 < c_end;
+        const RouteAt at0 = route_at(c0), at1 = route_at(c0 + 32);
         uint32_t r0[32], r1[32];
         if (have_acc) {
           tmem_load32_issue(lane_addr + uint32_t(c0), r0);
@@ -452,14 +476,14 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
           for (int j = 0; j < 32; ++j) r0[j] = r1[j] = 0u;
         }
         float v[32];
-        finish_values(c0, r0, v);
+        finish_values(c0, r0, v, at0);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           st_shared16(slab + uint32_t(lane * STAGING_ROW + 4 * j) * 4u, pack2(v[8 * j], v[8 * j + 1]), pack2(v[8 * j + 2], v[8 * j + 3]),
                       pack2(v[8 * j + 4], v[8 * j + 5]), pack2(v[8 * j + 6], v[8 * j + 7]));
         }
         if (two) {
-          finish_values(c0 + 32, r1, v);
+          finish_values(c0 + 32, r1, v, at1);
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             st_shared16(slab + uint32_t(lane * STAGING_ROW + 16 + 4 * j) * 4u, pack2(v[8 * j], v[8 * j + 1]), pack2(v[8 * j + 2], v[8 * j + 3]),
@@ -812,7 +836,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 
   // ---- epilogue: warps 2..5, each on the 32 accumulator lanes it may read ------------------
   bool acc_ok = true;
-  float bias_ahead = 0.f, res_ahead[32];  // feature-major epilogue: the lane's bias, and its residual for the first 32 tokens
+  float bias_ahead = 0.f, res_ahead[32];  // feature-major epilogue: the lane's bias, and its residual (or weights) for the first 32 tokens
 #pragma unroll
   for (int j = 0; j < 32; ++j) res_ahead[j] = 0.f;
   if (threadIdx.x == 64 && p.prefetch != nullptr) {
@@ -861,6 +885,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         if (p.residual != nullptr) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) res_ahead[j] = (j < p.bn && b0 + j < p.b_total) ? p.residual[size_t(b0 + j) * p.ldr + a] : 0.f;
+        } else if (p.route != nullptr) {   // (never both)
+          const float* weights = p.route + a / p.route_width;
+#pragma unroll
+          for (int j = 0; j < 32; ++j) res_ahead[j] = (j < p.bn && b0 + j < p.b_total) ? weights[size_t(b0 + j) * p.route_stride] : 0.f;
         }
       }
     }
@@ -965,6 +993,21 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           } else if (p.act == R2_ACT_GELU_ERF) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
+          }
+          if (p.route != nullptr) {
+            if (c0 == 0) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] *= res_ahead[j];
+            } else if (c0 == 16) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] *= res_ahead[16 + j];
+            } else {
+              const float* weights = p.route + a / p.route_width;
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                if (j < nb) v[j] *= weights[size_t(b0 + c0 + j) * p.route_stride];
+              }
+            }
           }
           if (p.residual != nullptr) {
             if (c0 == 0) {  // (asked for before the products ran: a chunk's residual read here costs it a round trip to L2)
@@ -1572,7 +1615,8 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
                           const float* residual, int ldr, void* out, int ldo, int m, int n, int k, int act,
                           int out_dtype, int* error_flag, const float* ln_x, int ln_ldx, const int32_t* ln_rows,
                           const float* ln_gamma, const float* ln_beta, float ln_eps, const void* prefetch,
-                          long long prefetch_bytes, const R2KvScatter* kv, int n_groups, cudaStream_t stream) {
+                          long long prefetch_bytes, const R2KvScatter* kv, int n_groups, const float* route, int route_stride, int route_width,
+                          cudaStream_t stream) {
   if (m <= 0 || n <= 0) return R2_OK;
   // (n_groups > 1: x [m, n_groups * k], the features' n / n_groups of group s on x's columns from s * k on)
   const int group_n = n_groups > 1 ? n / n_groups : 0;
@@ -1624,6 +1668,12 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
     p.kv_head_dim = kv->head_dim;
     p.kv_head_shift = (kv->head_dim & (kv->head_dim - 1)) == 0 ? page_shift_of(kv->head_dim) : -1;
   }
+  if (route != nullptr && (residual != nullptr || kv != nullptr || fused_ln || route_width < 32 || n % route_width != 0 || route_stride < n / route_width)) {
+    return R2_UNSUPPORTED;   // (32 columns lie in two blocks at most; the caller multiplies in a kernel of its own)
+  }
+  p.route = route;
+  p.route_stride = route_stride;
+  p.route_width = route_width;
   p.group_n = group_n;
   p.group_k = k;
   if (group_n > 0 && !pl.swapped && group_n % pl.bn != 0) return R2_UNSUPPORTED;
@@ -1711,7 +1761,7 @@ extern "C" int r2_gemm_tc(const void* x, int lda, const void* w, int ldw, int w_
                           const float* ln_gamma, const float* ln_beta, float ln_eps, const void* prefetch,
                           long long prefetch_bytes, const R2KvScatter* kv, cudaStream_t stream) {
   return gemm_tc_run(x, lda, w, ldw, w_is_nk, bias, residual, ldr, out, ldo, m, n, k, act, out_dtype, error_flag, ln_x, ln_ldx, ln_rows,
-                     ln_gamma, ln_beta, ln_eps, prefetch, prefetch_bytes, kv, 1, stream);
+                     ln_gamma, ln_beta, ln_eps, prefetch, prefetch_bytes, kv, 1, nullptr, 0, 1, stream);
 }
 
 // n_groups products in one launch: x [m, n_groups * k], w [n_groups * n, k] (the groups' matrices one after the other, stored
@@ -1721,5 +1771,14 @@ extern "C" int r2_gemm_tc_grouped(const void* x, int lda, const void* w, int ldw
                                   int out_dtype, int* error_flag, cudaStream_t stream) {
   if (n_groups < 1) return R2_BAD_SHAPE;
   return gemm_tc_run(x, lda, w, ldw, 1, nullptr, nullptr, 0, out, ldo, m, n * n_groups, k, R2_ACT_NONE, out_dtype, error_flag, nullptr, 0,
-                     nullptr, nullptr, nullptr, 0.f, nullptr, 0, nullptr, n_groups, stream);
+                     nullptr, nullptr, nullptr, 0.f, nullptr, 0, nullptr, n_groups, nullptr, 0, 1, stream);
+}
+
+// act(x @ w^T) with w [n, k] stored [out, in], each value times its token's weight for the block of route_width neighbouring features
+// that it lies in: route float [m, >= n / route_width], rows route_stride apart. Blocks narrower than 32: R2_UNSUPPORTED.
+extern "C" int r2_gemm_tc_routed(const void* x, int lda, const void* w, int ldw, void* out, int ldo, int m, int n, int k, int act,
+                                 const float* route, int route_stride, int route_width, int out_dtype, int* error_flag, cudaStream_t stream) {
+  if (route == nullptr) return R2_BAD_SHAPE;
+  return gemm_tc_run(x, lda, w, ldw, 1, nullptr, nullptr, 0, out, ldo, m, n, k, act, out_dtype, error_flag, nullptr, 0, nullptr, nullptr,
+                     nullptr, 0.f, nullptr, 0, nullptr, 1, route, route_stride, route_width, stream);
 }

@@ -143,7 +143,7 @@ def _lib(source: str) -> C.CDLL:
 def build_all(head_dims=()) -> None:
     """Compile every kernel library that does not depend on a model, and the attention kernels
     for the given head sizes (a model compiles its own head size at first use otherwise)."""
-    for source in ("rowwise", "recurrent", "state_scan", "streams", "routing", "gemm_simt", "gemm_tc", "attention_simt", "attention_prefill_tc", "latent_attention",
+    for source in ("rowwise", "recurrent", "state_scan", "decay_chunks", "streams", "routing", "gemm_simt", "gemm_tc", "attention_simt", "attention_prefill_tc", "latent_attention",
                    "sampling", "wait_selftest"):
         _lib(source)
     kernel_library("sfu_probe")  # (profiling/sfu_probe.py: a measurement, no part of a step)
@@ -547,6 +547,26 @@ def expert_unit(up: torch.Tensor, act: str, route: torch.Tensor, expert_width: i
     return out
 
 
+def routed_linear(a: torch.Tensor, w: torch.Tensor, act: str, route: torch.Tensor, expert_width: int) -> torch.Tensor:
+    """act(a @ w^T) times the row's weight for the column's expert: the first product of experts without gates whose matrices are
+    stacked (w [experts * expert_width, K], stored [out, in]), in a's dtype. The tensor-core kernel does it in its epilogue, from float32
+    values; else `expert_unit` does it to the product's result."""
+    _need(a, "a", dim=2)
+    _need(w, "w", a.dtype, 2)
+    _need(route, "route", torch.float32, 2)
+    m, k, n = a.shape[0], a.shape[1], w.shape[0]
+    if w.shape[1] != k or n % expert_width or route.shape[0] != m or route.shape[1] < n // expert_width or act not in ACTIVATIONS:
+        raise KernelError(f"routed_linear: a {tuple(a.shape)}, w {tuple(w.shape)}, experts of {expert_width}, route {tuple(route.shape)} do not fit")
+    if a.dtype == torch.bfloat16 and _tensor_core_gemm:
+        out = torch.empty(m, n, dtype=a.dtype, device=a.device)
+        status = _lib("gemm_tc").r2_gemm_tc_routed(_p(a), _rows(a, "a"), _p(w), _rows(w, "w"), _p(out), n, m, n, k, ACTIVATIONS[act], _p(route),
+                                                  _rows(route, "route"), expert_width, BF16, _p(_workspace(a.device).error), _stream())
+        if status != -4:
+            _check(status, "routed_linear (tensor cores)")
+            return out
+    return expert_unit(linear(a, w, None, w_is_nk=True), act, route, expert_width)
+
+
 def stream_join(x: torch.Tensor, read: torch.Tensor, gain: torch.Tensor | None = None, eps: float = 0.0, dtype: torch.dtype = torch.float32,
                 y: torch.Tensor | None = None, mix: torch.Tensor | None = None, join: torch.Tensor | None = None, keep: bool = True):
     """Several residual streams side by side: x float32 [T, S, D], or [T, D] for streams that all hold that row (S is then the length of
@@ -782,13 +802,28 @@ def route_scored(h: torch.Tensor, w: torch.Tensor, correction: torch.Tensor | No
     return (dense, chosen, weight, extra, carried) if n_identity else (dense, chosen, weight, extra)
 
 
+DECAY_CHUNK = 64
+_decay_chunks = os.environ.get("R2_DECAY_CHUNKS", "1") != "0"
+
+
+def use_decay_chunks(on: bool) -> bool:
+    """Whether linear attention with a fixed decay per head runs prompts in chunks on the tensor cores (bfloat16); off, row by row.
+    Returns the previous setting."""
+    global _decay_chunks
+    before, _decay_chunks = _decay_chunks, bool(on)
+    return before
+
+
 def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, k_scale: float,
                    inv_freq: torch.Tensor | None, rot_dims: int, positions: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor,
-                   state_slot: torch.Tensor, fresh: torch.Tensor, n_heads: int, dim: int, vdim: int, silu: bool = False) -> torch.Tensor:
+                   state_slot: torch.Tensor, fresh: torch.Tensor, n_heads: int, dim: int, vdim: int, silu: bool = False,
+                   n_tiles: int = 0) -> torch.Tensor:
     """Retention's recurrence S <- decay[h] S + k v^T, o = S^T q for every entry of a batch, from and to the entries' state
     slots. q, k [T, heads * dim], v [T, heads * vdim] (slices of a projection); the kernel rotates q and k by position on their
     way in (of each head the first rot_dims dimensions, i with i + rot_dims / 2, angle positions[t] * inv_freq[i], in float32)
-    and multiplies k by k_scale after that. `silu`: q, k and v pass silu on their way in (float32, instead of a rotation). decay float32 [heads]; state float32 [slots, heads * dim * vdim].
+    and multiplies k by k_scale after that. `silu`: q, k and v pass silu on their way in (float32, instead of a rotation).
+    With `n_tiles` (the sum over entries of ceil(rows / 64) or more) bfloat16 batches of 64 rows and more run in chunks of 64 rows on the tensor
+    cores (csrc/kernels/decay_chunks.cu; heads of up to 256 rows, no rotation) instead of row by row. decay float32 [heads]; state float32 [slots, heads * dim * vdim].
     -> float32 [T, heads * vdim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
     for name, t, width in (("q", q, n_heads * dim), ("k", k, n_heads * dim), ("v", v, n_heads * vdim)):
@@ -805,6 +840,17 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
         if rot_dims % 2 or rot_dims > dim or inv_freq.shape[0] != rot_dims // 2:
             raise KernelError(f"retention_scan: {rot_dims} rotated dimensions of {dim}, {tuple(inv_freq.shape)} frequencies")
     out = torch.empty(q.shape[0], n_heads * vdim, dtype=torch.float32, device=q.device)
+    if q.dtype == torch.bfloat16 and n_tiles > 0 and q.shape[0] >= DECAY_CHUNK and dim <= 256 and not rot_dims and _decay_chunks:
+        scratch = torch.empty(n_tiles * n_heads * dim * vdim, dtype=torch.float32, device=q.device)
+        status = _lib("decay_chunks").r2_decay_chunks(
+            _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), C.c_float(k_scale), int(bool(silu)), _p(state),
+            C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, n_tiles, _p(scratch), C.c_longlong(scratch.numel()), _p(out),
+            _rows(out, "out"), n_heads, dim, vdim, _stream())
+        if status != -4:
+            _check(status, "retention_scan (chunks)")
+            count_launches(2)  # the sums, the states, the outputs
+            _used("decay_chunks")
+            return out
     status = _lib("recurrent").r2_retention_scan(
         _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), C.c_float(k_scale), _p(inv_freq if rot_dims else None),
         rot_dims, _p(positions), _p(state), C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out),

@@ -83,10 +83,11 @@ def weight_spec(cfg: TagulixConfig) -> WeightSpec:
     return WeightSpec(tensors=tuple(tensors))
 
 
-def random_weights(cfg: TagulixConfig, seed: int, std: float = 0.05, norm_std: float = 0.1, bias_rows: int = 16) -> dict[str, torch.Tensor]:
+def random_weights(cfg: TagulixConfig, seed: int, std: float = 0.05, norm_std: float = 0.1, bias_rows: int = 16,
+                   correction_std: float | None = None) -> dict[str, torch.Tensor]:
     """Float32 draws from ONE CPU generator, in the order of `weight_spec`: matrices N(0, std), those over fewer inputs than the
     model's width by their input's size; the token table N(0, 1); gains 1 + N(0, norm_std); biases, sinks and bias tables N(0, 1) times a
-    size that lets them show; corrections a tenth of a score; streams read by weights that sum to about one, joined by weights
+    size that lets them show; corrections N(0, correction_std) (default: a tenth of a score); streams read by weights that sum to about one, joined by weights
     around one and mixed by a matrix near the identity. `bias_rows` is the size that a configuration leaves to the checkpoint."""
     gen = torch.Generator(device="cpu")
     gen.manual_seed(seed)
@@ -103,7 +104,7 @@ def random_weights(cfg: TagulixConfig, seed: int, std: float = 0.05, norm_std: f
         elif last == "router":
             out[name] = shape[1] ** -0.5 * draw
         elif last == "correction":
-            out[name] = 0.1 / shape[0] * draw
+            out[name] = (0.1 / shape[0] if correction_std is None else correction_std) * draw
         elif last == "rel" or last == "sink":
             out[name] = 0.7 * draw
         elif len(shape) == 2:

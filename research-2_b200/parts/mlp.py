@@ -234,7 +234,7 @@ class RoutedExperts:
         else:
             route, _, _ = ops.route_top_k(h, self.router, self.router_b, self.top)
         if not self.gated:
-            return ops.expert_unit(ops.linear(h, self.w_gate_up, None, w_is_nk=True), self.activation, route, self.expert_width), addend
+            return ops.routed_linear(h, self.w_gate_up, self.activation, route, self.expert_width), addend
         return ops.expert_act(ops.linear(h, self.w_gate_up, None, w_is_nk=True), self.activation, self.limit, self.alpha,
                               self.up_offset, route=route, n_experts=self.n_experts, expert_width=self.expert_width,
                               tail_limit=self.shared_limit, tail_gate=gate), addend

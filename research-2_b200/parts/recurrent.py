@@ -143,8 +143,9 @@ class DecayAttention:
         S' = decay S + k v^T   (S: [head_dim x v_head_dim], from zero),   o = S'^T q
         q = silu(W_q h), k = silu(W_k h), v = silu(W_v h)
 
-    The concatenated heads are RMS-normed as one row, times `norm`, times sigmoid(W_g h), and projected by W_o. silu and the
-    recurrence run in one kernel in float32: what enters the recurrence is the projections' values and nothing rounded after them.
+    The concatenated heads are RMS-normed as one row, times `norm`, times sigmoid(W_g h), and projected by W_o. silu is part of the
+    recurrence's kernels, in float32: what enters the recurrence is the projections' values. Decoded tokens, and everything in float32, walk
+    row by row; prompts in bfloat16 go in chunks of 64 rows on the tensor cores, operands as two bfloat16 terms, the state in float32.
 
     params: n_heads, head_dim, v_head_dim, decay (one number per head), norm_eps, out_scale (default 1: a factor on the gated outputs,
     folded into the norm's gains).
@@ -187,7 +188,8 @@ class DecayAttention:
             proj = ops.linear(h, self.w_in, None, w_is_nk=True)
         a, b = self.qk_width, 2 * self.qk_width
         o = ops.retention_scan(proj[:, :a], proj[:, a:b], proj[:, b: b + self.inner_width], self.decay, 1.0, None, 0, ctx.positions, state,
-                               ctx.q_start, ctx.state_slot, ctx.fresh, self.n_heads, self.head_dim, self.v_head_dim, silu=True)
+                               ctx.q_start, ctx.state_slot, ctx.fresh, self.n_heads, self.head_dim, self.v_head_dim, silu=True,
+                               n_tiles=ctx.n_attention_tiles)
         return ops.group_norm_gated(o, proj[:, b + self.inner_width:], self.norm, 1, self.norm_eps, False, proj.dtype, out=out)
 
     def mix(self, h, ctx, cache=None, state=None, writes_cache: bool = True):

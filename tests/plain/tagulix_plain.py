@@ -194,7 +194,10 @@ def mixture(h, w, p, cfg):
 
 # ---- several streams ---------------------------------------------------------------------------------
 def hyper(x, w, p, sublayer, m):
-    """x [T, s, D]; u = sum_a in[a] x_a is what the sublayer reads; x_b <- sum_a mix[a, b] x_a + m out[b] y."""
+    """x [T, s, D]; u = sum_a in[a] x_a is what the sublayer reads; x_b <- sum_a mix[a, b] x_a + m out[b] y. A model that says nothing of
+    streams has one, and no weights for it: x <- x + m y."""
+    if p + "in" not in w:
+        return x + m * sublayer(x[:, 0])[:, None, :]
     u = torch.einsum("a,tad->td", w[p + "in"].to(F64), x)
     y = sublayer(u)
     return torch.einsum("ab,tad->tbd", w[p + "mix"].to(F64), x) + m * w[p + "out"].to(F64)[None, :, None] * y[:, None, :]
@@ -207,7 +210,7 @@ def forward(config, w, tokens, layers_out=None):
 
     eps, m = config["norm"]["eps"], float(config.get("residual_mult", 1.0))
     x = w["embed"].to(F64)[torch.tensor(tokens)]
-    x = x[:, None, :].repeat(1, config["streams"], 1)
+    x = x[:, None, :].repeat(1, config.get("streams") or 1, 1)
     for i, layer in enumerate(config["layers"]):
         own = layer.get("weights_of")
         p, mix = f"l{i if own is None else own}.", layer["mixer"]
