@@ -22,7 +22,8 @@ A "step" is one decode step. The default run decodes a batch of 8 requests whose
 `--design bosenex` prints the same points for a Bosenex model beside a Zirunex model of equal layer sizes, and the
 design's kernels one by one; `--design zudalorn` a Zudalorn model beside a Bosenex model of equal layer sizes, likewise;
 `--design pidodra` a Pidodra model beside a Zudalorn model of equal layer sizes whose layers are all latent attention;
-`--design lagelorn` a Lagelorn model beside a Bosenex model of equal layer sizes with dense feed-forwards. `--design zirunex` prints, instead, the same decode and prefill points for Zirunex models with the layer sizes
+`--design lagelorn` a Lagelorn model beside a Bosenex model of equal layer sizes with dense feed-forwards; `--design tagulix` a
+Tagulix model beside a Zudalorn and a Bosenex model of equal layer sizes. `--design zirunex` prints, instead, the same decode and prefill points for Zirunex models with the layer sizes
 of `--model` beside GPT-2's, and the design's kernels one by one beside their likes.
 
 `--model gpt2-355M` and `--model gpt2-1.5B` run the same at those sizes (the 1.5B decode workload has
@@ -289,6 +290,8 @@ def prefill_point(model, cfg, pk: dict) -> dict:
         flops = zudalorn_flops(cfg, n_req, length)
     elif type(cfg).__name__ == "PidodraConfig":
         flops = pidodra_flops(cfg, n_req, length)
+    elif type(cfg).__name__ == "TagulixConfig":
+        flops = tagulix_flops(cfg, n_req, length)
     elif type(cfg).__name__ == "LagelornConfig":
         flops = lagelorn_flops(cfg, n_req, length)
     else:
@@ -1205,6 +1208,209 @@ def lagelorn_points(args, pk: dict) -> dict:
     return out
 
 
+def tagulix_config(size: str, n_layer: int) -> dict:
+    """A Tagulix configuration with the width, heads, head size, layers and vocabulary of a GPT-2 size, four streams: every other
+    layer is attention with a bias by distance (half the heads, about four query heads a key/value head) beside decay attention (half the
+    heads), the others attention inside a window of 256. Every layer routes each token to 3 of 8 experts and 2 identity outputs, in 2
+    groups of which 1 is kept; an expert's two matrices hold as many weights as the three of a gated expert of the other designs."""
+    g = SIZES[size]
+    d, h = g["n_embd"], g["n_head"]
+    hd, half = d // h, half_heads_for(h)
+    ff = max(128, round(2 * g["n_inner"] / 3 / 128) * 128)
+    left = {"heads": half, "kv_heads": kv_heads_for(half), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "bias_max": 128, "q_temp": {"coef": 0.1, "every": 256}}
+    right = {"heads": half, "dim": hd, "vdim": hd, "decay": [1.0 - 2.0 ** (-3.0 - 6.0 * i / max(1, half - 1)) for i in range(half)]}
+    pair = {"left": left, "left_scale": 0.7, "right": right, "right_scale": 0.7}
+    window = {"heads": h, "kv_heads": kv_heads_for(h), "dim": hd, "vdim": hd, "scale": 1.0, "mask": {"size": 256}, "rot": {"dims": hd, "base": 10000.0}}
+    moe = {"kind": "moe", "router": {"experts": 8, "identity": 2, "top": 3, "groups": {"count": 2, "keep": 1}, "scale": 1.5}, "expert": {"ff": 3 * ff // 8}}
+    layers = [{"type": "attention" if i % 2 else "parallel", "mixer": window if i % 2 else pair, "mlp": moe} for i in range(n_layer)]
+    return {"architecture": "Tagulix", "vocab": g["vocab_size"], "width": d, "norm": {"eps": 1e-5}, "streams": 4, "residual_mult": 0.7, "layers": layers}
+
+
+def tagulix_flops(cfg, n_req: int, length: int) -> float:
+    """Flops that one prefill step of n_req prompts of `length` tokens NEEDS in a Tagulix configuration: products with the weights
+    a token uses (its chosen outputs, not all), the recurrences, and the attention's seen pairs."""
+    t, d, total = n_req * length, cfg.width, 0.0
+    for layer in cfg.layers:
+        m = layer.mixer
+        a = getattr(m, "left", m)
+        q, kv, o = a.heads * a.dim, a.kv_heads * (a.dim + a.vdim), a.heads * a.vdim
+        total += 2 * t * d * (q + kv) + 2 * t * o * d
+        total += n_req * 2 * (q + o) * sum(min(i + 1, getattr(a, "window", 0) or length) for i in range(length))
+        if a is not m:
+            r = m.right
+            qk, v = r.heads * r.dim, r.heads * r.vdim
+            total += 2 * t * d * (2 * qk + 2 * v) + 2 * t * v * d + t * r.heads * 6 * r.dim * r.vdim
+        if layer.mlp is not None:
+            total += 2 * t * d * 2 * layer.mlp.top * layer.mlp.ff
+        total += 2 * t * d * 2 * cfg.streams * (cfg.streams + 2)
+    return total + 2 * n_req * d * cfg.vocab_size
+
+
+def tagulix_points(args, pk: dict) -> dict:
+    """`--design tagulix`: prefill and decode throughput of a Tagulix model with the layer sizes of `--model`, beside the closest of
+    the other models at that size (Zudalorn: linear attention with a fixed decay, experts inside the best groups; Bosenex: attention inside a
+    window beside a recurrence, pre-norm, experts) through the same loops, and the design's kernels one by one beside their likes."""
+    import torch
+    from research_2_b200.kernels import ops
+    from research_2_b200.profiling import kernel_cases
+
+    g = SIZES[args.model]
+    d, h = g["n_embd"], g["n_head"]
+    hd = d // h
+    variants = {"bosenex": bosenex_config(args.model, args.layers), "zudalorn": zudalorn_config(args.model, args.layers),
+                "tagulix": tagulix_config(args.model, args.layers)}
+    out = {"design": "tagulix", "sizes_of": args.model, "layers": args.layers, "prompt_len": PROMPT_LEN, "models": {}}
+    for name, data in variants.items():
+        model, cfg = build_gated_design(data, **({"bias_rows": 32} if name == "tagulix" else {}))
+        point = {"weights_MB": round(model.weight_bytes_per_step() / 1e6, 1)}
+        for batch in (8, 64):
+            steps = min(args.steps, 96)
+            value, ms, loop, kv_bytes = decode_point(model, batch, steps, args.warmup)
+            state_bytes = 2 * batch * sum(4 * int(torch.tensor(spec.shape).prod()) for spec in model.state_members)   # read and written
+            achieved = (model.weight_bytes_per_step() + kv_bytes + state_bytes) / (ms / 1e3) / 1e9
+            point[f"decode_b{batch}"] = {"tokens/s": round(value), "ms_per_step": round(ms, 4), "kernels_per_step": loop.graph.kernels,
+                                         "hbm_frac": round(achieved / pk["hbm_gbs"], 3)}
+            del loop
+            torch.cuda.empty_cache()
+        pre = prefill_point(model, cfg, pk)
+        point["prefill_2x1024"] = {"tokens/s": round(pre["value"]), "ms": round(pre["ms"], 3), "bf16_frac": round(pre["frac"], 3)}
+        out["models"][name] = point
+        del model
+        torch.cuda.empty_cache()
+
+    # the design's kernels one by one, at a prompt step (2 x 1,024 rows) and at decode steps (8 and 64 rows at position 1,023)
+    table = {}
+
+    def add(name, fn, n_bytes=0, flops=0):
+        us = kernel_cases.time_in_graph(fn)
+        entry = {"us": round(us, 2)}
+        if n_bytes:
+            entry.update(frac=round(n_bytes / us / 1e3 / pk["hbm_gbs"], 3), of="copy bandwidth")
+        if flops:
+            entry.update(flops_frac=round(flops / us / 1e6 / pk["bf16_tflops"], 4))
+        table[name] = entry
+
+    dev, bf = "cuda:0", torch.bfloat16
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)  # noqa: E731
+    page, length, window, streams = PAGE, 1024, 256, 4
+    sinks = torch.zeros(h, device=dev)
+    ff = max(128, round(2 * g["n_inner"] / 3 / 128) * 128)
+    for label, n_entries, rows_each in (("2 x 1,024 rows", 2, 1024), ("8 decoded rows", 8, 1), ("64 decoded rows", 64, 1)):
+        t = n_entries * rows_each
+        q_start = i32([i * rows_each for i in range(n_entries + 1)])
+        slots, fresh = i32(list(range(n_entries))), i32([0] * n_entries)
+        row_entry = i32([e for e in range(n_entries) for _ in range(rows_each)])
+        positions = i32([length - 1 if rows_each == 1 else p for _ in range(n_entries) for p in range(rows_each)])
+        seq_lens = i32([length] * n_entries)
+        slot_map = i32([e * length + p for e, p in zip(row_entry.tolist(), positions.tolist())])
+        n_tiles = n_entries * -(-rows_each // 64) if rows_each > 1 else 0
+        x32, y32, xs = torch.randn(t, d, device=dev), torch.randn(t, d, device=dev), torch.randn(t, streams, d, device=dev)
+        hrow = torch.randn(t, d, device=dev).to(bf)
+        gain = torch.ones(d, device=dev)
+        # the streams
+        read, join, mix = torch.full((streams,), 0.25, device=dev), torch.ones(streams, device=dev), torch.eye(streams, device=dev)
+        add(f"{streams} streams take a sublayer's output + the next norm, {label}", lambda: ops.stream_join(xs, read, gain, 1e-5, bf, y=y32, mix=mix, join=join),
+            n_bytes=t * d * (8 * streams + 6))
+        add(f"its like: a sublayer's output normed into one stream + the next norm (Zudalorn), {label}",
+            lambda: ops.norm_add(x32, y32, gain, 1e-5, gain, 1e-5, bf), n_bytes=t * d * 14)
+        add(f"the first sublayer's input from the embedding, {label}", lambda: ops.stream_join(x32, read, gain, 1e-5, bf), n_bytes=t * d * 6)
+        add(f"its like: the norm of a stream (any model), {label}", lambda: ops.rms_norm(x32, gain, 1e-5, bf), n_bytes=t * d * 6)
+        # the window attention's turned and normed heads
+        kvh = kv_heads_for(h)
+        qkv = torch.randn(t, (h + 2 * kvh) * hd, device=dev).to(bf)
+        pages_each = length // page
+        tables = torch.arange(n_entries * pages_each, dtype=torch.int32, device=dev).view(n_entries, pages_each).contiguous()
+        n_pages = n_entries * pages_each
+
+        def pool_of(kv):
+            return torch.randn(n_pages, 2 * kv * page * hd, device=dev).to(bf).view(-1)
+
+        pool = pool_of(kvh)
+        inv_freq = torch.tensor([10000.0 ** (-2.0 * i / hd) for i in range(hd // 2)], device=dev)
+        head_w = torch.ones(hd, device=dev)
+        scatter = ops.kv_scatter(slot_map, pool, pool[kvh * page * hd:], 2 * kvh * page * hd, page, n_pages, (h + kvh) * hd, kvh * hd, hd) if rows_each > 1 else None
+        turn = lambda inter: ops.rotate_half(qkv, h + kvh, hd, hd, inv_freq, positions, kv=scatter, n_kv_heads=kvh, k_col=h * hd, q_norm=head_w,  # noqa: E731
+                                             k_norm=head_w, n_q_heads=h, norm_eps=1e-5, interleaved=inter)
+        turn_bytes = t * (h + kvh) * hd * 4 + (t * kvh * hd * 6 if rows_each > 1 else 0)
+        add(f"window attention: {h + kvh} heads turned (neighbouring pairs) and normed, cache write in prompts, {label}", lambda: turn(True), n_bytes=turn_bytes)
+        add(f"its like: heads normed and turned by halves (Pidodra), {label}", lambda: turn(False), n_bytes=turn_bytes)
+
+        def attend(rows, kv_pool, heads, kv, win, **kw):
+            """Attention of `heads` query heads over `kv` in a stacked projection's rows."""
+            if rows_each > 1:
+                att_out = torch.empty(t, heads * hd, device=dev, dtype=bf)
+                return ops.paged_attention(rows[:, : heads * hd], kv_pool, kv_pool[kv * page * hd:], 2 * kv * page * hd, page, n_pages, tables, row_entry, positions,
+                                           seq_lens, heads, kv, hd, hd ** -0.5, win, out=att_out, max_context=length, q_start=q_start, n_tiles=n_tiles, **kw)
+            kw.pop("exact", None)
+            return ops.decode_attention_fused(rows[:, : heads * hd], rows[:, heads * hd: (heads + kv) * hd], rows[:, (heads + kv) * hd: (heads + 2 * kv) * hd], slot_map,
+                                              kv_pool, kv_pool[kv * page * hd:], 2 * kv * page * hd, page, n_pages, tables, row_entry, positions, seq_lens, heads, kv, hd,
+                                              hd ** -0.5, win, length, exact_weights=ops.exact_weights(), **kw)
+
+        windowed, all_seen = sum(min(p + 1, window) for p in positions.tolist()), sum(p + 1 for p in positions.tolist())
+        size = dict(n_bytes=t * h * hd * 4 + n_entries * (length if rows_each > 1 else window) * 2 * kvh * hd * 2, flops=4 * windowed * h * hd)
+        add(f"window attention of {window}, {h} heads of {hd} over {kvh}, {label}", lambda: attend(qkv, pool, h, kvh, window, exact=True), **size)
+        add(f"its like: window of {window}, capped scores, sinks (Bosenex), {label}",
+            lambda: attend(qkv, pool, h, kvh, window, softcap=30.0, sinks=sinks[:h]), **size)
+        # the two mixers side by side
+        half = half_heads_for(h)
+        kvl, inner = kv_heads_for(half), half * hd
+        left_w, right_w = (half + 2 * kvl) * hd, 4 * inner
+        proj = torch.randn(t, left_w + right_w, device=dev).to(bf)
+        w_in = (torch.randn(left_w + right_w, d, device=dev) * 0.02).to(bf)
+        add(f"side by side: one product for both inputs, {d} x {left_w + right_w:,}, {label}", lambda: ops.linear(hrow, w_in, None, w_is_nk=True),
+            n_bytes=t * (d + left_w + right_w) * 2 + w_in.numel() * 2, flops=2 * t * w_in.numel())
+        pool_l = pool_of(kvl)
+        scatter = ops.kv_scatter(slot_map, pool_l, pool_l[kvl * page * hd:], 2 * kvl * page * hd, page, n_pages, (half + kvl) * hd, kvl * hd, hd) if rows_each > 1 else None
+        norm_bytes = t * (half + kvl) * hd * 4 + (t * kvl * hd * 6 if rows_each > 1 else 0)
+        add(f"biased attention: {half + kvl} heads' norms, query temperature, cache write in prompts, {label}",
+            lambda: ops.head_norm(proj, half, kvl, hd, head_w, head_w, 1e-5, kv=scatter, temperature=(positions, 0.1, 256)), n_bytes=norm_bytes)
+        add(f"its like: heads' norms (Zirunex), {label}", lambda: ops.head_norm(proj, half, kvl, hd, head_w, head_w, 1e-5, kv=scatter), n_bytes=norm_bytes)
+        bias = torch.randn(half, 129, device=dev)
+        size = dict(n_bytes=t * inner * 4 + n_entries * length * 2 * kvl * hd * 2, flops=4 * all_seen * inner)
+        add(f"attention with a bias by distance and sinks over every earlier key, {half} heads of {hd} over {kvl}, {label}",
+            lambda: attend(proj, pool_l, half, kvl, 0, dist_bias=bias, sinks=sinks[:half], out_scale=0.7), **size)
+        add(f"its like: capped scores and sinks over every earlier key (Bosenex), {label}", lambda: attend(proj, pool_l, half, kvl, 0, softcap=30.0, sinks=sinks[:half]), **size)
+        rproj = proj[:, left_w:]
+        decay, state = torch.full((half,), 0.97, device=dev), torch.zeros(n_entries, half * hd * hd, device=dev)
+        scan_bytes = t * inner * (6 + 4) + 2 * state.numel() * 4
+        scan = lambda **kw: ops.retention_scan(rproj[:, :inner], rproj[:, inner: 2 * inner], rproj[:, 2 * inner: 3 * inner], decay, 1.0, None, 0,  # noqa: E731
+                                               positions, state, q_start, slots, fresh, half, hd, hd, **kw)
+        add(f"decay attention: silu and the recurrence, {half} heads of {hd} x {hd} (all launches), {label}", lambda: scan(silu=True, n_tiles=n_tiles), n_bytes=scan_bytes)
+        add(f"its like: retention's recurrence row by row with rotation (Zudalorn), {label}",
+            lambda: ops.retention_scan(rproj[:, :inner], rproj[:, inner: 2 * inner], rproj[:, 2 * inner: 3 * inner], decay, 1.0, inv_freq, hd, positions, state, q_start,
+                                       slots, fresh, half, hd, hd), n_bytes=scan_bytes)
+        o32 = torch.randn(t, inner, device=dev)
+        both = torch.empty(t, 2 * inner, device=dev, dtype=bf)
+        gate, gain_i = rproj[:, 3 * inner:], torch.ones(inner, device=dev)
+        add(f"decay attention: one norm over all heads and sigmoid gate, {label}",
+            lambda: ops.group_norm_gated(o32, gate, gain_i, 1, 1e-5, False, bf, out=both[:, inner:]), n_bytes=t * inner * 8)
+        add(f"its like: heads' norms and sigmoid gate (Bosenex), {label}", lambda: ops.group_norm_gated(o32, gate, gain_i, half, 1e-5, False, bf), n_bytes=t * inner * 8)
+        # the mixture
+        width = 3 * ff // 8
+        router, correction = torch.randn(10, d, device=dev) * 0.02, torch.randn(10, device=dev) * 0.1
+        pick = lambda: ops.route_scored(hrow, router, correction, 3, 2, 1, scoring="softmax", group_mark="best", weight_scale=1.5, n_identity=2)  # noqa: E731
+        route = pick()[0]
+        add(f"router: 8 + 2 corrected softmax scores in 32-bit, 1 of 2 groups, top 3, the identity outputs' share of the row, {label}", pick, n_bytes=t * d * 6)
+        add(f"its like: 8 sigmoid scores + a gate, 2 of 4 groups, top 2 (Zudalorn), {label}",
+            lambda: ops.route_scored(hrow, router[:9], correction[:8].contiguous(), 2, 4, 2, n_extra=1), n_bytes=t * d * 2)
+        w_up = (torch.randn(8 * width, d, device=dev) * 0.02).to(bf)
+        add(f"experts: first product with gelu and the routing weights inside, {d} x {8 * width:,}, {label}",
+            lambda: ops.routed_linear(hrow, w_up, "gelu", route, width), n_bytes=t * (d + 8 * width) * 2 + w_up.numel() * 2, flops=2 * t * w_up.numel())
+        gu = torch.randn(t, 8 * width, device=dev).to(bf)
+        add(f"its like: the same product alone (any model), {label}", lambda: ops.linear(hrow, w_up, None, w_is_nk=True),
+            n_bytes=t * (d + 8 * width) * 2 + w_up.numel() * 2, flops=2 * t * w_up.numel())
+        add(f"(gelu and routing weights as a kernel of their own, {8 * width:,} columns, {label})", lambda: ops.expert_unit(gu, "gelu", route, width), n_bytes=t * gu.shape[1] * 4)
+        zu = torch.randn(t, 2 * 9 * (ff // 4), device=dev).to(bf)
+        zroute, _, _, zg = ops.route_scored(hrow, router[:9], correction[:8].contiguous(), 2, 4, 2, n_extra=1)
+        add(f"(its like there: experts' gated silu unit, {zu.shape[1] // 2:,} columns (Zudalorn), {label})",
+            lambda: ops.expert_act(zu, "silu", route=zroute, n_experts=8, expert_width=ff // 4, tail_gate=zg), n_bytes=t * zu.shape[1] * 3)
+        w_down = (torch.randn(d, 8 * width, device=dev) * 0.02).to(bf)
+        add(f"experts: last product onto the identity outputs' share, {label}", lambda: ops.linear(gu, w_down, None, w_is_nk=True, residual=x32),
+            n_bytes=t * (8 * width * 2 + d * 8) + w_down.numel() * 2, flops=2 * t * w_down.numel())
+    out["kernels"] = table
+    return out
+
+
 def e2e_point(model, batch: int, steps: int, warmup: int) -> dict:
     """Through the Python entry point: submit prompts (host token lists), step, poll tokens."""
     import torch
@@ -1378,7 +1584,7 @@ def main() -> int:
     ap.add_argument("--phases", action="store_true", help="print where a layer's time goes inside the resident decode kernel at --batch rows, and stop")
     ap.add_argument("--logits-ctas", action="store_true", help="print when each CTA of a decode step's logits product starts and ends (its waves), and stop")
     ap.add_argument("--prefill", action="store_true", help="print the prefill point (2 x 1,024 tokens in one step) alone, and stop")
-    ap.add_argument("--design", default=None, choices=("zirunex", "bosenex", "zudalorn", "pidodra", "lagelorn"),
+    ap.add_argument("--design", default=None, choices=("zirunex", "bosenex", "zudalorn", "pidodra", "lagelorn", "tagulix"),
                     help="print prefill and decode throughput of that design at the layer sizes of --model beside GPT-2's, "
                          "and its kernels beside their likes, and stop (the default workload is GPT-2's)")
     args = ap.parse_args()
@@ -1413,7 +1619,8 @@ def main() -> int:
 
     pk, pk_source = peaks()
     if args.design:
-        points = {"bosenex": bosenex_points, "zudalorn": zudalorn_points, "pidodra": pidodra_points, "lagelorn": lagelorn_points}.get(args.design, design_points)
+        points = {"bosenex": bosenex_points, "zudalorn": zudalorn_points, "pidodra": pidodra_points, "lagelorn": lagelorn_points,
+                  "tagulix": tagulix_points}.get(args.design, design_points)
         print(json.dumps(points(args, pk)))
         return 0
     model, cfg = build_model(args.layers, size=args.model)

@@ -407,6 +407,35 @@ def test_decay_attention_alone(shape, dtype):
             assert torch.equal(portions[s], whole[s]) and torch.equal(single[s], whole[s]), f"{shape}: sequence {s} depends on its cutting"
 
 
+def test_decay_chunks_of_many_entries_beside_the_walk():
+    """Eighty entries, some without rows, some of one row: the two ways give the same outputs and states, and touch no slot of an
+    entry without rows."""
+    from research_2_b200.kernels import ops
+
+    gen = torch.Generator().manual_seed(6)
+    heads, dim, vdim = 3, 48, 40
+    lengths = [(0, 1, 63, 64, 65, 7, 130, 1)[i % 8] for i in range(80)]
+    starts = [sum(lengths[:i]) for i in range(81)]
+    x = torch.randn(starts[-1], heads * (2 * dim + vdim), generator=gen).to(torch.bfloat16).to(DEV)
+    q, k, v = x.split([heads * dim, heads * dim, heads * vdim], dim=1)
+    slots, fresh = torch.randperm(90, generator=gen)[:80].to(torch.int32), torch.randint(0, 2, (80,), generator=gen).to(torch.int32)
+    first = torch.randn(90, heads * dim * vdim, generator=gen)
+    decay = torch.tensor([0.9, 0.999, 0.2], device=DEV)
+    results = []
+    for chunks in (True, False):
+        state = first.to(DEV).clone()
+        old = ops.use_decay_chunks(chunks)
+        try:
+            out = ops.retention_scan(q, k, v, decay, 0.5, None, 0, i32([0] * starts[-1]), state, i32(starts), slots.to(DEV), fresh.to(DEV), heads, dim, vdim,
+                                     silu=True, n_tiles=sum(-(-n // 64) for n in lengths))
+        finally:
+            ops.use_decay_chunks(old)
+        results.append((out, state))
+    for a, b in zip(*results):
+        close(a, b.double().cpu(), 5e-5)
+    idle = [i for i in range(90) if i not in set(slots.tolist()) or lengths[slots.tolist().index(i)] == 0]
+    assert len(idle) == 20 and torch.equal(results[0][1][idle].cpu(), first[idle])
+
 # ---------------------------------------------------------------------------------------------
 # one key that stands out: in the window and out of it, at pages' borders, at the first token, far back in a cache and in a carried state
 
