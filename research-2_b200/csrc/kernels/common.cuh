@@ -78,6 +78,22 @@ __device__ __forceinline__ float gelu_erf(float x) {
   return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
 }
 
+// The same for results that are rounded to bfloat16. With Phi the normal distribution, gelu(x) = x Phi(x) = max(x, 0) - |x| (1 - Phi(|x|)),
+// and 1 - Phi(z) = erfc(z / sqrt 2) / 2 by formula 7.1.26 of Abramowitz and Stegun's Handbook of Mathematical Functions (Hastings'
+// rational approximation of the error function, within 1.5e-7): a polynomial of degree five in 1 / (1 + 0.3275911 z / sqrt 2), times
+// exp(-z^2 / 2).
+__device__ __forceinline__ float gelu_erf_rounded(float x) {
+  const float z = fabsf(x);
+  float t, e;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(fmaf(z, 0.3275911f * 0.7071067811865476f, 1.f)));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * x * (-0.5f * 1.4426950408889634f)));
+  float tail = fmaf(t, 0.5f * 1.061405429f, 0.5f * -1.453152027f);
+  tail = fmaf(t, tail, 0.5f * 1.421413741f);
+  tail = fmaf(t, tail, 0.5f * -0.284496736f);
+  tail = fmaf(t, tail, 0.5f * 0.254829592f);
+  return fmaf(-z, tail * t * e, fmaxf(x, 0.f));
+}
+
 __device__ __forceinline__ float activate(float x, int act) {
   if (act == R2_ACT_GELU_TANH) return gelu_tanh(x);
   if (act == R2_ACT_GELU_ERF) return gelu_erf(x);

@@ -12,6 +12,9 @@
 //   decay_chunk_states   entry by entry: every chunk's state at its start (written over U) and the request's new state; elementwise
 //   decay_chunk_outputs  o of every chunk: two products with a triangle of decays between them, and one with the chunk's first state
 //
+// and one for decode steps, in which (nearly) every entry is one row:
+//   decay_step           S and o of a row as they are written above, every load of the state in flight at once
+//
 // The products run on the warp-level tensor cores (mma.sync, bfloat16 with float sums). Everything that enters them is float: silu of
 // queries, keys and values (where asked for), powers of the decay, states, weighted scores; each operand is the sum of two bfloat16
 // terms (16 bits of mantissa), of whose four products three are taken. States and sums stay float.
@@ -69,7 +72,7 @@ __device__ __forceinline__ Tile find_tile(const int32_t* q_start, int n_entries,
 }
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return uint32_t(__cvta_generic_to_shared(p)); }
-__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }   // (a few units of the last place)
 __device__ __forceinline__ uint32_t pack_pair(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
@@ -356,6 +359,94 @@ decay_chunk_outputs_kernel(const ChunkArgs a) {
   }
 }
 
+// Decode steps. A CTA has one (entry, head, slice of the columns); a thread has V neighbouring columns of every row_groups-th row, and
+// the row groups' sums meet in shared memory, in order.
+constexpr int STEP_THREADS = 128, STEP_ROWS = 8;
+template <int V>
+__global__ void __launch_bounds__(STEP_THREADS)
+decay_step_kernel(const ChunkArgs a, int slice) {
+  pdl_launch_dependents();
+  __shared__ float qs[MAX_DIM], ks[MAX_DIM], sums[STEP_THREADS][V];
+  const int e = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * slice;
+  const int row0 = a.q_start[e], row1 = a.q_start[e + 1];
+  const bool is_fresh = a.fresh[e] != 0;
+  const float decay = a.decay[h];
+  const int groups = slice / V, row_groups = STEP_THREADS / groups;   // (groups divides the threads)
+  const int g = threadIdx.x % groups, rg = threadIdx.x / groups, j = col0 + g * V;
+  const bool mine = j < a.vdim;
+  float* head_state = a.state + size_t(a.state_slot[e]) * a.slot_stride + size_t(h) * a.dim * a.vdim;
+  pdl_wait();
+  for (int t = row0; t < row1; ++t) {
+    const bool zero = is_fresh && t == row0;
+    float s[STEP_ROWS][V], v[V], acc[V] = {};
+#pragma unroll
+    for (int i = 0; i < STEP_ROWS; ++i) {   // the first rows' states, asked for before anything is waited for
+      const int r = rg + i * row_groups;
+#pragma unroll
+      for (int u = 0; u < V; ++u) s[i][u] = 0.f;
+      if (mine && r < a.dim && !zero) {
+        const float* p = head_state + size_t(r) * a.vdim + j;
+        if (V == 4) {
+          const float4 f = *reinterpret_cast<const float4*>(p);
+          s[i][0] = f.x;
+          s[i][V > 1 ? 1 : 0] = f.y;
+          s[i][V > 2 ? 2 : 0] = f.z;
+          s[i][V > 3 ? 3 : 0] = f.w;
+        } else {
+          s[i][0] = *p;
+        }
+      }
+    }
+    const bf16* q = a.q + size_t(t) * a.q_stride + size_t(h) * a.dim;
+    const bf16* k = a.k + size_t(t) * a.k_stride + size_t(h) * a.dim;
+    for (int i = threadIdx.x; i < a.dim; i += STEP_THREADS) {
+      const float x = to_float(q[i]), y = to_float(k[i]);
+      qs[i] = a.silu_in ? silu(x) : x;
+      ks[i] = (a.silu_in ? silu(y) : y) * a.k_scale;
+    }
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+      const float x = mine ? to_float(a.v[size_t(t) * a.v_stride + size_t(h) * a.vdim + j + u]) : 0.f;
+      v[u] = a.silu_in ? silu(x) : x;
+    }
+    __syncthreads();
+    auto row = [&](int r, float (&state)[V]) {
+#pragma unroll
+      for (int u = 0; u < V; ++u) {
+        state[u] = fmaf(decay, state[u], ks[r] * v[u]);
+        acc[u] = fmaf(state[u], qs[r], acc[u]);
+      }
+      float* p = head_state + size_t(r) * a.vdim + j;
+      if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(state[0], state[V > 1 ? 1 : 0], state[V > 2 ? 2 : 0], state[V > 3 ? 3 : 0]);
+      else *p = state[0];
+    };
+    if (mine) {
+#pragma unroll
+      for (int i = 0; i < STEP_ROWS; ++i)
+        if (rg + i * row_groups < a.dim) row(rg + i * row_groups, s[i]);
+      for (int r = rg + STEP_ROWS * row_groups; r < a.dim; r += row_groups) {
+        const float* p = head_state + size_t(r) * a.vdim + j;
+        float state[V];
+#pragma unroll
+        for (int u = 0; u < V; ++u) state[u] = zero ? 0.f : p[u];
+        row(r, state);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < V; ++u) sums[threadIdx.x][u] = acc[u];
+    __syncthreads();
+    if (rg == 0 && mine) {
+#pragma unroll
+      for (int u = 0; u < V; ++u) {
+        float o = 0.f;
+        for (int i = 0; i < row_groups; ++i) o += sums[i * groups + g][u];
+        a.out[size_t(t) * a.out_stride + size_t(h) * a.vdim + j + u] = o;
+      }
+    }
+    __syncthreads();   // (the vectors and sums of the next row)
+  }
+}
+
 size_t split_bytes(int rows, int stride) { return size_t(rows) * stride * 2 * sizeof(bf16); }
 
 }  // namespace
@@ -397,5 +488,27 @@ extern "C" int r2_decay_chunks(const void* q, int q_stride, const void* k, int k
   r2_launch(decay_chunk_sums_kernel, grid, dim3(THREADS), smem_sums, stream, a);
   r2_launch(decay_chunk_states_kernel, dim3(n_entries, n_heads, (dim * vdim + 255) / 256), dim3(256), size_t(0), stream, a);
   r2_launch(decay_chunk_outputs_kernel, grid, dim3(THREADS), smem_out, stream, a);
+  return launch_status();
+}
+
+// The same for batches in which (nearly) every entry is one row: one launch, no scratch.
+extern "C" int r2_decay_step(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* decay, float k_scale,
+                             int silu_in, float* state, long long slot_stride, const int32_t* q_start, const int32_t* state_slot, const int32_t* fresh,
+                             int n_entries, float* out, int out_stride, int n_heads, int dim, int vdim, int n_sms, cudaStream_t stream) {
+  if (n_entries <= 0) return R2_OK;
+  if (n_heads < 1 || dim < 1 || vdim < 1 || n_sms < 1) return R2_BAD_SHAPE;
+  if (dim > MAX_DIM || n_heads > 65535) return R2_UNSUPPORTED;
+  ChunkArgs a = {};
+  a.q = (const bf16*)q; a.q_stride = q_stride; a.k = (const bf16*)k; a.k_stride = k_stride; a.v = (const bf16*)v; a.v_stride = v_stride;
+  a.decay = decay; a.k_scale = k_scale; a.silu_in = silu_in; a.state = state; a.slot_stride = slot_stride;
+  a.q_start = q_start; a.state_slot = state_slot; a.fresh = fresh; a.n_entries = n_entries; a.out = out; a.out_stride = out_stride;
+  a.n_heads = n_heads; a.dim = dim; a.vdim = vdim;
+  // as many columns a CTA as leave twice as many CTAs as the GPU has SMs
+  int slice = 64;
+  while (slice > 16 && (long long)n_entries * n_heads * ((vdim + slice - 1) / slice) < 2ll * n_sms) slice /= 2;
+  const dim3 grid(n_entries, n_heads, (vdim + slice - 1) / slice);
+  const bool quads = vdim % 4 == 0 && slot_stride % 4 == 0 && !(reinterpret_cast<uintptr_t>(state) & 15);
+  if (quads) r2_launch(decay_step_kernel<4>, grid, dim3(STEP_THREADS), size_t(0), stream, a, slice);
+  else r2_launch(decay_step_kernel<1>, grid, dim3(STEP_THREADS), size_t(0), stream, a, slice);
   return launch_status();
 }

@@ -425,8 +425,13 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
         for (int j = 0; j < 32; ++j) v[j] = gelu_tanh_fast(v[j]);
       }
     } else if (p.act == R2_ACT_GELU_ERF) {
+      if (p.out_is_bf16) {
 #pragma unroll
-      for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
+        for (int j = 0; j < 32; ++j) v[j] = gelu_erf_rounded(v[j]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
+      }
     }
     if (p.route != nullptr) {
 #pragma unroll
@@ -991,8 +996,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_tanh_fast(v[j]);
           } else if (p.act == R2_ACT_GELU_ERF) {
+            if (p.out_is_bf16) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
+              for (int j = 0; j < 16; ++j) v[j] = gelu_erf_rounded(v[j]);
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
+            }
           }
           if (p.route != nullptr) {
             if (c0 == 0) {

@@ -114,29 +114,64 @@ route_top_k_kernel(const T* __restrict__ h, int h_stride, const float* __restric
 // largest choice score alone. normalise = 0: the chosen s are not divided by their sum. The weights are multiplied by weight_scale.
 // n_identity: the last of the n_experts outputs stand for no expert but for the input row itself: carried[t] = their weights' sum
 // * h[t] (+ base[t] where given), float.
+// A warp has an output at a time; with `quads` its row of w comes as 16-byte pieces, the first ROUTE_AHEAD of them asked for before the
+// kernel before this one has ended (weights are no kernel's output).
+constexpr int ROUTE_AHEAD = 6, ROUTE_WARPS = 16;
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ w, const float* __restrict__ correction,
                     float* __restrict__ dense, int32_t* __restrict__ chosen, float* __restrict__ chosen_weight,
                     float* __restrict__ extra, int n_experts, int n_extra, int top, int n_groups, int keep, int width,
                     int softmax_scores, int mark_best_only, int normalise, float weight_scale, int n_identity,
-                    const float* __restrict__ base, float* __restrict__ carried) {
+                    const float* __restrict__ base, float* __restrict__ carried, int quads) {
   pdl_launch_dependents();
-  pdl_wait();
-  extern __shared__ float smem[];
+  extern __shared__ __align__(16) float smem[];
   __shared__ float identity_weight;
   float* row = smem;                    // [width]
-  float* score = smem + width;          // [n_experts] sigmoid of the logit
+  float* score = smem + width;          // [n_experts] the scores
   float* choice = score + n_experts;    // [n_experts] score + correction; -inf once picked or outside the kept groups
-  float* mark = choice + n_experts;     // [n_groups]
+  float* given = choice + n_experts;    // [n_experts] the weights, zero where not chosen
+  float* mark = given + n_experts;      // [n_groups]
+  float* pick_weight = mark + n_groups;                               // [top]
+  int* pick = reinterpret_cast<int*>(pick_weight + top);              // [top]
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  float4 ahead[ROUTE_AHEAD];
+  if (quads && warp < n_experts + n_extra) {
+#pragma unroll
+    for (int i = 0; i < ROUTE_AHEAD; ++i) {
+      const int k = 4 * lane + 128 * i;
+      ahead[i] = k < width ? *reinterpret_cast<const float4*>(w + size_t(warp) * width + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
+  for (int n = threadIdx.x; n < n_experts; n += blockDim.x) given[n] = 0.f;
+  pdl_wait();
   const T* hr = h + size_t(t) * h_stride;
   for (int k = threadIdx.x; k < width; k += blockDim.x) row[k] = to_float(hr[k]);
   __syncthreads();
   for (int n = warp; n < n_experts + n_extra; n += n_warps) {
     const float* wr = w + size_t(n) * width;
     float acc = 0.f;
-    for (int k = lane; k < width; k += 32) acc = fmaf(row[k], wr[k], acc);
+    if (quads) {
+      float sum[4] = {0.f, 0.f, 0.f, 0.f};
+      auto add = [&](const float4 a, int k) {
+        const float4 x = *reinterpret_cast<const float4*>(row + k);
+        sum[0] = fmaf(x.x, a.x, sum[0]);
+        sum[1] = fmaf(x.y, a.y, sum[1]);
+        sum[2] = fmaf(x.z, a.z, sum[2]);
+        sum[3] = fmaf(x.w, a.w, sum[3]);
+      };
+#pragma unroll
+      for (int i = 0; i < ROUTE_AHEAD; ++i) {
+        const int k = 4 * lane + 128 * i;
+        if (k < width) add(n == warp ? ahead[i] : *reinterpret_cast<const float4*>(wr + k), k);
+      }
+#pragma unroll 4
+      for (int k = 4 * lane + 128 * ROUTE_AHEAD; k < width; k += 128) add(*reinterpret_cast<const float4*>(wr + k), k);
+      acc = (sum[0] + sum[1]) + (sum[2] + sum[3]);
+    } else {
+#pragma unroll 4
+      for (int k = lane; k < width; k += 32) acc = fmaf(row[k], wr[k], acc);
+    }
     acc = warp_sum(acc);
     if (lane == 0) {
       if (n < n_experts) {
@@ -148,7 +183,6 @@ route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restri
       }
     }
   }
-  for (int n = threadIdx.x; n < n_experts; n += blockDim.x) dense[size_t(t) * n_experts + n] = 0.f;
   __syncthreads();
   if (warp == 0) {
     if (softmax_scores) {
@@ -216,28 +250,30 @@ route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restri
       const float s = score[at];
       sum += s;
       if (lane == 0) {
-        chosen[size_t(t) * top + c] = at;
-        chosen_weight[size_t(t) * top + c] = s;
+        pick[c] = at;
+        pick_weight[c] = s;
         choice[at] = -INFINITY;
       }
       __syncwarp();
     }
     const float inv = (normalise ? 1.f / (sum + 1e-20f) : 1.f) * weight_scale;
     for (int c = lane; c < top; c += 32) {
-      const float p = chosen_weight[size_t(t) * top + c] * inv;
+      const float p = pick_weight[c] * inv;
+      chosen[size_t(t) * top + c] = pick[c];
       chosen_weight[size_t(t) * top + c] = p;
-      dense[size_t(t) * n_experts + chosen[size_t(t) * top + c]] = p;
+      given[pick[c]] = p;
     }
+    __syncwarp();
     if (n_identity > 0) {
-      __syncwarp();   // (the warp's writes to the row of weights are seen by its lanes)
       float c = 0.f;
-      for (int n = n_experts - n_identity + lane; n < n_experts; n += 32) c += dense[size_t(t) * n_experts + n];
+      for (int n = n_experts - n_identity + lane; n < n_experts; n += 32) c += given[n];
       c = warp_sum(c);
       if (lane == 0) identity_weight = c;
     }
   }
-  if (n_identity == 0) return;
   __syncthreads();
+  for (int n = threadIdx.x; n < n_experts; n += blockDim.x) dense[size_t(t) * n_experts + n] = given[n];
+  if (n_identity == 0) return;
   const float share = identity_weight;
   for (int k = threadIdx.x; k < width; k += blockDim.x)
     carried[size_t(t) * width + k] = share * row[k] + (base != nullptr ? base[size_t(t) * width + k] : 0.f);
@@ -361,14 +397,18 @@ extern "C" int r2_route_scored(const void* h, int h_stride, const float* w, cons
   if (width < 1 || n_experts < 1 || n_experts > MAX_EXPERTS || top < 1 || n_groups < 1 || n_experts % n_groups != 0 || keep < 1 ||
       keep > n_groups || top > n_experts / n_groups * keep || n_extra < 0 || (n_extra > 0 && extra == nullptr) ||
       n_identity < 0 || n_identity > n_experts || (n_identity > 0 && carried == nullptr)) return R2_BAD_SHAPE;
-  const size_t smem = sizeof(float) * (size_t(width) + 2 * n_experts + n_groups);
-  if (smem > 48 * 1024) return R2_UNSUPPORTED;
+  const size_t smem = sizeof(float) * (size_t(width) + 3 * n_experts + n_groups + 2 * top);
+  if (smem > 47 * 1024) return R2_UNSUPPORTED;
+  const int quads = width % 4 == 0 && !(reinterpret_cast<uintptr_t>(w) & 15);
+  // a warp an output where there are few rows (a decode step waits for the slowest warp); many rows fill the SMs with fewer
+  const int outputs = n_experts + n_extra, most = n_rows <= 256 ? ROUTE_WARPS : 8;
+  const int threads = 32 * (outputs < 4 ? 4 : outputs < most ? outputs : most);
   if (dtype == R2_F32) {
-    r2_launch(route_scored_kernel<float>, dim3(n_rows), dim3(256), smem, stream, (const float*)h, h_stride, w, correction, dense, chosen,
-              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried);
+    r2_launch(route_scored_kernel<float>, dim3(n_rows), dim3(threads), smem, stream, (const float*)h, h_stride, w, correction, dense, chosen,
+              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried, quads);
   } else if (dtype == R2_BF16) {
-    r2_launch(route_scored_kernel<bf16>, dim3(n_rows), dim3(256), smem, stream, (const bf16*)h, h_stride, w, correction, dense, chosen,
-              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried);
+    r2_launch(route_scored_kernel<bf16>, dim3(n_rows), dim3(threads), smem, stream, (const bf16*)h, h_stride, w, correction, dense, chosen,
+              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried, quads);
   } else {
     return R2_BAD_DTYPE;
   }

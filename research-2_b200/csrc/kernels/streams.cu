@@ -113,7 +113,16 @@ stream_join_kernel(const StreamArgs a) {
     }
     return u;
   };
-  auto columns = [&](int d) { return joins ? joined(d) : summed(x, x_step, d); };
+  float read_all = 0.f;
+  for (int s = 0; s < n; ++s) read_all += read_s[s];
+  auto columns = [&](int d) {
+    if (joins) return joined(d);
+    if (!a.spread) return summed(x, x_step, d);
+    Pack<V> u = load_pack<V>(x + d);   // every stream holds this row
+#pragma unroll
+    for (int i = 0; i < V; ++i) u.v[i] *= read_all;
+    return u;
+  };
 
   const int step = blockDim.x * V, first = threadIdx.x * V;
   if (a.gain == nullptr) {   // u itself
@@ -149,7 +158,7 @@ stream_join_kernel(const StreamArgs a) {
     if (d < width) leave(d, keep[k]);
   }
   // (a thread's own columns again: of the new streams where they were stored, else of the ones that came)
-  for (int d = first + KEEP * step; d < width; d += step) leave(d, joins ? summed(x_out, width, d) : summed(x, x_step, d));
+  for (int d = first + KEEP * step; d < width; d += step) leave(d, joins ? summed(x_out, width, d) : columns(d));
 }
 
 template <int S, int V, typename O>

@@ -807,7 +807,7 @@ _decay_chunks = os.environ.get("R2_DECAY_CHUNKS", "1") != "0"
 
 
 def use_decay_chunks(on: bool) -> bool:
-    """Whether linear attention with a fixed decay per head runs prompts in chunks on the tensor cores (bfloat16); off, row by row.
+    """Whether linear attention with a fixed decay per head runs prompts in chunks on the tensor cores and decode steps on their own kernel (bfloat16); off, the general walk takes both.
     Returns the previous setting."""
     global _decay_chunks
     before, _decay_chunks = _decay_chunks, bool(on)
@@ -823,7 +823,7 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     way in (of each head the first rot_dims dimensions, i with i + rot_dims / 2, angle positions[t] * inv_freq[i], in float32)
     and multiplies k by k_scale after that. `silu`: q, k and v pass silu on their way in (float32, instead of a rotation).
     With `n_tiles` (the sum over entries of ceil(rows / 64) or more) bfloat16 batches of 64 rows and more run in chunks of 64 rows on the tensor
-    cores (csrc/kernels/decay_chunks.cu; heads of up to 256 rows, no rotation) instead of row by row. decay float32 [heads]; state float32 [slots, heads * dim * vdim].
+    cores (csrc/kernels/decay_chunks.cu; heads of up to 256 rows, no rotation) instead of row by row; there is a kernel for decode steps beside it. decay float32 [heads]; state float32 [slots, heads * dim * vdim].
     -> float32 [T, heads * vdim], the heads' outputs before their norm."""
     n = _entries(q_start, state_slot, fresh)
     for name, t, width in (("q", q, n_heads * dim), ("k", k, n_heads * dim), ("v", v, n_heads * vdim)):
@@ -840,7 +840,7 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
         if rot_dims % 2 or rot_dims > dim or inv_freq.shape[0] != rot_dims // 2:
             raise KernelError(f"retention_scan: {rot_dims} rotated dimensions of {dim}, {tuple(inv_freq.shape)} frequencies")
     out = torch.empty(q.shape[0], n_heads * vdim, dtype=torch.float32, device=q.device)
-    if q.dtype == torch.bfloat16 and n_tiles > 0 and q.shape[0] >= DECAY_CHUNK and dim <= 256 and not rot_dims and _decay_chunks:
+    if q.dtype == torch.bfloat16 and n_tiles > 0 and q.shape[0] >= DECAY_CHUNK and q.shape[0] > n and dim <= 256 and not rot_dims and _decay_chunks:
         scratch = torch.empty(n_tiles * n_heads * dim * vdim, dtype=torch.float32, device=q.device)
         status = _lib("decay_chunks").r2_decay_chunks(
             _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), C.c_float(k_scale), int(bool(silu)), _p(state),
@@ -850,6 +850,14 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
             _check(status, "retention_scan (chunks)")
             count_launches(2)  # the sums, the states, the outputs
             _used("decay_chunks")
+            return out
+    if q.dtype == torch.bfloat16 and q.shape[0] <= n and dim <= 256 and not rot_dims and _decay_chunks:
+        status = _lib("decay_chunks").r2_decay_step(
+            _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), C.c_float(k_scale), int(bool(silu)), _p(state),
+            C.c_longlong(state.shape[1]), _p(q_start), _p(state_slot), _p(fresh), n, _p(out), _rows(out, "out"), n_heads, dim, vdim, sm_count(q.device), _stream())
+        if status != -4:
+            _check(status, "retention_scan (step)")
+            _used("decay_step")
             return out
     status = _lib("recurrent").r2_retention_scan(
         _p(q), _rows(q, "q"), _p(k), _rows(k, "k"), _p(v), _rows(v, "v"), _p(decay), C.c_float(k_scale), _p(inv_freq if rot_dims else None),
