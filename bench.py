@@ -1313,8 +1313,6 @@ def tagulix_points(args, pk: dict) -> dict:
             n_bytes=t * d * (8 * streams + 6))
         add(f"its like: a sublayer's output normed into one stream + the next norm (Zudalorn), {label}",
             lambda: ops.norm_add(x32, y32, gain, 1e-5, gain, 1e-5, bf), n_bytes=t * d * 14)
-        add(f"the first sublayer's input from the embedding, {label}", lambda: ops.stream_join(x32, read, gain, 1e-5, bf), n_bytes=t * d * 6)
-        add(f"its like: the norm of a stream (any model), {label}", lambda: ops.rms_norm(x32, gain, 1e-5, bf), n_bytes=t * d * 6)
         # the window attention's turned and normed heads
         kvh = kv_heads_for(h)
         qkv = torch.randn(t, (h + 2 * kvh) * hd, device=dev).to(bf)

@@ -114,169 +114,252 @@ route_top_k_kernel(const T* __restrict__ h, int h_stride, const float* __restric
 // largest choice score alone. normalise = 0: the chosen s are not divided by their sum. The weights are multiplied by weight_scale.
 // n_identity: the last of the n_experts outputs stand for no expert but for the input row itself: carried[t] = their weights' sum
 // * h[t] (+ base[t] where given), float.
-// A warp has an output at a time; with `quads` its row of w comes as 16-byte pieces, the first ROUTE_AHEAD of them asked for before the
-// kernel before this one has ended (weights are no kernel's output).
-constexpr int ROUTE_AHEAD = 6, ROUTE_WARPS = 16;
-template <typename T>
-__global__ void __launch_bounds__(ROUTE_WARPS * 32)
-route_scored_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ w, const float* __restrict__ correction,
-                    float* __restrict__ dense, int32_t* __restrict__ chosen, float* __restrict__ chosen_weight,
-                    float* __restrict__ extra, int n_experts, int n_extra, int top, int n_groups, int keep, int width,
-                    int softmax_scores, int mark_best_only, int normalise, float weight_scale, int n_identity,
-                    const float* __restrict__ base, float* __restrict__ carried, int quads) {
-  pdl_launch_dependents();
-  extern __shared__ __align__(16) float smem[];
-  __shared__ float identity_weight;
-  float* row = smem;                    // [width]
-  float* score = smem + width;          // [n_experts] the scores
-  float* choice = score + n_experts;    // [n_experts] score + correction; -inf once picked or outside the kept groups
-  float* given = choice + n_experts;    // [n_experts] the weights, zero where not chosen
-  float* mark = given + n_experts;      // [n_groups]
-  float* pick_weight = mark + n_groups;                               // [top]
-  int* pick = reinterpret_cast<int*>(pick_weight + top);              // [top]
-  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
-  float4 ahead[ROUTE_AHEAD];
-  if (quads && warp < n_experts + n_extra) {
-#pragma unroll
-    for (int i = 0; i < ROUTE_AHEAD; ++i) {
-      const int k = 4 * lane + 128 * i;
-      ahead[i] = k < width ? *reinterpret_cast<const float4*>(w + size_t(warp) * width + k) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
+struct RouteArgs {
+  const void* h; int h_stride;
+  const float* w; const float* correction;
+  float* dense; int32_t* chosen; float* chosen_weight; float* extra;
+  int n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise;
+  float weight_scale;
+  int n_identity; const float* base; float* carried;
+  int quads;   // rows of w start on 16-byte boundaries and hold a multiple of four numbers
+};
+
+// What a row's choice works on, in shared memory.
+struct RouteRow {
+  float* row;          // [width]
+  float* score;        // [n_experts] the scores
+  float* choice;       // [n_experts] score + correction; -inf once picked or outside the kept groups
+  float* given;        // [n_experts] the weights, zero where not chosen
+  float* mark;         // [n_groups]
+  float* pick_weight;  // [top]
+  int* pick;           // [top]
+};
+__device__ __host__ __forceinline__ size_t route_row_floats(int width, int n_experts, int n_groups, int top) {
+  return (size_t(width) + 3 * n_experts + n_groups + 2 * top + 3) / 4 * 4;
+}
+__device__ __forceinline__ RouteRow route_row(float* at, const RouteArgs& a) {
+  RouteRow r;
+  r.row = at;
+  r.score = at + a.width;
+  r.choice = r.score + a.n_experts;
+  r.given = r.choice + a.n_experts;
+  r.mark = r.given + a.n_experts;
+  r.pick_weight = r.mark + a.n_groups;
+  r.pick = reinterpret_cast<int*>(r.pick_weight + a.top);
+  return r;
+}
+
+// a logit: what becomes of it
+__device__ __forceinline__ void put_logit(const RouteArgs& a, const RouteRow& r, int t, int n, float z) {
+  if (n < a.n_experts) {
+    const float s = a.softmax_scores ? z : 1.f / (1.f + expf(-z));   // (the softmax follows once all logits are there)
+    r.score[n] = s;
+    r.choice[n] = s + (a.correction != nullptr ? a.correction[n] : 0.f);
+  } else {
+    a.extra[size_t(t) * a.n_extra + (n - a.n_experts)] = z;
   }
-  for (int n = threadIdx.x; n < n_experts; n += blockDim.x) given[n] = 0.f;
-  pdl_wait();
-  const T* hr = h + size_t(t) * h_stride;
-  for (int k = threadIdx.x; k < width; k += blockDim.x) row[k] = to_float(hr[k]);
-  __syncthreads();
-  for (int n = warp; n < n_experts + n_extra; n += n_warps) {
-    const float* wr = w + size_t(n) * width;
-    float acc = 0.f;
-    if (quads) {
-      float sum[4] = {0.f, 0.f, 0.f, 0.f};
-      auto add = [&](const float4 a, int k) {
-        const float4 x = *reinterpret_cast<const float4*>(row + k);
-        sum[0] = fmaf(x.x, a.x, sum[0]);
-        sum[1] = fmaf(x.y, a.y, sum[1]);
-        sum[2] = fmaf(x.z, a.z, sum[2]);
-        sum[3] = fmaf(x.w, a.w, sum[3]);
-      };
-#pragma unroll
-      for (int i = 0; i < ROUTE_AHEAD; ++i) {
-        const int k = 4 * lane + 128 * i;
-        if (k < width) add(n == warp ? ahead[i] : *reinterpret_cast<const float4*>(wr + k), k);
-      }
-#pragma unroll 4
-      for (int k = 4 * lane + 128 * ROUTE_AHEAD; k < width; k += 128) add(*reinterpret_cast<const float4*>(wr + k), k);
-      acc = (sum[0] + sum[1]) + (sum[2] + sum[3]);
-    } else {
-#pragma unroll 4
-      for (int k = lane; k < width; k += 32) acc = fmaf(row[k], wr[k], acc);
+}
+
+// One warp: scores, groups, picks and weights of row t, from its logits. -> the identity outputs' weights' sum
+__device__ __forceinline__ float choose_experts(const RouteArgs& a, const RouteRow& r, int t, int lane) {
+  if (a.softmax_scores) {
+    // s = exp(z - max) / sum over all experts, one warp, sums in a fixed order
+    float top_z = -INFINITY;
+    for (int n = lane; n < a.n_experts; n += 32) top_z = fmaxf(top_z, r.score[n]);
+    for (int o = 16; o > 0; o >>= 1) top_z = fmaxf(top_z, __shfl_xor_sync(0xffffffffu, top_z, o));
+    float total = 0.f;
+    for (int n = lane; n < a.n_experts; n += 32) {
+      const float e = expf(r.score[n] - top_z);
+      r.score[n] = e;
+      total += e;
     }
-    acc = warp_sum(acc);
-    if (lane == 0) {
-      if (n < n_experts) {
-        const float s = softmax_scores ? acc : 1.f / (1.f + expf(-acc));   // (the softmax follows once all logits are there)
-        score[n] = s;
-        choice[n] = s + (correction != nullptr ? correction[n] : 0.f);
-      } else {
-        extra[size_t(t) * n_extra + (n - n_experts)] = acc;
-      }
+    total = warp_sum(total);
+    const float inv_total = 1.f / total;
+    for (int n = lane; n < a.n_experts; n += 32) {
+      const float s = r.score[n] * inv_total;
+      r.score[n] = s;
+      r.choice[n] = s + (a.correction != nullptr ? a.correction[n] : 0.f);
     }
+    __syncwarp();
   }
-  __syncthreads();
-  if (warp == 0) {
-    if (softmax_scores) {
-      // s = exp(z - max) / sum over all experts, one warp, sums in a fixed order
-      float top_z = -INFINITY;
-      for (int n = lane; n < n_experts; n += 32) top_z = fmaxf(top_z, score[n]);
-      for (int o = 16; o > 0; o >>= 1) top_z = fmaxf(top_z, __shfl_xor_sync(0xffffffffu, top_z, o));
-      float total = 0.f;
-      for (int n = lane; n < n_experts; n += 32) {
-        const float e = expf(score[n] - top_z);
-        score[n] = e;
-        total += e;
+  const int size = a.n_experts / a.n_groups;
+  if (a.keep < a.n_groups) {
+    for (int g = lane; g < a.n_groups; g += 32) {
+      float best = -INFINITY, second = -INFINITY;   // the group's largest and second largest
+      for (int n = g * size; n < (g + 1) * size; ++n) {
+        const float c = r.choice[n];
+        if (c > best) { second = best; best = c; }
+        else if (c > second) second = c;
       }
-      total = warp_sum(total);
-      const float inv_total = 1.f / total;
-      for (int n = lane; n < n_experts; n += 32) {
-        const float s = score[n] * inv_total;
-        score[n] = s;
-        choice[n] = s + (correction != nullptr ? correction[n] : 0.f);
-      }
-      __syncwarp();
+      r.mark[g] = (size > 1 && !a.mark_best_only) ? best + second : best;
     }
-    const int size = n_experts / n_groups;
-    if (keep < n_groups) {
-      for (int g = lane; g < n_groups; g += 32) {
-        float a = -INFINITY, b = -INFINITY;   // the group's largest and second largest
-        for (int n = g * size; n < (g + 1) * size; ++n) {
-          const float c = choice[n];
-          if (c > a) { b = a; a = c; }
-          else if (c > b) b = c;
-        }
-        mark[g] = (size > 1 && !mark_best_only) ? a + b : a;
-      }
-      __syncwarp();
-      // the kept groups: `keep` times the largest mark; a kept group's mark becomes +inf, and what is not +inf at the end is out
-      for (int c = 0; c < keep; ++c) {
-        float v = -INFINITY;
-        int at = n_groups;
-        for (int g = lane; g < n_groups; g += 32)
-          if (mark[g] != INFINITY && (mark[g] > v || at == n_groups)) { v = mark[g]; at = g; }
-        for (int o = 16; o > 0; o >>= 1) {
-          const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-          const int oat = __shfl_xor_sync(0xffffffffu, at, o);
-          if (oat < n_groups && (at == n_groups || ov > v || (ov == v && oat < at))) { v = ov; at = oat; }
-        }
-        if (lane == 0 && at < n_groups) mark[at] = INFINITY;
-        __syncwarp();
-      }
-      for (int n = lane; n < n_experts; n += 32)
-        if (mark[n / size] != INFINITY) choice[n] = -INFINITY;
-      __syncwarp();
-    }
-    float sum = 0.f;
-    for (int c = 0; c < top; ++c) {
+    __syncwarp();
+    // the kept groups: `keep` times the largest mark; a kept group's mark becomes +inf, and what is not +inf at the end is out
+    for (int c = 0; c < a.keep; ++c) {
       float v = -INFINITY;
-      int at = n_experts;
-      for (int n = lane; n < n_experts; n += 32)
-        if (choice[n] > v) { v = choice[n]; at = n; }
+      int at = a.n_groups;
+      for (int g = lane; g < a.n_groups; g += 32)
+        if (r.mark[g] != INFINITY && (r.mark[g] > v || at == a.n_groups)) { v = r.mark[g]; at = g; }
       for (int o = 16; o > 0; o >>= 1) {
         const float ov = __shfl_xor_sync(0xffffffffu, v, o);
         const int oat = __shfl_xor_sync(0xffffffffu, at, o);
-        if (ov > v || (ov == v && oat < at)) { v = ov; at = oat; }
+        if (oat < a.n_groups && (at == a.n_groups || ov > v || (ov == v && oat < at))) { v = ov; at = oat; }
       }
-      if (at >= n_experts) at = c;   // scores that are not numbers: no index may leave the row
-      const float s = score[at];
-      sum += s;
-      if (lane == 0) {
-        pick[c] = at;
-        pick_weight[c] = s;
-        choice[at] = -INFINITY;
-      }
+      if (lane == 0 && at < a.n_groups) r.mark[at] = INFINITY;
       __syncwarp();
     }
-    const float inv = (normalise ? 1.f / (sum + 1e-20f) : 1.f) * weight_scale;
-    for (int c = lane; c < top; c += 32) {
-      const float p = pick_weight[c] * inv;
-      chosen[size_t(t) * top + c] = pick[c];
-      chosen_weight[size_t(t) * top + c] = p;
-      given[pick[c]] = p;
+    for (int n = lane; n < a.n_experts; n += 32)
+      if (r.mark[n / size] != INFINITY) r.choice[n] = -INFINITY;
+    __syncwarp();
+  }
+  float sum = 0.f;
+  for (int c = 0; c < a.top; ++c) {
+    float v = -INFINITY;
+    int at = a.n_experts;
+    for (int n = lane; n < a.n_experts; n += 32)
+      if (r.choice[n] > v) { v = r.choice[n]; at = n; }
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+      const int oat = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ov > v || (ov == v && oat < at)) { v = ov; at = oat; }
+    }
+    if (at >= a.n_experts) at = c;   // scores that are not numbers: no index may leave the row
+    const float s = r.score[at];
+    sum += s;
+    if (lane == 0) {
+      r.pick[c] = at;
+      r.pick_weight[c] = s;
+      r.choice[at] = -INFINITY;
     }
     __syncwarp();
-    if (n_identity > 0) {
-      float c = 0.f;
-      for (int n = n_experts - n_identity + lane; n < n_experts; n += 32) c += given[n];
-      c = warp_sum(c);
-      if (lane == 0) identity_weight = c;
+  }
+  const float inv = (a.normalise ? 1.f / (sum + 1e-20f) : 1.f) * a.weight_scale;
+  for (int c = lane; c < a.top; c += 32) {
+    const float p = r.pick_weight[c] * inv;
+    a.chosen[size_t(t) * a.top + c] = r.pick[c];
+    a.chosen_weight[size_t(t) * a.top + c] = p;
+    r.given[r.pick[c]] = p;
+  }
+  __syncwarp();
+  float share = 0.f;
+  for (int n = a.n_experts - a.n_identity + lane; n < a.n_experts; n += 32) share += r.given[n];
+  return warp_sum(share);
+}
+
+// four neighbouring products into four sums: the order in which a logit's terms are added is the same in both forms below
+__device__ __forceinline__ void add_quad(float (&sum)[4], const float4 x, const float4 w) {
+  sum[0] = fmaf(x.x, w.x, sum[0]);
+  sum[1] = fmaf(x.y, w.y, sum[1]);
+  sum[2] = fmaf(x.z, w.z, sum[2]);
+  sum[3] = fmaf(x.w, w.w, sum[3]);
+}
+
+// A CTA a row. A warp has an output at a time; with `quads` its row of w comes as 16-byte pieces, the first ROUTE_AHEAD of them asked for
+// before the kernel before this one has ended (weights are no kernel's output).
+constexpr int ROUTE_AHEAD = 6, ROUTE_WARPS = 16;
+template <typename T>
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+route_scored_kernel(const RouteArgs a) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float smem[];
+  __shared__ float identity_weight;
+  const RouteRow r = route_row(smem, a);
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5, width = a.width;
+  float4 ahead[ROUTE_AHEAD];
+  if (a.quads && warp < a.n_experts + a.n_extra) {
+#pragma unroll
+    for (int i = 0; i < ROUTE_AHEAD; ++i) {
+      const int k = 4 * lane + 128 * i;
+      ahead[i] = k < width ? *reinterpret_cast<const float4*>(a.w + size_t(warp) * width + k) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   }
+  for (int n = threadIdx.x; n < a.n_experts; n += blockDim.x) r.given[n] = 0.f;
+  pdl_wait();
+  const T* hr = static_cast<const T*>(a.h) + size_t(t) * a.h_stride;
+  for (int k = threadIdx.x; k < width; k += blockDim.x) r.row[k] = to_float(hr[k]);
   __syncthreads();
-  for (int n = threadIdx.x; n < n_experts; n += blockDim.x) dense[size_t(t) * n_experts + n] = given[n];
-  if (n_identity == 0) return;
+  for (int n = warp; n < a.n_experts + a.n_extra; n += n_warps) {
+    const float* wr = a.w + size_t(n) * width;
+    float acc = 0.f;
+    if (a.quads) {
+      float sum[4] = {0.f, 0.f, 0.f, 0.f};
+      auto at = [&](const float* p, int k) { return *reinterpret_cast<const float4*>(p + k); };
+#pragma unroll
+      for (int i = 0; i < ROUTE_AHEAD; ++i) {
+        const int k = 4 * lane + 128 * i;
+        if (k < width) add_quad(sum, at(r.row, k), n == warp ? ahead[i] : at(wr, k));
+      }
+#pragma unroll 4
+      for (int k = 4 * lane + 128 * ROUTE_AHEAD; k < width; k += 128) add_quad(sum, at(r.row, k), at(wr, k));
+      acc = (sum[0] + sum[1]) + (sum[2] + sum[3]);
+    } else {
+#pragma unroll 4
+      for (int k = lane; k < width; k += 32) acc = fmaf(r.row[k], wr[k], acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) put_logit(a, r, t, n, acc);
+  }
+  __syncthreads();
+  if (warp == 0) {
+    const float share = choose_experts(a, r, t, lane);
+    if (lane == 0) identity_weight = share;
+  }
+  __syncthreads();
+  for (int n = threadIdx.x; n < a.n_experts; n += blockDim.x) a.dense[size_t(t) * a.n_experts + n] = r.given[n];
+  if (a.n_identity == 0) return;
   const float share = identity_weight;
   for (int k = threadIdx.x; k < width; k += blockDim.x)
-    carried[size_t(t) * width + k] = share * row[k] + (base != nullptr ? base[size_t(t) * width + k] : 0.f);
+    a.carried[size_t(t) * width + k] = share * r.row[k] + (a.base != nullptr ? a.base[size_t(t) * width + k] : 0.f);
+}
+
+// A warp a row, for many rows: the weights are in shared memory once a CTA, whose warps take row after row. (`quads` only.)
+constexpr int ROUTE_ROWS = 8;
+template <typename T>
+__global__ void __launch_bounds__(ROUTE_ROWS * 32)
+route_scored_rows_kernel(const RouteArgs a, int n_rows) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float smem[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, width = a.width, outputs = a.n_experts + a.n_extra;
+  float* ws = smem;   // [outputs][width]
+  const RouteRow r = route_row(smem + size_t(outputs) * width + warp * route_row_floats(width, a.n_experts, a.n_groups, a.top), a);
+  for (int i = threadIdx.x; i < outputs * width / 4; i += blockDim.x) reinterpret_cast<float4*>(ws)[i] = reinterpret_cast<const float4*>(a.w)[i];
+  __syncthreads();
+  pdl_wait();
+  for (int t = blockIdx.x * ROUTE_ROWS + warp; t < n_rows; t += gridDim.x * ROUTE_ROWS) {
+    const T* hr = static_cast<const T*>(a.h) + size_t(t) * a.h_stride;
+    for (int k = lane; k < width; k += 32) r.row[k] = to_float(hr[k]);
+    for (int n = lane; n < a.n_experts; n += 32) r.given[n] = 0.f;
+    __syncwarp();
+    for (int n0 = 0; n0 < outputs; n0 += 4) {   // four outputs at a time: the row's numbers are read once for them
+      float sum[4][4] = {};
+      const float* wr[4];
+#pragma unroll
+      for (int o = 0; o < 4; ++o) wr[o] = ws + size_t(min(n0 + o, outputs - 1)) * width;
+#pragma unroll 2
+      for (int k = 4 * lane; k < width; k += 128) {
+        const float4 x = *reinterpret_cast<const float4*>(r.row + k);
+#pragma unroll
+        for (int o = 0; o < 4; ++o) add_quad(sum[o], x, *reinterpret_cast<const float4*>(wr[o] + k));
+      }
+#pragma unroll
+      for (int o = 0; o < 4; ++o) {
+        const float acc = warp_sum((sum[o][0] + sum[o][1]) + (sum[o][2] + sum[o][3]));
+        if (lane == 0 && n0 + o < outputs) put_logit(a, r, t, n0 + o, acc);
+      }
+    }
+    __syncwarp();
+    const float share = choose_experts(a, r, t, lane);
+    for (int n = lane; n < a.n_experts; n += 32) a.dense[size_t(t) * a.n_experts + n] = r.given[n];
+    if (a.n_identity > 0) {
+      for (int k = 4 * lane; k < width; k += 128) {
+        const float4 x = *reinterpret_cast<const float4*>(r.row + k);
+        const size_t at = size_t(t) * width + k;
+        const float4 b = a.base != nullptr ? *reinterpret_cast<const float4*>(a.base + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+        *reinterpret_cast<float4*>(a.carried + at) = make_float4(share * x.x + b.x, share * x.y + b.y, share * x.z + b.z, share * x.w + b.w);
+      }
+    }
+    __syncwarp();   // (the warp's next row)
+  }
 }
 
 constexpr int KIND_CLAMPED_SWISH = 0, KIND_RELU = 1, KIND_SILU = 2, KIND_GELU_TANH = 3;
@@ -397,21 +480,36 @@ extern "C" int r2_route_scored(const void* h, int h_stride, const float* w, cons
   if (width < 1 || n_experts < 1 || n_experts > MAX_EXPERTS || top < 1 || n_groups < 1 || n_experts % n_groups != 0 || keep < 1 ||
       keep > n_groups || top > n_experts / n_groups * keep || n_extra < 0 || (n_extra > 0 && extra == nullptr) ||
       n_identity < 0 || n_identity > n_experts || (n_identity > 0 && carried == nullptr)) return R2_BAD_SHAPE;
-  const size_t smem = sizeof(float) * (size_t(width) + 3 * n_experts + n_groups + 2 * top);
-  if (smem > 47 * 1024) return R2_UNSUPPORTED;
-  const int quads = width % 4 == 0 && !(reinterpret_cast<uintptr_t>(w) & 15);
-  // a warp an output where there are few rows (a decode step waits for the slowest warp); many rows fill the SMs with fewer
-  const int outputs = n_experts + n_extra, most = n_rows <= 256 ? ROUTE_WARPS : 8;
-  const int threads = 32 * (outputs < 4 ? 4 : outputs < most ? outputs : most);
-  if (dtype == R2_F32) {
-    r2_launch(route_scored_kernel<float>, dim3(n_rows), dim3(threads), smem, stream, (const float*)h, h_stride, w, correction, dense, chosen,
-              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried, quads);
-  } else if (dtype == R2_BF16) {
-    r2_launch(route_scored_kernel<bf16>, dim3(n_rows), dim3(threads), smem, stream, (const bf16*)h, h_stride, w, correction, dense, chosen,
-              chosen_weight, extra, n_experts, n_extra, top, n_groups, keep, width, softmax_scores, mark_best_only, normalise, weight_scale, n_identity, base, carried, quads);
-  } else {
-    return R2_BAD_DTYPE;
+  RouteArgs a = {};
+  a.h = h; a.h_stride = h_stride; a.w = w; a.correction = correction; a.dense = dense; a.chosen = chosen; a.chosen_weight = chosen_weight; a.extra = extra;
+  a.n_experts = n_experts; a.n_extra = n_extra; a.top = top; a.n_groups = n_groups; a.keep = keep; a.width = width; a.softmax_scores = softmax_scores;
+  a.mark_best_only = mark_best_only; a.normalise = normalise; a.weight_scale = weight_scale; a.n_identity = n_identity; a.base = base; a.carried = carried;
+  auto on16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  a.quads = width % 4 == 0 && on16(w);
+  if (dtype != R2_F32 && dtype != R2_BF16) return R2_BAD_DTYPE;
+  const size_t per_row = sizeof(float) * route_row_floats(width, n_experts, n_groups, top);
+  const int outputs = n_experts + n_extra;
+  const size_t many = sizeof(float) * size_t(outputs) * width + ROUTE_ROWS * per_row;
+  constexpr size_t MOST = 110 * 1024;   // (two CTAs an SM)
+  if (n_rows >= 512 && a.quads && many <= MOST && on16(base) && on16(carried)) {
+    static bool configured = false;
+    if (!configured) {
+      cudaError_t e = cudaFuncSetAttribute(route_scored_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(MOST));
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(route_scored_rows_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(MOST));
+      if (e != cudaSuccess) return int(e);
+      configured = true;
+    }
+    const dim3 grid(min((n_rows + ROUTE_ROWS - 1) / ROUTE_ROWS, 2048));
+    if (dtype == R2_F32) r2_launch(route_scored_rows_kernel<float>, grid, dim3(ROUTE_ROWS * 32), many, stream, a, n_rows);
+    else r2_launch(route_scored_rows_kernel<bf16>, grid, dim3(ROUTE_ROWS * 32), many, stream, a, n_rows);
+    return launch_status();
   }
+  if (per_row > 47 * 1024) return R2_UNSUPPORTED;
+  // a warp an output where there are few rows (a decode step waits for the slowest warp); many rows fill the SMs with fewer
+  const int most = n_rows <= 256 ? ROUTE_WARPS : 8;
+  const dim3 threads(32 * (outputs < 4 ? 4 : outputs < most ? outputs : most));
+  if (dtype == R2_F32) r2_launch(route_scored_kernel<float>, dim3(n_rows), threads, per_row, stream, a);
+  else r2_launch(route_scored_kernel<bf16>, dim3(n_rows), threads, per_row, stream, a);
   return launch_status();
 }
 

@@ -208,6 +208,9 @@ class StreamsBlock:
                 raise ValueError(f"streams: in {tuple(read.shape)}, out {tuple(join.shape)} and mix {tuple(mix.shape)} do not fit each other")
             self.ways.append((read, mix, join * float(factor)))
         self.sum = torch.ones_like(self.ways[0][0])
+        # Streams that all hold the row e: u = c e with c = sum_s in_1[s], and u / rms(u) is e / sqrt(mean(e^2) + eps / c^2) with c's sign
+        total = float(self.ways[0][0].double().sum())
+        self.first = None if total == 0.0 else (norm_1.gain if total > 0 else -norm_1.gain, norm_1.eps / total ** 2)
 
     @property
     def n_streams(self) -> int:
@@ -222,7 +225,10 @@ class StreamsBlock:
         if carried is not None and carried[0] is x:
             h = carried[1]
         else:
-            _, h = ops.stream_join(x, self.ways[0][0], self.norm_1.gain, self.norm_1.eps, self.compute_dtype)
+            if x.dim() == 2 and self.first is not None:
+                h = ops.rms_norm(x, *self.first, self.compute_dtype)
+            else:
+                _, h = ops.stream_join(x, self.ways[0][0], self.norm_1.gain, self.norm_1.eps, self.compute_dtype)
         ctx.stream_input = None
         follows = isinstance(upcoming, StreamsBlock) and upcoming.n_streams == self.n_streams
         after = (upcoming.ways[0][0], upcoming.norm_1) if follows else (self.sum, None)
