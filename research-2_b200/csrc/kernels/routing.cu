@@ -490,7 +490,7 @@ extern "C" int r2_route_scored(const void* h, int h_stride, const float* w, cons
   const size_t per_row = sizeof(float) * route_row_floats(width, n_experts, n_groups, top);
   const int outputs = n_experts + n_extra;
   const size_t many = sizeof(float) * size_t(outputs) * width + ROUTE_ROWS * per_row;
-  constexpr size_t MOST = 110 * 1024;   // (two CTAs an SM)
+  constexpr size_t MOST = 200 * 1024;   // (two CTAs an SM up to 113 KB)
   if (n_rows >= 512 && a.quads && many <= MOST && on16(base) && on16(carried)) {
     static bool configured = false;
     if (!configured) {
