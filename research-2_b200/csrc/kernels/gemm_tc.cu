@@ -387,6 +387,9 @@ constexpr int BIAS_SLOTS = 256;                       // floats: the widest tile
 // `bias_s` holds the tile's bias (zeros without one), 16-byte aligned. bfloat16 output without a
 // residual moves 64 columns a group as packed pairs; everything else 32 columns as floats.
 // `slab` is the warp's 32 x STAGING_ROW words of shared memory, as a shared-space address.
+// ROUTED: values are multiplied by their token's weight for their block of features (a form of its own: the other products' epilogues stay
+// as short as they are).
+template <bool ROUTED>
 __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t lane_addr, uint32_t slab, const float* bias_s,
                                                  int row0, int col0, int c_begin, int c_end, int lane, bool have_acc) {
   const int rows = min(32, p.a_total - row0);        // rows of this slab that exist
@@ -396,7 +399,7 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
   struct RouteAt { float first, second; int n_first; };
   auto route_at = [&](int c) {
     RouteAt at = {1.f, 1.f, 32};
-    if (p.route != nullptr) {
+    if constexpr (ROUTED) {
       const int block = (col0 + c) / p.route_width, last = p.b_total / p.route_width - 1;
       const float* weights = p.route + size_t(min(row0 + lane, p.a_total - 1)) * p.route_stride;
       at.n_first = (block + 1) * p.route_width - (col0 + c);
@@ -425,7 +428,7 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
         for (int j = 0; j < 32; ++j) v[j] = gelu_tanh_fast(v[j]);
       }
     } else if (p.act == R2_ACT_GELU_ERF) {
-      if (p.out_is_bf16) {
+      if (ROUTED && p.out_is_bf16) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) v[j] = gelu_erf_rounded(v[j]);
       } else {
@@ -433,7 +436,7 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
         for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
       }
     }
-    if (p.route != nullptr) {
+    if constexpr (ROUTED) {
 #pragma unroll
       for (int j = 0; j < 32; ++j) v[j] *= j < at.n_first ? at.first : at.second;
     }
@@ -651,7 +654,7 @@ __device__ __forceinline__ void finish_tile_rows(const GemmParams& p, uint32_t l
 // A_MN / B_MN: the operand's tile in shared memory is MN-major (rows of 64 MN-elements, one row
 // per k) instead of K-major (rows of 64 k-elements, one row per MN index).
 // TRANSPOSED: the a side is the features and the b side the tokens.
-template <bool A_MN, bool B_MN, bool TRANSPOSED, bool FUSED_LN = false>
+template <bool A_MN, bool B_MN, bool TRANSPOSED, bool FUSED_LN = false, bool ROUTED = false>
 __global__ void __launch_bounds__(THREADS, (TRANSPOSED && !FUSED_LN) ? 1 : 2)  // token-major tiles run two CTAs to an SM, and so does the form with the norm inside (the logits' 393 CTAs)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmParams p) {
   extern __shared__ uint8_t smem_raw[];
@@ -890,7 +893,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         if (p.residual != nullptr) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) res_ahead[j] = (j < p.bn && b0 + j < p.b_total) ? p.residual[size_t(b0 + j) * p.ldr + a] : 0.f;
-        } else if (p.route != nullptr) {   // (never both)
+        } else if (ROUTED) {   // (never both)
           const float* weights = p.route + a / p.route_width;
 #pragma unroll
           for (int j = 0; j < 32; ++j) res_ahead[j] = (j < p.bn && b0 + j < p.b_total) ? weights[size_t(b0 + j) * p.route_stride] : 0.f;
@@ -953,7 +956,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     if constexpr (!TRANSPOSED) {
       // every product has completed: the first tiles' shared memory serves as the warps' slabs
       if (ok && a0 + q * 32 < p.a_total) {
-        finish_tile_rows(p, lane_addr, smem_u32(a_tiles) + uint32_t(q * STAGING_WORDS) * 4u, reduce, a0 + q * 32, b0, 0, p.bn, lane, n_kb > 0);
+        finish_tile_rows<ROUTED>(p, lane_addr, smem_u32(a_tiles) + uint32_t(q * STAGING_WORDS) * 4u, reduce, a0 + q * 32, b0, 0, p.bn, lane, n_kb > 0);
       }
     } else if (ok) {
       const bool a_ok = a < p.a_total;
@@ -996,7 +999,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_tanh_fast(v[j]);
           } else if (p.act == R2_ACT_GELU_ERF) {
-            if (p.out_is_bf16) {
+            if (ROUTED && p.out_is_bf16) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] = gelu_erf_rounded(v[j]);
             } else {
@@ -1004,7 +1007,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
               for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
             }
           }
-          if (p.route != nullptr) {
+          if constexpr (ROUTED) {
             if (c0 == 0) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] *= res_ahead[j];
@@ -1118,7 +1121,7 @@ constexpr int PAIR_THREADS = 320;        // warp 0: TMA, warp 1: MMA + tensor me
 constexpr int PAIR_EPILOGUE_WARPS = 8;
 constexpr int PAIR_SLAB_BYTES = PAIR_EPILOGUE_WARPS * STAGING_WORDS * 4;
 
-template <bool B_MN>
+template <bool B_MN, bool ROUTED = false>
 __global__ void __launch_bounds__(PAIR_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmParams p) {
   extern __shared__ uint8_t smem_raw[];
@@ -1307,7 +1310,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       if (ok && a0 + q * 32 < p.a_total) {
         const uint32_t lane_addr = tmem_base + buf * uint32_t(p.bn) + (uint32_t(q * 32) << 16);
-        finish_tile_rows(p, lane_addr, slab, bias_s, a0 + q * 32, b_tile0, side * half, (side + 1) * half, lane, true);
+        finish_tile_rows<ROUTED>(p, lane_addr, slab, bias_s, a0 + q * 32, b_tile0, side * half, (side + 1) * half, lane, true);
       }
       // this warp has read the accumulator: the leader may overwrite it with the tile after next
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -1335,9 +1338,9 @@ bool make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer
   return r2::encode_bf16_map(map, base, 2, dims, strides, box);
 }
 
-template <bool A_MN, bool B_MN, bool TRANSPOSED, bool FUSED_LN = false>
+template <bool A_MN, bool B_MN, bool TRANSPOSED, bool FUSED_LN = false, bool ROUTED = false>
 int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, dim3 grid, size_t smem, cudaStream_t stream) {
-  auto kernel = gemm_tc_kernel<A_MN, B_MN, TRANSPOSED, FUSED_LN>;
+  auto kernel = gemm_tc_kernel<A_MN, B_MN, TRANSPOSED, FUSED_LN, ROUTED>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
@@ -1549,9 +1552,9 @@ PairPlan make_pair_plan(int m, int n, int k, int w_is_nk, bool always) {
   return pl;
 }
 
-template <bool B_MN>
+template <bool B_MN, bool ROUTED = false>
 int launch_pair(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, const PairPlan& pl, cudaStream_t stream) {
-  auto kernel = gemm_tc_pair_kernel<B_MN>;
+  auto kernel = gemm_tc_pair_kernel<B_MN, ROUTED>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
@@ -1678,7 +1681,7 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
     p.kv_head_dim = kv->head_dim;
     p.kv_head_shift = (kv->head_dim & (kv->head_dim - 1)) == 0 ? page_shift_of(kv->head_dim) : -1;
   }
-  if (route != nullptr && (residual != nullptr || kv != nullptr || fused_ln || route_width < 32 || n % route_width != 0 || route_stride < n / route_width)) {
+  if (route != nullptr && (!w_is_nk || residual != nullptr || kv != nullptr || fused_ln || route_width < 32 || n % route_width != 0 || route_stride < n / route_width)) {
     return R2_UNSUPPORTED;   // (32 columns lie in two blocks at most; the caller multiplies in a kernel of its own)
   }
   p.route = route;
@@ -1722,7 +1725,7 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
       bool maps = make_map(&pa, x, x_cols, uint64_t(m), uint64_t(lda), BK, BM);
       if (w_is_nk) {
         maps = maps && make_map(&pb, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, uint32_t(pp.bn / 2));
-        if (maps) return launch_pair<false>(pa, pb, p, pp, stream);
+        if (maps) return route != nullptr ? launch_pair<false, true>(pa, pb, p, pp, stream) : launch_pair<false>(pa, pb, p, pp, stream);
       } else {
         maps = maps && make_map(&pb, w, uint64_t(n), uint64_t(k), uint64_t(ldw), 64, BK);
         if (maps) return launch_pair<true>(pa, pb, p, pp, stream);
@@ -1743,7 +1746,8 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
     if (w_is_nk) {
       ok = ok && make_map(&mb, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, uint32_t(bn));
       if (!ok) return R2_UNSUPPORTED;
-      return launch<false, false, false>(ma, mb, p, grid, smem, stream);
+      return route != nullptr ? launch<false, false, false, false, true>(ma, mb, p, grid, smem, stream)
+                              : launch<false, false, false>(ma, mb, p, grid, smem, stream);
     }
     ok = ok && make_map(&mb, w, uint64_t(n), uint64_t(k), uint64_t(ldw), 64, BK);
     if (!ok) return R2_UNSUPPORTED;
@@ -1755,6 +1759,7 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
   if (w_is_nk) {
     ok = ok && make_map(&ma, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, BM);
     if (!ok) return R2_UNSUPPORTED;
+    if (route != nullptr) return launch<false, false, true, false, true>(ma, mb, p, grid, smem, stream);
     return fused_ln ? launch<false, false, true, true>(ma, mb, p, grid, smem, stream)
                     : launch<false, false, true>(ma, mb, p, grid, smem, stream);
   }
