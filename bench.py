@@ -1392,12 +1392,12 @@ def tagulix_points(args, pk: dict) -> dict:
         add(f"its like: 8 sigmoid scores + a gate, 2 of 4 groups, top 2 (Zudalorn), {label}",
             lambda: ops.route_scored(hrow, router[:9], correction[:8].contiguous(), 2, 4, 2, n_extra=1), n_bytes=t * d * 2)
         w_up = (torch.randn(8 * width, d, device=dev) * 0.02).to(bf)
-        add(f"experts: first product with gelu and the routing weights inside, {d} x {8 * width:,}, {label}",
+        add(f"experts: first product, gelu and routing weights (one launch from 65 rows on, else two), {d} x {8 * width:,}, {label}",
             lambda: ops.routed_linear(hrow, w_up, "gelu", route, width), n_bytes=t * (d + 8 * width) * 2 + w_up.numel() * 2, flops=2 * t * w_up.numel())
         gu = torch.randn(t, 8 * width, device=dev).to(bf)
         add(f"its like: the same product alone (any model), {label}", lambda: ops.linear(hrow, w_up, None, w_is_nk=True),
             n_bytes=t * (d + 8 * width) * 2 + w_up.numel() * 2, flops=2 * t * w_up.numel())
-        add(f"(gelu and routing weights as a kernel of their own, {8 * width:,} columns, {label})", lambda: ops.expert_unit(gu, "gelu", route, width), n_bytes=t * gu.shape[1] * 4)
+        add(f"(gelu and routing weights alone, {8 * width:,} columns, {label})", lambda: ops.expert_unit(gu, "gelu", route, width), n_bytes=t * gu.shape[1] * 4)
         zu = torch.randn(t, 2 * 9 * (ff // 4), device=dev).to(bf)
         zroute, _, _, zg = ops.route_scored(hrow, router[:9], correction[:8].contiguous(), 2, 4, 2, n_extra=1)
         add(f"(its like there: experts' gated silu unit, {zu.shape[1] // 2:,} columns (Zudalorn), {label})",

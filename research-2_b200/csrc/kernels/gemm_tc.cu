@@ -844,7 +844,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 
   // ---- epilogue: warps 2..5, each on the 32 accumulator lanes it may read ------------------
   bool acc_ok = true;
-  float bias_ahead = 0.f, res_ahead[32];  // feature-major epilogue: the lane's bias, and its residual (or weights) for the first 32 tokens
+  float bias_ahead = 0.f, res_ahead[32];  // feature-major epilogue: the lane's bias, and its residual for the first 32 tokens
 #pragma unroll
   for (int j = 0; j < 32; ++j) res_ahead[j] = 0.f;
   if (threadIdx.x == 64 && p.prefetch != nullptr) {
@@ -893,10 +893,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         if (p.residual != nullptr) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) res_ahead[j] = (j < p.bn && b0 + j < p.b_total) ? p.residual[size_t(b0 + j) * p.ldr + a] : 0.f;
-        } else if (ROUTED) {   // (never both)
-          const float* weights = p.route + a / p.route_width;
-#pragma unroll
-          for (int j = 0; j < 32; ++j) res_ahead[j] = (j < p.bn && b0 + j < p.b_total) ? weights[size_t(b0 + j) * p.route_stride] : 0.f;
         }
       }
     }
@@ -999,28 +995,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_tanh_fast(v[j]);
           } else if (p.act == R2_ACT_GELU_ERF) {
-            if (ROUTED && p.out_is_bf16) {
 #pragma unroll
-              for (int j = 0; j < 16; ++j) v[j] = gelu_erf_rounded(v[j]);
-            } else {
-#pragma unroll
-              for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
-            }
-          }
-          if constexpr (ROUTED) {
-            if (c0 == 0) {
-#pragma unroll
-              for (int j = 0; j < 16; ++j) v[j] *= res_ahead[j];
-            } else if (c0 == 16) {
-#pragma unroll
-              for (int j = 0; j < 16; ++j) v[j] *= res_ahead[16 + j];
-            } else {
-              const float* weights = p.route + a / p.route_width;
-#pragma unroll
-              for (int j = 0; j < 16; ++j) {
-                if (j < nb) v[j] *= weights[size_t(b0 + c0 + j) * p.route_stride];
-              }
-            }
+            for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
           }
           if (p.residual != nullptr) {
             if (c0 == 0) {  // (asked for before the products ran: a chunk's residual read here costs it a round trip to L2)
@@ -1681,8 +1657,8 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
     p.kv_head_dim = kv->head_dim;
     p.kv_head_shift = (kv->head_dim & (kv->head_dim - 1)) == 0 ? page_shift_of(kv->head_dim) : -1;
   }
-  if (route != nullptr && (!w_is_nk || residual != nullptr || kv != nullptr || fused_ln || route_width < 32 || n % route_width != 0 || route_stride < n / route_width)) {
-    return R2_UNSUPPORTED;   // (32 columns lie in two blocks at most; the caller multiplies in a kernel of its own)
+  if (route != nullptr && (!w_is_nk || pl.swapped || residual != nullptr || kv != nullptr || fused_ln || route_width < 32 || n % route_width != 0 || route_stride < n / route_width)) {
+    return R2_UNSUPPORTED;   // (token-major tiles, whose 32 columns lie in two blocks at most; the caller multiplies in a kernel of its own)
   }
   p.route = route;
   p.route_stride = route_stride;
@@ -1759,7 +1735,6 @@ int gemm_tc_run(const void* x, int lda, const void* w, int ldw, int w_is_nk, con
   if (w_is_nk) {
     ok = ok && make_map(&ma, w, uint64_t(k), uint64_t(n), uint64_t(ldw), BK, BM);
     if (!ok) return R2_UNSUPPORTED;
-    if (route != nullptr) return launch<false, false, true, false, true>(ma, mb, p, grid, smem, stream);
     return fused_ln ? launch<false, false, true, true>(ma, mb, p, grid, smem, stream)
                     : launch<false, false, true>(ma, mb, p, grid, smem, stream);
   }
@@ -1790,7 +1765,7 @@ extern "C" int r2_gemm_tc_grouped(const void* x, int lda, const void* w, int ldw
 }
 
 // act(x @ w^T) with w [n, k] stored [out, in], each value times its token's weight for the block of route_width neighbouring features
-// that it lies in: route float [m, >= n / route_width], rows route_stride apart. Blocks narrower than 32: R2_UNSUPPORTED.
+// that it lies in: route float [m, >= n / route_width], rows route_stride apart. Blocks narrower than 32, and few tokens (features in the tile's rows): R2_UNSUPPORTED.
 extern "C" int r2_gemm_tc_routed(const void* x, int lda, const void* w, int ldw, void* out, int ldo, int m, int n, int k, int act,
                                  const float* route, int route_stride, int route_width, int out_dtype, int* error_flag, cudaStream_t stream) {
   if (route == nullptr) return R2_BAD_SHAPE;

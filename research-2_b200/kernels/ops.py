@@ -549,16 +549,16 @@ def expert_unit(up: torch.Tensor, act: str, route: torch.Tensor, expert_width: i
 
 def routed_linear(a: torch.Tensor, w: torch.Tensor, act: str, route: torch.Tensor, expert_width: int) -> torch.Tensor:
     """act(a @ w^T) times the row's weight for the column's expert: the first product of experts without gates whose matrices are
-    stacked (w [experts * expert_width, K], stored [out, in]), in a's dtype. The tensor-core kernel does it in its epilogue, from float32
-    values; else `expert_unit` does it to the product's result."""
+    stacked (w [experts * expert_width, K], stored [out, in]), in a's dtype. For more than 64 rows the tensor-core kernel does it in its
+    epilogue, from float32 values; else `expert_unit` does it to the product's result."""
     _need(a, "a", dim=2)
     _need(w, "w", a.dtype, 2)
     _need(route, "route", torch.float32, 2)
     m, k, n = a.shape[0], a.shape[1], w.shape[0]
     if w.shape[1] != k or n % expert_width or route.shape[0] != m or route.shape[1] < n // expert_width or act not in ACTIVATIONS:
         raise KernelError(f"routed_linear: a {tuple(a.shape)}, w {tuple(w.shape)}, experts of {expert_width}, route {tuple(route.shape)} do not fit")
-    # (33 to 64 rows: two launches, 9.7 us at 768 x 6,144 columns; in the epilogue, whose threads have a feature each, 10.9)
-    if a.dtype == torch.bfloat16 and _tensor_core_gemm and not 32 < m <= 64:
+    # (few rows: two launches; inside the product a decode step of 12 layers and 8 rows took 0.71 ms against 0.67)
+    if a.dtype == torch.bfloat16 and _tensor_core_gemm and m > 64:
         out = torch.empty(m, n, dtype=a.dtype, device=a.device)
         status = _lib("gemm_tc").r2_gemm_tc_routed(_p(a), _rows(a, "a"), _p(w), _rows(w, "w"), _p(out), n, m, n, k, ACTIVATIONS[act], _p(route),
                                                   _rows(route, "route"), expert_width, BF16, _p(_workspace(a.device).error), _stream())
